@@ -19,8 +19,8 @@ that place.  Pages are handed out last-freed-first (kv.go:29-40), so reuse is
 immediate.
 
 Beside the pages, every request holds one state slot.  A mixer with per-request
-state of fixed size (``StateNeed``) gets a tensor [max_requests, *shape] per layer,
-and the slot's rows are zeroed when a request opens.  Models without such a mixer
+state of fixed size (``StateNeed``) gets a tensor [max_requests, *shape] per layer
+(a layer may ask for several, told apart by name), and the slot's rows are zeroed when a request opens.  Models without such a mixer
 hold and return their slots all the same.
 """
 from __future__ import annotations
@@ -128,6 +128,7 @@ class CacheManager:
         self.slot_group: Dict[int, int] = {}       # cache slot -> group index
         self.slot_layer: Dict[int, int] = {}       # cache slot -> index inside its group
         self.state: Dict[int, torch.Tensor] = {}   # cache slot -> [max_requests, *shape]
+        self.named_states: Dict[int, Dict[str, torch.Tensor]] = {}     # cache slot -> name -> the same, of further states
         self.n_slots = len(needs)
         by_key: Dict[tuple, CacheGroup] = {}
         for slot, need in enumerate(needs):
@@ -155,11 +156,15 @@ class CacheManager:
                     self.slot_layer[slot] = len(g.slots)
                     g.slots.append(slot)
                 elif isinstance(item, StateNeed):
+                    t = None
                     if allocate:
-                        self.state[slot] = torch.zeros((max_requests,) + tuple(item.shape),
-                                                       dtype=getattr(torch, item.dtype), device=self.device)
-                    else:
-                        self.state[slot] = None
+                        t = torch.zeros((max_requests,) + tuple(item.shape), dtype=getattr(torch, item.dtype),
+                                        device=self.device)
+                    held = self.named_states.setdefault(slot, {}) if item.name else self.state
+                    key = item.name or slot
+                    if key in held:
+                        raise ValueError(f"cache slot {slot} asks for two states named {item.name!r}")
+                    held[key] = t
                 else:
                     raise TypeError(f"cache slot {slot}: unknown need {item!r}")
         if allocate:
@@ -246,7 +251,7 @@ class CacheManager:
         if rid in self.live:
             raise CacheError(f"request {rid} is already open")
         (slot,) = self.state_slots.take(1)
-        for t in self.state.values():
+        for t in list(self.state.values()) + [t for named in self.named_states.values() for t in named.values()]:
             if t is not None:
                 t[slot].zero_()
         req = RequestCache(rid=rid, state_slot=slot, tables=[[] for _ in self.groups])
@@ -351,7 +356,7 @@ class CacheManager:
                 k, v = g.k_store[layer], g.v_store[layer]
                 table = block_tables[g.index]
             out.append(LayerCache(k=k, v=v, block_table=table, state=self.state.get(slot),
-                                  writes=True, page_size=self.page_size))
+                                  writes=True, page_size=self.page_size, states=self.named_states.get(slot, {})))
         return out
 
     # ---- checks for tests and debugging -------------------------------------

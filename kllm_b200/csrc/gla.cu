@@ -1,0 +1,705 @@
+// Linear attention with a decaying state, for mixed batches of prompt portions and single tokens, with
+// the state of every request in a slot of a state tensor.
+//
+// Per head, with dk key channels d, dv value channels e and a state S [dk][dv] that starts at zero for
+// a new request:
+//
+//     S_t[d][e] = alpha_t[d] S_(t-1)[d][e] + k_t[d] v_t[e]          o_t[e] = sum_d S_t[d][e] q_t[d]
+//     y_t       = o_t / rms(o_t over the head's dv values) * gain * silu(g_t)
+//
+// The decay alpha has two forms.  Gated: alpha = sigmoid(z)^(1 / tau) per key channel, z = W2 low_t + b, the
+// outer half of a low-rank product whose inner half `low` comes with the projections.  Fixed: one number per
+// head.  q and k may be rotated first (the pairs (i, i + rot / 2), i < rot / 2, by position * freq[i], the angle
+// formed in double precision) and are multiplied by q_scale and k_scale.  Everything is float32: the
+// projections arrive unrounded, the decay, the state and every sum; y alone is stored in the model's type.
+//
+// Steps in which every request brings one row take one kernel (step_kernel): a cluster of CTAs per (head,
+// request), each CTA with a slice of the value channels; the state's slice is on its way from HBM before the
+// projections are waited for, is updated in registers and written back, and the cluster's CTAs join their sums
+// of squares through distributed shared memory for the head's norm.
+//
+// Steps with portions take three kernels.  A request's rows are cut into chunks of kC rows.  Since the
+// recurrence is linear in the state, with the cumulative decay A_i = alpha_first ... alpha_i of a chunk
+//
+//     o_i = local_i + sum_d (q_i A_i)[d] S_in[d]           S_out = A_last S_in + S_local
+//
+// where local and S_local belong to the same rows run from a zero state:
+//   local_kernel   every chunk at once: the recurrence row by row from a zero state; leaves local_i, S_local,
+//                  q_i A_i and A_last
+//   carry_kernel   the states at the chunks' starts, element by element over a request's chunks in order;
+//                  moves the slot on
+//   apply_kernel   every chunk at once: o, the head's norm and the gate
+// No quotient of decays is ever formed: every factor is a product of numbers in [0, 1], so a decay that reaches
+// zero inside a chunk is harmless.  Where a prompt is cut changes the order of float32 sums and nothing else.
+#include "common.cuh"
+
+KLLM_EXPORT_LAST_ERROR(gla)
+
+namespace {
+
+constexpr int kC = 64;          // rows of a chunk
+constexpr int kTS = 16;         // rows staged in shared memory at a time
+constexpr int kSl = 64;         // value channels of a CTA of the local kernel
+constexpr int kThreads = 256;
+constexpr int kMaxRot = 256;
+
+struct GlaArgs {
+    const float *q, *k, *v, *g;             // rows of the projections, float32, at `stride`
+    int64_t stride;
+    const float* low;                       // gated decay: [n][R] at `stride`; null: fixed decay
+    const void* w2;                         // [H * dk][R] in the model's type
+    const float* w2_bias;                   // [H * dk]
+    int R;
+    float inv_tau;
+    const float* decay;                     // fixed decay: [H]
+    const double* freq;                     // [rot / 2], or null
+    int rot;
+    float amplitude, q_scale, k_scale;
+    const int* positions;
+    const int *q_start, *state_slots;
+    int n_requests, heads, dk, dv;
+    float* state;
+    int64_t state_stride;
+    const float* gain;                      // [H * dv]
+    float eps;
+    void* y;
+    int64_t y_stride;
+    // work of the three-kernel form
+    float *o, *qa, *a_last, *s_in;          // [n][H dv], [n][H dk], [chunks][H dk], [chunks][H][dk][dv]
+    const int* start_pos;
+};
+
+__device__ __forceinline__ void cluster_sync_all() {
+    asm volatile("barrier.cluster.arrive.release.aligned;\n" ::: "memory");
+    asm volatile("barrier.cluster.wait.acquire.aligned;\n" ::: "memory");
+}
+
+__device__ __forceinline__ float peer_f32(const float* p, int rank) {
+    unsigned a = (unsigned)__cvta_generic_to_shared(p), r;
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;\n" : "=r"(r) : "r"(a), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];\n" : "=f"(v) : "r"(r) : "memory");
+    return v;
+}
+
+__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+
+// sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau)
+__device__ __forceinline__ float gated_alpha(float z, float inv_tau) {
+    return expf(-(log1pf(expf(-fabsf(z))) + fmaxf(-z, 0.f)) * inv_tau);
+}
+
+// element d of a head's row, turned by the row's angles (cos [half], sin [half])
+__device__ __forceinline__ float turned(const float* row, int d, int rot, const float* cs) {
+    const float x = row[d];
+    if (d >= rot) return x;
+    const int half = rot >> 1;
+    return d < half ? x * cs[d] - row[d + half] * cs[half + d] : x * cs[d - half] + row[d - half] * cs[d];
+}
+
+template <int V> struct Vec { float x[V]; };
+template <int V> __device__ __forceinline__ Vec<V> load_vec(const float* p) {
+    Vec<V> r;
+    if constexpr (V == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        r.x[0] = t.x; r.x[1] = t.y; r.x[2] = t.z; r.x[3] = t.w;
+    } else {
+#pragma unroll
+        for (int i = 0; i < V; i++) r.x[i] = p[i];
+    }
+    return r;
+}
+template <int V> __device__ __forceinline__ void store_vec(float* p, const Vec<V>& r) {
+    if constexpr (V == 4) {
+        *reinterpret_cast<float4*>(p) = make_float4(r.x[0], r.x[1], r.x[2], r.x[3]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < V; i++) p[i] = r.x[i];
+    }
+}
+
+// ---- one row per request -----------------------------------------------------------------------------------
+// grid (slices, heads, requests), cluster (slices, 1, 1).  Thread (cg, dl): V value channels e0 + cg V ..., key
+// channels dl, dl + lanes, ...  Shared memory: partial sums [kThreads * V], o [sl], q, k, alpha [dk] each,
+// cos / sin [rot], W2 [dk][R + 1] (gated).  Started early, the kernel reads the state before the kernel in front of it
+// has ended: that kernel must not write the state.
+template <typename T, int V>
+__global__ void __launch_bounds__(kThreads)
+step_kernel(const GlaArgs a, int sl) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[32];
+    __shared__ float part;
+    constexpr int NB = V == 4 ? 8 : 16;                     // key channels in flight per thread
+    const int tid = threadIdx.x, slice = blockIdx.x, head = blockIdx.y, req = blockIdx.z;
+    const int dk = a.dk, dv = a.dv, R = a.R;
+    float* ps = sm;                                         // [kThreads * V], 16-byte aligned
+    float* ob = ps + kThreads * V;                          // [sl]
+    float* qs = ob + sl;
+    float* ks = qs + dk;
+    float* as = ks + dk;
+    float* cs = as + dk;                                    // [rot]
+    float* w2s = cs + a.rot;                                // [dk][R + 1]
+    const int t = a.q_start[req];
+    const int groups = sl / V, lanes = kThreads / groups, cg = tid % groups, dl = tid / groups;
+    const bool on = dl < lanes;
+    const int e = slice * sl + cg * V;
+    float* Sg = a.state + (int64_t)a.state_slots[req] * a.state_stride + (int64_t)head * dk * dv + e;
+    // what no kernel right before this one writes: the state, the decay's matrix, the angles
+    Vec<V> s[NB];
+#pragma unroll
+    for (int i = 0; i < NB; i++) {
+        const int d = dl + i * lanes;
+        if (on && d < dk) s[i] = load_vec<V>(Sg + (int64_t)d * dv);
+    }
+    if (a.low) {
+        const T* w2 = reinterpret_cast<const T*>(a.w2) + (int64_t)head * dk * R;
+        for (int i = tid; i < dk * R; i += kThreads) w2s[(i / R) * (R + 1) + i % R] = to_f32(w2[i]);
+    }
+    const int half = a.rot >> 1;
+    for (int i = tid; i < half; i += kThreads) {
+        double sn, c;
+        sincos((double)a.positions[t] * a.freq[i], &sn, &c);
+        cs[i] = (float)c * a.amplitude;
+        cs[half + i] = (float)sn * a.amplitude;
+    }
+    __syncthreads();
+    griddep_wait();
+    griddep_launch();
+    const float* qr = a.q + (int64_t)t * a.stride + head * dk;
+    const float* kr = a.k + (int64_t)t * a.stride + head * dk;
+    for (int d = tid; d < dk; d += kThreads) {
+        qs[d] = turned(qr, d, a.rot, cs) * a.q_scale;
+        ks[d] = turned(kr, d, a.rot, cs) * a.k_scale;
+        float al;
+        if (a.low) {
+            const float* lr = a.low + (int64_t)t * a.stride;
+            float z = 0.f;
+#pragma unroll 8
+            for (int r = 0; r < R; r++) z = fmaf(lr[r], w2s[d * (R + 1) + r], z);
+            al = gated_alpha(z + a.w2_bias[head * dk + d], a.inv_tau);
+        } else {
+            al = a.decay[head];
+        }
+        as[d] = al;
+    }
+    Vec<V> vv, acc;
+#pragma unroll
+    for (int j = 0; j < V; j++) acc.x[j] = 0.f;
+    if (on) vv = load_vec<V>(a.v + (int64_t)t * a.stride + head * dv + e);
+    __syncthreads();
+    if (on) {
+        for (int d0 = dl; d0 < dk; d0 += NB * lanes) {
+            if (d0 != dl) {
+#pragma unroll
+                for (int i = 0; i < NB; i++) {
+                    const int d = d0 + i * lanes;
+                    if (d < dk) s[i] = load_vec<V>(Sg + (int64_t)d * dv);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < NB; i++) {
+                const int d = d0 + i * lanes;
+                if (d < dk) {
+                    const float al = as[d], kd = ks[d], qd = qs[d];
+#pragma unroll
+                    for (int j = 0; j < V; j++) {
+                        s[i].x[j] = fmaf(al, s[i].x[j], kd * vv.x[j]);
+                        acc.x[j] = fmaf(qd, s[i].x[j], acc.x[j]);
+                    }
+                    store_vec<V>(Sg + (int64_t)d * dv, s[i]);
+                }
+            }
+        }
+        store_vec<V>(ps + dl * sl + cg * V, acc);
+    }
+    __syncthreads();
+    float ss = 0.f;
+    for (int c = tid; c < sl; c += kThreads) {
+        float o = 0.f;
+        for (int l = 0; l < lanes; l++) o += ps[l * sl + c];
+        ob[c] = o;
+        ss += o * o;
+    }
+    ss = block_sum(ss, red);
+    if (tid == 0) part = ss;
+    cluster_sync_all();
+    float tot = 0.f;
+    for (int r = 0; r < (int)gridDim.x; r++) tot += peer_f32(&part, r);
+    const float scale = rsqrtf(tot / (float)dv + a.eps);
+    T* yr = reinterpret_cast<T*>(a.y) + (int64_t)t * a.y_stride + head * dv + slice * sl;
+    const float* gr = a.g + (int64_t)t * a.stride + head * dv + slice * sl;
+    const float* gn = a.gain + head * dv + slice * sl;
+    for (int c = tid; c < sl; c += kThreads) yr[c] = from_f32<T>(ob[c] * scale * gn[c] * silu_f(gr[c]));
+    cluster_sync_all();                                     // no CTA leaves while another may still read its sum
+}
+
+// ---- portions ------------------------------------------------------------------------------------------------
+
+// The request and first row of the step's chunk number `chunk`; false beyond the last chunk.
+__device__ __forceinline__ bool find_chunk(const GlaArgs& a, int chunk, int& req, int& row0, int& rows, int& index) {
+    for (req = 0; req < a.n_requests; req++) {
+        const int lo = a.q_start[req], len = a.q_start[req + 1] - lo, chunks = (len + kC - 1) / kC;
+        if (chunk < chunks) {
+            index = chunk;
+            row0 = lo + chunk * kC;
+            rows = min(kC, len - chunk * kC);
+            return true;
+        }
+        chunk -= chunks;
+    }
+    return false;
+}
+
+// grid (chunk bound, heads, slices of kSl value channels).  Thread (cg, l): value channels 4 cg .. 4 cg + 3 of the
+// slice, key channels of lane l = tid % 16: (i * 16 + l) * W + j, i < DPT / W, j < W.
+// Shared memory: q, k, alpha [kTS][16 DPT], v [kTS][kSl], cumulative decay [16 DPT], cos / sin [kTS][rot],
+// gated: W2 [dk][R + 1], low [kTS][R].
+template <typename T, int DPT>
+__global__ void __launch_bounds__(kThreads)
+local_kernel(const GlaArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int W = DPT < 4 ? DPT : 4, P = 16 * DPT, NI = DPT / W;
+    griddep_wait();
+    griddep_launch();
+    const int tid = threadIdx.x, l = tid & 15, cg = tid >> 4, lane = tid & 31;
+    const int head = blockIdx.y, e0 = blockIdx.z * kSl, dk = a.dk, dv = a.dv, R = a.R, rot = a.rot, half = rot >> 1;
+    const int ne = min(kSl, dv - e0);
+    int req, row0, rows, index;
+    if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
+    float* qs = sm;
+    float* ks = qs + kTS * P;
+    float* as = ks + kTS * P;
+    float* vs = as + kTS * P;
+    float* cum = vs + kTS * kSl;
+    float* cs = cum + P;
+    float* lows = cs + kTS * rot;
+    float* w2s = lows + kTS * R;
+    if (a.low) {
+        const T* w2 = reinterpret_cast<const T*>(a.w2) + (int64_t)head * dk * R;
+        for (int i = tid; i < dk * R; i += kThreads) w2s[(i / R) * (R + 1) + i % R] = to_f32(w2[i]);
+    }
+    for (int i = tid; i < P; i += kThreads) cum[i] = 1.f;
+    float S[4][DPT];
+#pragma unroll
+    for (int c = 0; c < 4; c++)
+#pragma unroll
+        for (int i = 0; i < DPT; i++) S[c][i] = 0.f;
+    const int A_w = a.heads * dk, B_w = a.heads * dv;
+    for (int b0 = 0; b0 < rows; b0 += kTS) {
+        const int nr = min(kTS, rows - b0), r0 = row0 + b0;
+        for (int i = tid; i < nr * half; i += kThreads) {
+            const int r = i / half, j = i - r * half;
+            double sn, c;
+            sincos((double)a.positions[r0 + r] * a.freq[j], &sn, &c);
+            cs[r * rot + j] = (float)c * a.amplitude;
+            cs[r * rot + half + j] = (float)sn * a.amplitude;
+        }
+        if (a.low)
+            for (int i = tid; i < nr * R; i += kThreads) lows[i] = a.low[(int64_t)(r0 + i / R) * a.stride + i % R];
+        __syncthreads();                    // angles and low rows are there; the batch before has been used up
+        for (int i = tid; i < kTS * P; i += kThreads) {
+            const int r = i / P, d = i - r * P;
+            float q = 0.f, k = 0.f, al = 1.f;
+            if (r < nr && d < dk) {
+                const int64_t off = (int64_t)(r0 + r) * a.stride + head * dk;
+                q = turned(a.q + off, d, rot, cs + r * rot) * a.q_scale;
+                k = turned(a.k + off, d, rot, cs + r * rot) * a.k_scale;
+                if (a.low) {
+                    float z = 0.f;
+#pragma unroll 4
+                    for (int j = 0; j < R; j++) z = fmaf(lows[r * R + j], w2s[d * (R + 1) + j], z);
+                    al = gated_alpha(z + a.w2_bias[head * dk + d], a.inv_tau);
+                } else {
+                    al = a.decay[head];
+                }
+            }
+            qs[i] = q;
+            ks[i] = k;
+            as[i] = al;
+        }
+        for (int i = tid; i < kTS * kSl; i += kThreads) {
+            const int r = i / kSl, c = i - r * kSl;
+            vs[i] = (r < nr && c < ne) ? a.v[(int64_t)(r0 + r) * a.stride + head * dv + e0 + c] : 0.f;
+        }
+        __syncthreads();
+        if (blockIdx.z == 0) {              // q_i A_i, once per (chunk, head)
+            for (int d = tid; d < dk; d += kThreads) {
+                float c = cum[d];
+                for (int r = 0; r < nr; r++) {
+                    c *= as[r * P + d];
+                    a.qa[(int64_t)(r0 + r) * A_w + head * dk + d] = qs[r * P + d] * c;
+                }
+                cum[d] = c;
+            }
+        }
+        // rows in fours (those beyond the batch have q = k = v = 0, alpha = 1 and change nothing)
+        for (int rb = 0; rb < nr; rb += 4) {
+            float acc[16];                  // [row of the four][value channel of the four]
+#pragma unroll
+            for (int p = 0; p < 4; p++) {
+                const int r = rb + p;
+                const float4 v4 = *reinterpret_cast<const float4*>(vs + r * kSl + cg * 4);
+                const float vv[4] = {v4.x, v4.y, v4.z, v4.w};
+#pragma unroll
+                for (int c = 0; c < 4; c++) acc[p * 4 + c] = 0.f;
+#pragma unroll
+                for (int i = 0; i < NI; i++) {
+                    const int d = r * P + (i * 16 + l) * W;
+                    float q[W], k[W], al[W];
+                    if constexpr (W == 4) {
+                        const float4 q4 = *reinterpret_cast<const float4*>(qs + d), k4 = *reinterpret_cast<const float4*>(ks + d),
+                                     a4 = *reinterpret_cast<const float4*>(as + d);
+                        q[0] = q4.x; q[1] = q4.y; q[2] = q4.z; q[3] = q4.w;
+                        k[0] = k4.x; k[1] = k4.y; k[2] = k4.z; k[3] = k4.w;
+                        al[0] = a4.x; al[1] = a4.y; al[2] = a4.z; al[3] = a4.w;
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < W; j++) { q[j] = qs[d + j]; k[j] = ks[d + j]; al[j] = as[d + j]; }
+                    }
+#pragma unroll
+                    for (int j = 0; j < W; j++)
+#pragma unroll
+                        for (int c = 0; c < 4; c++) {
+                            float& s = S[c][i * W + j];
+                            s = fmaf(al[j], s, k[j] * vv[c]);
+                            acc[p * 4 + c] = fmaf(q[j], s, acc[p * 4 + c]);
+                        }
+                }
+            }
+            // sixteen sums over sixteen lanes by halving: lane l ends with the sum number l
+#pragma unroll
+            for (int o = 8; o >= 1; o >>= 1) {
+                const bool upper = (lane & o) != 0;
+#pragma unroll
+                for (int j = 0; j < o; j++) {
+                    const float send = upper ? acc[j] : acc[j + o];
+                    const float keep = upper ? acc[j + o] : acc[j];
+                    acc[j] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                }
+            }
+            const int r = rb + (l >> 2), c = cg * 4 + (l & 3);
+            if (r < nr && c < ne) a.o[(int64_t)(r0 + r) * B_w + head * dv + e0 + c] = acc[0];
+        }
+        __syncthreads();
+    }
+    if (blockIdx.z == 0)
+        for (int d = tid; d < dk; d += kThreads) a.a_last[(int64_t)blockIdx.x * A_w + head * dk + d] = cum[d];
+    float* dst = a.s_in + ((int64_t)blockIdx.x * a.heads + head) * dk * dv + e0 + cg * 4;
+    const bool whole = (dv & 3) == 0 && cg * 4 + 4 <= ne;
+#pragma unroll
+    for (int i = 0; i < DPT; i++) {
+        const int d = (i / W * 16 + l) * W + i % W;
+        if (d >= dk) continue;
+        if (whole) {
+            *reinterpret_cast<float4*>(dst + (int64_t)d * dv) = make_float4(S[0][i], S[1][i], S[2][i], S[3][i]);
+        } else {
+#pragma unroll
+            for (int c = 0; c < 4; c++)
+                if (cg * 4 + c < ne) dst[(int64_t)d * dv + c] = S[c][i];
+        }
+    }
+}
+
+// grid (pieces of kThreads * V state elements, heads, requests): s_in turns from the chunks' own states into the
+// states at their starts.
+template <int V>
+__global__ void __launch_bounds__(kThreads)
+carry_kernel(const GlaArgs a) {
+    griddep_wait();
+    griddep_launch();
+    const int head = blockIdx.y, req = blockIdx.z, dk = a.dk, dv = a.dv;
+    const int64_t i = ((int64_t)blockIdx.x * kThreads + threadIdx.x) * V;
+    if (i >= (int64_t)dk * dv) return;
+    int chunk = 0;
+    for (int r = 0; r < req; r++) chunk += (a.q_start[r + 1] - a.q_start[r] + kC - 1) / kC;
+    const int chunks = (a.q_start[req + 1] - a.q_start[req] + kC - 1) / kC;
+    float* slot = a.state + (int64_t)a.state_slots[req] * a.state_stride + (int64_t)head * dk * dv + i;
+    float* w = a.s_in + ((int64_t)chunk * a.heads + head) * dk * dv + i;
+    const float* al = a.a_last + (int64_t)chunk * a.heads * dk + head * dk + i / dv;
+    const int64_t step = (int64_t)a.heads * dk * dv;
+    const int a_step = a.heads * dk;
+    Vec<V> s = load_vec<V>(slot);
+    constexpr int AHEAD = 8;
+    for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+        Vec<V> loc[AHEAD];
+        float d[AHEAD];
+#pragma unroll
+        for (int u = 0; u < AHEAD; u++)
+            if (c0 + u < chunks) {
+                loc[u] = load_vec<V>(w + (c0 + u) * step);
+                d[u] = al[(int64_t)(c0 + u) * a_step];
+            }
+#pragma unroll
+        for (int u = 0; u < AHEAD; u++)
+            if (c0 + u < chunks) {
+                store_vec<V>(w + (c0 + u) * step, s);
+#pragma unroll
+                for (int j = 0; j < V; j++) s.x[j] = fmaf(d[u], s.x[j], loc[u].x[j]);
+            }
+    }
+    store_vec<V>(slot, s);
+}
+
+// grid (chunk bound, heads, column blocks of 64 NJ).  Thread (rg, cg): rows 4 rg .. 4 rg + 3, value channels
+// j * 64 + 4 cg .. + 3.  NORM: the columns are all of the head's (grid.z is 1) and the row is normed, gated and stored
+// in y; otherwise o is written back.  Shared memory: q A [kC][36], S [32][64 NJ].
+template <typename T, int NJ, bool NORM>
+__global__ void __launch_bounds__(kThreads)
+apply_kernel(const GlaArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int DB = 32, QP = DB + 4, CW = 64 * NJ;
+    griddep_wait();
+    griddep_launch();
+    const int tid = threadIdx.x, cg = tid & 15, rg = tid >> 4;
+    const int head = blockIdx.y, e0 = blockIdx.z * CW, dk = a.dk, dv = a.dv;
+    const int ne = min(CW, dv - e0);
+    int req, row0, rows, index;
+    if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
+    float* qs = sm;                         // [kC][QP]
+    float* ss = qs + kC * QP;               // [DB][CW]
+    float acc[4][NJ * 4];
+#pragma unroll
+    for (int r = 0; r < 4; r++)
+#pragma unroll
+        for (int j = 0; j < NJ * 4; j++) acc[r][j] = 0.f;
+    const int A_w = a.heads * dk, B_w = a.heads * dv;
+    const float* S = a.s_in + ((int64_t)blockIdx.x * a.heads + head) * dk * dv + e0;
+    const bool from_zero = index == 0 && a.start_pos[req] == 0;        // the state in front of a request's first chunk
+    for (int d0 = 0; d0 < dk && !from_zero; d0 += DB) {
+        const int nd = min(DB, dk - d0);
+        __syncthreads();
+        for (int i = tid; i < kC * DB; i += kThreads) {
+            const int r = i / DB, d = i - r * DB;
+            qs[r * QP + d] = (r < rows && d < nd) ? a.qa[(int64_t)(row0 + r) * A_w + head * dk + d0 + d] : 0.f;
+        }
+        if ((dv & 3) == 0) {
+            for (int i = tid; i < DB * CW / 4; i += kThreads) {
+                const int d = i / (CW / 4), c = (i - d * (CW / 4)) * 4;
+                *reinterpret_cast<float4*>(ss + d * CW + c) =
+                    (d < nd && c < ne) ? *reinterpret_cast<const float4*>(S + (int64_t)(d0 + d) * dv + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+        } else {
+            for (int i = tid; i < DB * CW; i += kThreads) {
+                const int d = i / CW, c = i - d * CW;
+                ss[i] = (d < nd && c < ne) ? S[(int64_t)(d0 + d) * dv + c] : 0.f;
+            }
+        }
+        __syncthreads();
+#pragma unroll 2
+        for (int d = 0; d < DB; d += 4) {
+            float q[4][4];
+#pragma unroll
+            for (int r = 0; r < 4; r++) {
+                const float4 q4 = *reinterpret_cast<const float4*>(qs + (rg * 4 + r) * QP + d);
+                q[r][0] = q4.x; q[r][1] = q4.y; q[r][2] = q4.z; q[r][3] = q4.w;
+            }
+#pragma unroll
+            for (int j = 0; j < NJ; j++)
+#pragma unroll
+                for (int u = 0; u < 4; u++) {
+                    const float4 s4 = *reinterpret_cast<const float4*>(ss + (d + u) * CW + j * 64 + cg * 4);
+#pragma unroll
+                    for (int r = 0; r < 4; r++) {
+                        acc[r][j * 4 + 0] = fmaf(q[r][u], s4.x, acc[r][j * 4 + 0]);
+                        acc[r][j * 4 + 1] = fmaf(q[r][u], s4.y, acc[r][j * 4 + 1]);
+                        acc[r][j * 4 + 2] = fmaf(q[r][u], s4.z, acc[r][j * 4 + 2]);
+                        acc[r][j * 4 + 3] = fmaf(q[r][u], s4.w, acc[r][j * 4 + 3]);
+                    }
+                }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < 4; r++) {
+        const int row = rg * 4 + r;
+        float* orow = a.o + (int64_t)(row0 + min(row, rows - 1)) * B_w + head * dv + e0;
+        float sq = 0.f;
+#pragma unroll
+        for (int j = 0; j < NJ; j++)
+#pragma unroll
+            for (int c = 0; c < 4; c++) {
+                const int col = j * 64 + cg * 4 + c;
+                float& x = acc[r][j * 4 + c];
+                x = col < ne ? x + orow[col] : 0.f;
+                sq += x * x;
+            }
+        if constexpr (NORM) {
+#pragma unroll
+            for (int o = 8; o >= 1; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+            if (row < rows) {
+                const float scale = rsqrtf(sq / (float)dv + a.eps);
+                T* yr = reinterpret_cast<T*>(a.y) + (int64_t)(row0 + row) * a.y_stride + head * dv;
+                const float* gr = a.g + (int64_t)(row0 + row) * a.stride + head * dv;
+#pragma unroll
+                for (int j = 0; j < NJ; j++)
+#pragma unroll
+                    for (int c = 0; c < 4; c++) {
+                        const int col = j * 64 + cg * 4 + c;
+                        if (col < ne) yr[col] = from_f32<T>(acc[r][j * 4 + c] * scale * a.gain[head * dv + col] * silu_f(gr[col]));
+                    }
+            }
+        } else if (row < rows) {
+#pragma unroll
+            for (int j = 0; j < NJ; j++)
+#pragma unroll
+                for (int c = 0; c < 4; c++) {
+                    const int col = j * 64 + cg * 4 + c;
+                    if (col < ne) orow[col] = acc[r][j * 4 + c];
+                }
+        }
+    }
+}
+
+// a head wider than one apply CTA: norm and gate in a kernel of their own, one warp per (row, head)
+template <typename T>
+__global__ void __launch_bounds__(kThreads)
+norm_gate_kernel(const GlaArgs a, int n) {
+    griddep_wait();
+    griddep_launch();
+    const int lane = threadIdx.x & 31, dv = a.dv;
+    const int64_t item = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
+    if (item >= (int64_t)n * a.heads) return;
+    const int64_t t = item / a.heads;
+    const int head = (int)(item - t * a.heads);
+    const float* orow = a.o + item * dv;
+    float sq = 0.f;
+    for (int c = lane; c < dv; c += 32) sq += orow[c] * orow[c];
+    const float scale = rsqrtf(warp_sum(sq) / (float)dv + a.eps);
+    const float* gr = a.g + t * a.stride + head * dv;
+    T* yr = reinterpret_cast<T*>(a.y) + t * a.y_stride + head * dv;
+    for (int c = lane; c < dv; c += 32) yr[c] = from_f32<T>(orow[c] * scale * a.gain[head * dv + c] * silu_f(gr[c]));
+}
+
+template <int V> size_t step_smem(const GlaArgs& a, int sl) {
+    return sizeof(float) * ((size_t)3 * a.dk + a.rot + sl + (size_t)kThreads * V + (a.low ? (size_t)a.dk * (a.R + 1) : 0));
+}
+
+template <typename T, int V>
+int launch_step(const GlaArgs& a, bool early, cudaStream_t s) {
+    // slices: a power of two up to a portable cluster's 8 CTAs, more of them while the launch would leave SMs idle
+    int slices = 1;
+    auto splits = [&](int n) { return a.dv % (n * V) == 0; };
+    while (a.dv / slices / V > kThreads && slices < 8 && splits(slices * 2)) slices *= 2;
+    while (slices < 8 && splits(slices * 2) && a.dv / (slices * 2) >= 16 && (int64_t)slices * a.heads * a.n_requests < 148) slices *= 2;
+    const int sl = a.dv / slices;
+    if (sl / V > kThreads) KLLM_FAIL("gla step: a head of %d value channels does not fit", a.dv);
+    const size_t smem = step_smem<V>(a, sl);
+    if (smem > 200 * 1024) KLLM_FAIL("gla step: a head of %d key channels with a decay of rank %d does not fit shared memory", a.dk, a.R);
+    auto kern = step_kernel<T, V>;
+    static bool raised = false;
+    if (!raised) {
+        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        if (e != cudaSuccess) KLLM_FAIL("gla step: %s", cudaGetErrorString(e));
+        raised = true;
+    }
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(slices, a.heads, a.n_requests);
+    cfg.blockDim = dim3(kThreads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = s;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = slices;
+    attr[0].val.clusterDim.y = 1;
+    attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = (early && kllm_pdl_enabled()) ? 2 : 1;
+    cudaError_t e = cudaLaunchKernelEx(&cfg, kern, a, sl);
+    if (e != cudaSuccess) KLLM_FAIL("gla step: %s", cudaGetErrorString(e));
+    KLLM_LAUNCH_STATUS();
+}
+
+template <typename T, int DPT>
+int launch_local(const GlaArgs& a, int chunk_bound, cudaStream_t s) {
+    const size_t smem = sizeof(float) * ((size_t)3 * kTS * 16 * DPT + kTS * kSl + 16 * DPT + (size_t)kTS * a.rot +
+                                         (a.low ? (size_t)kTS * a.R + (size_t)a.dk * (a.R + 1) : 0));
+    if (smem > 200 * 1024) KLLM_FAIL("gla: a head of %d key channels with a decay of rank %d does not fit shared memory", a.dk, a.R);
+    auto kern = local_kernel<T, DPT>;
+    static bool raised = false;
+    if (!raised) {
+        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        if (e != cudaSuccess) KLLM_FAIL("gla: %s", cudaGetErrorString(e));
+        raised = true;
+    }
+    kllm_launch_dep(false, (kern), dim3(chunk_bound, a.heads, (a.dv + kSl - 1) / kSl), dim3(kThreads), smem, s, a);
+    KLLM_LAUNCH_STATUS();
+}
+
+template <typename T, int NJ, bool NORM>
+int launch_apply(const GlaArgs& a, int chunk_bound, cudaStream_t s) {
+    const size_t smem = sizeof(float) * (kC * 36 + 32 * 64 * NJ);
+    kllm_launch_dep(false, (apply_kernel<T, NJ, NORM>), dim3(chunk_bound, a.heads, NORM ? 1 : (a.dv + 64 * NJ - 1) / (64 * NJ)),
+                    dim3(kThreads), smem, s, a);
+    KLLM_LAUNCH_STATUS();
+}
+
+template <typename T>
+int run(const GlaArgs& a, int n, bool single, bool early, int chunk_bound, cudaStream_t s) {
+    const bool vec = a.dv % 4 == 0 && a.stride % 4 == 0 && a.state_stride % 4 == 0 &&
+                     !(((uintptr_t)a.state | (uintptr_t)a.v | (uintptr_t)a.s_in) & 15);
+    if (single) return vec ? launch_step<T, 4>(a, early, s) : launch_step<T, 1>(a, early, s);
+    if (a.dv % 4 == 0 && ((uintptr_t)a.s_in & 15)) KLLM_FAIL("gla: the work buffer must be 16-byte aligned");
+    int rc;
+    if (a.dk <= 16) rc = launch_local<T, 1>(a, chunk_bound, s);
+    else if (a.dk <= 32) rc = launch_local<T, 2>(a, chunk_bound, s);
+    else if (a.dk <= 64) rc = launch_local<T, 4>(a, chunk_bound, s);
+    else if (a.dk <= 128) rc = launch_local<T, 8>(a, chunk_bound, s);
+    else rc = launch_local<T, 16>(a, chunk_bound, s);
+    if (rc) return rc;
+    const int64_t elems = (int64_t)a.dk * a.dv;
+    if (vec)
+        kllm_launch_dep(false, (carry_kernel<4>), dim3((unsigned)((elems / 4 + kThreads - 1) / kThreads), a.heads, a.n_requests),
+                        dim3(kThreads), 0, s, a);
+    else
+        kllm_launch_dep(false, (carry_kernel<1>), dim3((unsigned)((elems + kThreads - 1) / kThreads), a.heads, a.n_requests),
+                        dim3(kThreads), 0, s, a);
+    cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) KLLM_FAIL("gla: %s", cudaGetErrorString(e));
+    if (a.dv <= 64) return launch_apply<T, 1, true>(a, chunk_bound, s);
+    if (a.dv <= 128) return launch_apply<T, 2, true>(a, chunk_bound, s);
+    if (a.dv <= 256) return launch_apply<T, 4, true>(a, chunk_bound, s);
+    rc = launch_apply<T, 4, false>(a, chunk_bound, s);
+    if (rc) return rc;
+    const int64_t items = (int64_t)n * a.heads;
+    kllm_launch((norm_gate_kernel<T>), dim3((unsigned)((items + 7) / 8)), dim3(kThreads), 0, s, a, n);
+    KLLM_LAUNCH_STATUS();
+}
+
+}  // namespace
+
+extern "C" int kllm_gla_chunk_rows() { return kC; }
+
+// q, k float32 rows of heads * dk, v, g rows of heads * dv, low rows of R values (null: the fixed decay), all at row
+// stride `stride`; w2 [heads * dk][R] in the element type `dtype`, w2_bias float32 [heads * dk]; decay float32 [heads];
+// freq double [rot / 2] or null; state float32 [slots][state_stride] whose first heads * dk * dv values are S as
+// [heads][dk][dv]; gain float32 [heads * dv]; y in `dtype` at row stride y_stride.  single: every request brings one
+// row; otherwise the work buffers o [n][heads dv], qa [n][heads dk], a_last [chunk_bound][heads dk], s_in
+// [chunk_bound][heads][dk][dv] are float32 and chunk_bound an upper bound of the chunks (sum over requests of
+// ceil(rows / kllm_gla_chunk_rows())).  early (single): the kernel may start beside the end of the one before it in the
+// stream, which must not write the state.
+extern "C" int kllm_gla(void* y, int64_t y_stride, const float* q, const float* k, const float* v, const float* g, int64_t stride,
+                        const float* low, const void* w2, const float* w2_bias, int R, float inv_tau, const float* decay,
+                        const double* freq, int rot, float amplitude, float q_scale, float k_scale, const int* positions,
+                        const int* q_start, const int* start_pos, const int* state_slots, float* state, int64_t state_stride,
+                        const float* gain, float eps, int n, int n_requests, int heads, int dk, int dv, int single,
+                        int early, int chunk_bound, float* o, float* qa, float* a_last, float* s_in, int dtype, void* stream) {
+    if (n <= 0 || n_requests <= 0) return 0;
+    if (heads <= 0 || dk <= 0 || dk > 256 || dv <= 0) KLLM_FAIL("gla: %d heads of sizes %d (up to 256), %d", heads, dk, dv);
+    if (heads > 65535 || n_requests > 65535) KLLM_FAIL("gla: %d heads, %d requests in one launch", heads, n_requests);
+    if (rot < 0 || (rot & 1) || rot > dk || rot > kMaxRot || (rot > 0 && !freq)) KLLM_FAIL("gla: rotary width %d invalid for head size %d", rot, dk);
+    if (low ? (!w2 || !w2_bias || R <= 0) : !decay) KLLM_FAIL("gla: a decay needs its matrix and bias, or one number per head");
+    if (state_stride < (int64_t)heads * dk * dv) KLLM_FAIL("gla: a state slot of %lld values is too small", (long long)state_stride);
+    if (single && n != n_requests) KLLM_FAIL("gla: %d rows of %d requests that bring one row each", n, n_requests);
+    if (!single && (!o || !qa || !a_last || !s_in || chunk_bound <= 0)) KLLM_FAIL("gla: portions need work buffers");
+    GlaArgs a;
+    a.q = q; a.k = k; a.v = v; a.g = g; a.stride = stride; a.low = low; a.w2 = w2; a.w2_bias = w2_bias; a.R = low ? R : 0;
+    a.inv_tau = inv_tau; a.decay = decay; a.freq = freq; a.rot = rot; a.amplitude = amplitude; a.q_scale = q_scale;
+    a.k_scale = k_scale; a.positions = positions; a.q_start = q_start; a.state_slots = state_slots; a.n_requests = n_requests;
+    a.heads = heads; a.dk = dk; a.dv = dv; a.state = state; a.state_stride = state_stride; a.gain = gain; a.eps = eps; a.y = y;
+    a.y_stride = y_stride; a.o = o; a.qa = qa; a.a_last = a_last; a.s_in = s_in; a.start_pos = start_pos;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == KLLM_F32) return run<float>(a, n, single != 0, early != 0, chunk_bound, s);
+    if (dtype == KLLM_BF16) return run<bf16>(a, n, single != 0, early != 0, chunk_bound, s);
+    KLLM_FAIL("gla: unknown element type %d", dtype);
+}

@@ -6,8 +6,8 @@
 //   divides every query and key head by its root mean square over its dk values and multiplies by
 //   a gain [dk] that all heads share (optional),
 //   turns the pairs (i, i + rot / 2), i < rot / 2, of every query and key head by the angle
-//   p * freq[i] (rotate-half layout; the dims from rot on pass unchanged), cos and sin times
-//   `amplitude`,
+//   p * freq[i] (rotate-half layout; `interleaved`: the pairs (2i, 2i + 1); the dims from rot on
+//   pass unchanged), cos and sin times `amplitude`,
 //   stores the queries dense in the model's element type and writes keys and values into the paged
 //   caches [pages][k heads][page_size][dk] and [pages][v heads][page_size][dv] at position p.
 //
@@ -33,7 +33,7 @@ __global__ void __launch_bounds__(kWarps * 32)
 headnorm_rope_append_kernel(T* __restrict__ q_out, const float* __restrict__ qkv, int64_t qkv_stride,
                             const float* __restrict__ bias, const float* __restrict__ q_gain,
                             const float* __restrict__ k_gain, float eps, const double* __restrict__ freq,
-                            float amplitude, int rot, const int* __restrict__ positions,
+                            float amplitude, int rot, int interleaved, const int* __restrict__ positions,
                             const int* __restrict__ token_req, const int* __restrict__ block_table, int max_blocks,
                             T* __restrict__ kcache, T* __restrict__ vcache, int q_heads, int k_heads, int v_heads,
                             int dk, int dv, int page_size) {
@@ -77,9 +77,11 @@ headnorm_rope_append_kernel(T* __restrict__ q_out, const float* __restrict__ qkv
         for (int i = lane; i < dk; i += 32) {
             float v = buf[warp][i] * scale * (gain ? gain[i] : 1.f);
             if (i < rot) {
-                const int j = i < half ? i : i - half, o = i < half ? i + half : i - half;
+                const bool first = interleaved ? !(i & 1) : i < half;
+                const int j = interleaved ? i >> 1 : (first ? i : i - half);
+                const int o = interleaved ? (i ^ 1) : (first ? i + half : i - half);
                 const float w = buf[warp][o] * scale * (gain ? gain[o] : 1.f);
-                v = i < half ? v * cs[j] - w * cs[half + j] : v * cs[j] + w * cs[half + j];
+                v = first ? v * cs[j] - w * cs[half + j] : v * cs[j] + w * cs[half + j];
             }
             dst[i] = from_f32<T>(v);
         }
@@ -134,7 +136,7 @@ maps_combine_kernel(T* __restrict__ out, const float* __restrict__ a, int n, int
 // type `dtype`, which is also the caches'.  kcache NULL: only the queries are produced.
 extern "C" int kllm_headnorm_rope_append(void* q_out, const float* qkv, int64_t qkv_stride, const float* bias,
                                          const float* q_gain, const float* k_gain, float eps, const double* freq,
-                                         float amplitude, int rot, const int* positions, const int* token_req,
+                                         float amplitude, int rot, int interleaved, const int* positions, const int* token_req,
                                          const int* block_table, int max_blocks, void* kcache, void* vcache, int n,
                                          int q_heads, int k_heads, int v_heads, int dk, int dv, int page_size, int dtype,
                                          void* stream) {
@@ -147,11 +149,11 @@ extern "C" int kllm_headnorm_rope_append(void* q_out, const float* qkv, int64_t 
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == KLLM_F32)
         kllm_launch((headnorm_rope_append_kernel<float>), dim3(n), dim3(kWarps * 32), 0, s, (float*)q_out, qkv, qkv_stride,
-                    bias, q_gain, k_gain, eps, freq, amplitude, rot, positions, token_req, block_table, max_blocks,
+                    bias, q_gain, k_gain, eps, freq, amplitude, rot, interleaved, positions, token_req, block_table, max_blocks,
                     (float*)kcache, (float*)vcache, q_heads, k_heads, v_heads, dk, dv, page_size);
     else if (dtype == KLLM_BF16)
         kllm_launch((headnorm_rope_append_kernel<bf16>), dim3(n), dim3(kWarps * 32), 0, s, (bf16*)q_out, qkv, qkv_stride,
-                    bias, q_gain, k_gain, eps, freq, amplitude, rot, positions, token_req, block_table, max_blocks,
+                    bias, q_gain, k_gain, eps, freq, amplitude, rot, interleaved, positions, token_req, block_table, max_blocks,
                     (bf16*)kcache, (bf16*)vcache, q_heads, k_heads, v_heads, dk, dv, page_size);
     else
         KLLM_FAIL("head norm: unknown element type %d", dtype);

@@ -17,7 +17,8 @@
 //             ADD_F32     Y is added into a float32 matrix (the residual stream)
 //             SWIGLU      W holds a gate and an up matrix [F, K] each; the output is
 //                         silu(gate row) * (up row) as bfloat16 [n, F]
-//                         (backend/model.cu:477-483, :1112-1114)
+//                         (backend/model.cu:477-483, :1112-1114); optionally with biases on both
+//                         rows' sums and with the tanh gelu in place of silu
 //
 // Layout of the work: a tile is 16 weight rows (for SWIGLU 8 gate rows and the 8 up
 // rows that go with them).  A CTA of 16 warps, one per SM, walks tiles tile = blockIdx.x,
@@ -59,6 +60,9 @@ struct Args {
     bf16* y_bf16;         // STORE_BF16, SWIGLU
     float* y_f32;         // STORE_F32, ADD_F32
     int64_t y_stride;
+    const float* bias;      // optional [N]: ADD_F32 adds it with the product; SWIGLU: to the gate rows' sums
+    const float* bias_up;   // optional [N], SWIGLU: to the up rows' sums
+    int gelu;               // SWIGLU: the activation is the gelu with tanh instead of silu
     int tl_slot;            // timeline row of this launch (-1: none)
     const void* prefetch;   // optional: weights of a later kernel, to be brought into L2
     int64_t prefetch_bytes;
@@ -333,12 +337,17 @@ skinny_gemm_kernel(const Args a) {
                     float u = 0.f;
 #pragma unroll
                     for (int w = 0; w < WARPS; w++) u += red[(w * 16 + r + 8) * 8 * NT + c];
-                    a.y_bf16[(int64_t)c * a.y_stride + col] = __float2bfloat16_rn((v / (1.f + expf(-v))) * u);
+                    if (a.bias) v += a.bias[col];
+                    if (a.bias_up) u += a.bias_up[col];
+                    const float act = a.gelu ? 0.5f * v * (1.f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)))
+                                             : v / (1.f + expf(-v));
+                    a.y_bf16[(int64_t)c * a.y_stride + col] = __float2bfloat16_rn(act * u);
                 } else if (EPI == STORE_BF16) {
                     a.y_bf16[(int64_t)c * a.y_stride + col] = __float2bfloat16_rn(v);
                 } else if (EPI == STORE_F32) {
                     a.y_f32[(int64_t)c * a.y_stride + col] = v;
                 } else {
+                    if (a.bias) v += a.bias[col];
                     a.y_f32[(int64_t)c * a.y_stride + col] += v;
                 }
             }
@@ -428,12 +437,15 @@ extern "C" int kllm_skinny_gemm_fits(int n, int K) {
 // w_stride: elements from one weight row to the next (>= K; more than K when the call
 // multiplies a slice of the columns of a wider matrix, which is how a K too long for
 // shared memory is taken: one call per slice, each adding into y_f32).
+// bias, bias_up: optional float32 [N] (epilogue 2: bias joins the sum; 3: the gate's and the up rows' biases); gelu:
+// epilogue 3 with the tanh gelu instead of silu.
 // prefetch: optional, `prefetch_bytes` bytes that a later kernel will stream; they are
 // requested into L2 before this kernel's own work.
 extern "C" int kllm_skinny_gemm(const void* w, const void* w_up, int64_t w_stride, int N, int K, int n, const void* x_bf16,
                                 int64_t x_stride, const float* x_f32, const float* gain, const int* rows,
                                 float eps, void* y_bf16, float* y_f32, int64_t y_stride, int prologue,
-                                int epilogue, const void* prefetch, int64_t prefetch_bytes, void* stream) {
+                                int epilogue, const float* bias, const float* bias_up, int gelu,
+                                const void* prefetch, int64_t prefetch_bytes, void* stream) {
     if (n <= 0 || N <= 0) return 0;
     if (!kllm_skinny_gemm_fits(n, K))
         KLLM_FAIL("skinny_gemm: %d rows of width %d not supported (1..16 rows, width a multiple of 32 that fits "
@@ -452,6 +464,7 @@ extern "C" int kllm_skinny_gemm(const void* w, const void* w_up, int64_t w_strid
     a.y_bf16 = (bf16*)y_bf16; a.y_f32 = y_f32; a.y_stride = y_stride;
     if (prefetch && ((uintptr_t)prefetch & 15)) KLLM_FAIL("skinny_gemm: the matrix to prefetch must be 16-byte aligned");
     a.prefetch = prefetch; a.prefetch_bytes = prefetch ? prefetch_bytes : 0;
+    a.bias = bias; a.bias_up = bias_up; a.gelu = gelu;
     a.tl_slot = TL_SLOT();
     cudaStream_t s = (cudaStream_t)stream;
     if (n <= 8) {

@@ -49,6 +49,9 @@ struct Args {
     float eps;
     float* y;             // [n, N] at y_stride
     int64_t y_stride;
+    const float* bias;    // optional [N]: ADD adds it with the product; SWIGLU: to the gate rows' sums
+    const float* bias_up; // optional [N], SWIGLU: to the up rows' sums
+    int gelu;             // SWIGLU: the activation is the gelu with tanh instead of silu
 };
 
 __device__ __forceinline__ float4 ldg_stream(const float* p) {
@@ -196,8 +199,12 @@ skinny_f32_kernel(const Args a) {
                 const int col = EPI == SWIGLU ? tile * WR + r : tile * GROUPS * WR + g2 * WR + r;
                 if (c < n && col < N) {
                     float* dst = a.y + (int64_t)c * a.y_stride + col;
-                    if (EPI == SWIGLU) *dst = (v / (1.f + expf(-v))) * up;
-                    else if (EPI == ADD) *dst += v;
+                    if (EPI == SWIGLU) {
+                        if (a.bias) v += a.bias[col];
+                        if (a.bias_up) up += a.bias_up[col];
+                        *dst = (a.gelu ? 0.5f * v * (1.f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)))
+                                       : v / (1.f + expf(-v))) * up;
+                    } else if (EPI == ADD) *dst += v + (a.bias ? a.bias[col] : 0.f);
                     else *dst = v;
                 }
             }
@@ -248,9 +255,11 @@ extern "C" int kllm_skinny_gemm_f32_fits(int n, int K) {
 // given) normalised with gain [K] and eps.  epilogue 0: y written; 1: y += result; 2: w = gate
 // [N, K], w_up = up [N, K], y = silu(gate) * up.  w_stride: elements from one weight row to the
 // next (more than K when the call multiplies a slice of the columns of a wider matrix).
+// bias, bias_up, gelu: as in skinny_gemm.cu.
 extern "C" int kllm_skinny_gemm_f32(const float* w, const float* w_up, int64_t w_stride, int N, int K, int n,
                                     const float* x, int64_t x_stride, const float* gain, const int* rows, float eps,
-                                    float* y, int64_t y_stride, int prologue, int epilogue, void* stream) {
+                                    float* y, int64_t y_stride, int prologue, int epilogue, const float* bias,
+                                    const float* bias_up, int gelu, void* stream) {
     if (n <= 0 || N <= 0) return 0;
     if (!kllm_skinny_gemm_f32_fits(n, K))
         KLLM_FAIL("skinny_gemm_f32: %d rows of width %d not supported (1..8 rows, width a multiple of 128 that fits "
@@ -262,6 +271,7 @@ extern "C" int kllm_skinny_gemm_f32(const float* w, const float* w_up, int64_t w
     Args a;
     a.w = w; a.w_up = w_up; a.w_stride = w_stride; a.N = N; a.K = K; a.n = n; a.x = x; a.x_stride = x_stride;
     a.gain = gain; a.rows = rows; a.eps = eps; a.y = y; a.y_stride = y_stride;
+    a.bias = bias; a.bias_up = bias_up; a.gelu = gelu;
     cudaStream_t s = (cudaStream_t)stream;
 #define KLLM_F32_CASE(P, E) if (prologue == P && epilogue == E) return launch<P, E>(a, s)
     KLLM_F32_CASE(X_PLAIN, STORE); KLLM_F32_CASE(X_PLAIN, ADD); KLLM_F32_CASE(X_PLAIN, SWIGLU);

@@ -302,12 +302,13 @@ def headnorm_rope_append(q_out: torch.Tensor, qkv: torch.Tensor, bias: Optional[
                          q_gain: Optional[torch.Tensor], k_gain: Optional[torch.Tensor], eps: float,
                          freq: Optional[torch.Tensor], amplitude: float, rot: int, positions: torch.Tensor,
                          token_req: torch.Tensor, block_table: Optional[torch.Tensor], kcache: Optional[torch.Tensor],
-                         vcache: Optional[torch.Tensor], q_heads: int, k_heads: int, v_heads: int, dk: int, dv: int) -> None:
+                         vcache: Optional[torch.Tensor], q_heads: int, k_heads: int, v_heads: int, dk: int, dv: int,
+                         interleaved: bool = False) -> None:
     """Bias, RMS norm per head with a gain [dk] that all heads share, rotation of the first ``rot`` values
     of every query and key head, and the cache write, in one kernel (csrc/qk_headnorm.cu).  ``qkv`` float32
     [n, (q_heads + k_heads) dk + v_heads dv]; ``bias`` float32 of a row's length or None; ``q_gain`` /
-    ``k_gain`` float32 [dk] or None (no norm); ``freq`` float64 [rot / 2] (pair (i, i + rot / 2) turns by
-    position * freq[i], cos and sin times ``amplitude``); ``q_out`` [n, q_heads dk] in the model dtype;
+    ``k_gain`` float32 [dk] or None (no norm); ``freq`` float64 [rot / 2] (pair (i, i + rot / 2), or with
+    ``interleaved`` pair (2i, 2i + 1), turns by position * freq[i], cos and sin times ``amplitude``); ``q_out`` [n, q_heads dk] in the model dtype;
     caches [pages, k_heads, page_size, dk] and [pages, v_heads, page_size, dv].  With ``kcache`` None ``qkv``
     holds queries only."""
     _cuda(q_out, qkv, bias, q_gain, k_gain, freq, positions, token_req, block_table, kcache, vcache)
@@ -334,9 +335,9 @@ def headnorm_rope_append(q_out: torch.Tensor, qkv: torch.Tensor, bias: Optional[
             raise KernelError("headnorm_rope_append: caches must be [pages, heads, page_size, size] in q_out's dtype")
     lib = load_library("qk_headnorm")
     rc = lib.kllm_headnorm_rope_append(_p(q_out), _p(qkv), ctypes.c_int64(qkv.stride(0)), _p(bias), _p(q_gain), _p(k_gain),
-                                       ctypes.c_float(eps), _p(freq), ctypes.c_float(amplitude), int(rot), _p(positions),
-                                       _p(token_req), _p(block_table), max_blocks, _p(kcache), _p(vcache), n, q_heads,
-                                       k_heads, v_heads, dk, dv, page_size, dtype_code(q_out.dtype), _stream())
+                                       ctypes.c_float(eps), _p(freq), ctypes.c_float(amplitude), int(rot), int(interleaved),
+                                       _p(positions), _p(token_req), _p(block_table), max_blocks, _p(kcache), _p(vcache), n,
+                                       q_heads, k_heads, v_heads, dk, dv, page_size, dtype_code(q_out.dtype), _stream())
     _check(lib, "qk_headnorm", rc)
 
 
@@ -356,19 +357,21 @@ def maps_combine(out: torch.Tensor, a: torch.Tensor, kv_heads: int, group: int, 
     _check(lib, "qk_headnorm", rc)
 
 
-def sigmoid_gate(out: torch.Tensor, a: torch.Tensor, gate: torch.Tensor) -> None:
-    """out = a * sigmoid(gate): a and out in the model dtype, gate float32 logits; dense rows, strided rows
-    allowed (csrc/activation.cu)."""
+def sigmoid_gate(out: torch.Tensor, a: torch.Tensor, gate: torch.Tensor, factor: float = 1.0) -> None:
+    """out = a * sigmoid(gate) * factor: out in the model dtype, a in it or float32, gate float32 logits; dense rows,
+    strided rows allowed (csrc/activation.cu)."""
     _cuda(out, a, gate)
-    if gate.dtype != torch.float32 or a.dtype != out.dtype or a.shape != out.shape or gate.shape != out.shape:
-        raise KernelError("sigmoid_gate: a and out of one dtype and shape, gate float32 of that shape")
+    if gate.dtype != torch.float32 or a.dtype not in (out.dtype, torch.float32) or a.shape != out.shape \
+            or gate.shape != out.shape:
+        raise KernelError("sigmoid_gate: a of out's dtype or float32, gate float32, all of one shape")
     for t in (out, a, gate):
         if t.stride(1) != 1:
             raise KernelError("sigmoid_gate: operands must have dense rows")
     n, f = out.shape
     lib = load_library("activation")
     rc = lib.kllm_sigmoid_gate(_p(out), ctypes.c_int64(out.stride(0)), _p(a), ctypes.c_int64(a.stride(0)), _p(gate),
-                               ctypes.c_int64(gate.stride(0)), n, f, dtype_code(out.dtype), _stream())
+                               ctypes.c_int64(gate.stride(0)), n, f, ctypes.c_float(factor), dtype_code(out.dtype),
+                               dtype_code(a.dtype), _stream())
     _check(lib, "activation", rc)
 
 
@@ -952,6 +955,30 @@ def clamped_glu(out: torch.Tensor, gate: torch.Tensor, up: torch.Tensor, limit: 
     _check(lib, "activation", rc)
 
 
+def biased_glu(out: torch.Tensor, gate: torch.Tensor, up: torch.Tensor, bias_gate: Optional[torch.Tensor] = None,
+               bias_up: Optional[torch.Tensor] = None, activation: str = "silu") -> None:
+    """out = act(gate + bias_gate) * (up + bias_up), ``activation`` "silu" or "gelu_tanh"; float32 gate and up with dense
+    rows (strided rows allowed), float32 biases [f] or None, out in float32 or bfloat16."""
+    _cuda(out, gate, up, bias_gate, bias_up)
+    n, f = out.shape
+    for t in (out, gate, up):
+        if t.stride(1) != 1 or t.shape != out.shape:
+            raise KernelError("biased_glu: operands must have dense rows and out's shape")
+    if gate.dtype != torch.float32 or up.dtype != torch.float32 or activation not in ("silu", "gelu_tanh"):
+        raise KernelError("biased_glu: gate and up must be float32, the activation silu or gelu_tanh")
+    _bias(bias_gate, f, "biased_glu"); _bias(bias_up, f, "biased_glu")
+    lib = load_library("activation")
+    rc = lib.kllm_biased_glu(_p(out), ctypes.c_int64(out.stride(0)), _p(gate), ctypes.c_int64(gate.stride(0)), _p(up),
+                             ctypes.c_int64(up.stride(0)), _p(bias_gate), _p(bias_up), n, f, int(activation == "gelu_tanh"),
+                             dtype_code(out.dtype), _stream())
+    _check(lib, "activation", rc)
+
+
+def _bias(t: Optional[torch.Tensor], n: int, what: str):
+    if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or t.numel() != n):
+        raise KernelError(f"{what}: a bias must be contiguous float32 [{n}]")
+
+
 def sample(out: torch.Tensor, logits: torch.Tensor, temperature: Optional[torch.Tensor],
            uniform: Optional[torch.Tensor], last_token: Optional[torch.Tensor] = None,
            slots: Optional[torch.Tensor] = None, host_out: Optional[torch.Tensor] = None) -> None:
@@ -1020,7 +1047,9 @@ def _prefetch_args(t: Optional[torch.Tensor]):
 def skinny_gemm(weight: torch.Tensor, *, x: Optional[torch.Tensor] = None, x_f32: Optional[torch.Tensor] = None,
                 gain: Optional[torch.Tensor] = None, eps: float = 0.0, rows: Optional[torch.Tensor] = None,
                 n_rows: Optional[int] = None, weight_up: Optional[torch.Tensor] = None, epilogue: str = "bf16",
-                out: Optional[torch.Tensor] = None, prefetch: Optional[torch.Tensor] = None) -> torch.Tensor:
+                out: Optional[torch.Tensor] = None, prefetch: Optional[torch.Tensor] = None,
+                bias: Optional[torch.Tensor] = None, bias_up: Optional[torch.Tensor] = None,
+                activation: str = "silu") -> torch.Tensor:
     """y = X @ weight^T for at most 16 rows, the weights streamed once (csrc/skinny_gemm.cu
     for bfloat16 weights, csrc/skinny_gemm_f32.cu for float32 weights: true float32 FMAs,
     at most 8 rows).
@@ -1029,19 +1058,26 @@ def skinny_gemm(weight: torch.Tensor, *, x: Optional[torch.Tensor] = None, x_f32
     inside the kernel (rows ``rows`` of x_f32 when given).  ``epilogue``: "store" stores y
     [n, N] in the weights' dtype ("bf16" / "f32" name the dtype); "add" adds y into the
     float32 ``out``; "swiglu" takes ``weight`` as gate and ``weight_up`` as up matrix and
-    stores silu(gate) * up [n, N] in the weights' dtype.
+    stores silu(gate) * up [n, N] in the weights' dtype.  ``bias`` (float32 [N]) joins the sum of
+    "add", or the gate's sums of "swiglu" (``bias_up``: the up sums'); ``activation`` "gelu_tanh" takes
+    silu's place there.
     ``prefetch``: a contiguous tensor that a later kernel will stream (the next weight
     matrix); the kernel asks for it to be brought into L2 before its own work.
     A width K too long for shared memory is taken in column slices, one launch each, when
     X is bfloat16 and the epilogue is "add" (the slices' sums meet in ``out``, always in
     the same order).
     """
-    _cuda(weight, x, x_f32, gain, rows, weight_up, out, prefetch)
+    _cuda(weight, x, x_f32, gain, rows, weight_up, out, prefetch, bias, bias_up)
     N, K = weight.shape
+    _bias(bias, N, "skinny_gemm"); _bias(bias_up, N, "skinny_gemm")
+    if (bias is not None and epilogue not in ("add", "swiglu")) or (bias_up is not None and epilogue != "swiglu") \
+            or activation not in ("silu", "gelu_tanh"):
+        raise KernelError("skinny_gemm: biases go with 'add' and 'swiglu', the activation is silu or gelu_tanh")
     if epilogue == "store":
         epilogue = "f32" if weight.dtype == torch.float32 else "bf16"
     if weight.dtype == torch.float32:
-        return _skinny_gemm_f32(weight, x, x_f32, gain, eps, rows, n_rows, weight_up, epilogue, out)
+        return _skinny_gemm_f32(weight, x, x_f32, gain, eps, rows, n_rows, weight_up, epilogue, out, bias, bias_up,
+                                activation)
     if weight.dtype != torch.bfloat16 or weight.stride(1) != 1 or weight.stride(0) % 8:
         raise KernelError("skinny_gemm: the weight must be bfloat16 with dense rows at a stride that is a multiple of 8")
     if weight_up is not None and weight_up.stride() != weight.stride():
@@ -1054,7 +1090,7 @@ def skinny_gemm(weight: torch.Tensor, *, x: Optional[torch.Tensor] = None, x_f32
         for lo in range(0, K, width):
             hi = min(K, lo + width)
             skinny_gemm(weight[:, lo:hi], x=x[:, lo:hi], epilogue="add", out=out,
-                        prefetch=prefetch if hi == K else None)
+                        prefetch=prefetch if hi == K else None, bias=bias if hi == K else None)
         return out
     if x is not None:
         pro, n = 0, x.shape[0]
@@ -1088,12 +1124,13 @@ def skinny_gemm(weight: torch.Tensor, *, x: Optional[torch.Tensor] = None, x_f32
     rc = lib.kllm_skinny_gemm(_p(weight), _p(weight_up), ctypes.c_int64(weight.stride(0)), N, K, n, _p(x),
                               ctypes.c_int64(x.stride(0) if x is not None else 0), _p(x_f32), _p(gain), _p(rows),
                               ctypes.c_float(eps), _p(y16), _p(y32), ctypes.c_int64(out.stride(0)), pro, epi,
-                              *_prefetch_args(prefetch), _stream())
+                              _p(bias), _p(bias_up), int(activation == "gelu_tanh"), *_prefetch_args(prefetch), _stream())
     _check(lib, "skinny_gemm", rc)
     return out
 
 
-def _skinny_gemm_f32(weight, x, x_f32, gain, eps, rows, n_rows, weight_up, epilogue, out):
+def _skinny_gemm_f32(weight, x, x_f32, gain, eps, rows, n_rows, weight_up, epilogue, out, bias=None, bias_up=None,
+                     activation="silu"):
     """The float32 form of ``skinny_gemm`` (same arguments; no prefetch hint)."""
     N, K = weight.shape
     if weight.stride(1) != 1 or weight.stride(0) % 4:
@@ -1109,7 +1146,8 @@ def _skinny_gemm_f32(weight, x, x_f32, gain, eps, rows, n_rows, weight_up, epilo
             width = -(-K // parts // 128) * 128
             for lo in range(0, K, width):
                 hi = min(K, lo + width)
-                _skinny_gemm_f32(weight[:, lo:hi], x[:, lo:hi], None, None, 0.0, None, None, None, "add", out)
+                _skinny_gemm_f32(weight[:, lo:hi], x[:, lo:hi], None, None, 0.0, None, None, None, "add", out,
+                                 bias if hi == K else None)
             return out
         src, pro, stride = x, 0, x.stride(0)
     else:
@@ -1133,7 +1171,8 @@ def _skinny_gemm_f32(weight, x, x_f32, gain, eps, rows, n_rows, weight_up, epilo
     lib = load_library("skinny_gemm_f32")
     rc = lib.kllm_skinny_gemm_f32(_p(weight), _p(weight_up), ctypes.c_int64(weight.stride(0)), N, K, n, _p(src),
                                   ctypes.c_int64(stride), _p(gain), _p(rows), ctypes.c_float(eps), _p(out),
-                                  ctypes.c_int64(out.stride(0)), pro, {"f32": 0, "add": 1, "swiglu": 2}[epilogue], _stream())
+                                  ctypes.c_int64(out.stride(0)), pro, {"f32": 0, "add": 1, "swiglu": 2}[epilogue],
+                                  _p(bias), _p(bias_up), int(activation == "gelu_tanh"), _stream())
     _check(lib, "skinny_gemm_f32", rc)
     return out
 
@@ -1151,6 +1190,22 @@ def linear_add(acc: torch.Tensor, x: torch.Tensor, weight: torch.Tensor) -> None
         torch.addmm(acc, x, weight.t(), out=acc)
     else:
         torch.addmm(acc, x, weight.t(), out_dtype=torch.float32, out=acc)
+
+
+def linear_into(acc: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None,
+                prefetch: Optional[torch.Tensor] = None) -> None:
+    """acc += x @ weight^T (+ bias in every row), acc the float32 residual stream: the weight-streaming product for
+    a step of a few rows, else the library's (``linear_add``) and a kernel for the bias."""
+    if (skinny_fits(x.shape[0], x.shape[1], x.dtype, sliced=True) and x.stride(1) == 1 and weight.stride(1) == 1
+            and weight.stride(0) % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0):
+        skinny_gemm(weight, x=x, epilogue="add", out=acc, bias=bias, prefetch=prefetch)
+        return
+    linear_add(acc, x, weight)
+    if bias is not None:
+        _cuda(acc, bias)
+        _bias(bias, acc.shape[1], "linear_into")
+        lib = load_library("activation")
+        _check(lib, "activation", lib.kllm_add_row(_p(acc), _p(bias), acc.shape[0], acc.shape[1], _stream()))
 
 
 def _gemm_args(x, weight, weight_up, out, epilogue):
@@ -1465,6 +1520,103 @@ def lightning_gate_norm(o: torch.Tensor, g: torch.Tensor, gain: torch.Tensor, ep
     return y
 
 
+# ---- linear attention with a decaying state (csrc/gla.cu) ------------------------------------
+
+def gla(y: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, state: torch.Tensor, ctx,
+        heads: int, dk: int, dv: int, gain: torch.Tensor, eps: float, *, low: Optional[torch.Tensor] = None,
+        w2: Optional[torch.Tensor] = None, w2_bias: Optional[torch.Tensor] = None, tau: float = 1.0,
+        decay: Optional[torch.Tensor] = None, freq: Optional[torch.Tensor] = None, amplitude: float = 1.0,
+        q_scale: float = 1.0, k_scale: float = 1.0, early: bool = False) -> None:
+    """y [n, heads * dv] (model dtype, dense rows) = o / rms(o over each head) * gain * silu(g) of the recurrence
+    S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head.  q, k (rows of heads * dk), v, g (heads * dv) and
+    ``low`` (R) are columns of one float32 matrix of projections.  The decay is gated, alpha = sigmoid(low @ w2^T +
+    w2_bias)^(1 / tau) per key channel (``w2`` [heads * dk, R] in the model dtype), or ``decay``, one float32 number per
+    head.  With ``freq`` (float64) q and k are rotated first (pair (i, i + len(freq)) by position * freq[i], cos and sin
+    times ``amplitude``); they are multiplied by ``q_scale`` and ``k_scale``.  ``state`` float32 [slots, >= heads * dk * dv]
+    holds S as [heads, dk, dv] per request slot and is carried on.  ``early``: a step of one row per request may
+    read the state beside the end of the kernel before it, which then must not write it."""
+    _cuda(y, q, k, v, g, state, gain, low, w2, w2_bias, decay, freq)
+    n = q.shape[0]
+    for t, cols, what in ((q, heads * dk, "q"), (k, heads * dk, "k"), (v, heads * dv, "v"), (g, heads * dv, "g")):
+        _f32_rows(t, cols, "gla: " + what)
+        if t.shape[0] != n or t.stride(0) != q.stride(0):
+            raise KernelError("gla: q, k, v and g must be columns of one matrix")
+    if y.shape != (n, heads * dv) or y.stride(1) != 1 or gain.dtype != torch.float32 or gain.numel() != heads * dv \
+            or not gain.is_contiguous():
+        raise KernelError("gla: y [n, heads * dv] with dense rows, gain contiguous float32 [heads * dv]")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < heads * dk * dv:
+        raise KernelError("gla: the state must be float32 [slots, >= heads * dk * dv]")
+    R = 0
+    if low is not None:
+        R = low.shape[1]
+        _f32_rows(low, R, "gla: low")
+        if low.stride(0) != q.stride(0) or w2.dtype != y.dtype or tuple(w2.shape) != (heads * dk, R) or not w2.is_contiguous():
+            raise KernelError("gla: low must be columns of the projections, w2 contiguous [heads * dk, R] in y's dtype")
+        _bias(w2_bias, heads * dk, "gla")
+        if w2_bias is None or not tau > 0:
+            raise KernelError("gla: a gated decay has a bias and a positive tau")
+    elif decay is None or decay.dtype != torch.float32 or decay.numel() != heads or not decay.is_contiguous():
+        raise KernelError("gla: one float32 decay per head")
+    _f64(freq, "gla: freq")
+    _i32(ctx.q_start, "q_start"); _i32(ctx.state_slots, "state_slots"); _i32(ctx.positions, "positions")
+    _i32(ctx.start_pos, "start_pos")
+    lib = load_library("gla")
+    o = qa = a_last = s_in = None
+    bound = 0
+    if not ctx.all_single:
+        f32 = dict(dtype=torch.float32, device=q.device)
+        bound = n // lib.kllm_gla_chunk_rows() + ctx.n_requests
+        o, qa = torch.empty((n, heads * dv), **f32), torch.empty((n, heads * dk), **f32)
+        a_last, s_in = torch.empty((bound, heads * dk), **f32), torch.empty((bound, heads, dk, dv), **f32)
+    rc = lib.kllm_gla(_p(y), ctypes.c_int64(y.stride(0)), _p(q), _p(k), _p(v), _p(g), ctypes.c_int64(q.stride(0)), _p(low),
+                      _p(w2), _p(w2_bias), R, ctypes.c_float(1.0 / tau), _p(decay), _p(freq),
+                      2 * freq.numel() if freq is not None else 0, ctypes.c_float(amplitude), ctypes.c_float(q_scale),
+                      ctypes.c_float(k_scale), _p(ctx.positions), _p(ctx.q_start), _p(ctx.start_pos), _p(ctx.state_slots),
+                      _p(state), ctypes.c_int64(state.stride(0)), _p(gain), ctypes.c_float(eps), n, ctx.n_requests, heads,
+                      dk, dv, int(ctx.all_single), int(early), bound, _p(o), _p(qa), _p(a_last), _p(s_in),
+                      dtype_code(y.dtype), _stream())
+    _check(lib, "gla", rc)
+    if not ctx.all_single:
+        global launches
+        launches += 2 if dv <= 256 else 3
+
+
+# ---- what stands in front of a layer (csrc/shift_norm.cu) --------------------------------------
+
+def norm_shift(x: torch.Tensor, gain: torch.Tensor, eps: float, mu: torch.Tensor, state: torch.Tensor, ctx,
+               dtype: torch.dtype):
+    """(h, hs) [n, d] in ``dtype``: h = rmsnorm(x) * gain of the float32 stream x, hs = h + (h_prev - h) * mu with
+    h_prev the row before in the same request, for a request's first row of the step what ``state[slot, :d]`` (float32)
+    holds, which is then replaced by the request's last row."""
+    _cuda(x, gain, mu, state)
+    n, d = x.shape
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise KernelError("norm_shift: x must be contiguous float32 [n, d]")
+    _bias(gain, d, "norm_shift"); _bias(mu, d, "norm_shift")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < d:
+        raise KernelError("norm_shift: the state must be float32 [slots, >= d]")
+    h, hs = (torch.empty((n, d), dtype=dtype, device=x.device) for _ in range(2))
+    lib = load_library("shift_norm")
+    rc = lib.kllm_norm_shift(_p(h), _p(hs), _p(x), _p(gain), _p(mu), ctypes.c_float(eps), _p(state),
+                             ctypes.c_int64(state.stride(0)), _p(ctx.q_start), _p(ctx.token_req), _p(ctx.state_slots), n, d,
+                             dtype_code(dtype), _stream())
+    _check(lib, "shift_norm", rc)
+    return h, hs
+
+
+def stream_entry(cat: torch.Tensor, x: torch.Tensor, row: torch.Tensor, copy_x0: bool) -> None:
+    """cat[:, :d] = x in cat's dtype (``copy_x0``: cat[:, d:] too), then x = ``row`` in every row; cat [n, 2 d], x
+    float32 [n, d], row float32 [d]."""
+    _cuda(cat, x, row)
+    n, d = x.shape
+    if x.dtype != torch.float32 or not x.is_contiguous() or not cat.is_contiguous() or tuple(cat.shape) != (n, 2 * d):
+        raise KernelError("stream_entry: x contiguous float32 [n, d], cat contiguous [n, 2 d]")
+    _bias(row, d, "stream_entry")
+    lib = load_library("shift_norm")
+    rc = lib.kllm_stream_entry(_p(cat), _p(x), _p(row), n, d, int(copy_x0), dtype_code(cat.dtype), _stream())
+    _check(lib, "shift_norm", rc)
+
+
 # ---- attention with scores mixed across the heads (csrc/attention_mixed.cu) ---------------
 
 _mixed_tile_rows = {}
@@ -1670,13 +1822,15 @@ def moe_gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, pe
 
 
 def moe_combine(parts: torch.Tensor, top: int, shared: Optional[torch.Tensor] = None,
-                gate: Optional[torch.Tensor] = None, scale: float = 1.0) -> torch.Tensor:
+                gate: Optional[torch.Tensor] = None, scale: float = 1.0,
+                into: Optional[torch.Tensor] = None) -> torch.Tensor:
     """y[t] = sum of parts[t * top + j] over j in order; float32.  With ``shared`` (float32
     [n, d], the output of an expert that every token runs) also + shared[t] * sigmoid(gate[t]),
     ``gate`` being a float32 column of one logit per token (None: the rows are added as they are).
-    ``scale`` multiplies the sum over j (one weight that all of a token's choices share)."""
-    _cuda(parts, shared, gate)
-    if top == 1 and shared is None and scale == 1.0:
+    ``scale`` multiplies the sum over j (one weight that all of a token's choices share).  ``into``: a float32
+    [n, d] matrix (the residual stream) to which the sum is added; it is what is returned."""
+    _cuda(parts, shared, gate, into)
+    if top == 1 and shared is None and scale == 1.0 and into is None:
         return parts            # nothing to add up: the rows themselves
     n, d = parts.shape[0] // top, parts.shape[1]
     if not parts.is_contiguous() or parts.dtype != torch.float32:
@@ -1685,10 +1839,13 @@ def moe_combine(parts: torch.Tensor, top: int, shared: Optional[torch.Tensor] = 
         raise KernelError("moe_combine: the shared expert's rows must be contiguous float32 [n, d]")
     if gate is not None and (shared is None or gate.dtype != torch.float32 or gate.dim() != 2 or gate.shape[0] != n):
         raise KernelError("moe_combine: the gate is a float32 column [n, 1] beside a shared expert")
-    y = torch.empty((n, d), dtype=torch.float32, device=parts.device)
+    if into is not None and (into.dtype != torch.float32 or not into.is_contiguous() or into.shape != (n, d)):
+        raise KernelError("moe_combine: the matrix added into must be contiguous float32 [n, d]")
+    y = into if into is not None else torch.empty((n, d), dtype=torch.float32, device=parts.device)
     lib = load_library("moe")
     rc = lib.kllm_moe_combine(_p(y), _p(parts), n, d, int(top), _p(shared), _p(gate),
-                              ctypes.c_int64(gate.stride(0) if gate is not None else 0), ctypes.c_float(scale), _stream())
+                              ctypes.c_int64(gate.stride(0) if gate is not None else 0), ctypes.c_float(scale),
+                              int(into is not None), _stream())
     _check(lib, "moe", rc)
     return y
 

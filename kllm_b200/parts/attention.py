@@ -38,10 +38,14 @@ which holds all heads of a tile of rows in one CTA, and needs a ``qk_transform``
 ``sink`` ("zero": a term exp(0) = 1 joins every head's softmax denominator, a sink without key, value or tensor;
 or the full name of a float32 tensor [H] of learned sink scores; taken by the mixed kernel and by the kernels
 that take ``sinks``).
+``out_gate`` (the full name of a matrix [H*vd, d]: the heads' outputs are multiplied element by element with
+sigmoid(W_g xn) before the output projection) and ``out_factor`` (a number that multiplies them too, default 1): both in one
+kernel behind the attention; they need a ``qk_transform`` with ``prepare``.
 Tensors: ``<prefix>.{q,k,v,o}_proj.weight`` with shapes [H*hd, d], [G*hd, d],
 [G*vd, d], [d, H*vd]; no bias (reference backend/model.cu:1090-1104).  At bind time
 q, k and v are stacked into one [(H+2G)*hd, d] matrix so the three projections are
-one product.
+one product; a gate's rows stand in front of them.  A layer whose ``qk_transform`` has ``prepare``
+offers the split form of a mixer (``gla.py``), so that it may run beside another mixer.
 
 Interface of a mixer part:
   ``cache_need()`` -> PagedKVNeed | StateNeed | None
@@ -64,6 +68,7 @@ import math
 import torch
 
 from .. import kernels
+from .gla import SplitMixer, stack_rows
 from .spec import BuildEnv, PagedKVNeed, PartSpec, TensorSpec, part_factory, register_part
 
 
@@ -114,6 +119,10 @@ class PagedAttention:
                              "without differential maps, segments and score slopes")
         if self.sink_name and not self._prepares:
             raise ValueError("attention: a sink needs a qk_transform that stores keys and values (prepare)")
+        self.gate_name = p.get("out_gate")
+        self.out_factor = float(p.get("out_factor", 1.0))
+        if (self.gate_name or self.out_factor != 1.0) and not self._prepares:
+            raise ValueError("attention: a gate or factor on the output needs a qk_transform with prepare")
         slopes = p.get("score_slopes")
         if slopes == "geometric":
             # the slopes 2^(-8 (h + 1) / H) of a bias that grows with the distance, head by head
@@ -154,6 +163,8 @@ class PagedAttention:
             out.append(TensorSpec(self.mix_name, (self.n_heads, self.n_heads), store="float32", init="eye"))
         if self.sink_name and self.sink_name != "zero":
             out.append(TensorSpec(self.sink_name, (self.n_heads,), store="float32", init="zeros"))
+        if self.gate_name:
+            out.append(TensorSpec(self.gate_name, (self.o_dim, self.hidden)))
         return out + (self.position.tensor_specs() if self.position else []) + \
             (self.qk_transform.tensor_specs() if self.qk_transform else [])
 
@@ -169,7 +180,12 @@ class PagedAttention:
 
     def bind(self, tensors):
         n = self._names()
-        self.w_qkv = torch.cat([self._by_key_head(tensors[n["q"]]), tensors[n["k"]], tensors[n["v"]]], dim=0).contiguous()
+        rows = [self._by_key_head(tensors[n["q"]]), tensors[n["k"]], tensors[n["v"]]]
+        if self.gate_name:
+            self.w_in = stack_rows([tensors[self.gate_name]] + rows)
+            self.w_qkv = self.w_in[self.o_dim:self.o_dim + self.q_dim + self.kv_dim + self.v_dim]
+        else:
+            self.w_qkv = self.w_in = torch.cat(rows, dim=0).contiguous()
         self.w_o = tensors[n["o"]]
         if self.has_bias:
             self.bias = torch.cat([self._by_key_head(tensors[n["q_bias"]]), tensors[n["k_bias"]],
@@ -274,7 +290,32 @@ class PagedAttention:
                           v_head_dim=self.v_head_dim, exact_weights=self.exact_weights, segment=self.segment)
         return attn
 
+    @property
+    def out_dim(self):
+        return self.o_dim
+
+    @property
+    def w_out(self):
+        return self.w_o
+
+    @w_out.setter
+    def w_out(self, w):
+        self.w_o = w
+
+    def core(self, proj, ctx, cache, y):
+        """The split form (``gla.py``): ``proj`` holds the gate's logits, if there is a gate, then q, k and v."""
+        if not (self._prepares and cache.writes):
+            raise ValueError("attention: the split form is for layers with a qk_transform's prepare and a cache of their own")
+        off = self.o_dim if self.gate_name else 0
+        attn = self._attend_prepared(proj[:, off:off + self.q_dim + self.kv_dim + self.v_dim], ctx, cache)
+        if self.gate_name:
+            kernels.sigmoid_gate(y, attn, proj[:, :off], self.out_factor)
+        else:
+            torch.mul(attn, self.out_factor, out=y)
+
     def forward(self, xn, ctx, cache):
+        if self.gate_name or self.out_factor != 1.0:
+            return SplitMixer.forward(self, xn, ctx, cache)
         # a layer that reads another layer's cache projects its queries only
         w = self.w_qkv if cache.writes else self.w_qkv[:self.q_dim]
         if self._prepares:
@@ -284,6 +325,8 @@ class PagedAttention:
         attn = self._attend(q, k, v, ctx, cache)
         # float32 out: the result goes into the residual stream unrounded
         return kernels.linear(attn, self.w_o, out_dtype=torch.float32)
+
+    _rows = SplitMixer._rows
 
     def forward_residual(self, x, norm, ctx, cache):
         n = x.shape[0]

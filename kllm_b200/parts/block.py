@@ -8,6 +8,8 @@ first norm, or the model's final norm), as the reference does
 ``output_norm``: x += norm1(mixer(x)); x += norm2(ff(x)), the sublayers reading the stream itself, with an
 optional third sublayer that reads the step's token ids (``OutputNormBlock``).
 
+``parallel``: x += mixer(shift(h)) + ff(h) with h = norm(x), both sublayers reading one norm (``ParallelBlock``).
+
 Interface of a block: ``forward(x, pending, ctx, cache) -> pending'``.  x is the
 float32 residual stream, updated in place; ``pending`` (float32 or model dtype, or
 None) is what is still to be added to x.
@@ -27,7 +29,7 @@ block's mixer through ``set_successor``.  A part without them is left alone.
 """
 from __future__ import annotations
 
-from .spec import BlockSpec, BuildEnv, part_factory, register_part
+from .spec import BlockSpec, BuildEnv, StateNeed, TensorSpec, part_factory, register_part
 
 
 class PreNormBlock:
@@ -245,6 +247,74 @@ class OutputNormBlock:
         return y if y.dtype == torch.float32 and y.is_contiguous() else y.float().contiguous()
 
 
+class ParallelBlock:
+    """``parallel``: one norm, both sublayers side by side,
+
+        h = norm(x);  x += mixer(s(h)) + ff(h)
+
+    ``BlockSpec.mixer_norm`` is the norm (an RMS norm with ``gain`` and ``eps``), ``ff_norm`` is None and ``feed_forward`` may
+    be.  ``params``: ``shift`` (the full name of a float32 tensor mu [hidden], or absent): the mixer reads
+    s(h)_t = h_t + (h_(t-1) - h_t) * mu, the row in front of a request's first token being zeros; the request's last row
+    of h, unrounded, is a state of the layer (``StateNeed`` named "shift").  Norm and shift are one kernel
+    (csrc/shift_norm.cu).  The sublayers add their results into x themselves where they offer ``forward_add(x, h, ctx[,
+    cache])``; the block hands nothing on."""
+
+    def __init__(self, spec: BlockSpec, env: BuildEnv):
+        self.mixer = part_factory("mixer", spec.mixer.kind)(spec.mixer, env)
+        self.norm = part_factory("norm", spec.mixer_norm.kind)(spec.mixer_norm, env)
+        self.feed_forward = None
+        if spec.feed_forward is not None:
+            self.feed_forward = part_factory("feed_forward", spec.feed_forward.kind)(spec.feed_forward, env)
+        self.shift_name, self.shift = spec.params.get("shift"), None
+        self.width, self.dtype = env.hidden_size, env.dtype
+
+    def parts(self):
+        return [p for p in (self.norm, self.mixer, self.feed_forward) if p is not None]
+
+    def tensor_specs(self):
+        own = [TensorSpec(self.shift_name, (self.width,), store="float32", init="uniform:0:1")] if self.shift_name else []
+        return own + [s for p in self.parts() for s in p.tensor_specs()]
+
+    @property
+    def graph_safe(self):
+        return all(getattr(p, "graph_safe", True) for p in self.parts())
+
+    def bind(self, tensors):
+        for p in self.parts():
+            p.bind(tensors)
+        self.shift = tensors[self.shift_name].contiguous() if self.shift_name else None
+
+    def cache_need(self):
+        need = self.mixer.cache_need()
+        need = list(need) if isinstance(need, (list, tuple)) else [need]
+        if self.shift_name:
+            need.append(StateNeed((-(-self.width // 4) * 4,), "float32", name="shift"))     # whole 16-byte units per slot
+        return need
+
+    def forward(self, x, pending, ctx, cache):
+        if hasattr(pending, "settle"):
+            pending = pending.settle(x)
+        if pending is not None:
+            x.add_(pending.float())
+        if self.shift is None:
+            h = hs = self.norm.forward(x, None)
+        else:
+            from .. import kernels
+            h, hs = kernels.norm_shift(x, self.norm.gain, self.norm.eps, self.shift, cache.states["shift"], ctx, self.dtype)
+        self._add(self.mixer, x, hs, ctx, cache)
+        if self.feed_forward is not None:
+            self._add(self.feed_forward, x, h, ctx)
+        return None
+
+    @staticmethod
+    def _add(part, x, h, *args):
+        if hasattr(part, "forward_add"):
+            part.forward_add(x, h, *args)
+        else:
+            x.add_(part.forward(h, *args).float())
+
+
+register_part("block", "parallel", ParallelBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "output_norm", OutputNormBlock)
 register_part("block", "sandwich_norm", SandwichNormBlock)

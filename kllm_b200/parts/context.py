@@ -55,3 +55,4 @@ class LayerCache:
     state: Optional[torch.Tensor]        # [slots, *state shape]
     writes: bool = True
     page_size: int = 0
+    states: Dict[str, torch.Tensor] = field(default_factory=dict)   # further states of the layer by name, [slots, *shape]

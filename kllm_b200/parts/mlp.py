@@ -1,9 +1,10 @@
 """Gated feed-forward (SwiGLU): down( act(x Wg^T) * (x Wu^T) ).
 
-params: ``hidden``, ``intermediate``, ``activation`` ("silu"), optional ``tensors`` (gate, up,
-down -> full names).  Tensors:
+params: ``hidden``, ``intermediate``, ``activation`` ("silu"; "gelu_tanh": the tanh form of the gelu), optional
+``tensors`` (gate, up, down -> full names), ``bias`` (True: all three projections have float32 biases,
+``<weight name>.b``).  Tensors:
 ``<prefix>.{gate,up}_proj.weight`` [f, d] and ``<prefix>.down_proj.weight`` [d, f],
-no bias (reference backend/model.cu:1112-1115, activation :477-483).  Gate and up
+no bias by default (reference backend/model.cu:1112-1115, activation :477-483).  Gate and up
 are stacked into one [2f, d] matrix at bind time so both are one product.
 
 Optional ``forward_residual(x, norm, ctx) -> bool``: as for mixers, the part reads
@@ -13,6 +14,8 @@ product carries the norm as prologue and the activation as epilogue, the down
 product adds into x (csrc/skinny_gemm.cu).  Large portions in bfloat16 run gate, up
 and the activation as one tensor-core kernel (csrc/gemm_tcgen05.cu) where its tiles
 fill the GPU; everything else uses the library product and the activation kernel.
+
+``forward_add(x, h, ctx)``: x += ff(h) for a normed input h that another sublayer reads too (the ``parallel`` block).
 
 Interface of a feed-forward part: ``forward(xn, ctx) -> [n, hidden]`` in float32 or
 the model dtype.
@@ -31,8 +34,11 @@ class GatedMLP:
         self.hidden = int(p["hidden"])
         self.inter = int(p["intermediate"])
         self.activation = p.get("activation", "silu")
-        if self.activation != "silu":
-            raise ValueError(f"gated feed-forward: activation {self.activation!r} has no kernel (silu only)")
+        if self.activation not in ("silu", "gelu_tanh"):
+            raise ValueError(f"gated feed-forward: activation {self.activation!r} has no kernel (silu, gelu_tanh)")
+        self.has_bias = bool(p.get("bias", False))
+        self.plain = self.activation == "silu" and not self.has_bias
+        self.b_gate = self.b_up = self.b_down = None
         self.prefix = spec.prefix
         names = dict(p.get("tensors") or {})
         self.names = {k: names.get(k) or f"{self.prefix}.{k}_proj.weight" for k in ("gate", "up", "down")}
@@ -42,13 +48,19 @@ class GatedMLP:
         self._after = []           # weights streamed right after this part (see set_prefetch_targets)
 
     def tensor_specs(self):
-        return [TensorSpec(self.names["gate"], (self.inter, self.hidden)),
-                TensorSpec(self.names["up"], (self.inter, self.hidden)),
-                TensorSpec(self.names["down"], (self.hidden, self.inter))]
+        out = [TensorSpec(self.names["gate"], (self.inter, self.hidden)),
+               TensorSpec(self.names["up"], (self.inter, self.hidden)),
+               TensorSpec(self.names["down"], (self.hidden, self.inter))]
+        if self.has_bias:
+            out += [TensorSpec(self.names[k] + ".b", (size,), store="float32")
+                    for k, size in (("gate", self.inter), ("up", self.inter), ("down", self.hidden))]
+        return out
 
     def bind(self, tensors):
         self.w_gate_up = torch.cat([tensors[self.names["gate"]], tensors[self.names["up"]]], dim=0).contiguous()
         self.w_down = tensors[self.names["down"]]
+        if self.has_bias:
+            self.b_gate, self.b_up, self.b_down = (tensors[self.names[k] + ".b"].contiguous() for k in ("gate", "up", "down"))
 
     def streamed_weights(self):
         """The matrices this part streams in a small step, in kernel order."""
@@ -68,19 +80,34 @@ class GatedMLP:
         n = xn.shape[0]
         act = torch.empty((n, self.inter), dtype=self.dtype, device=xn.device)
         w_gate, w_up = self.w_gate_up[:self.inter], self.w_gate_up[self.inter:]
-        if (self.dtype == torch.bfloat16 and kernels.gemm_pays(n, self.inter, "swiglu")
+        if (kernels.skinny_fits(n, self.hidden, self.dtype) and xn.is_contiguous() and xn.data_ptr() % 16 == 0
+                and w_gate.data_ptr() % 16 == 0 and w_up.data_ptr() % 16 == 0):
+            # a step of a few rows: the weights streamed once, biases and activation in the product's epilogue
+            return kernels.skinny_gemm(w_gate, weight_up=w_up, x=xn, epilogue="swiglu", prefetch=self._target(0),
+                                       bias=self.b_gate, bias_up=self.b_up, activation=self.activation)
+        if (self.plain and self.dtype == torch.bfloat16 and kernels.gemm_pays(n, self.inter, "swiglu")
                 and kernels.gemm_fits(xn, w_gate, act, "swiglu", w_up)):
             # large portions: both products and the activation in one tcgen05 kernel
             kernels.gemm(xn, w_gate, weight_up=w_up, epilogue="swiglu", out=act)
         else:
             gu = kernels.linear(xn, self.w_gate_up, out_dtype=torch.float32)
-            kernels.silu_mul(act, gu[:, :self.inter], gu[:, self.inter:])
+            if self.plain:
+                kernels.silu_mul(act, gu[:, :self.inter], gu[:, self.inter:])
+            else:
+                kernels.biased_glu(act, gu[:, :self.inter], gu[:, self.inter:], self.b_gate, self.b_up, self.activation)
         return act
+
+    def forward_add(self, x, h, ctx):
+        kernels.linear_into(x, self._activation(h), self.w_down, bias=self.b_down, prefetch=self._target(1))
 
     def forward(self, xn, ctx):
         # gate and up stay float32 until the activation has been applied; the down
         # projection's float32 result goes into the residual stream unrounded
         n = xn.shape[0]
+        if not self.plain:
+            y = torch.zeros((n, self.hidden), dtype=torch.float32, device=xn.device)
+            self.forward_add(y, xn, ctx)
+            return y
         if (kernels.skinny_fits(n, self.hidden, self.dtype) and kernels.skinny_fits(n, self.inter, self.dtype)
                 and xn.is_contiguous()):
             # a step of a few rows: both products stream their weights once, the activation in the first one's epilogue
@@ -90,9 +117,11 @@ class GatedMLP:
         act = self._activation(xn)
         return kernels.linear(act, self.w_down, out_dtype=torch.float32)
 
-
     def forward_residual(self, x, norm, ctx):
         n = x.shape[0]
+        if not self.plain:
+            self.forward_add(x, norm.forward(x, None), ctx)
+            return True
         if not (getattr(norm, "fusable_rmsnorm", False) and kernels.skinny_fits(n, self.hidden, self.dtype)
                 and kernels.skinny_fits(n, self.inter, self.dtype, sliced=True)):
             # larger steps: the down product adds into the residual stream

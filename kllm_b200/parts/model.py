@@ -14,8 +14,8 @@ from typing import Dict, List, Optional
 import torch
 
 # registering the built-in part kinds
-from . import (attention, block, embedding, latent_attention, lightning, mlp, moe, norm, qk_norm, rotary,  # noqa: F401
-               side_input, streams, wkv)
+from . import (attention, block, embedding, gla, latent_attention, lightning, mlp, moe, norm, qk_norm, rotary,  # noqa: F401
+               side_by_side, side_input, stream_entry, streams, wkv)
 from .context import LayerCache, StepContext
 from .spec import BuildEnv, ModelSpec, PagedKVNeed, StateNeed, TensorSpec, part_factory
 
@@ -32,6 +32,7 @@ class DecoderModel:
         self.blocks = [part_factory("block", b.kind)(b, env) for b in spec.blocks]
         self.final_norm = part_factory("norm", spec.final_norm.kind)(spec.final_norm, env)
         self.head = part_factory("head", spec.head.kind)(spec.head, env)
+        self.entries = [part_factory("stream_entry", e.kind)(e, env) for e in spec.entries]
         self.schedule = list(spec.schedule)
         self.tap = None         # debugging: tap(i, x) is called with the residual stream after schedule entry i
         self._check_schedule()
@@ -41,6 +42,8 @@ class DecoderModel:
         for i, call in enumerate(self.schedule):
             if not (0 <= call.block < len(self.blocks)):
                 raise ValueError(f"schedule entry {i} names block {call.block} of {len(self.blocks)}")
+            if call.entry is not None and not (0 <= call.entry[0] < len(self.entries)):
+                raise ValueError(f"schedule entry {i} names stream entry {call.entry[0]} of {len(self.entries)}")
             if call.writes_cache:
                 if call.cache in writers:
                     raise ValueError(f"cache slot {call.cache} is written by schedule entries "
@@ -57,7 +60,7 @@ class DecoderModel:
 
     # ---- weights ---------------------------------------------------------
     def parts(self):
-        return [self.embedding] + self.blocks + [self.final_norm, self.head]
+        return [self.embedding] + self.entries + self.blocks + [self.final_norm, self.head]
 
     def tensor_specs(self) -> List[TensorSpec]:
         seen: Dict[str, TensorSpec] = {}
@@ -89,11 +92,12 @@ class DecoderModel:
 
     # ---- cache -----------------------------------------------------------
     def cache_needs(self):
-        """For every cache slot, what the mixer that writes it asks for."""
+        """For every cache slot, what the layer that writes it asks for: its mixer, or its block where
+        the arrangement keeps something of its own."""
         needs = []
         for slot in range(self.n_cache_slots):
-            mixer = self.blocks[self._writer_block[slot]].mixer
-            needs.append(mixer.cache_need())
+            block = self.blocks[self._writer_block[slot]]
+            needs.append((block if hasattr(block, "cache_need") else block.mixer).cache_need())
         return needs
 
     # ---- one step --------------------------------------------------------
@@ -102,12 +106,21 @@ class DecoderModel:
         is wanted; the cache is still filled)."""
         x = self.embedding.forward(ctx.token_ids, ctx.last_token)
         pending = None
+        held = [e.begin(x, bool(self.schedule) and self.schedule[0].entry is not None
+                        and self.schedule[0].entry[0] == j) for j, e in enumerate(self.entries)]
         for i, call in enumerate(self.schedule):
             cache = caches[call.cache]
             if cache.writes != call.writes_cache:
                 cache = LayerCache(cache.k, cache.v, cache.block_table, cache.state,
-                                   writes=call.writes_cache, page_size=cache.page_size)
+                                   writes=call.writes_cache, page_size=cache.page_size, states=cache.states)
             block = self.blocks[call.block]
+            if call.entry is not None:
+                if hasattr(pending, "settle"):
+                    pending = pending.settle(x)
+                if pending is not None:
+                    x.add_(pending)
+                    pending = None
+                self.entries[call.entry[0]].apply(x, held[call.entry[0]], call.entry[1])
             if hasattr(pending, "settle") and not getattr(block, getattr(pending, "accepted_by", "accepts_deferred_norm"),
                                                            False):
                 pending = pending.settle(x)

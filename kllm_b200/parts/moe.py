@@ -132,17 +132,32 @@ class RoutedExperts:
                                       for e in range(self.experts)]).contiguous()
         self.w_down = torch.stack([tensors[self._name(e, "down")] for e in range(self.experts)]).contiguous()
 
-    def _shared(self, xn):
-        """(rows float32 [n, d], gate logits float32 [n, 1] or None) of the expert that every token runs."""
+    def _shared_act(self, xn):
+        """(activation rows [n, f], gate logits float32 [n, 1] or None) of the expert that every token runs."""
         sh, f = self.shared, self.shared["ff"]
+        w = sh["w_in"]
+        if sh["act"]["activation"] == "silu" and w.shape[0] == 2 * f and xn.is_contiguous():
+            # no gate logit among the rows: the activation in the product's epilogue
+            w_gate, w_up = w[:f], w[f:]
+            aligned = xn.data_ptr() % 16 == 0 and w_gate.data_ptr() % 16 == 0 and w_up.data_ptr() % 16 == 0
+            if aligned and kernels.skinny_fits(xn.shape[0], self.hidden, self.dtype):
+                return kernels.skinny_gemm(w_gate, weight_up=w_up, x=xn, epilogue="swiglu"), None
+            if self.dtype == torch.bfloat16 and kernels.gemm_pays(xn.shape[0], f, "swiglu"):
+                act = torch.empty((xn.shape[0], f), dtype=self.dtype, device=xn.device)
+                if kernels.gemm_fits(xn, w_gate, act, "swiglu", w_up):
+                    return kernels.gemm(xn, w_gate, weight_up=w_up, epilogue="swiglu", out=act), None
         gu = kernels.linear(xn, sh["w_in"], out_dtype=torch.float32, small_ok=True)
         act = torch.empty((xn.shape[0], f), dtype=self.dtype, device=xn.device)
         if sh["act"]["activation"] == "clamped":
             kernels.clamped_glu(act, gu[:, :f], gu[:, f:2 * f], sh["act"]["limit"], sh["act"]["alpha"])
         else:
             kernels.silu_mul(act, gu[:, :f], gu[:, f:2 * f])
-        rows = kernels.linear(act, sh["w_down"], out_dtype=torch.float32, small_ok=True)
-        return rows, (gu[:, 2 * f:] if gu.shape[1] > 2 * f else None)
+        return act, (gu[:, 2 * f:] if gu.shape[1] > 2 * f else None)
+
+    def _shared(self, xn):
+        """(rows float32 [n, d], gate logits float32 [n, 1] or None) of the expert that every token runs."""
+        act, logit = self._shared_act(xn)
+        return kernels.linear(act, self.shared["w_down"], out_dtype=torch.float32, small_ok=True), logit
 
     def _plan(self, ctx, n):
         """The host's sort of a step's (token, choice) pairs by expert, for a table and ids that the host knows:
@@ -190,12 +205,30 @@ class RoutedExperts:
         shared, logit = self._shared(xn) if self.shared is not None else (None, None)
         return kernels.moe_combine(parts, top, shared=shared, gate=logit, scale=self.table_weight)
 
+    def forward_add(self, x, h, ctx):
+        """x += ff(h), x the float32 residual stream."""
+        if self.routing == "table" or (self.shared and self.shared["names"].get("gate_logit")):
+            x.add_(self.forward(h, ctx))
+            return
+        kernels.moe_combine(self._routed(h, ctx), self.top, into=x)
+        if self.shared is not None:
+            act, _ = self._shared_act(h)
+            kernels.linear_into(x, act, self.shared["w_down"])
+
     def forward(self, xn, ctx):
         if (self.routing == "table" and self.weight_on == "output" and getattr(ctx, "host_token_ids", None) is not None
                 and xn.shape[0] * self.top >= self.planned_rows * self.experts):
             plan = self._plan(ctx, xn.shape[0])
             if plan is not None:
                 return self._forward_planned(xn, plan)
+        parts = self._routed(xn, ctx)
+        if self.shared is None:
+            return kernels.moe_combine(parts, self.top)
+        rows, logit = self._shared(xn)
+        return kernels.moe_combine(parts, self.top, shared=rows, gate=logit)
+
+    def _routed(self, xn, ctx):
+        """Float32 rows token * top + choice of the chosen experts' weighted outputs."""
         if self.routing == "table":
             idx, wt = kernels.moe_table_route(ctx.token_ids, self.table, self.experts, self.table_weight, ctx.last_token)
         else:
@@ -206,14 +239,9 @@ class RoutedExperts:
         if kernels.moe_gemm_tcgen05_pays(xn, self.w_gate_up, perm.numel(), True, on_input):
             # a large step in bfloat16: tiles of 128 rows per expert on the tcgen05 tensor cores
             act = kernels.moe_gemm_tcgen05(xn, self.w_gate_up, offsets, perm, wt, self.top, gated=True, **self.act)
-            parts = kernels.moe_gemm_tcgen05(act, self.w_down, offsets, perm, wt, self.top, gated=False, scale_out=True)
-        else:
-            act = kernels.moe_gemm(xn, self.w_gate_up, offsets, perm, wt, self.top, gated=True, scale_in=on_input, **self.act)
-            parts = kernels.moe_gemm(act, self.w_down, offsets, perm, wt, self.top, gated=False, scale_out=not on_input)
-        if self.shared is None:
-            return kernels.moe_combine(parts, self.top)
-        rows, logit = self._shared(xn)
-        return kernels.moe_combine(parts, self.top, shared=rows, gate=logit)
+            return kernels.moe_gemm_tcgen05(act, self.w_down, offsets, perm, wt, self.top, gated=False, scale_out=True)
+        act = kernels.moe_gemm(xn, self.w_gate_up, offsets, perm, wt, self.top, gated=True, scale_in=on_input, **self.act)
+        return kernels.moe_gemm(act, self.w_down, offsets, perm, wt, self.top, gated=False, scale_out=not on_input)
 
 
 register_part("feed_forward", "routed_experts", RoutedExperts)

@@ -67,7 +67,7 @@ class HeadNormRotary:
     ``head_dim`` values and multiplied by a gain [head_dim] that all heads share (``q_gain`` /
     ``k_gain``: full tensor names, float32; None: no norm on that side), then the first ``rotary_dim``
     values of every head are rotated (pair (i, i + rotary_dim / 2), angle position * f_i; ``theta``,
-    ``scaling`` as in ``rotary.rotary_frequencies``), before which the projections' biases are added
+    ``scaling`` as in ``rotary.rotary_frequencies``; ``interleaved``: pair (2i, 2i + 1) instead), before which the projections' biases are added
     (the attention's ``bias``).  It offers ``prepare``: it takes the float32 result of the stacked
     projection, so biases, sums, scales and the rotation are float32 and the angle is formed in double
     precision on the device (no table, no bound on the position); it returns the queries in the model
@@ -83,6 +83,7 @@ class HeadNormRotary:
         self.rot = int(p.get("rotary_dim") or 0)
         if self.rot % 2 or self.rot > self.head_dim:
             raise ValueError(f"rotary_dim {self.rot} must be even and within head_dim {self.head_dim}")
+        self.interleaved = bool(p.get("interleaved", False))
         self.freq, self.amplitude = None, 1.0
         if self.rot:
             freq, self.amplitude = rotary_frequencies(self.rot, float(p["theta"]), p.get("scaling"))
@@ -104,7 +105,7 @@ class HeadNormRotary:
         kernels.headnorm_rope_append(q, qkv, attn.bias, self.q_gain, self.k_gain, self.eps, self.freq, self.amplitude,
                                      self.rot, ctx.positions, ctx.token_req, cache.block_table if writes else None,
                                      cache.k if writes else None, cache.v if writes else None, q_heads, k_heads,
-                                     attn.n_kv, self.head_dim, attn.v_head_dim)
+                                     attn.n_kv, self.head_dim, attn.v_head_dim, interleaved=self.interleaved)
         return q
 
 

@@ -71,6 +71,7 @@ class LayerCall:
     block: int
     cache: int
     writes_cache: bool = True
+    entry: Optional[Tuple[int, int]] = None     # (index into ModelSpec.entries, its argument): done to the stream before the layer
 
 
 @dataclass
@@ -84,6 +85,7 @@ class ModelSpec:
     final_norm: PartSpec
     head: PartSpec
     eos_token_ids: Tuple[int, ...] = ()
+    entries: List[PartSpec] = field(default_factory=list)   # parts of the stream_entry family that schedule entries name
 
 
 # ---- what a mixer asks of the cache manager ---------------------------------
@@ -129,22 +131,24 @@ class PagedKVNeed:
 @dataclass(frozen=True)
 class StateNeed:
     """Per-request state of fixed size, one slot per live request, zero at the
-    start of a request."""
+    start of a request.  A layer that asks for several gives all but one a ``name``
+    (``LayerCache.states[name]``; the one without is ``LayerCache.state``)."""
     shape: Tuple[int, ...]
     dtype: str = "float32"
+    name: str = ""
 
 
 # ---- registries -----------------------------------------------------------
 
 _KINDS: Dict[str, Dict[str, Callable]] = {
     "mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "qk_transform": {}, "block": {},
-    "embedding": {}, "head": {}, "side_input": {},
+    "embedding": {}, "head": {}, "side_input": {}, "stream_entry": {},
 }
 
 
 def register_part(family: str, kind: str, factory: Callable) -> None:
     """``factory(spec: PartSpec, env: BuildEnv)`` returns the part.  ``family`` is one
-    of mixer, feed_forward, norm, position, qk_transform, block, embedding, head, side_input."""
+    of mixer, feed_forward, norm, position, qk_transform, block, embedding, head, side_input, stream_entry."""
     if family not in _KINDS:
         raise KeyError(f"unknown part family {family!r}; families: {sorted(_KINDS)}")
     _KINDS[family][kind] = factory
