@@ -50,6 +50,8 @@ attention through a latent with a rotated key part, layer norms, experts chosen 
 attention through a latent that a later layer reads again, linear attention with a fixed decay per head,
 output norms, a token side input) beside a dense Sozarax model of equal size, the closest existing design
 (a recurrent mixer, attention with norms over the whole projections, a plain feed-forward), and beside a Llama.
+``--design dirarax`` measures the Dirarax design (gated linear attention, attention and retention side by side, one norm
+for both sublayers with a token shift, biased and routed feed-forwards) beside a Sozarax and a Llama.
 """
 from __future__ import annotations
 
@@ -256,8 +258,8 @@ def main():
     ap.add_argument("--workload", default="", choices=["", "llama2-7b-mixed"],
                     help="llama2-7b-mixed: 32 requests, prompts uniform in [128, 3072], 128 new tokens each, through "
                          "the scheduler (a record of its own, not the bench line)")
-    ap.add_argument("--design", default="", choices=["", "sozarax", "nutizen", "ronurax", "senulix"],
-                    help="sozarax, nutizen, ronurax: prefill and decode of that design at two layer sizes beside a Llama of equal size, and "
+    ap.add_argument("--design", default="", choices=["", "sozarax", "nutizen", "ronurax", "senulix", "dirarax"],
+                    help="sozarax, nutizen, ronurax, senulix, dirarax: prefill and decode of that design at two layer sizes beside a Llama of equal size, and "
                          "its kernels against their rooflines (a record of its own, not the bench line)")
     args = ap.parse_args()
     if args.timeline:
@@ -696,6 +698,28 @@ def senulix_config(width, layers, heads, kv_heads, head_dim, ff, vocab, kv_rank,
             out.append({"type": "latent_attention", "mixer": dict(lat, kv_from=i - 2), "mlp": dict(dense)})
     return {"architecture": "Senulix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
             "token_side": {"dim": side_dim}, "logit_softcap": 30.0, "layers": out}
+
+
+def dirarax_config(width, layers, heads, kv_heads, head_dim, ff, experts, top, expert_ff, vocab):
+    """A Dirarax model of ``layers`` layers in the pattern of three gated linear-attention layers and one that runs softmax
+    attention and retention side by side; dense and routed feed-forwards in turn; every layer runs once, as one
+    pass of the loop (its mix with the embedding's output included).  The recurrent heads have twice as many value
+    channels as key channels, the attention's half as many; the side-by-side mixers have half the width each."""
+    gh = width // 256
+    gla = {"heads": gh, "dim": 128, "vdim": 256, "tau": 16.0}
+    par = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": head_dim,
+                    "vdim": head_dim // 2, "scale": head_dim ** -0.5,
+                    "rot": {"base": 50000.0, "dims": head_dim // 2,
+                            "scaling": {"factor": 2.0, "original": 1024, "fast": 32.0, "slow": 1.0}}},
+           "right": {"heads": gh, "dim": 128, "vdim": 128, "rot": {"base": 1000000.0, "dims": 128},
+                     "decay": [1.0 - 2.0 ** (-5.0 - 6.0 * h / max(1, gh - 1)) for h in range(gh)]},
+           "left_scale": 0.7, "right_scale": 0.7}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": expert_ff}}
+    return {"architecture": "Dirarax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [{"type": "parallel" if i % 4 == 3 else "gla", "mixer": dict(par if i % 4 == 3 else gla),
+                        "mlp": dict(dense if i % 2 == 0 else moe)} for i in range(layers)],
+            "loop": {"start": 0, "stop": layers, "times": 1}}
 
 
 SENULIX_EXTRA = {
@@ -1354,8 +1378,175 @@ def design_comparison(args):
             del caches
         return rows
 
+    def dirarax_rows(width, heads, kv, hd, ff):
+        """The Dirarax design's own kernels, each beside the kernels of the closest design that do the like work."""
+        import itertools
+        import types
+        rows = []
+        dev, f32 = "cuda", torch.float32
+        A = heads * hd
+        esz = 2 if dtype == "bfloat16" else 4
+        hbm, tens = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+        cores = 2 * 128 * kernels.sm_count() * 1.9e9        # float32 operations a second of the CUDA cores
+
+        def ctx_of(n_new, start):
+            S = len(n_new)
+            qs = torch.tensor([0] + list(itertools.accumulate(n_new)), dtype=torch.int32, device=dev)
+            return types.SimpleNamespace(
+                n_tokens=sum(n_new), n_requests=S, q_start=qs,
+                token_req=torch.repeat_interleave(torch.arange(S, dtype=torch.int32), torch.tensor(n_new)).to(dev),
+                start_pos=torch.tensor(start, dtype=torch.int32, device=dev),
+                positions=torch.cat([torch.arange(s, s + c, dtype=torch.int32) for s, c in zip(start, n_new)]).to(dev),
+                state_slots=torch.arange(S, dtype=torch.int32, device=dev), host_n_new=list(n_new),
+                host_start_pos=list(start), all_single=all(c == 1 for c in n_new),
+                max_ctx=max(s + c for s, c in zip(start, n_new)), split_bound=0, max_new=max(n_new))
+
+        def row(name, us, by, like=None, tensor=0.0, core=0.0):
+            floor, bound = max((by / hbm * 1e6, "memory"), (tensor / tens * 1e6 if dtype == "bfloat16" else 0.0, "tensor"),
+                               (core / cores * 1e6, "float32 cores"))
+            rows.append({"kernel": name, "us": round(us, 1), "floor_us": round(floor, 2), "bound": bound,
+                         "times_floor": round(us / floor, 1), "like": like})
+
+        def each(call, inner=4):
+            it = [0]
+
+            def fn():
+                it[0] += 1
+                call(it[0])
+            return timed(fn, inner=inner) * 1e3
+        gh, gk, gv, R = width // 256, 128, 256, 16
+        for name, n_new, start in (("prefill", [T], [0]), ("decode", [1] * B, [ctx - 1] * B)):
+            c, S, n = ctx_of(n_new, start), len(n_new), sum(n_new)
+            # ---- recurrences with their decay, unit norm and gate: the state read and written once, the rows read and
+            # written once, and four float32 operations per state element and row on the CUDA cores ----
+            for what, dv in (("gated linear attention", gv), ("retention", 128)):
+                KA, VB = gh * gk, gh * dv
+                P = 2 * KA + 2 * VB + (R if dv == gv else 0)
+                projs = rotate(lambda: torch.randn(n, P, device=dev) * 0.3, 4 * n * P)
+                states = rotate(lambda: torch.zeros(S, KA * dv, device=dev), 4 * S * KA * dv)
+                w2, b2 = (torch.randn(KA, R, device=dev) * 0.1).to(tdt), torch.full((KA,), 4.0, device=dev)
+                dec, gain = torch.linspace(0.96, 0.999, gh, device=dev), torch.ones(VB, device=dev)
+                freq = (1e6 ** (-2.0 * torch.arange(64, dtype=torch.float64) / 128)).to(dev)
+                y = torch.empty((n, VB), dtype=tdt, device=dev)
+
+                def rec(i):
+                    p = projs[i % len(projs)]
+                    kw = dict(low=p[:, P - R:], w2=w2, w2_bias=b2, tau=16.0) if dv == gv else dict(decay=dec, freq=freq)
+                    kernels.gla(y, p[:, :KA], p[:, KA:2 * KA], p[:, 2 * KA:2 * KA + VB], p[:, 2 * KA + VB:2 * (KA + VB)],
+                                states[i % len(states)], c, gh, gk, dv, gain, 1e-6, q_scale=gk ** -0.5, **kw)
+                row(f"{what} {name}", each(rec), 8.0 * S * KA * dv + 4.0 * n * P + esz * n * VB, like=f"wkv {name}",
+                    core=4.0 * n * KA * dv)
+                del projs, states
+            sets = rotate(lambda: [torch.randn(n, A, device=dev) * 0.1 for _ in range(4)] + [torch.randn(n, 64, device=dev)], 16 * n * A)
+            states = rotate(lambda: torch.zeros(S, A * hd + width, device=dev), 4 * S * A * hd)
+            wo, w0, u = (torch.randn(A, 64, device=dev) * 0.1).to(tdt), torch.zeros(A, device=dev), torch.zeros(A, device=dev)
+            one = torch.ones(A, device=dev)
+
+            def wkv(i):
+                r, k, v, gt, lo = sets[i % len(sets)]
+                o = kernels.wkv_scan(r, k, v, kernels.wkv_decay_outer(lo, wo), w0, u, states[i % len(states)], c, heads, hd)
+                kernels.wkv_gate_norm(o, gt, one, 1e-6, heads, hd, tdt)
+            row(f"wkv {name} (decay, scan, norm and gate)", each(wkv), 8.0 * S * A * hd + 16.0 * n * A + 256.0 * n + esz * n * A,
+                core=4.0 * n * A * hd)
+            del sets, states
+            # ---- norm and token shift ----
+            xs = rotate(lambda: torch.randn(n, width, device=dev), 4 * n * width)
+            sh = torch.zeros(S, width, device=dev)
+            gain, mu = torch.ones(width, device=dev), torch.full((width,), 0.5, device=dev)
+            row(f"norm and token shift {name}", each(lambda i: kernels.norm_shift(xs[i % len(xs)], gain, 1e-6, mu, sh, c, tdt)),
+                n * width * (4 + 2 * esz) + 8.0 * S * width, like=f"sozarax norm, then shift {name}")
+
+            def norm_then_shift(i):
+                h = torch.empty((n, width), dtype=tdt, device=dev)
+                kernels.add_rmsnorm(xs[i % len(xs)], None, h, gain, 1e-6)
+                kernels.wkv_shift_mix(h, mu.view(1, -1), sh, 0, c)
+            row(f"sozarax norm, then shift {name}", each(norm_then_shift), n * width * (4 + 3 * esz) + 8.0 * S * width)
+            # ---- attention with values half as wide as the keys, float32 weights ----
+            vd = hd // 2
+            per = -(-max(s + m for s, m in zip(start, n_new)) // page)
+            table = torch.arange(S * per, dtype=torch.int32, device=dev).view(S, per).contiguous()
+            caches = rotate(lambda: tuple(torch.randn(S * per, kv, page, z, device=dev).to(tdt) for z in (hd, vd, hd)),
+                            S * per * kv * page * (2 * hd + vd) * esz)
+            q = (torch.randn(n, A, device=dev) * 0.2).to(tdt)
+            out_v, out = (torch.empty(n, heads * z, device=dev, dtype=tdt) for z in (vd, hd))
+            pairs = sum(p + 1 for s, m in zip(start, n_new) for p in range(s, s + m))
+            keys = sum(s + m for s, m in zip(start, n_new))
+            slopes = torch.linspace(-0.1, -0.001, heads, device=dev)
+            row(f"gated attention's softmax part {name} (values of {vd})",
+                each(lambda i: kernels.attention(out_v, q, caches[i % len(caches)][0], caches[i % len(caches)][1], c, table, heads,
+                                                 kv, hd, 0, hd ** -0.5, v_head_dim=vd, exact_weights=True)),
+                keys * kv * (hd + vd) * esz + n * (A + heads * vd) * esz, like=f"sozarax attention {name}",
+                tensor=2.0 * pairs * heads * (hd + vd))
+            for what, kw in (("sozarax attention", dict(score_slopes=slopes, exact_weights=True)), ("llama attention", {})):
+                row(f"{what} {name} (values of {hd})",
+                    each(lambda i: kernels.attention(out, q, caches[i % len(caches)][0], caches[i % len(caches)][2], c, table, heads,
+                                                     kv, hd, 0, hd ** -0.5, **kw)),
+                    keys * kv * 2 * hd * esz + 2 * n * A * esz, tensor=4.0 * pairs * heads * hd)
+            # ---- rotation and cache write, output gate ----
+            W = A + kv * (hd + vd)
+            projs = rotate(lambda: torch.randn(n, W, device=dev), 4 * n * W)
+            freq = (5e4 ** (-2.0 * torch.arange(hd // 4, dtype=torch.float64) / (hd // 2))).to(dev)
+            qo = torch.empty((n, A), dtype=tdt, device=dev)
+            row(f"rotation and cache write {name}",
+                each(lambda i: kernels.headnorm_rope_append(qo, projs[i % len(projs)], None, None, None, 0.0, freq, 1.07, hd // 2,
+                                                            c.positions, c.token_req, table, caches[0][0], caches[0][1], heads, kv,
+                                                            kv, hd, vd, interleaved=True)),
+                n * W * (4 + esz), like=f"sozarax norm and cache write {name}")
+            W2 = A + 2 * kv * hd
+            projs2 = rotate(lambda: torch.randn(n, W2, device=dev), 4 * n * W2)
+            qg, kg = torch.ones(A, device=dev), torch.ones(kv * hd, device=dev)
+            row(f"sozarax norm and cache write {name}",
+                each(lambda i: kernels.qknorm_append(qo, projs2[i % len(projs2)], qg, kg, 1e-6, 0.1, 64, c.positions, c.token_req,
+                                                     table, caches[0][0], caches[0][2], heads, kv, hd, hd)), n * W2 * (4 + esz))
+            del caches, projs, projs2
+            # ---- the gate and up half of the dense feed-forward: biases and gelu, beside Llama's silu ----
+            wgu = rotate(lambda: (torch.randn(2 * ff, width, device=dev) * 0.02).to(tdt), 2 * ff * width * esz)
+            h = (torch.randn(n, width, device=dev)).to(tdt)
+            bias = torch.zeros(ff, device=dev)
+
+            def glu(act, b):
+                def call(i):
+                    w = wgu[i % len(wgu)]
+                    if kernels.skinny_fits(n, width, tdt):
+                        kernels.skinny_gemm(w[:ff], weight_up=w[ff:], x=h, epilogue="swiglu", bias=b, bias_up=b, activation=act)
+                        return
+                    o = torch.empty((n, ff), dtype=tdt, device=dev)
+                    if b is None and tdt == torch.bfloat16 and kernels.gemm_pays(n, ff, "swiglu"):
+                        kernels.gemm(h, w[:ff], weight_up=w[ff:], epilogue="swiglu", out=o)
+                        return
+                    gu = kernels.linear(h, w, out_dtype=f32)
+                    if b is None:
+                        kernels.silu_mul(o, gu[:, :ff], gu[:, ff:])
+                    else:
+                        kernels.biased_glu(o, gu[:, :ff], gu[:, ff:], b, b, act)
+                return call
+            by, fl = 2.0 * ff * width * esz + n * (width + ff) * esz, 4.0 * n * ff * width
+            row(f"gate and up with biases and gelu {name}", each(glu("gelu_tanh", bias)), by, like=f"llama gate and up {name}", tensor=fl)
+            row(f"llama gate and up {name}", each(glu("silu", None)), by, tensor=fl)
+            del wgu
+        return rows
+
     sizes = {}
     for name, (width, layers, heads, kv, hd, ff, E, top, eff, vocab) in DESIGN_SIZES.items():
+        if args.design == "dirarax":
+            dira = dirarax_config(width, layers, heads, kv, hd, ff, E, top, eff, vocab)
+            soz = sozarax_config(width, layers, heads, kv, hd, ff, E, top, eff, vocab)
+            llama = dict(TINYLLAMA, num_hidden_layers=layers, hidden_size=width, num_attention_heads=heads,
+                         num_key_value_heads=kv, head_dim=hd, intermediate_size=ff, vocab_size=vocab,
+                         max_position_embeddings=max(ctx, T))
+            left = dira["layers"][3]["mixer"]["left"]
+            rec = {"layers": layers, "recurrent_heads": f"{width // 256} of 128 x 256",
+                   "side_by_side": f"{left['heads']} heads of {hd} (values {hd // 2}) over {kv} kv heads, "
+                                   f"{width // 256} retention heads of 128 x 128",
+                   "ff": ff, "experts": f"{top} of {E} x {eff} + shared {eff}"}
+            for key, cfg in (("dirarax", dira), ("sozarax", soz), ("llama", llama)):
+                print(f"[bench] {name}: {key}", file=sys.stderr, flush=True)
+                rec[key] = model_run(cfg, vocab)
+            print(f"[bench] {name}: kernels", file=sys.stderr, flush=True)
+            rec["kernels"] = dirarax_rows(width, heads, kv, hd, ff)
+            sizes[name] = rec
+            torch.cuda.empty_cache()
+            continue
         if args.design == "senulix":
             R, dr, window, side = SENULIX_EXTRA[name]
             sen = senulix_config(width, layers, heads, kv, hd, ff, vocab, R, dr, window, side)
@@ -1424,7 +1615,7 @@ def design_comparison(args):
         sizes[name] = rec
         torch.cuda.empty_cache()
     sampler.stop()
-    beside = "a dense Sozarax and a Llama" if args.design == "senulix" else "a Llama"
+    beside = {"senulix": "a dense Sozarax and a Llama", "dirarax": "a Sozarax and a Llama"}.get(args.design, "a Llama")
     print(json.dumps({"partial": f"{args.design.capitalize()} beside {beside} of equal size", "dtype": dtype, "prefill_tokens": T,
                       "decode_batch": B, "decode_context": ctx, "data": "synthetic, random weights",
                       "peaks": pk, "clocks": sampler.summary(t_begin, time.time()), "sizes": sizes}))
