@@ -43,8 +43,8 @@
 #ifndef KLLM_HD
 #error "compile with -DKLLM_HD=<head size>"
 #endif
-// Values of another size than the keys: -DKLLM_VD=<value size>.  Such a library holds the prefill
-// kernel alone (the decode kernels are built for values as wide as the keys).
+// Values of another size than the keys: -DKLLM_VD=<value size>.  Such a library holds the prefill kernel
+// and the plain decode kernel (the fused one is built for values as wide as the keys).
 #ifndef KLLM_VD
 #define KLLM_VD KLLM_HD
 #endif
@@ -70,7 +70,7 @@ constexpr int STAGE_ELEMS = TILE * (ROW + ROWV);                  // K tile then
 // the more of the range is in flight at once (with 5 stages a range of 256 keys is
 // requested whole before the first tile is used).  Prefill keeps 3 stages and more
 // CTAs per SM.
-constexpr int DEC_STAGES_DEEP = HD <= 64 ? 5 : (HD <= 96 ? 4 : 3);   // few CTAs: everything in flight at once
+constexpr int DEC_STAGES_DEEP = HD + VD <= 128 ? 5 : (HD + VD <= 192 ? 4 : 3);   // few CTAs: everything in flight at once
 constexpr int DEC_PAGES = 256;                                        // block-table entries of a range kept in shared memory
 constexpr int DEC_STAGES_WIDE = 3;                                    // many CTAs: more of them per SM
 constexpr int PRE_STAGES = 3;
@@ -118,14 +118,45 @@ __device__ __forceinline__ void load_tile(bf16* stage, const bf16* __restrict__ 
     const int lp0 = key0 / page_size, in_page = key0 - lp0 * page_size;
     if (in_page + TILE <= page_size) {
         // the whole tile lies in one page: one look-up, rows one after the other
-        const int64_t base = (((int64_t)table[lp0 - page_base] * n_kv + g) * page_size + in_page) * HD;
+        const int64_t base = ((int64_t)table[lp0 - page_base] * n_kv + g) * page_size + in_page;
+        if constexpr (VD == HD) {
 #pragma unroll
-        for (int c = threadIdx.x; c < TILE * CHUNKS; c += THREADS) {
-            const int row = c / CHUNKS, ch = c - row * CHUNKS;
-            const bool valid = key0 + row < hi;
-            const int64_t off = valid ? base + row * HD + ch * 8 : 0;
-            cp_async16(sk + row * ROW + ch * 8, kcache + off, valid);
-            cp_async16(sv + row * ROW + ch * 8, vcache + off, valid);
+            for (int c = threadIdx.x; c < TILE * CHUNKS; c += THREADS) {
+                const int row = c / CHUNKS, ch = c - row * CHUNKS;
+                const bool valid = key0 + row < hi;
+                const int64_t off = valid ? (base + row) * HD + ch * 8 : 0;
+                cp_async16(sk + row * ROW + ch * 8, kcache + off, valid);
+                cp_async16(sv + row * ROW + ch * 8, vcache + off, valid);
+            }
+        } else {
+#pragma unroll
+            for (int c = threadIdx.x; c < TILE * CHUNKS; c += THREADS) {
+                const int row = c / CHUNKS, ch = c - row * CHUNKS;
+                const bool valid = key0 + row < hi;
+                cp_async16(sk + row * ROW + ch * 8, kcache + (valid ? (base + row) * HD + ch * 8 : 0), valid);
+            }
+#pragma unroll
+            for (int c = threadIdx.x; c < TILE * VCHUNKS; c += THREADS) {
+                const int row = c / VCHUNKS, ch = c - row * VCHUNKS;
+                const bool valid = key0 + row < hi;
+                cp_async16(sv + row * ROWV + ch * 8, vcache + (valid ? (base + row) * VD + ch * 8 : 0), valid);
+            }
+        }
+        return;
+    }
+    if constexpr (VD != HD) {
+        for (int c = threadIdx.x; c < TILE * (CHUNKS + VCHUNKS); c += THREADS) {
+            const bool is_k = c < TILE * CHUNKS;
+            const int e = is_k ? c : c - TILE * CHUNKS, per = is_k ? CHUNKS : VCHUNKS;
+            const int row = e / per, ch = e - row * per, key = key0 + row;
+            const bool valid = key < hi;
+            int64_t slot = 0;
+            if (valid) {
+                const int lp = key / page_size;
+                slot = ((int64_t)table[lp - page_base] * n_kv + g) * page_size + (key - lp * page_size);
+            }
+            if (is_k) cp_async16(sk + row * ROW + ch * 8, kcache + (valid ? slot * HD + ch * 8 : 0), valid);
+            else cp_async16(sv + row * ROWV + ch * 8, vcache + (valid ? slot * VD + ch * 8 : 0), valid);
         }
         return;
     }
@@ -199,7 +230,6 @@ __device__ __forceinline__ void load_tile_wide(bf16* stage, const bf16* __restri
 // what rounding to bfloat16 leaves of x
 __device__ __forceinline__ float bf16_rest(float x) { return x - __bfloat162float(__float2bfloat16_rn(x)); }
 
-#if KLLM_VD == KLLM_HD
 // Scores of 16 rows against keys [16*slice, 16*slice+16) of a K tile.
 __device__ __forceinline__ void scores16(float (&s)[2][4], const uint32_t (&qa)[KSTEPS][4], const bf16* sk,
                                          int slice, int lane) {
@@ -223,9 +253,9 @@ __device__ __forceinline__ void scores16(float (&s)[2][4], const uint32_t (&qa)[
 __device__ __forceinline__ void accumulate16(float (&o)[DTILES][4], const uint32_t (&pa)[4], const bf16* sv,
                                              int slice, int lane) {
     const int mi = lane >> 3;
-    const bf16* base = sv + (16 * slice + (mi & 1) * 8 + (lane & 7)) * ROW + (mi >> 1) * 8;
+    const bf16* base = sv + (16 * slice + (mi & 1) * 8 + (lane & 7)) * ROWV + (mi >> 1) * 8;
 #pragma unroll
-    for (int dp = 0; dp < HD / 16; dp++) {
+    for (int dp = 0; dp < VD / 16; dp++) {
         uint32_t v[4];
         ldmatrix_x4_trans(v, base + dp * 16);
         mma_bf16(o[2 * dp], pa, v[0], v[1]);
@@ -542,20 +572,20 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     float* sm_m = reinterpret_cast<float*>(smem_raw);       // [4][16]
     float* sm_l = sm_m + 64;                                // [4][16]
-    float* sm_o = sm_l + 64;                                // [4][16][HD]
+    float* sm_o = sm_l + 64;                                // [4][16][VD]
     if (tq == 0) {
         sm_m[warp * 16 + gid] = m0; sm_m[warp * 16 + gid + 8] = m1;
         sm_l[warp * 16 + gid] = l0; sm_l[warp * 16 + gid + 8] = l1;
     }
 #pragma unroll
     for (int dt = 0; dt < DTILES; dt++) {
-        float* r0 = sm_o + (warp * 16 + gid) * HD + dt * 8 + 2 * tq;
-        float* r1 = sm_o + (warp * 16 + gid + 8) * HD + dt * 8 + 2 * tq;
+        float* r0 = sm_o + (warp * 16 + gid) * VD + dt * 8 + 2 * tq;
+        float* r1 = sm_o + (warp * 16 + gid + 8) * VD + dt * 8 + 2 * tq;
         r0[0] = o[dt][0]; r0[1] = o[dt][1]; r1[0] = o[dt][2]; r1[1] = o[dt][3];
     }
     __syncthreads();
-    for (int e = threadIdx.x; e < gs * HD; e += THREADS) {
-        const int r = e / HD, d = e - r * HD;
+    for (int e = threadIdx.x; e < gs * VD; e += THREADS) {
+        const int r = e / VD, d = e - r * VD;
         float M = -INFINITY;
 #pragma unroll
         for (int w = 0; w < 4; w++) M = fmaxf(M, sm_m[w * 16 + r]);
@@ -568,16 +598,16 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
             for (int w = 0; w < 4; w++) {
                 const float f = exp2f((sm_m[w * 16 + r] - M) * scale_log2e);   // 0 for a warp without keys
                 L += sm_l[w * 16 + r] * f;
-                O += sm_o[(w * 16 + r) * HD + d] * f;
+                O += sm_o[(w * 16 + r) * VD + d] * f;
             }
             if (sk > -INFINITY) L += exp2f((sk - M) * scale_log2e);
         }
         const int h = g * gs + r;
         if (num_splits == 1) {
-            out[(int64_t)t * n_heads * HD + (int64_t)h * HD + d] = __float2bfloat16_rn(O / L);
+            out[(int64_t)t * n_heads * VD + (int64_t)h * VD + d] = __float2bfloat16_rn(O / L);
         } else {
             const int64_t slot = ((int64_t)t * n_heads + h) * num_splits + split;
-            part_o[slot * HD + d] = O;
+            part_o[slot * VD + d] = O;
             if (d == 0) { part_ml[slot * 2] = M * scale_log2e; part_ml[slot * 2 + 1] = L; }
         }
     }
@@ -616,15 +646,13 @@ __global__ void attn_combine_kernel(bf16* __restrict__ out, const float* __restr
     for (int j = 0; j < num_splits; j++) M = fmaxf(M, ml[2 * j]);
     float L = 0.f;
     for (int j = 0; j < num_splits; j++) L += ml[2 * j + 1] * exp2f(ml[2 * j] - M);
-    for (int d = threadIdx.x; d < HD; d += blockDim.x) {
+    for (int d = threadIdx.x; d < VD; d += blockDim.x) {
         float O = 0.f;
         for (int j = 0; j < num_splits; j++)
-            O += part_o[(th * num_splits + j) * HD + d] * exp2f(ml[2 * j] - M);
-        out[th * HD + d] = __float2bfloat16_rn(O / L);
+            O += part_o[(th * num_splits + j) * VD + d] * exp2f(ml[2 * j] - M);
+        out[th * VD + d] = __float2bfloat16_rn(O / L);
     }
 }
-
-#endif  // KLLM_VD == KLLM_HD
 
 // ---- prefill ------------------------------------------------------------------
 
@@ -979,10 +1007,10 @@ int set_attributes() {
     auto raise = [&](auto kernel, int bytes) {
         if (e == cudaSuccess) e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
     };
-#if KLLM_VD == KLLM_HD
     raise(attn_decode_kernel<false, DEC_STAGES_DEEP>, dec_smem_bytes(DEC_STAGES_DEEP));
-    raise(attn_decode_kernel<true, DEC_STAGES_DEEP>, dec_smem_bytes(DEC_STAGES_DEEP));
     raise(attn_decode_kernel<false, DEC_STAGES_WIDE>, dec_smem_bytes(DEC_STAGES_WIDE));
+#if KLLM_VD == KLLM_HD
+    raise(attn_decode_kernel<true, DEC_STAGES_DEEP>, dec_smem_bytes(DEC_STAGES_DEEP));
     raise(attn_decode_kernel<true, DEC_STAGES_WIDE>, dec_smem_bytes(DEC_STAGES_WIDE));
 #endif
     raise(attn_prefill_kernel, PRE_SMEM_BYTES);
@@ -1008,10 +1036,9 @@ int check_common(int n_heads, int n_kv, int hd, int page_size, const void* q, in
 extern "C" int kllm_attention_tc_head_dim() { return HD; }
 extern "C" int kllm_attention_tc_value_dim() { return VD; }
 
-#if KLLM_VD == KLLM_HD
-
 // Decode form: every token on its own (any batch is valid, one token per request
-// is what it is made for).  part_o [n_tokens, n_heads, num_splits, HD] float32 and
+// is what it is made for).  out [n_tokens, n_heads * VD]; vcache [pages, n_kv, page_size, VD];
+// part_o [n_tokens, n_heads, num_splits, VD] float32 and
 // part_ml [n_tokens, n_heads, num_splits, 2] float32 are scratch for num_splits > 1.
 extern "C" int kllm_attention_decode(void* out, void* part_o, void* part_ml, const void* q, int64_t q_stride,
                                      const void* kcache, const void* vcache, const int* positions,
@@ -1054,10 +1081,12 @@ extern "C" int kllm_attention_decode(void* out, void* part_o, void* part_ml, con
         (bf16*)vcache, positions, token_req, block_table, max_blocks, n_heads, n_kv, page_size, window, sl2e,
         num_splits, extra);
     if (num_splits > 1)
-        kllm_launch((attn_combine_kernel), dim3(n_tokens * n_heads), dim3(HD < 64 ? 32 : 64), 0, s, (bf16*)out, (const float*)part_o,
+        kllm_launch((attn_combine_kernel), dim3(n_tokens * n_heads), dim3(VD < 64 ? 32 : 64), 0, s, (bf16*)out, (const float*)part_o,
                                                                           (const float*)part_ml, num_splits);
     KLLM_LAUNCH_STATUS();
 }
+
+#if KLLM_VD == KLLM_HD
 
 // Decode form with the step's rotary encoding, cache write and split merge inside
 // (one token per request).  q [n, n_heads*HD], k_new and v_new [n, n_kv*HD] are this

@@ -18,19 +18,20 @@
 // projections are waited for, is updated in registers and written back, and the cluster's CTAs join their sums
 // of squares through distributed shared memory for the head's norm.
 //
-// Steps with portions take three kernels.  A request's rows are cut into chunks of kC rows.  Since the
-// recurrence is linear in the state, with the cumulative decay A_i = alpha_first ... alpha_i of a chunk
+// Steps with portions take four kernels.  A request's rows are cut into chunks of kC rows.  With the cumulative decay
+// D_ij = alpha_(j+1) ... alpha_i per key channel (D_ii = 1) and A_i = alpha_first ... alpha_i inside a chunk,
 //
-//     o_i = local_i + sum_d (q_i A_i)[d] S_in[d]           S_out = A_last S_in + S_local
+//     o_i   = sum_d (q_i A_i)[d] S_in[d] + sum over j <= i of W_ij v_j        W_ij = sum_d q_i[d] D_ij[d] k_j[d]
+//     S_out = A_last S_in + sum over j of (k_j D_last,j) v_j^T
 //
-// where local and S_local belong to the same rows run from a zero state:
-//   local_kernel   every chunk at once: the recurrence row by row from a zero state; leaves local_i, S_local,
-//                  q_i A_i and A_last
+//   chunk_kernel   every (chunk, head) at once: W, q_i A_i, k_j D_last,j and A_last.  A thread carries k_j times its
+//                  running decay from row to row, so no quotient of decays is ever formed: every factor is a product of
+//                  numbers in [0, 1], and a decay that reaches zero inside a chunk is harmless
+//   outer_kernel   every chunk at once: the chunk's own addition to the state
 //   carry_kernel   the states at the chunks' starts, element by element over a request's chunks in order;
 //                  moves the slot on
 //   apply_kernel   every chunk at once: o, the head's norm and the gate
-// No quotient of decays is ever formed: every factor is a product of numbers in [0, 1], so a decay that reaches
-// zero inside a chunk is harmless.  Where a prompt is cut changes the order of float32 sums and nothing else.
+// Where a prompt is cut changes the order of float32 sums and nothing else.
 #include "common.cuh"
 
 KLLM_EXPORT_LAST_ERROR(gla)
@@ -38,8 +39,7 @@ KLLM_EXPORT_LAST_ERROR(gla)
 namespace {
 
 constexpr int kC = 64;          // rows of a chunk
-constexpr int kTS = 16;         // rows staged in shared memory at a time
-constexpr int kSl = 64;         // value channels of a CTA of the local kernel
+constexpr int kTS = 16;         // rows whose angles are in shared memory at a time
 constexpr int kThreads = 256;
 constexpr int kMaxRot = 256;
 
@@ -64,8 +64,9 @@ struct GlaArgs {
     float eps;
     void* y;
     int64_t y_stride;
-    // work of the three-kernel form
-    float *o, *qa, *a_last, *s_in;          // [n][H dv], [n][H dk], [chunks][H dk], [chunks][H][dk][dv]
+    // work of the form for portions
+    float *o, *qa, *kd, *a_last, *w, *s_in; // [n][H dv], [n][H dk] twice, [chunks][H dk], [chunks][H][kC][kC], [chunks][H][dk][dv]
+    bool vec;                               // sizes and addresses allow 16-byte accesses throughout
     const int* start_pos;
 };
 
@@ -250,152 +251,229 @@ __device__ __forceinline__ bool find_chunk(const GlaArgs& a, int chunk, int& req
     return false;
 }
 
-// grid (chunk bound, heads, slices of kSl value channels).  Thread (cg, l): value channels 4 cg .. 4 cg + 3 of the
-// slice, key channels of lane l = tid % 16: (i * 16 + l) * W + j, i < DPT / W, j < W.
-// Shared memory: q, k, alpha [kTS][16 DPT], v [kTS][kSl], cumulative decay [16 DPT], cos / sin [kTS][rot],
-// gated: W2 [dk][R + 1], low [kTS][R].
-template <typename T, int DPT>
+__device__ __forceinline__ void cp_async16(float* smem, const float* gmem, bool valid) {
+    const unsigned dst = (unsigned)__cvta_generic_to_shared(smem);
+    const int bytes = valid ? 16 : 0;                     // 0: the 16 bytes are filled with zeros, nothing is read
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst), "l"(gmem), "r"(bytes));
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
+
+// grid (chunk bound, heads).  Thread (j, g): row j of the chunk as a key, key channels (i * 4 + g) * 4 + 0 .. 3,
+// i < DPT / 4.  Shared memory: k, then alpha [kC][4 DPT]; q [kC][4 DPT]; cos / sin [kTS][rot]; gated: W2 [dk][R + 1],
+// low [kC][R].
+template <typename T, int DPT, bool GATED>
 __global__ void __launch_bounds__(kThreads)
-local_kernel(const GlaArgs a) {
+chunk_kernel(const GlaArgs a) {
     extern __shared__ __align__(16) float sm[];
-    constexpr int W = DPT < 4 ? DPT : 4, P = 16 * DPT, NI = DPT / W;
+    constexpr int P = 4 * DPT;
     griddep_wait();
     griddep_launch();
-    const int tid = threadIdx.x, l = tid & 15, cg = tid >> 4, lane = tid & 31;
-    const int head = blockIdx.y, e0 = blockIdx.z * kSl, dk = a.dk, dv = a.dv, R = a.R, rot = a.rot, half = rot >> 1;
-    const int ne = min(kSl, dv - e0);
+    const int tid = threadIdx.x, j = tid >> 2, g = tid & 3, warp = tid >> 5;
+    const int head = blockIdx.y, dk = a.dk, R = a.R, rot = a.rot, half = rot >> 1;
     int req, row0, rows, index;
     if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
-    float* qs = sm;
-    float* ks = qs + kTS * P;
-    float* as = ks + kTS * P;
-    float* vs = as + kTS * P;
-    float* cum = vs + kTS * kSl;
-    float* cs = cum + P;
-    float* lows = cs + kTS * rot;
-    float* w2s = lows + kTS * R;
-    if (a.low) {
+    float* xs = sm;
+    float* qs = xs + kC * P;
+    float* cs = qs + kC * P;
+    float* w2s = cs + kTS * rot;
+    float* lows = w2s + (GATED ? dk * (R + 1) : 0);
+    if (GATED) {
         const T* w2 = reinterpret_cast<const T*>(a.w2) + (int64_t)head * dk * R;
         for (int i = tid; i < dk * R; i += kThreads) w2s[(i / R) * (R + 1) + i % R] = to_f32(w2[i]);
+        for (int i = tid; i < rows * R; i += kThreads) lows[i] = a.low[(int64_t)(row0 + i / R) * a.stride + i % R];
     }
-    for (int i = tid; i < P; i += kThreads) cum[i] = 1.f;
-    float S[4][DPT];
-#pragma unroll
-    for (int c = 0; c < 4; c++)
-#pragma unroll
-        for (int i = 0; i < DPT; i++) S[c][i] = 0.f;
-    const int A_w = a.heads * dk, B_w = a.heads * dv;
-    for (int b0 = 0; b0 < rows; b0 += kTS) {
-        const int nr = min(kTS, rows - b0), r0 = row0 + b0;
-        for (int i = tid; i < nr * half; i += kThreads) {
-            const int r = i / half, j = i - r * half;
-            double sn, c;
-            sincos((double)a.positions[r0 + r] * a.freq[j], &sn, &c);
-            cs[r * rot + j] = (float)c * a.amplitude;
-            cs[r * rot + half + j] = (float)sn * a.amplitude;
+    for (int b0 = 0; b0 < kC; b0 += kTS) {
+        const int nr = max(0, min(kTS, rows - b0));
+        if (rot) {
+            __syncthreads();                // the angles before have been used up
+            for (int i = tid; i < nr * half; i += kThreads) {
+                const int r = i / half, d = i - r * half;
+                double sn, c;
+                sincos((double)a.positions[row0 + b0 + r] * a.freq[d], &sn, &c);
+                cs[r * rot + d] = (float)c * a.amplitude;
+                cs[r * rot + half + d] = (float)sn * a.amplitude;
+            }
+            __syncthreads();
         }
-        if (a.low)
-            for (int i = tid; i < nr * R; i += kThreads) lows[i] = a.low[(int64_t)(r0 + i / R) * a.stride + i % R];
-        __syncthreads();                    // angles and low rows are there; the batch before has been used up
         for (int i = tid; i < kTS * P; i += kThreads) {
             const int r = i / P, d = i - r * P;
-            float q = 0.f, k = 0.f, al = 1.f;
+            float q = 0.f, k = 0.f;
             if (r < nr && d < dk) {
-                const int64_t off = (int64_t)(r0 + r) * a.stride + head * dk;
+                const int64_t off = (int64_t)(row0 + b0 + r) * a.stride + head * dk;
                 q = turned(a.q + off, d, rot, cs + r * rot) * a.q_scale;
                 k = turned(a.k + off, d, rot, cs + r * rot) * a.k_scale;
-                if (a.low) {
-                    float z = 0.f;
+            }
+            qs[b0 * P + i] = q;
+            xs[b0 * P + i] = k;
+        }
+    }
+    __syncthreads();
+    float w[DPT];
+#pragma unroll
+    for (int i = 0; i < DPT; i += 4) {
+        const float4 k4 = *reinterpret_cast<const float4*>(xs + j * P + (i + g) * 4);
+        w[i] = k4.x; w[i + 1] = k4.y; w[i + 2] = k4.z; w[i + 3] = k4.w;
+    }
+    const float fixed = GATED ? 1.f : a.decay[head];
+    if (GATED) {
+        __syncthreads();                    // everyone has its keys: their place takes the decays
+        for (int i = tid; i < rows * P; i += kThreads) {
+            const int r = i / P, d = i - r * P;
+            float al = 1.f;
+            if (d < dk) {
+                float z = 0.f;
 #pragma unroll 4
-                    for (int j = 0; j < R; j++) z = fmaf(lows[r * R + j], w2s[d * (R + 1) + j], z);
-                    al = gated_alpha(z + a.w2_bias[head * dk + d], a.inv_tau);
-                } else {
-                    al = a.decay[head];
-                }
+                for (int u = 0; u < R; u++) z = fmaf(lows[r * R + u], w2s[d * (R + 1) + u], z);
+                al = gated_alpha(z + a.w2_bias[head * dk + d], a.inv_tau);
             }
-            qs[i] = q;
-            ks[i] = k;
-            as[i] = al;
-        }
-        for (int i = tid; i < kTS * kSl; i += kThreads) {
-            const int r = i / kSl, c = i - r * kSl;
-            vs[i] = (r < nr && c < ne) ? a.v[(int64_t)(r0 + r) * a.stride + head * dv + e0 + c] : 0.f;
-        }
-        __syncthreads();
-        if (blockIdx.z == 0) {              // q_i A_i, once per (chunk, head)
-            for (int d = tid; d < dk; d += kThreads) {
-                float c = cum[d];
-                for (int r = 0; r < nr; r++) {
-                    c *= as[r * P + d];
-                    a.qa[(int64_t)(r0 + r) * A_w + head * dk + d] = qs[r * P + d] * c;
-                }
-                cum[d] = c;
-            }
-        }
-        // rows in fours (those beyond the batch have q = k = v = 0, alpha = 1 and change nothing)
-        for (int rb = 0; rb < nr; rb += 4) {
-            float acc[16];                  // [row of the four][value channel of the four]
-#pragma unroll
-            for (int p = 0; p < 4; p++) {
-                const int r = rb + p;
-                const float4 v4 = *reinterpret_cast<const float4*>(vs + r * kSl + cg * 4);
-                const float vv[4] = {v4.x, v4.y, v4.z, v4.w};
-#pragma unroll
-                for (int c = 0; c < 4; c++) acc[p * 4 + c] = 0.f;
-#pragma unroll
-                for (int i = 0; i < NI; i++) {
-                    const int d = r * P + (i * 16 + l) * W;
-                    float q[W], k[W], al[W];
-                    if constexpr (W == 4) {
-                        const float4 q4 = *reinterpret_cast<const float4*>(qs + d), k4 = *reinterpret_cast<const float4*>(ks + d),
-                                     a4 = *reinterpret_cast<const float4*>(as + d);
-                        q[0] = q4.x; q[1] = q4.y; q[2] = q4.z; q[3] = q4.w;
-                        k[0] = k4.x; k[1] = k4.y; k[2] = k4.z; k[3] = k4.w;
-                        al[0] = a4.x; al[1] = a4.y; al[2] = a4.z; al[3] = a4.w;
-                    } else {
-#pragma unroll
-                        for (int j = 0; j < W; j++) { q[j] = qs[d + j]; k[j] = ks[d + j]; al[j] = as[d + j]; }
-                    }
-#pragma unroll
-                    for (int j = 0; j < W; j++)
-#pragma unroll
-                        for (int c = 0; c < 4; c++) {
-                            float& s = S[c][i * W + j];
-                            s = fmaf(al[j], s, k[j] * vv[c]);
-                            acc[p * 4 + c] = fmaf(q[j], s, acc[p * 4 + c]);
-                        }
-                }
-            }
-            // sixteen sums over sixteen lanes by halving: lane l ends with the sum number l
-#pragma unroll
-            for (int o = 8; o >= 1; o >>= 1) {
-                const bool upper = (lane & o) != 0;
-#pragma unroll
-                for (int j = 0; j < o; j++) {
-                    const float send = upper ? acc[j] : acc[j + o];
-                    const float keep = upper ? acc[j + o] : acc[j];
-                    acc[j] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-                }
-            }
-            const int r = rb + (l >> 2), c = cg * 4 + (l & 3);
-            if (r < nr && c < ne) a.o[(int64_t)(r0 + r) * B_w + head * dv + e0 + c] = acc[0];
+            xs[i] = al;
         }
         __syncthreads();
     }
-    if (blockIdx.z == 0)
-        for (int d = tid; d < dk; d += kThreads) a.a_last[(int64_t)blockIdx.x * A_w + head * dk + d] = cum[d];
-    float* dst = a.s_in + ((int64_t)blockIdx.x * a.heads + head) * dk * dv + e0 + cg * 4;
-    const bool whole = (dv & 3) == 0 && cg * 4 + 4 <= ne;
+    const int A_w = a.heads * dk;
+    // q_i A_i and A_last, by the half of the threads whose keys have the fewer rows behind them
+    if (tid >= kThreads / 2) {
+        for (int d = tid - kThreads / 2; d < dk; d += kThreads / 2) {
+            float c = 1.f;
+            for (int r = 0; r < rows; r++) {
+                c *= GATED ? xs[r * P + d] : fixed;
+                a.qa[(int64_t)(row0 + r) * A_w + head * dk + d] = qs[r * P + d] * c;
+            }
+            a.a_last[(int64_t)blockIdx.x * A_w + head * dk + d] = c;
+        }
+    }
+    float* Wr = a.w + ((int64_t)blockIdx.x * a.heads + head) * kC * kC + j;
+    const int jmin = warp * 8, jmax = jmin + 7;
+    if (g == 0)
+        for (int i = 0; i < min(jmin, rows); i++) Wr[i * kC] = 0.f;
+    for (int i = jmin; i < rows; i++) {
+        float acc = 0.f, acc2 = 0.f;
+        const bool on = i > j;
 #pragma unroll
-    for (int i = 0; i < DPT; i++) {
-        const int d = (i / W * 16 + l) * W + i % W;
-        if (d >= dk) continue;
-        if (whole) {
-            *reinterpret_cast<float4*>(dst + (int64_t)d * dv) = make_float4(S[0][i], S[1][i], S[2][i], S[3][i]);
+        for (int u = 0; u < DPT; u += 4) {
+            const float4 q4 = *reinterpret_cast<const float4*>(qs + i * P + (u + g) * 4);
+            float4 al = make_float4(fixed, fixed, fixed, fixed);
+            if (GATED) al = *reinterpret_cast<const float4*>(xs + i * P + (u + g) * 4);
+            if (i > jmax) {                 // the same for the whole warp
+                w[u] *= al.x; w[u + 1] *= al.y; w[u + 2] *= al.z; w[u + 3] *= al.w;
+            } else if (on) {
+                w[u] *= al.x; w[u + 1] *= al.y; w[u + 2] *= al.z; w[u + 3] *= al.w;
+            }
+            acc = fmaf(q4.x, w[u], acc);
+            acc2 = fmaf(q4.y, w[u + 1], acc2);
+            acc = fmaf(q4.z, w[u + 2], acc);
+            acc2 = fmaf(q4.w, w[u + 3], acc2);
+        }
+        acc += acc2;
+        acc += __shfl_xor_sync(0xffffffffu, acc, 1);
+        acc += __shfl_xor_sync(0xffffffffu, acc, 2);
+        if (g == 0) Wr[i * kC] = i >= j ? acc : 0.f;
+    }
+    if (j < rows) {
+        float* dst = a.kd + (int64_t)(row0 + j) * A_w + head * dk;
+#pragma unroll
+        for (int i = 0; i < DPT; i += 4) {
+            const int d = (i + g) * 4;
+            if (a.vec) {
+                if (d < dk) *reinterpret_cast<float4*>(dst + d) = make_float4(w[i], w[i + 1], w[i + 2], w[i + 3]);
+            } else {
+#pragma unroll
+                for (int u = 0; u < 4; u++)
+                    if (d + u < dk) dst[d + u] = w[i + u];
+            }
+        }
+    }
+}
+
+// N consecutive values of shared memory as the register tile of thread `t` of 16: fours at 64 u + 4 t (N 4, 8), or two at 2 t
+template <int N> __device__ __forceinline__ int tile_at(int t, int i) { return N == 2 ? 2 * t + i : (i >> 2) * 64 + 4 * t + (i & 3); }
+
+// grid (chunk bound, heads, tiles of 16 RM key channels by 16 RN value channels): s_in = sum over the chunk's rows of
+// kd_j v_j^T.  Thread (ty, tx): an RM x RN tile.  Shared memory: kd [kC][16 RM], v [kC][16 RN].
+template <int RM, int RN>
+__global__ void __launch_bounds__(kThreads)
+outer_kernel(const GlaArgs a, int e_tiles) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int TM = 16 * RM, TN = 16 * RN;
+    griddep_wait();
+    griddep_launch();
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    const int head = blockIdx.y, d0 = blockIdx.z / e_tiles * TM, e0 = blockIdx.z % e_tiles * TN, dk = a.dk, dv = a.dv;
+    int req, row0, rows, index;
+    if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
+    float* ks = sm;
+    float* vs = ks + kC * TM;
+    const int A_w = a.heads * dk;
+    const float* kg = a.kd + (int64_t)row0 * A_w + head * dk + d0;
+    const float* vg = a.v + (int64_t)row0 * a.stride + head * dv + e0;
+    if (a.vec) {
+        for (int i = tid; i < rows * (TM / 4); i += kThreads) {
+            const int r = i / (TM / 4), d = (i - r * (TM / 4)) * 4;
+            cp_async16(ks + r * TM + d, kg + (d0 + d < dk ? (int64_t)r * A_w + d : 0), d0 + d < dk);
+        }
+        for (int i = tid; i < rows * (TN / 4); i += kThreads) {
+            const int r = i / (TN / 4), c = (i - r * (TN / 4)) * 4;
+            cp_async16(vs + r * TN + c, vg + (e0 + c < dv ? (int64_t)r * a.stride + c : 0), e0 + c < dv);
+        }
+        cp_async_commit();
+        cp_async_wait<0>();
+    } else {
+        for (int i = tid; i < rows * TM; i += kThreads) {
+            const int r = i / TM, d = i - r * TM;
+            ks[i] = d0 + d < dk ? kg[(int64_t)r * A_w + d] : 0.f;
+        }
+        for (int i = tid; i < rows * TN; i += kThreads) {
+            const int r = i / TN, c = i - r * TN;
+            vs[i] = e0 + c < dv ? vg[(int64_t)r * a.stride + c] : 0.f;
+        }
+    }
+    __syncthreads();
+    float acc[RM][RN];
+#pragma unroll
+    for (int m = 0; m < RM; m++)
+#pragma unroll
+        for (int n = 0; n < RN; n++) acc[m][n] = 0.f;
+#pragma unroll 2
+    for (int r = 0; r < rows; r++) {
+        float k[RM], v[RN];
+        if constexpr (RM == 2) {
+            const float2 t = *reinterpret_cast<const float2*>(ks + r * TM + 2 * ty);
+            k[0] = t.x; k[1] = t.y;
         } else {
 #pragma unroll
-            for (int c = 0; c < 4; c++)
-                if (cg * 4 + c < ne) dst[(int64_t)d * dv + c] = S[c][i];
+            for (int u = 0; u < RM / 4; u++) {
+                const float4 t = *reinterpret_cast<const float4*>(ks + r * TM + u * 64 + 4 * ty);
+                k[4 * u] = t.x; k[4 * u + 1] = t.y; k[4 * u + 2] = t.z; k[4 * u + 3] = t.w;
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < RN / 4; u++) {
+            const float4 t = *reinterpret_cast<const float4*>(vs + r * TN + u * 64 + 4 * tx);
+            v[4 * u] = t.x; v[4 * u + 1] = t.y; v[4 * u + 2] = t.z; v[4 * u + 3] = t.w;
+        }
+#pragma unroll
+        for (int m = 0; m < RM; m++)
+#pragma unroll
+            for (int n = 0; n < RN; n++) acc[m][n] = fmaf(k[m], v[n], acc[m][n]);
+    }
+    float* S = a.s_in + ((int64_t)blockIdx.x * a.heads + head) * dk * dv;
+#pragma unroll
+    for (int m = 0; m < RM; m++) {
+        const int d = d0 + tile_at<RM>(ty, m);
+        if (d >= dk) continue;
+#pragma unroll
+        for (int u = 0; u < RN / 4; u++) {
+            const int e = e0 + u * 64 + 4 * tx;
+            if (a.vec) {
+                if (e < dv)
+                    *reinterpret_cast<float4*>(S + (int64_t)d * dv + e) =
+                        make_float4(acc[m][4 * u], acc[m][4 * u + 1], acc[m][4 * u + 2], acc[m][4 * u + 3]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < 4; i++)
+                    if (e + i < dv) S[(int64_t)d * dv + e + i] = acc[m][4 * u + i];
+            }
         }
     }
 }
@@ -440,14 +518,17 @@ carry_kernel(const GlaArgs a) {
     store_vec<V>(slot, s);
 }
 
-// grid (chunk bound, heads, column blocks of 64 NJ).  Thread (rg, cg): rows 4 rg .. 4 rg + 3, value channels
-// j * 64 + 4 cg .. + 3.  NORM: the columns are all of the head's (grid.z is 1) and the row is normed, gated and stored
-// in y; otherwise o is written back.  Shared memory: q A [kC][36], S [32][64 NJ].
+// grid (chunk bound, heads, column blocks of 64 NJ): o = [q A | W] [S_in ; v], in blocks of kKB inner elements, two of them
+// in shared memory.  Thread (rg, cg): rows 4 rg .. 4 rg + 3, value channels j * 64 + 4 cg .. + 3.  NORM: the columns are all
+// of the head's (grid.z is 1) and the row is normed, gated and stored in y; otherwise o is stored.
+// Shared memory, twice: left [kC][kKB + 4], right [kKB][64 NJ].
+constexpr int kKB = 32;
+
 template <typename T, int NJ, bool NORM>
 __global__ void __launch_bounds__(kThreads)
 apply_kernel(const GlaArgs a) {
     extern __shared__ __align__(16) float sm[];
-    constexpr int DB = 32, QP = DB + 4, CW = 64 * NJ;
+    constexpr int QP = kKB + 4, CW = 64 * NJ, STAGE = kC * QP + kKB * CW;
     griddep_wait();
     griddep_launch();
     const int tid = threadIdx.x, cg = tid & 15, rg = tid >> 4;
@@ -455,38 +536,60 @@ apply_kernel(const GlaArgs a) {
     const int ne = min(CW, dv - e0);
     int req, row0, rows, index;
     if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
-    float* qs = sm;                         // [kC][QP]
-    float* ss = qs + kC * QP;               // [DB][CW]
     float acc[4][NJ * 4];
 #pragma unroll
     for (int r = 0; r < 4; r++)
 #pragma unroll
         for (int j = 0; j < NJ * 4; j++) acc[r][j] = 0.f;
     const int A_w = a.heads * dk, B_w = a.heads * dv;
-    const float* S = a.s_in + ((int64_t)blockIdx.x * a.heads + head) * dk * dv + e0;
     const bool from_zero = index == 0 && a.start_pos[req] == 0;        // the state in front of a request's first chunk
-    for (int d0 = 0; d0 < dk && !from_zero; d0 += DB) {
-        const int nd = min(DB, dk - d0);
-        __syncthreads();
-        for (int i = tid; i < kC * DB; i += kThreads) {
-            const int r = i / DB, d = i - r * DB;
-            qs[r * QP + d] = (r < rows && d < nd) ? a.qa[(int64_t)(row0 + r) * A_w + head * dk + d0 + d] : 0.f;
-        }
-        if ((dv & 3) == 0) {
-            for (int i = tid; i < DB * CW / 4; i += kThreads) {
-                const int d = i / (CW / 4), c = (i - d * (CW / 4)) * 4;
-                *reinterpret_cast<float4*>(ss + d * CW + c) =
-                    (d < nd && c < ne) ? *reinterpret_cast<const float4*>(S + (int64_t)(d0 + d) * dv + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const int nb_s = from_zero ? 0 : (dk + kKB - 1) / kKB, nb = nb_s + (rows + kKB - 1) / kKB;
+    const float* S = a.s_in + ((int64_t)blockIdx.x * a.heads + head) * dk * dv + e0;
+    const float* W = a.w + ((int64_t)blockIdx.x * a.heads + head) * kC * kC;
+    auto load = [&](int b) {                // inner elements k0 .. k0 + kKB - 1 of the state's part, then of the chunk's own
+        float* left = sm + (b & 1) * STAGE;
+        float* right = left + kC * QP;
+        const bool state = b < nb_s;
+        const int k0 = (state ? b : b - nb_s) * kKB, nk = min(kKB, (state ? dk : rows) - k0);
+        const float* lg = state ? a.qa + (int64_t)row0 * A_w + head * dk + k0 : W + k0;
+        const float* rg_ = state ? S + (int64_t)k0 * dv : a.v + (int64_t)(row0 + k0) * a.stride + head * dv + e0;
+        const int64_t ls = state ? A_w : kC, rs = state ? dv : a.stride;
+        if (a.vec) {
+            for (int i = tid; i < kC * (kKB / 4); i += kThreads) {
+                const int r = i / (kKB / 4), k = (i - r * (kKB / 4)) * 4;
+                const bool in = r < rows && (state ? k < nk : true);      // W's rows are whole: zeros beyond the diagonal
+                cp_async16(left + r * QP + k, lg + (in ? r * ls + k : 0), in);
+            }
+            for (int i = tid; i < kKB * (CW / 4); i += kThreads) {
+                const int k = i / (CW / 4), c = (i - k * (CW / 4)) * 4;
+                const bool in = k < nk && c < ne;
+                cp_async16(right + k * CW + c, rg_ + (in ? k * rs + c : 0), in);
             }
         } else {
-            for (int i = tid; i < DB * CW; i += kThreads) {
-                const int d = i / CW, c = i - d * CW;
-                ss[i] = (d < nd && c < ne) ? S[(int64_t)(d0 + d) * dv + c] : 0.f;
+            for (int i = tid; i < kC * kKB; i += kThreads) {
+                const int r = i / kKB, k = i - r * kKB;
+                left[r * QP + k] = (r < rows && k < nk) ? lg[r * ls + k] : 0.f;
+            }
+            for (int i = tid; i < kKB * CW; i += kThreads) {
+                const int k = i / CW, c = i - k * CW;
+                right[i] = (k < nk && c < ne) ? rg_[k * rs + c] : 0.f;
             }
         }
+        cp_async_commit();
+    };
+    load(0);
+    for (int b = 0; b < nb; b++) {
+        if (b + 1 < nb) {
+            load(b + 1);
+            cp_async_wait<1>();
+        } else {
+            cp_async_wait<0>();
+        }
         __syncthreads();
+        const float* qs = sm + (b & 1) * STAGE;
+        const float* ss = qs + kC * QP;
 #pragma unroll 2
-        for (int d = 0; d < DB; d += 4) {
+        for (int d = 0; d < kKB; d += 4) {
             float q[4][4];
 #pragma unroll
             for (int r = 0; r < 4; r++) {
@@ -507,20 +610,19 @@ apply_kernel(const GlaArgs a) {
                     }
                 }
         }
+        __syncthreads();                    // this stage may be loaded again
     }
 #pragma unroll
     for (int r = 0; r < 4; r++) {
         const int row = rg * 4 + r;
-        float* orow = a.o + (int64_t)(row0 + min(row, rows - 1)) * B_w + head * dv + e0;
         float sq = 0.f;
 #pragma unroll
         for (int j = 0; j < NJ; j++)
 #pragma unroll
             for (int c = 0; c < 4; c++) {
                 const int col = j * 64 + cg * 4 + c;
-                float& x = acc[r][j * 4 + c];
-                x = col < ne ? x + orow[col] : 0.f;
-                sq += x * x;
+                if (col >= ne) acc[r][j * 4 + c] = 0.f;
+                sq += acc[r][j * 4 + c] * acc[r][j * 4 + c];
             }
         if constexpr (NORM) {
 #pragma unroll
@@ -538,6 +640,7 @@ apply_kernel(const GlaArgs a) {
                     }
             }
         } else if (row < rows) {
+            float* orow = a.o + (int64_t)(row0 + row) * B_w + head * dv + e0;
 #pragma unroll
             for (int j = 0; j < NJ; j++)
 #pragma unroll
@@ -610,42 +713,70 @@ int launch_step(const GlaArgs& a, bool early, cudaStream_t s) {
     KLLM_LAUNCH_STATUS();
 }
 
-template <typename T, int DPT>
-int launch_local(const GlaArgs& a, int chunk_bound, cudaStream_t s) {
-    const size_t smem = sizeof(float) * ((size_t)3 * kTS * 16 * DPT + kTS * kSl + 16 * DPT + (size_t)kTS * a.rot +
-                                         (a.low ? (size_t)kTS * a.R + (size_t)a.dk * (a.R + 1) : 0));
-    if (smem > 200 * 1024) KLLM_FAIL("gla: a head of %d key channels with a decay of rank %d does not fit shared memory", a.dk, a.R);
-    auto kern = local_kernel<T, DPT>;
+template <typename K>
+int raise_smem(K kern, bool& raised) {
+    if (raised) return 0;
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+    if (e != cudaSuccess) KLLM_FAIL("gla: %s", cudaGetErrorString(e));
+    raised = true;
+    return 0;
+}
+
+template <typename T, int DPT, bool GATED>
+int launch_chunk(const GlaArgs& a, int chunk_bound, cudaStream_t s) {
+    const size_t smem = sizeof(float) * ((size_t)2 * kC * 4 * DPT + (size_t)kTS * a.rot +
+                                         (GATED ? (size_t)kC * a.R + (size_t)a.dk * (a.R + 1) : 0));
+    if (smem > 220 * 1024) KLLM_FAIL("gla: a head of %d key channels with a decay of rank %d does not fit shared memory", a.dk, a.R);
     static bool raised = false;
-    if (!raised) {
-        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        if (e != cudaSuccess) KLLM_FAIL("gla: %s", cudaGetErrorString(e));
-        raised = true;
-    }
-    kllm_launch_dep(false, (kern), dim3(chunk_bound, a.heads, (a.dv + kSl - 1) / kSl), dim3(kThreads), smem, s, a);
+    int rc = raise_smem(chunk_kernel<T, DPT, GATED>, raised);
+    if (rc) return rc;
+    kllm_launch_dep(false, (chunk_kernel<T, DPT, GATED>), dim3(chunk_bound, a.heads), dim3(kThreads), smem, s, a);
+    KLLM_LAUNCH_STATUS();
+}
+
+template <typename T, int DPT>
+int launch_chunk(const GlaArgs& a, int chunk_bound, cudaStream_t s) {
+    return a.low ? launch_chunk<T, DPT, true>(a, chunk_bound, s) : launch_chunk<T, DPT, false>(a, chunk_bound, s);
+}
+
+template <int RM, int RN>
+int launch_outer(const GlaArgs& a, int chunk_bound, cudaStream_t s) {
+    const int e_tiles = (a.dv + 16 * RN - 1) / (16 * RN), d_tiles = (a.dk + 16 * RM - 1) / (16 * RM);
+    static bool raised = false;
+    int rc = raise_smem(outer_kernel<RM, RN>, raised);
+    if (rc) return rc;
+    kllm_launch_dep(false, (outer_kernel<RM, RN>), dim3(chunk_bound, a.heads, e_tiles * d_tiles), dim3(kThreads),
+                    sizeof(float) * kC * 16 * (RM + RN), s, a, e_tiles);
     KLLM_LAUNCH_STATUS();
 }
 
 template <typename T, int NJ, bool NORM>
 int launch_apply(const GlaArgs& a, int chunk_bound, cudaStream_t s) {
-    const size_t smem = sizeof(float) * (kC * 36 + 32 * 64 * NJ);
+    const size_t smem = sizeof(float) * 2 * (kC * (kKB + 4) + kKB * 64 * NJ);
+    static bool raised = false;
+    int rc = raise_smem(apply_kernel<T, NJ, NORM>, raised);
+    if (rc) return rc;
     kllm_launch_dep(false, (apply_kernel<T, NJ, NORM>), dim3(chunk_bound, a.heads, NORM ? 1 : (a.dv + 64 * NJ - 1) / (64 * NJ)),
                     dim3(kThreads), smem, s, a);
     KLLM_LAUNCH_STATUS();
 }
 
 template <typename T>
-int run(const GlaArgs& a, int n, bool single, bool early, int chunk_bound, cudaStream_t s) {
-    const bool vec = a.dv % 4 == 0 && a.stride % 4 == 0 && a.state_stride % 4 == 0 &&
-                     !(((uintptr_t)a.state | (uintptr_t)a.v | (uintptr_t)a.s_in) & 15);
-    if (single) return vec ? launch_step<T, 4>(a, early, s) : launch_step<T, 1>(a, early, s);
-    if (a.dv % 4 == 0 && ((uintptr_t)a.s_in & 15)) KLLM_FAIL("gla: the work buffer must be 16-byte aligned");
+int run(GlaArgs a, int n, bool single, bool early, int chunk_bound, cudaStream_t s) {
+    const bool rows_vec = a.dv % 4 == 0 && a.stride % 4 == 0 && a.state_stride % 4 == 0 &&
+                          !(((uintptr_t)a.state | (uintptr_t)a.v) & 15);
+    if (single) return rows_vec ? launch_step<T, 4>(a, early, s) : launch_step<T, 1>(a, early, s);
+    a.vec = rows_vec && a.dk % 4 == 0 && !(((uintptr_t)a.s_in | (uintptr_t)a.qa | (uintptr_t)a.kd | (uintptr_t)a.w) & 15);
+    const bool vec = a.vec;
     int rc;
-    if (a.dk <= 16) rc = launch_local<T, 1>(a, chunk_bound, s);
-    else if (a.dk <= 32) rc = launch_local<T, 2>(a, chunk_bound, s);
-    else if (a.dk <= 64) rc = launch_local<T, 4>(a, chunk_bound, s);
-    else if (a.dk <= 128) rc = launch_local<T, 8>(a, chunk_bound, s);
-    else rc = launch_local<T, 16>(a, chunk_bound, s);
+    if (a.dk <= 32) rc = launch_chunk<T, 8>(a, chunk_bound, s);
+    else if (a.dk <= 64) rc = launch_chunk<T, 16>(a, chunk_bound, s);
+    else if (a.dk <= 128) rc = launch_chunk<T, 32>(a, chunk_bound, s);
+    else rc = launch_chunk<T, 64>(a, chunk_bound, s);
+    if (rc) return rc;
+    if (a.dk <= 32) rc = a.dv <= 64 ? launch_outer<2, 4>(a, chunk_bound, s) : launch_outer<2, 8>(a, chunk_bound, s);
+    else if (a.dk <= 64) rc = a.dv <= 64 ? launch_outer<4, 4>(a, chunk_bound, s) : launch_outer<4, 8>(a, chunk_bound, s);
+    else rc = a.dv <= 64 ? launch_outer<8, 4>(a, chunk_bound, s) : launch_outer<8, 8>(a, chunk_bound, s);
     if (rc) return rc;
     const int64_t elems = (int64_t)a.dk * a.dv;
     if (vec)
@@ -674,8 +805,8 @@ extern "C" int kllm_gla_chunk_rows() { return kC; }
 // stride `stride`; w2 [heads * dk][R] in the element type `dtype`, w2_bias float32 [heads * dk]; decay float32 [heads];
 // freq double [rot / 2] or null; state float32 [slots][state_stride] whose first heads * dk * dv values are S as
 // [heads][dk][dv]; gain float32 [heads * dv]; y in `dtype` at row stride y_stride.  single: every request brings one
-// row; otherwise the work buffers o [n][heads dv], qa [n][heads dk], a_last [chunk_bound][heads dk], s_in
-// [chunk_bound][heads][dk][dv] are float32 and chunk_bound an upper bound of the chunks (sum over requests of
+// row; otherwise the work buffers qa, kd [n][heads dk], a_last [chunk_bound][heads dk], w [chunk_bound][heads][C][C] (C:
+// rows of a chunk), s_in [chunk_bound][heads][dk][dv] and, for dv above 256, o [n][heads dv] are float32 and chunk_bound an upper bound of the chunks (sum over requests of
 // ceil(rows / kllm_gla_chunk_rows())).  early (single): the kernel may start beside the end of the one before it in the
 // stream, which must not write the state.
 extern "C" int kllm_gla(void* y, int64_t y_stride, const float* q, const float* k, const float* v, const float* g, int64_t stride,
@@ -683,7 +814,7 @@ extern "C" int kllm_gla(void* y, int64_t y_stride, const float* q, const float* 
                         const double* freq, int rot, float amplitude, float q_scale, float k_scale, const int* positions,
                         const int* q_start, const int* start_pos, const int* state_slots, float* state, int64_t state_stride,
                         const float* gain, float eps, int n, int n_requests, int heads, int dk, int dv, int single,
-                        int early, int chunk_bound, float* o, float* qa, float* a_last, float* s_in, int dtype, void* stream) {
+                        int early, int chunk_bound, float* o, float* qa, float* kd, float* a_last, float* w, float* s_in, int dtype, void* stream) {
     if (n <= 0 || n_requests <= 0) return 0;
     if (heads <= 0 || dk <= 0 || dk > 256 || dv <= 0) KLLM_FAIL("gla: %d heads of sizes %d (up to 256), %d", heads, dk, dv);
     if (heads > 65535 || n_requests > 65535) KLLM_FAIL("gla: %d heads, %d requests in one launch", heads, n_requests);
@@ -691,13 +822,13 @@ extern "C" int kllm_gla(void* y, int64_t y_stride, const float* q, const float* 
     if (low ? (!w2 || !w2_bias || R <= 0) : !decay) KLLM_FAIL("gla: a decay needs its matrix and bias, or one number per head");
     if (state_stride < (int64_t)heads * dk * dv) KLLM_FAIL("gla: a state slot of %lld values is too small", (long long)state_stride);
     if (single && n != n_requests) KLLM_FAIL("gla: %d rows of %d requests that bring one row each", n, n_requests);
-    if (!single && (!o || !qa || !a_last || !s_in || chunk_bound <= 0)) KLLM_FAIL("gla: portions need work buffers");
+    if (!single && (!qa || !kd || !a_last || !w || !s_in || (dv > 256 && !o) || chunk_bound <= 0)) KLLM_FAIL("gla: portions need work buffers");
     GlaArgs a;
     a.q = q; a.k = k; a.v = v; a.g = g; a.stride = stride; a.low = low; a.w2 = w2; a.w2_bias = w2_bias; a.R = low ? R : 0;
     a.inv_tau = inv_tau; a.decay = decay; a.freq = freq; a.rot = rot; a.amplitude = amplitude; a.q_scale = q_scale;
     a.k_scale = k_scale; a.positions = positions; a.q_start = q_start; a.state_slots = state_slots; a.n_requests = n_requests;
     a.heads = heads; a.dk = dk; a.dv = dv; a.state = state; a.state_stride = state_stride; a.gain = gain; a.eps = eps; a.y = y;
-    a.y_stride = y_stride; a.o = o; a.qa = qa; a.a_last = a_last; a.s_in = s_in; a.start_pos = start_pos;
+    a.y_stride = y_stride; a.o = o; a.qa = qa; a.kd = kd; a.a_last = a_last; a.w = w; a.s_in = s_in; a.vec = false; a.start_pos = start_pos;
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == KLLM_F32) return run<float>(a, n, single != 0, early != 0, chunk_bound, s);
     if (dtype == KLLM_BF16) return run<bf16>(a, n, single != 0, early != 0, chunk_bound, s);

@@ -656,13 +656,28 @@ def attention(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: 
             and vd % 16 == 0 and 16 <= vd <= 256 and group <= 64 and not (special and scale <= 0)
             and vcache.dim() == 4 and vcache.shape[3] % 8 == 0)
     short = min(int(segment or (1 << 30)), int(window or (1 << 30))) <= WIDE_SINGLE_KEYS
+    # the decode kernel takes 16 heads per CTA: more heads on a kv head are cut into groups of equal size
+    groups = n_kv * next((s for s in range(1, group + 1) if group % s == 0 and group // s <= 16), 1)
+    # single tokens of the wide form: the decode kernel where the values have a plain store of their own size
+    wide_decode = wide and not segment and plain_values
+
+    def decode(singles, bound):
+        # token t of the first `singles` is request t: no token-to-request table needed
+        attention_decode(out[:singles], q[:singles], kcache, vcache, ctx.positions[:singles], None, block_table[:singles],
+                         n_heads, n_kv, head_dim, window, scale,
+                         decode_splits(singles, groups, min(bound, window or (1 << 30))), slopes=score_slopes,
+                         split_weights=exact_weights, sinks=sinks, v_head_dim=vd)
     if wide and not short and (ctx.all_single or not ctx.host_n_new):
+        if wide_decode and ctx.all_single:
+            return decode(ctx.n_tokens, ctx.split_bound or ctx.max_ctx)
         wide = False
     if wide:
         singles = 0
         while not short and singles < ctx.n_requests and ctx.host_n_new[singles] == 1:
             singles += 1
-        if singles:
+        if singles and wide_decode:
+            decode(singles, ctx.max_ctx)
+        elif singles:
             if not simt_fits(q, n_heads, n_kv, head_dim, vd):
                 wide = False
             else:
@@ -682,8 +697,6 @@ def attention(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: 
                                      head_dim, window, scale, score_slopes, vd, sinks, segment)
         return attention_simt(out, q, kcache, vcache, ctx, block_table, n_heads, n_kv, head_dim, window, scale,
                               score_slopes, vd, sinks, segment)
-    # the decode kernel takes 16 heads per CTA: more heads on a kv head are cut into groups of equal size
-    groups = n_kv * next(s for s in range(1, group + 1) if group % s == 0 and group // s <= 16)
     if tc and ctx.all_single and group <= 64:
         return attention_decode(out, q, kcache, vcache, ctx.positions, ctx.token_req, block_table, n_heads,
                                 n_kv, head_dim, window, scale,
@@ -694,11 +707,7 @@ def attention(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: 
         while singles < ctx.n_requests and ctx.host_n_new[singles] == 1:
             singles += 1
     if 0 < singles < ctx.n_requests:
-        # token t of the first `singles` is request t: no token-to-request table needed
-        attention_decode(out[:singles], q[:singles], kcache, vcache, ctx.positions[:singles], None,
-                         block_table[:singles], n_heads, n_kv, head_dim, window, scale,
-                         decode_splits(singles, groups, min(ctx.max_ctx, window or (1 << 30))), slopes=score_slopes,
-                         split_weights=exact_weights, sinks=sinks)
+        decode(singles, ctx.max_ctx)
     q_start, start_pos, table, n_req = ctx.q_start, ctx.start_pos, block_table, ctx.n_requests
     if 0 < singles < ctx.n_requests:
         q_start, start_pos, table, n_req = q_start[singles:], start_pos[singles:], block_table[singles:], n_req - singles
@@ -717,12 +726,13 @@ def attention(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: 
                              head_dim, window, scale)
 
 
-def _check_attention(out, q, kcache, vcache, block_table, n_kv, head_dim):
+def _check_attention(out, q, kcache, vcache, block_table, n_kv, head_dim, vd=None):
     if q.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or kcache.dtype != torch.bfloat16:
         raise KernelError("tensor-core attention takes bfloat16 operands")
     if q.stride(1) != 1 or not out.is_contiguous() or not kcache.is_contiguous() or not vcache.is_contiguous():
         raise KernelError("attention: out and caches contiguous, q rows dense")
-    if kcache.shape[1] != n_kv or kcache.shape[3] != head_dim or kcache.shape != vcache.shape:
+    if kcache.shape[1] != n_kv or kcache.shape[3] != head_dim or vcache.shape[3] != (vd or head_dim) \
+            or kcache.shape[:3] != vcache.shape[:3]:
         raise KernelError("attention: cache layout must be [pages, n_kv, page_size, head_dim]")
     _i32(block_table, "block_table")
 
@@ -735,21 +745,26 @@ def _slopes_arg(slopes, n_heads, what="score slopes"):
 
 def attention_decode(out, q, kcache, vcache, positions, token_req, block_table, n_heads, n_kv, head_dim,
                      window, scale, num_splits: int, slopes: Optional[torch.Tensor] = None,
-                     split_weights: bool = False, sinks: Optional[torch.Tensor] = None) -> None:
+                     split_weights: bool = False, sinks: Optional[torch.Tensor] = None,
+                     v_head_dim: Optional[int] = None) -> None:
     """Tensor-core decode attention: every token attends on its own, its keys cut
     into ``num_splits`` ranges that are merged in a fixed order.  ``slopes`` (float32 [heads]):
     slope[h] * (key position - query position) is added to the scaled scores; ``split_weights``:
     the probabilities enter the second product as two bfloat16 terms instead of one; ``sinks``
-    (float32 [heads]): exp(sinks[h]) joins the denominator of head h's softmax."""
+    (float32 [heads]): exp(sinks[h]) joins the denominator of head h's softmax; ``v_head_dim``: values of another
+    size than the keys (a library of its own per pair of sizes)."""
     _cuda(out, q, kcache, vcache, positions, token_req, block_table, slopes, sinks)
-    _check_attention(out, q, kcache, vcache, block_table, n_kv, head_dim)
+    vd = int(v_head_dim or head_dim)
+    _check_attention(out, q, kcache, vcache, block_table, n_kv, head_dim, vd)
+    if out.shape[1] != n_heads * vd:
+        raise KernelError("attention: out must be [n, heads * value size]")
     _i32(positions, "positions"); _i32(token_req, "token_req")
     n = q.shape[0]
     part_o = part_ml = None
     if num_splits > 1:
-        part_o = torch.empty((n, n_heads, num_splits, head_dim), dtype=torch.float32, device=q.device)
+        part_o = torch.empty((n, n_heads, num_splits, vd), dtype=torch.float32, device=q.device)
         part_ml = torch.empty((n, n_heads, num_splits, 2), dtype=torch.float32, device=q.device)
-    lib = load_library("attention_tc", {"KLLM_HD": head_dim})
+    lib = load_library("attention_tc", {"KLLM_HD": head_dim} if vd == head_dim else {"KLLM_HD": head_dim, "KLLM_VD": vd})
     rc = lib.kllm_attention_decode(_p(out), _p(part_o), _p(part_ml), _p(q), ctypes.c_int64(q.stride(0)),
                                    _p(kcache), _p(vcache), _p(positions), _p(token_req), _p(block_table),
                                    block_table.shape[1], n, n_heads, n_kv, head_dim, kcache.shape[2],
@@ -1561,24 +1576,27 @@ def gla(y: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: t
     _i32(ctx.q_start, "q_start"); _i32(ctx.state_slots, "state_slots"); _i32(ctx.positions, "positions")
     _i32(ctx.start_pos, "start_pos")
     lib = load_library("gla")
-    o = qa = a_last = s_in = None
+    o = qa = kd = a_last = w = s_in = None
     bound = 0
     if not ctx.all_single:
         f32 = dict(dtype=torch.float32, device=q.device)
-        bound = n // lib.kllm_gla_chunk_rows() + ctx.n_requests
-        o, qa = torch.empty((n, heads * dv), **f32), torch.empty((n, heads * dk), **f32)
+        C = lib.kllm_gla_chunk_rows()
+        bound = n // C + ctx.n_requests
+        qa, kd = torch.empty((n, heads * dk), **f32), torch.empty((n, heads * dk), **f32)
         a_last, s_in = torch.empty((bound, heads * dk), **f32), torch.empty((bound, heads, dk, dv), **f32)
+        w = torch.empty((bound, heads, C, C), **f32)
+        o = torch.empty((n, heads * dv), **f32) if dv > 256 else None
     rc = lib.kllm_gla(_p(y), ctypes.c_int64(y.stride(0)), _p(q), _p(k), _p(v), _p(g), ctypes.c_int64(q.stride(0)), _p(low),
                       _p(w2), _p(w2_bias), R, ctypes.c_float(1.0 / tau), _p(decay), _p(freq),
                       2 * freq.numel() if freq is not None else 0, ctypes.c_float(amplitude), ctypes.c_float(q_scale),
                       ctypes.c_float(k_scale), _p(ctx.positions), _p(ctx.q_start), _p(ctx.start_pos), _p(ctx.state_slots),
                       _p(state), ctypes.c_int64(state.stride(0)), _p(gain), ctypes.c_float(eps), n, ctx.n_requests, heads,
-                      dk, dv, int(ctx.all_single), int(early), bound, _p(o), _p(qa), _p(a_last), _p(s_in),
-                      dtype_code(y.dtype), _stream())
+                      dk, dv, int(ctx.all_single), int(early), bound, _p(o), _p(qa), _p(kd), _p(a_last),
+                      _p(w), _p(s_in), dtype_code(y.dtype), _stream())
     _check(lib, "gla", rc)
     if not ctx.all_single:
         global launches
-        launches += 2 if dv <= 256 else 3
+        launches += 3 if dv <= 256 else 4
 
 
 # ---- what stands in front of a layer (csrc/shift_norm.cu) --------------------------------------
