@@ -39,7 +39,6 @@ KLLM_EXPORT_LAST_ERROR(gla)
 namespace {
 
 constexpr int kC = 64;          // rows of a chunk
-constexpr int kTS = 16;         // rows whose angles are in shared memory at a time
 constexpr int kThreads = 256;
 constexpr int kMaxRot = 256;
 
@@ -67,6 +66,7 @@ struct GlaArgs {
     // work of the form for portions
     float *o, *qa, *kd, *a_last, *w, *s_in; // [n][H dv], [n][H dk] twice, [chunks][H dk], [chunks][H][kC][kC], [chunks][H][dk][dv]
     bool vec;                               // sizes and addresses allow 16-byte accesses throughout
+    bool vec_out;                           // ... and four values of g, gain and y at once
     const int* start_pos;
 };
 
@@ -88,6 +88,12 @@ __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); 
 // sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau)
 __device__ __forceinline__ float gated_alpha(float z, float inv_tau) {
     return expf(-(log1pf(expf(-fabsf(z))) + fmaxf(-z, 0.f)) * inv_tau);
+}
+
+// cos and sin of position * f in float32: the angle and its rest from whole turns in double precision
+__device__ __forceinline__ void turn(int position, double f, float& c, float& s) {
+    const double ang = (double)position * f;
+    sincosf((float)(ang - rint(ang * 0.15915494309189533577) * 6.28318530717958647693), &s, &c);
 }
 
 // element d of a head's row, turned by the row's angles (cos [half], sin [half])
@@ -158,10 +164,10 @@ step_kernel(const GlaArgs a, int sl) {
     }
     const int half = a.rot >> 1;
     for (int i = tid; i < half; i += kThreads) {
-        double sn, c;
-        sincos((double)a.positions[t] * a.freq[i], &sn, &c);
-        cs[i] = (float)c * a.amplitude;
-        cs[half + i] = (float)sn * a.amplitude;
+        float c, sn;
+        turn(a.positions[t], a.freq[i], c, sn);
+        cs[i] = c * a.amplitude;
+        cs[half + i] = sn * a.amplitude;
     }
     __syncthreads();
     griddep_wait();
@@ -260,8 +266,7 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
 
 // grid (chunk bound, heads).  Thread (j, g): row j of the chunk as a key, key channels (i * 4 + g) * 4 + 0 .. 3,
-// i < DPT / 4.  Shared memory: k, then alpha [kC][4 DPT]; q [kC][4 DPT]; cos / sin [kTS][rot]; gated: W2 [dk][R + 1],
-// low [kC][R].
+// i < DPT / 4.  Shared memory: k, then alpha [kC][4 DPT]; q [kC][4 DPT]; gated: W2 [dk][R + 1], low [kC][R].
 template <typename T, int DPT, bool GATED>
 __global__ void __launch_bounds__(kThreads)
 chunk_kernel(const GlaArgs a) {
@@ -275,45 +280,54 @@ chunk_kernel(const GlaArgs a) {
     if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
     float* xs = sm;
     float* qs = xs + kC * P;
-    float* cs = qs + kC * P;
-    float* w2s = cs + kTS * rot;
+    float* w2s = qs + kC * P;
     float* lows = w2s + (GATED ? dk * (R + 1) : 0);
+    const float* qg = a.q + (int64_t)row0 * a.stride + head * dk;
+    const float* kg = a.k + (int64_t)row0 * a.stride + head * dk;
+    if (a.vec) {
+        for (int i = tid; i < kC * (P / 4); i += kThreads) {
+            const int r = i / (P / 4), d = (i - r * (P / 4)) * 4;
+            const bool in = r < rows && d < dk;
+            const int64_t off = in ? r * a.stride + d : 0;
+            cp_async16(qs + i * 4, qg + off, in);
+            cp_async16(xs + i * 4, kg + off, in);
+        }
+    } else {
+        for (int i = tid; i < kC * P; i += kThreads) {
+            const int r = i / P, d = i - r * P;
+            const bool in = r < rows && d < dk;
+            qs[i] = in ? qg[r * a.stride + d] : 0.f;
+            xs[i] = in ? kg[r * a.stride + d] : 0.f;
+        }
+    }
+    cp_async_commit();
     if (GATED) {
         const T* w2 = reinterpret_cast<const T*>(a.w2) + (int64_t)head * dk * R;
         for (int i = tid; i < dk * R; i += kThreads) w2s[(i / R) * (R + 1) + i % R] = to_f32(w2[i]);
         for (int i = tid; i < rows * R; i += kThreads) lows[i] = a.low[(int64_t)(row0 + i / R) * a.stride + i % R];
     }
-    for (int b0 = 0; b0 < kC; b0 += kTS) {
-        const int nr = max(0, min(kTS, rows - b0));
-        if (rot) {
-            __syncthreads();                // the angles before have been used up
-            for (int i = tid; i < nr * half; i += kThreads) {
-                const int r = i / half, d = i - r * half;
-                double sn, c;
-                sincos((double)a.positions[row0 + b0 + r] * a.freq[d], &sn, &c);
-                cs[r * rot + d] = (float)c * a.amplitude;
-                cs[r * rot + half + d] = (float)sn * a.amplitude;
-            }
-            __syncthreads();
-        }
-        for (int i = tid; i < kTS * P; i += kThreads) {
-            const int r = i / P, d = i - r * P;
-            float q = 0.f, k = 0.f;
-            if (r < nr && d < dk) {
-                const int64_t off = (int64_t)(row0 + b0 + r) * a.stride + head * dk;
-                q = turned(a.q + off, d, rot, cs + r * rot) * a.q_scale;
-                k = turned(a.k + off, d, rot, cs + r * rot) * a.k_scale;
-            }
-            qs[b0 * P + i] = q;
-            xs[b0 * P + i] = k;
-        }
-    }
+    cp_async_wait<0>();
     __syncthreads();
+    if (half) {
+        for (int i = tid; i < rows * half; i += kThreads) {
+            const int r = i / half, d = i - r * half;
+            float c, sn;
+            turn(a.positions[row0 + r], a.freq[d], c, sn);
+            c *= a.amplitude;
+            sn *= a.amplitude;
+            for (float* row : {qs + r * P, xs + r * P}) {
+                const float u = row[d], v = row[d + half];
+                row[d] = u * c - v * sn;
+                row[d + half] = v * c + u * sn;
+            }
+        }
+        __syncthreads();
+    }
     float w[DPT];
 #pragma unroll
     for (int i = 0; i < DPT; i += 4) {
         const float4 k4 = *reinterpret_cast<const float4*>(xs + j * P + (i + g) * 4);
-        w[i] = k4.x; w[i + 1] = k4.y; w[i + 2] = k4.z; w[i + 3] = k4.w;
+        w[i] = k4.x * a.k_scale; w[i + 1] = k4.y * a.k_scale; w[i + 2] = k4.z * a.k_scale; w[i + 3] = k4.w * a.k_scale;
     }
     const float fixed = GATED ? 1.f : a.decay[head];
     if (GATED) {
@@ -336,9 +350,11 @@ chunk_kernel(const GlaArgs a) {
     if (tid >= kThreads / 2) {
         for (int d = tid - kThreads / 2; d < dk; d += kThreads / 2) {
             float c = 1.f;
+            float* dst = a.qa + (int64_t)row0 * A_w + head * dk + d;
+#pragma unroll 4
             for (int r = 0; r < rows; r++) {
                 c *= GATED ? xs[r * P + d] : fixed;
-                a.qa[(int64_t)(row0 + r) * A_w + head * dk + d] = qs[r * P + d] * c;
+                dst[(int64_t)r * A_w] = qs[r * P + d] * a.q_scale * c;
             }
             a.a_last[(int64_t)blockIdx.x * A_w + head * dk + d] = c;
         }
@@ -368,7 +384,7 @@ chunk_kernel(const GlaArgs a) {
         acc += acc2;
         acc += __shfl_xor_sync(0xffffffffu, acc, 1);
         acc += __shfl_xor_sync(0xffffffffu, acc, 2);
-        if (g == 0) Wr[i * kC] = i >= j ? acc : 0.f;
+        if (g == 0) Wr[i * kC] = i >= j ? acc * a.q_scale : 0.f;
     }
     if (j < rows) {
         float* dst = a.kd + (int64_t)(row0 + j) * A_w + head * dk;
@@ -631,13 +647,31 @@ apply_kernel(const GlaArgs a) {
                 const float scale = rsqrtf(sq / (float)dv + a.eps);
                 T* yr = reinterpret_cast<T*>(a.y) + (int64_t)(row0 + row) * a.y_stride + head * dv;
                 const float* gr = a.g + (int64_t)(row0 + row) * a.stride + head * dv;
+                const float* gn = a.gain + head * dv;
 #pragma unroll
-                for (int j = 0; j < NJ; j++)
+                for (int j = 0; j < NJ; j++) {
+                    const int col = j * 64 + cg * 4;
+                    float v[4] = {acc[r][j * 4] * scale, acc[r][j * 4 + 1] * scale, acc[r][j * 4 + 2] * scale, acc[r][j * 4 + 3] * scale};
+                    if (a.vec_out) {
+                        if (col >= ne) continue;
+                        const float4 g4 = *reinterpret_cast<const float4*>(gr + col), n4 = *reinterpret_cast<const float4*>(gn + col);
+                        v[0] *= n4.x * silu_f(g4.x); v[1] *= n4.y * silu_f(g4.y);
+                        v[2] *= n4.z * silu_f(g4.z); v[3] *= n4.w * silu_f(g4.w);
+                        if constexpr (sizeof(T) == 4) {
+                            *reinterpret_cast<float4*>(yr + col) = make_float4(v[0], v[1], v[2], v[3]);
+                        } else {
+                            __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+                            uint2 pk;
+                            pk.x = *reinterpret_cast<uint32_t*>(&lo);
+                            pk.y = *reinterpret_cast<uint32_t*>(&hi);
+                            *reinterpret_cast<uint2*>(yr + col) = pk;
+                        }
+                    } else {
 #pragma unroll
-                    for (int c = 0; c < 4; c++) {
-                        const int col = j * 64 + cg * 4 + c;
-                        if (col < ne) yr[col] = from_f32<T>(acc[r][j * 4 + c] * scale * a.gain[head * dv + col] * silu_f(gr[col]));
+                        for (int c = 0; c < 4; c++)
+                            if (col + c < ne) yr[col + c] = from_f32<T>(v[c] * gn[col + c] * silu_f(gr[col + c]));
                     }
+                }
             }
         } else if (row < rows) {
             float* orow = a.o + (int64_t)(row0 + row) * B_w + head * dv + e0;
@@ -724,7 +758,7 @@ int raise_smem(K kern, bool& raised) {
 
 template <typename T, int DPT, bool GATED>
 int launch_chunk(const GlaArgs& a, int chunk_bound, cudaStream_t s) {
-    const size_t smem = sizeof(float) * ((size_t)2 * kC * 4 * DPT + (size_t)kTS * a.rot +
+    const size_t smem = sizeof(float) * ((size_t)2 * kC * 4 * DPT +
                                          (GATED ? (size_t)kC * a.R + (size_t)a.dk * (a.R + 1) : 0));
     if (smem > 220 * 1024) KLLM_FAIL("gla: a head of %d key channels with a decay of rank %d does not fit shared memory", a.dk, a.R);
     static bool raised = false;
@@ -766,7 +800,8 @@ int run(GlaArgs a, int n, bool single, bool early, int chunk_bound, cudaStream_t
     const bool rows_vec = a.dv % 4 == 0 && a.stride % 4 == 0 && a.state_stride % 4 == 0 &&
                           !(((uintptr_t)a.state | (uintptr_t)a.v) & 15);
     if (single) return rows_vec ? launch_step<T, 4>(a, early, s) : launch_step<T, 1>(a, early, s);
-    a.vec = rows_vec && a.dk % 4 == 0 && !(((uintptr_t)a.s_in | (uintptr_t)a.qa | (uintptr_t)a.kd | (uintptr_t)a.w) & 15);
+    a.vec = rows_vec && a.dk % 4 == 0 && !(((uintptr_t)a.s_in | (uintptr_t)a.qa | (uintptr_t)a.kd | (uintptr_t)a.w | (uintptr_t)a.q | (uintptr_t)a.k) & 15);
+    a.vec_out = a.vec && a.y_stride % 4 == 0 && !(((uintptr_t)a.g | (uintptr_t)a.gain | (uintptr_t)a.y) & 15);
     const bool vec = a.vec;
     int rc;
     if (a.dk <= 32) rc = launch_chunk<T, 8>(a, chunk_bound, s);
@@ -828,7 +863,7 @@ extern "C" int kllm_gla(void* y, int64_t y_stride, const float* q, const float* 
     a.inv_tau = inv_tau; a.decay = decay; a.freq = freq; a.rot = rot; a.amplitude = amplitude; a.q_scale = q_scale;
     a.k_scale = k_scale; a.positions = positions; a.q_start = q_start; a.state_slots = state_slots; a.n_requests = n_requests;
     a.heads = heads; a.dk = dk; a.dv = dv; a.state = state; a.state_stride = state_stride; a.gain = gain; a.eps = eps; a.y = y;
-    a.y_stride = y_stride; a.o = o; a.qa = qa; a.kd = kd; a.a_last = a_last; a.w = w; a.s_in = s_in; a.vec = false; a.start_pos = start_pos;
+    a.y_stride = y_stride; a.o = o; a.qa = qa; a.kd = kd; a.a_last = a_last; a.w = w; a.s_in = s_in; a.vec = a.vec_out = false; a.start_pos = start_pos;
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == KLLM_F32) return run<float>(a, n, single != 0, early != 0, chunk_bound, s);
     if (dtype == KLLM_BF16) return run<bf16>(a, n, single != 0, early != 0, chunk_bound, s);
