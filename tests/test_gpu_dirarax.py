@@ -634,3 +634,76 @@ def test_passes_keep_states_of_their_own(tmp_path):
             check_rows(run_cut(eng, ids, [20, 1, 2, 30, 1]), want, "float32", f"passes {i}")
         finally:
             eng.close()
+
+
+def _drawn(seed):
+    """A configuration drawn at random: sizes in steps of 2 to 16, any order of layers, any loop."""
+    rng = np.random.default_rng(1000 + seed)
+
+    def pick(*xs):
+        return xs[int(rng.integers(len(xs)))]
+    step = pick(2, 4, 8, 16)
+
+    def size(lo, hi):
+        return max(step, int(rng.integers(lo, hi + 1)) // step * step)
+
+    def rot(dim, scaled):
+        dims = max(2, int(rng.integers(1, dim // 2 + 1)) * 2)
+        return pick(_rot(dims, float(rng.integers(10, 20000)), (pick(2.0, 8.0), int(rng.integers(16, 100)), pick(8.0, 32.0), 1.0)
+                         if scaled and rng.random() < 0.7 else None), _rot(dim // 2 * 2, 500.0))
+    layers = []
+    for _ in range(int(rng.integers(2, 5))):
+        if rng.random() < 0.5:
+            layer = _gla(int(rng.integers(1, 6)), size(4, 72), size(4, 90), float(rng.uniform(1, 16)))
+        else:
+            g, dk, dim = int(rng.integers(1, 4)), size(4, 80), size(4, 72)
+            layer = _parallel((g * int(rng.integers(1, 4)), g, dk, size(4, 72), float(rng.uniform(0.1, 0.4)), rot(dk, True)),
+                              (dim, size(4, 72), rng.uniform(0.6, 1.0, int(rng.integers(1, 5))).tolist(), rot(dim, False)),
+                              float(rng.uniform(-1.5, 1.5)), float(rng.uniform(-1.5, 1.5)))
+        kind = rng.random()
+        if kind < 0.4:
+            layer = _dense(layer, size(8, 120))
+        elif kind < 0.85:
+            e = int(rng.integers(1, 9))
+            layer = _moe(layer, e, int(rng.integers(1, e + 1)), size(4, 64), pick(None, size(4, 80)))
+        else:
+            layer = _alone(layer)
+        layers.append(layer)
+    cfg = {"architecture": "Dirarax", "vocab": int(rng.integers(30, 200)), "width": size(16, 160), "norm": {"eps": pick(1e-6, 1e-5)},
+           "layers": layers}
+    if rng.random() < 0.75:
+        a = int(rng.integers(0, len(layers)))
+        cfg["loop"] = {"start": a, "stop": int(rng.integers(a + 1, len(layers) + 1)), "times": int(rng.integers(1, 4))}
+    return cfg, int(rng.integers(1, 20)), rng
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("seed", range(12))
+def test_configurations_drawn_at_random(tmp_path, seed, dtype):
+    """Whole, cut, decoded and two in a batch."""
+    from kllm_b200.engine.step import StepEntry
+    cfg, rank, rng = _drawn(seed)
+    if dtype == "bfloat16":
+        for L in cfg["layers"]:                          # no close call of a router between two runs (see make_model)
+            if L["mlp"] and L["mlp"]["kind"] == "moe":
+                L["mlp"]["router"]["top"] = L["mlp"]["router"]["experts"]
+    w = P.random_weights(cfg, seed, rank=rank)
+    d = write_model_dir(str(tmp_path / "drawn"), cfg, {k: np.asarray(v, dtype=np.float32) for k, v in w.items()})
+    a, b = (rng.integers(0, cfg["vocab"], size=n).tolist() for n in (140, 33))
+    want_a, want_b = P.forward(w, cfg, a), P.forward(w, cfg, b)
+    eng = engine_for(d, dtype, block_size=8, num_blocks=64)
+    try:
+        check_rows(run_cut(eng, a, [140]), want_a, dtype, "whole")
+        check_rows(run_cut(eng, a, [70, 2, 1, 1, 40, 1]), want_a, dtype, "cut")
+        ca, cb = eng.cache.open(), eng.cache.open()
+        got_a, got_b = [], []
+        for n, m in ((100, 1), (1, 20), (38, 11), (1, 1)):
+            pa, pb = len(np.concatenate(got_a)) if got_a else 0, len(np.concatenate(got_b)) if got_b else 0
+            lg = eng.runner.run([StepEntry(cb, b[pb:pb + m], list(range(m))), StepEntry(ca, a[pa:pa + n], list(range(n)))])
+            lg = lg.float().cpu().numpy().copy()
+            got_b.append(lg[:m])
+            got_a.append(lg[m:])
+        check_rows(np.concatenate(got_a), want_a, dtype, "first of two")
+        check_rows(np.concatenate(got_b), want_b, dtype, "second of two")
+    finally:
+        eng.close()
