@@ -118,17 +118,18 @@ __device__ __forceinline__ void load_tile(bf16* stage, const bf16* __restrict__ 
     const int lp0 = key0 / page_size, in_page = key0 - lp0 * page_size;
     if (in_page + TILE <= page_size) {
         // the whole tile lies in one page: one look-up, rows one after the other
-        const int64_t base = ((int64_t)table[lp0 - page_base] * n_kv + g) * page_size + in_page;
         if constexpr (VD == HD) {
+            const int64_t base = (((int64_t)table[lp0 - page_base] * n_kv + g) * page_size + in_page) * HD;
 #pragma unroll
             for (int c = threadIdx.x; c < TILE * CHUNKS; c += THREADS) {
                 const int row = c / CHUNKS, ch = c - row * CHUNKS;
                 const bool valid = key0 + row < hi;
-                const int64_t off = valid ? (base + row) * HD + ch * 8 : 0;
+                const int64_t off = valid ? base + row * HD + ch * 8 : 0;
                 cp_async16(sk + row * ROW + ch * 8, kcache + off, valid);
                 cp_async16(sv + row * ROW + ch * 8, vcache + off, valid);
             }
         } else {
+            const int64_t base = ((int64_t)table[lp0 - page_base] * n_kv + g) * page_size + in_page;
 #pragma unroll
             for (int c = threadIdx.x; c < TILE * CHUNKS; c += THREADS) {
                 const int row = c / CHUNKS, ch = c - row * CHUNKS;

@@ -17,8 +17,10 @@
 //             ADD_F32     Y is added into a float32 matrix (the residual stream)
 //             SWIGLU      W holds a gate and an up matrix [F, K] each; the output is
 //                         silu(gate row) * (up row) as bfloat16 [n, F]
-//                         (backend/model.cu:477-483, :1112-1114); optionally with biases on both
-//                         rows' sums and with the tanh gelu in place of silu
+//                         (backend/model.cu:477-483, :1112-1114)
+// Compiled with -DKLLM_BIAS=1 (a library of its own, so that the plain kernels keep their code) the
+// adding epilogue also adds a bias, and the gated one adds biases to both rows' sums and may take
+// the tanh gelu in place of silu.
 //
 // Layout of the work: a tile is 16 weight rows (for SWIGLU 8 gate rows and the 8 up
 // rows that go with them).  A CTA of 16 warps, one per SM, walks tiles tile = blockIdx.x,
@@ -60,12 +62,14 @@ struct Args {
     bf16* y_bf16;         // STORE_BF16, SWIGLU
     float* y_f32;         // STORE_F32, ADD_F32
     int64_t y_stride;
-    const float* bias;      // optional [N]: ADD_F32 adds it with the product; SWIGLU: to the gate rows' sums
-    const float* bias_up;   // optional [N], SWIGLU: to the up rows' sums
-    int gelu;               // SWIGLU: the activation is the gelu with tanh instead of silu
     int tl_slot;            // timeline row of this launch (-1: none)
     const void* prefetch;   // optional: weights of a later kernel, to be brought into L2
     int64_t prefetch_bytes;
+#ifdef KLLM_BIAS
+    const float* bias;      // ADD_F32: optional [N], joins the sum; SWIGLU: optional [N], to the gate rows' sums
+    const float* bias_up;   // SWIGLU: optional [N], to the up rows' sums
+    int gelu;               // SWIGLU: the activation is the gelu with tanh instead of silu
+#endif
 };
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
@@ -337,17 +341,24 @@ skinny_gemm_kernel(const Args a) {
                     float u = 0.f;
 #pragma unroll
                     for (int w = 0; w < WARPS; w++) u += red[(w * 16 + r + 8) * 8 * NT + c];
+#ifdef KLLM_BIAS
                     if (a.bias) v += a.bias[col];
                     if (a.bias_up) u += a.bias_up[col];
-                    const float act = a.gelu ? 0.5f * v * (1.f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)))
-                                             : v / (1.f + expf(-v));
-                    a.y_bf16[(int64_t)c * a.y_stride + col] = __float2bfloat16_rn(act * u);
+                    if (a.gelu) {
+                        const float act = 0.5f * v * (1.f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)));
+                        a.y_bf16[(int64_t)c * a.y_stride + col] = __float2bfloat16_rn(act * u);
+                        continue;
+                    }
+#endif
+                    a.y_bf16[(int64_t)c * a.y_stride + col] = __float2bfloat16_rn((v / (1.f + expf(-v))) * u);
                 } else if (EPI == STORE_BF16) {
                     a.y_bf16[(int64_t)c * a.y_stride + col] = __float2bfloat16_rn(v);
                 } else if (EPI == STORE_F32) {
                     a.y_f32[(int64_t)c * a.y_stride + col] = v;
                 } else {
+#ifdef KLLM_BIAS
                     if (a.bias) v += a.bias[col];
+#endif
                     a.y_f32[(int64_t)c * a.y_stride + col] += v;
                 }
             }
@@ -437,8 +448,7 @@ extern "C" int kllm_skinny_gemm_fits(int n, int K) {
 // w_stride: elements from one weight row to the next (>= K; more than K when the call
 // multiplies a slice of the columns of a wider matrix, which is how a K too long for
 // shared memory is taken: one call per slice, each adding into y_f32).
-// bias, bias_up: optional float32 [N] (epilogue 2: bias joins the sum; 3: the gate's and the up rows' biases); gelu:
-// epilogue 3 with the tanh gelu instead of silu.
+// bias, bias_up, gelu: see Args; refused by a library compiled without KLLM_BIAS.
 // prefetch: optional, `prefetch_bytes` bytes that a later kernel will stream; they are
 // requested into L2 before this kernel's own work.
 extern "C" int kllm_skinny_gemm(const void* w, const void* w_up, int64_t w_stride, int N, int K, int n, const void* x_bf16,
@@ -464,7 +474,11 @@ extern "C" int kllm_skinny_gemm(const void* w, const void* w_up, int64_t w_strid
     a.y_bf16 = (bf16*)y_bf16; a.y_f32 = y_f32; a.y_stride = y_stride;
     if (prefetch && ((uintptr_t)prefetch & 15)) KLLM_FAIL("skinny_gemm: the matrix to prefetch must be 16-byte aligned");
     a.prefetch = prefetch; a.prefetch_bytes = prefetch ? prefetch_bytes : 0;
+#ifdef KLLM_BIAS
     a.bias = bias; a.bias_up = bias_up; a.gelu = gelu;
+#else
+    if (bias || bias_up || gelu) KLLM_FAIL("skinny_gemm: this library was built without biases");
+#endif
     a.tl_slot = TL_SLOT();
     cudaStream_t s = (cudaStream_t)stream;
     if (n <= 8) {

@@ -49,9 +49,11 @@ struct Args {
     float eps;
     float* y;             // [n, N] at y_stride
     int64_t y_stride;
-    const float* bias;    // optional [N]: ADD adds it with the product; SWIGLU: to the gate rows' sums
-    const float* bias_up; // optional [N], SWIGLU: to the up rows' sums
+#ifdef KLLM_BIAS
+    const float* bias;    // ADD: optional [N], joins the sum; SWIGLU: optional [N], to the gate rows' sums
+    const float* bias_up; // SWIGLU: optional [N], to the up rows' sums
     int gelu;             // SWIGLU: the activation is the gelu with tanh instead of silu
+#endif
 };
 
 __device__ __forceinline__ float4 ldg_stream(const float* p) {
@@ -199,12 +201,15 @@ skinny_f32_kernel(const Args a) {
                 const int col = EPI == SWIGLU ? tile * WR + r : tile * GROUPS * WR + g2 * WR + r;
                 if (c < n && col < N) {
                     float* dst = a.y + (int64_t)c * a.y_stride + col;
-                    if (EPI == SWIGLU) {
-                        if (a.bias) v += a.bias[col];
-                        if (a.bias_up) up += a.bias_up[col];
-                        *dst = (a.gelu ? 0.5f * v * (1.f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)))
-                                       : v / (1.f + expf(-v))) * up;
-                    } else if (EPI == ADD) *dst += v + (a.bias ? a.bias[col] : 0.f);
+#ifdef KLLM_BIAS
+                    if (EPI != STORE && a.bias) v += a.bias[col];
+                    if (EPI == SWIGLU && a.bias_up) up += a.bias_up[col];
+                    if (EPI == SWIGLU && a.gelu)
+                        *dst = 0.5f * v * (1.f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v))) * up;
+                    else
+#endif
+                    if (EPI == SWIGLU) *dst = (v / (1.f + expf(-v))) * up;
+                    else if (EPI == ADD) *dst += v;
                     else *dst = v;
                 }
             }
@@ -255,7 +260,7 @@ extern "C" int kllm_skinny_gemm_f32_fits(int n, int K) {
 // given) normalised with gain [K] and eps.  epilogue 0: y written; 1: y += result; 2: w = gate
 // [N, K], w_up = up [N, K], y = silu(gate) * up.  w_stride: elements from one weight row to the
 // next (more than K when the call multiplies a slice of the columns of a wider matrix).
-// bias, bias_up, gelu: as in skinny_gemm.cu.
+// bias, bias_up, gelu: see Args; refused by a library compiled without KLLM_BIAS (as in skinny_gemm.cu).
 extern "C" int kllm_skinny_gemm_f32(const float* w, const float* w_up, int64_t w_stride, int N, int K, int n,
                                     const float* x, int64_t x_stride, const float* gain, const int* rows, float eps,
                                     float* y, int64_t y_stride, int prologue, int epilogue, const float* bias,
@@ -271,7 +276,11 @@ extern "C" int kllm_skinny_gemm_f32(const float* w, const float* w_up, int64_t w
     Args a;
     a.w = w; a.w_up = w_up; a.w_stride = w_stride; a.N = N; a.K = K; a.n = n; a.x = x; a.x_stride = x_stride;
     a.gain = gain; a.rows = rows; a.eps = eps; a.y = y; a.y_stride = y_stride;
+#ifdef KLLM_BIAS
     a.bias = bias; a.bias_up = bias_up; a.gelu = gelu;
+#else
+    if (bias || bias_up || gelu) KLLM_FAIL("skinny_gemm_f32: this library was built without biases");
+#endif
     cudaStream_t s = (cudaStream_t)stream;
 #define KLLM_F32_CASE(P, E) if (prologue == P && epilogue == E) return launch<P, E>(a, s)
     KLLM_F32_CASE(X_PLAIN, STORE); KLLM_F32_CASE(X_PLAIN, ADD); KLLM_F32_CASE(X_PLAIN, SWIGLU);

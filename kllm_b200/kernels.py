@@ -989,6 +989,12 @@ def biased_glu(out: torch.Tensor, gate: torch.Tensor, up: torch.Tensor, bias_gat
     _check(lib, "activation", rc)
 
 
+def _bias_form(bias, bias_up, activation):
+    """Compile-time definitions of the weight-streaming library that a call takes: the plain kernels are a library
+    without biases and the gelu."""
+    return {"KLLM_BIAS": 1} if bias is not None or bias_up is not None or activation != "silu" else None
+
+
 def _bias(t: Optional[torch.Tensor], n: int, what: str):
     if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or t.numel() != n):
         raise KernelError(f"{what}: a bias must be contiguous float32 [{n}]")
@@ -1133,7 +1139,7 @@ def skinny_gemm(weight: torch.Tensor, *, x: Optional[torch.Tensor] = None, x_f32
     want = torch.float32 if epilogue in ("f32", "add") else torch.bfloat16
     if out.dtype != want or out.stride(1) != 1 or out.shape[0] < n or out.shape[1] != N:
         raise KernelError("skinny_gemm: out has the wrong dtype or shape")
-    lib = load_library("skinny_gemm")
+    lib = load_library("skinny_gemm", _bias_form(bias, bias_up, activation))
     y16 = out if want == torch.bfloat16 else None
     y32 = out if want == torch.float32 else None
     rc = lib.kllm_skinny_gemm(_p(weight), _p(weight_up), ctypes.c_int64(weight.stride(0)), N, K, n, _p(x),
@@ -1183,7 +1189,7 @@ def _skinny_gemm_f32(weight, x, x_f32, gain, eps, rows, n_rows, weight_up, epilo
         out = torch.empty((n, N), dtype=torch.float32, device=weight.device)
     if out.dtype != torch.float32 or out.stride(1) != 1 or out.shape[0] < n or out.shape[1] != N:
         raise KernelError("skinny_gemm: out has the wrong dtype or shape")
-    lib = load_library("skinny_gemm_f32")
+    lib = load_library("skinny_gemm_f32", _bias_form(bias, bias_up, activation))
     rc = lib.kllm_skinny_gemm_f32(_p(weight), _p(weight_up), ctypes.c_int64(weight.stride(0)), N, K, n, _p(src),
                                   ctypes.c_int64(stride), _p(gain), _p(rows), ctypes.c_float(eps), _p(out),
                                   ctypes.c_int64(out.stride(0)), pro, {"f32": 0, "add": 1, "swiglu": 2}[epilogue],
