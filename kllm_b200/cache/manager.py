@@ -3,7 +3,7 @@ slots for per-request state of fixed size.
 
 Layers are put into groups by what they need: layers that keep every key of a
 request form one group, layers that only ever read a window of the last W keys
-form another (one per distinct W and shape).  A group has a page pool of its own,
+form another (one per distinct W and shape; such a layer may keep the first keys of a request beside its window).  A group has a page pool of its own,
 a device tensor [layers of the group, 2 (k, v), pages, kv heads, page_size,
 head_dim], and a block table per request, so one page id addresses the same slot
 in every layer of its group (as in the reference's pool,
@@ -14,8 +14,8 @@ Protocol, as in the reference (engine/kv/kv.go:54-74; engine/engine.go:160-168):
 ``commit(req, n)`` after it advances the length, ``close(req)`` gives everything
 back.  Unlike the reference, a reservation is all-or-nothing over all groups: when
 pages run out nothing is held that was not held before.  A window group gives a
-page back as soon as the window has passed it (at commit); its table keeps -1 in
-that place.  Pages are handed out last-freed-first (kv.go:29-40), so reuse is
+page back as soon as the window has passed it (at commit), unless it holds first keys
+that stay; its table keeps -1 in that place.  Pages are handed out last-freed-first (kv.go:29-40), so reuse is
 immediate.
 
 Beside the pages, every request holds one state slot.  A mixer with per-request
@@ -139,12 +139,14 @@ class CacheManager:
                 if isinstance(item, PagedKVNeed):
                     if item.window is not None and item.window <= 0:
                         raise ValueError(f"cache slot {slot}: window {item.window} must be positive")
+                    if item.keep_first < 0 or (item.keep_first and item.window is None):
+                        raise ValueError(f"cache slot {slot}: {item.keep_first} kept first keys beside a window of {item.window}")
                     if item.n_kv_heads % item.value_heads or (item.values_are_keys and (
                             item.value_heads != item.n_kv_heads or item.value_dim > item.head_dim)):
                         raise ValueError(f"cache slot {slot}: {item.value_heads} value heads of {item.value_dim} under "
                                          f"{item.n_kv_heads} key heads of {item.head_dim}")
                     key = (item.n_kv_heads, item.head_dim, item.window, item.value_dim, item.values_are_keys,
-                           item.value_heads)
+                           item.value_heads, item.keep_first)
                     g = by_key.get(key)
                     if g is None:
                         g = CacheGroup(len(self.groups), item, [], page_size, IdPool(num_pages, "page"))
@@ -228,12 +230,13 @@ class CacheManager:
         needs a page for each ``page_size`` tokens; a window group only the pages that the
         window of one query can touch (the window's width, whatever its alignment, plus the
         page of the token being written), since the pages behind the window come back at
-        every commit.  A model without any paged group needs none."""
+        every commit, and the pages of the first keys that stay.  A model without any paged group needs none."""
         out = []
         for g in self.groups:
             pages = -(-int(total_tokens) // self.page_size)
             if g.window is not None:
-                pages = min(pages, (g.window - 1) // self.page_size + 2)
+                kept = -(-g.need.keep_first // self.page_size)
+                pages = min(pages, (g.window - 1) // self.page_size + 2 + kept)
             out.append(pages)
         return out
 
@@ -316,7 +319,8 @@ class CacheManager:
                 continue
             first_needed = total + 1 - g.window      # earliest key the next query reads
             dead = max(0, first_needed) // self.page_size
-            for j in range(min(dead, len(table))):
+            kept = -(-g.need.keep_first // self.page_size)     # pages of the first keys that stay
+            for j in range(kept, min(dead, len(table))):
                 if table[j] >= 0:
                     g.pool.give([table[j]])
                     table[j] = -1

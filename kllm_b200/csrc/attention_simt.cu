@@ -66,7 +66,7 @@ attn_simt_kernel(T* __restrict__ out, float* __restrict__ part_o, float* __restr
                  const int* __restrict__ block_table, int max_blocks, int n_requests, int n_heads, int n_kv, int hd,
                  int vd, int page_size, int window, float scale, int qt, int chunk, int max_splits,
                  const float* __restrict__ slopes, const float* __restrict__ sinks, int segment, int v_heads,
-                 int v_row, int out_f32) {
+                 int v_row, int out_f32, int keep) {
     extern __shared__ __align__(16) float sm[];
     const int ld = hd + 4, ldv = vd + 4;
     float* Qs = sm;
@@ -105,12 +105,13 @@ attn_simt_kernel(T* __restrict__ out, float* __restrict__ part_o, float* __restr
     const int p0 = start_pos[s] + q0;                       // position of the tile's first token
     int lo_all = (window > 0 && p0 + 1 > window) ? p0 + 1 - window : 0;
     if (segment > 0) lo_all = max(lo_all, p0 - p0 % segment);      // the first token's segment starts no later than the others'
-    const int hi_all = p0 + nq;
-    int lo = lo_all, hi = hi_all;
+    const KeyLine line(lo_all, p0 + nq, keep, KEYS);        // kept keys, then the window
+    const int total = line.total();
+    int lo = 0, hi = total;                                 // this CTA's range of the line; chunks are whole tiles
     if (chunk > 0) {
-        lo = lo_all + split * chunk;
-        hi = min(hi_all, lo + chunk);
-        if (lo >= hi_all) return;
+        lo = split * chunk;
+        hi = min(total, lo + chunk);
+        if (lo >= total) return;
     }
     const int* table = block_table + (int64_t)s * max_blocks;
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
@@ -147,12 +148,13 @@ attn_simt_kernel(T* __restrict__ out, float* __restrict__ part_o, float* __restr
     const bool active = ty < R;                             // row ty exists; the thread's other rows may not
     const int ri = (R + 15) >> 4;                           // row slots i < ri hold rows of this tile (the same for all threads)
 
-    for (int key0 = lo; key0 < hi; key0 += KEYS) {
+    for (int v0 = lo; v0 < hi; v0 += KEYS) {
+        const int key0 = line.key(v0), lim = line.limit(v0);
         __syncthreads();                                    // the tile before is no longer read
         {
             // four threads per key: one look-up of the key's page, then independent 16-byte loads
             const int k = tid >> 2, kp = key0 + k;
-            const bool ok = kp < hi;
+            const bool ok = kp < lim;
             int64_t off = 0, offv = 0;
             if (ok) {
                 const int lp = kp / page_size;
@@ -209,7 +211,7 @@ attn_simt_kernel(T* __restrict__ out, float* __restrict__ part_o, float* __restr
 #pragma unroll
             for (int j = 0; j < 4; j++) {
                 const int kp = key0 + tx + 16 * j;
-                vis[j] = kp < hi && kp <= pos[i] && kp >= wlo[i];
+                vis[j] = kp < lim && kp <= pos[i] && (kp >= wlo[i] || kp < keep);
                 sc[i][j] = vis[j] ? sc[i][j] * scale + slope[i] * (float)(kp - pos[i]) : -INFINITY;
                 mx = fmaxf(mx, sc[i][j]);
             }
@@ -236,7 +238,7 @@ attn_simt_kernel(T* __restrict__ out, float* __restrict__ part_o, float* __restr
         }
         __syncthreads();
         if (active) {
-            const int nk = min(KEYS, hi - key0);
+            const int nk = min(KEYS, lim - key0);
             for (int k = 0; k < nk; k += 4) {
                 float4 p4[4];
 #pragma unroll
@@ -514,7 +516,7 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 attn_simt_merge_kernel(T* __restrict__ out, const float* __restrict__ part_o, const float* __restrict__ part_ml,
                        const int* __restrict__ positions, int n_rows, int n_heads, int hd, int window, int chunk,
-                       int max_splits, const float* __restrict__ sinks, int segment, int out_f32) {
+                       int max_splits, const float* __restrict__ sinks, int segment, int out_f32, int keep) {
     griddep_wait();
     griddep_launch();
     const int lane = threadIdx.x & 31;
@@ -523,7 +525,7 @@ attn_simt_merge_kernel(T* __restrict__ out, const float* __restrict__ part_o, co
     const int p = positions[row / n_heads];
     int lo_all = (window > 0 && p + 1 > window) ? p + 1 - window : 0;
     if (segment > 0) lo_all = max(lo_all, p - p % segment);
-    const int ns = (p + 1 - lo_all + chunk - 1) / chunk;
+    const int ns = (KeyLine(lo_all, p + 1, keep, KEYS).total() + chunk - 1) / chunk;
     // the chunks' maxima first (all loads at once), then their weights, then the sums in chunk order
     const float sink = sinks ? sinks[row % n_heads] : -INFINITY;
     float M = sink;
@@ -577,7 +579,7 @@ int launch(void* out, float* part_o, float* part_ml, const void* q, int64_t q_st
            const void* vcache, const int* q_start, const int* start_pos, const int* block_table, int max_blocks,
            int n_requests, int max_tiles, int n_heads, int n_kv, int hd, int vd, int page_size, int window, float scale,
            int qt, int chunk, int max_splits, const float* slopes, const float* sinks, int segment, int v_heads,
-           int v_row, int out_f32, cudaStream_t s) {
+           int v_row, int out_f32, int keep, cudaStream_t s) {
     auto kern = attn_simt_kernel<T, NC>;
     static bool raised = false;
     const size_t smem = smem_bytes(hd, vd);
@@ -592,7 +594,7 @@ int launch(void* out, float* part_o, float* part_ml, const void* q, int64_t q_st
     kllm_launch(kern, dim3(max_tiles * n_kv, 1, chunk > 0 ? max_splits : 1), dim3(THREADS), smem, s, (T*)out, part_o,
                 part_ml, (const T*)q, q_stride, (const T*)kcache, (const T*)vcache, q_start, start_pos, block_table,
                 max_blocks, n_requests, n_heads, n_kv, hd, vd, page_size, window, scale, qt, chunk, max_splits, slopes, sinks,
-                segment, v_heads, v_row, out_f32);
+                segment, v_heads, v_row, out_f32, keep);
     KLLM_LAUNCH_STATUS();
 }
 
@@ -614,13 +616,14 @@ int launch(void* out, float* part_o, float* part_ml, const void* q, int64_t q_st
 // keys of its own segment (beside the causal rule and the window).  v_heads: heads of the value store
 // (n_kv / v_heads neighbouring key heads read one value head); v_row: elements between two value rows
 // (vd, or more when a value row is the head of a longer row, e.g. of the key row itself).
-// out_f32: `out` is float32 whatever the operands' type.
+// out_f32: `out` is float32 whatever the operands' type.  keep (beside a window): the first `keep` keys of a
+// sequence stay visible.
 extern "C" int kllm_attention_simt(void* out, void* part_o, void* part_ml, const void* q, int64_t q_stride,
                                    const void* kcache, const void* vcache, const int* q_start, const int* start_pos,
                                    const int* block_table, int max_blocks, int n_requests, int max_tiles,
                                    int n_heads, int n_kv, int hd, int vd, int page_size, int window, float scale, int qt,
                                    int chunk, int max_splits, const float* slopes, const float* sinks, int segment,
-                                   int v_heads, int v_row, int out_f32, int dtype, void* stream) {
+                                   int v_heads, int v_row, int out_f32, int keep, int dtype, void* stream) {
     if (n_requests <= 0 || max_tiles <= 0) return 0;
     if (hd <= 0 || hd > 256 || hd % 4) KLLM_FAIL("attention (simt): head size %d is not a multiple of 4 up to 256", hd);
     if (vd <= 0 || vd > 256 || vd % 4) KLLM_FAIL("attention (simt): value size %d is not a multiple of 4 up to 256", vd);
@@ -631,6 +634,8 @@ extern "C" int kllm_attention_simt(void* out, void* part_o, void* part_ml, const
                   segment, v_heads, n_kv, vd, v_row);
     if (qt < 1 || qt * gs > ROWS) KLLM_FAIL("attention (simt): %d tokens x %d heads exceed the %d rows of a tile", qt, gs, ROWS);
     if (page_size <= 0) KLLM_FAIL("attention (simt): page size %d", page_size);
+    if (keep < 0 || (keep > 0 && (window <= 0 || segment > 0)) || chunk % KEYS)
+        KLLM_FAIL("attention (simt): %d kept keys beside a window of %d, segments of %d, chunks of %d keys", keep, window, segment, chunk);
     if (chunk < 0 || (chunk > 0 && (qt != 1 || max_splits < 1 || !part_o || !part_ml || n_kv > 65535 || max_splits > 65535)))
         KLLM_FAIL("attention (simt): chunks of keys need one token per tile, scratch buffers and a split count");
     const int esize = dtype == KLLM_F32 ? 4 : 2;
@@ -639,7 +644,7 @@ extern "C" int kllm_attention_simt(void* out, void* part_o, void* part_ml, const
     cudaStream_t s = (cudaStream_t)stream;
     // decoding tokens in float32 at the common head sizes and group widths: the kernel in which every thread works
     if (chunk > 0 && dtype == KLLM_F32 && (hd == 64 || hd == 128) && vd == hd && n_requests == max_tiles && segment == 0 &&
-        v_heads == n_kv && v_row == vd) {
+        v_heads == n_kv && v_row == vd && keep == 0) {
 #define KLLM_SIMT_DEC(HD_, GS_)                                                                                        \
     if (hd == HD_ && gs == GS_)                                                                                       \
         return launch_decode<HD_, GS_>((float*)part_o, (float*)part_ml, q, q_stride, kcache, vcache, q_start, start_pos, \
@@ -652,7 +657,7 @@ extern "C" int kllm_attention_simt(void* out, void* part_o, void* part_ml, const
 #define KLLM_SIMT(T, NC)                                                                                              \
     return launch<T, NC>(out, (float*)part_o, (float*)part_ml, q, q_stride, kcache, vcache, q_start, start_pos,      \
                          block_table, max_blocks, n_requests, max_tiles, n_heads, n_kv, hd, vd, page_size, window,    \
-                         scale, qt, chunk, max_splits, slopes, sinks, segment, v_heads, v_row, out_f32, s)
+                         scale, qt, chunk, max_splits, slopes, sinks, segment, v_heads, v_row, out_f32, keep, s)
     if (dtype == KLLM_F32) {
         if (vd <= 64) KLLM_SIMT(float, 1);
         if (vd <= 128) KLLM_SIMT(float, 2);
@@ -668,19 +673,19 @@ extern "C" int kllm_attention_simt(void* out, void* part_o, void* part_ml, const
 
 extern "C" int kllm_attention_simt_merge(void* out, const void* part_o, const void* part_ml, const int* positions,
                                          int n_tokens, int n_heads, int hd, int window, int chunk, int max_splits,
-                                         const float* sinks, int segment, int out_f32, int dtype, void* stream) {
+                                         const float* sinks, int segment, int out_f32, int keep, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
-    if (hd <= 0 || hd > 256 || chunk <= 0 || max_splits < 1) KLLM_FAIL("attention merge (simt): bad sizes");
+    if (hd <= 0 || hd > 256 || chunk <= 0 || max_splits < 1 || keep < 0) KLLM_FAIL("attention merge (simt): bad sizes");
     cudaStream_t s = (cudaStream_t)stream;
     const int n_rows = n_tokens * n_heads;
     if (dtype == KLLM_F32)
         kllm_launch((attn_simt_merge_kernel<float>), dim3((n_rows + 3) / 4), dim3(128), 0, s, (float*)out,
                     (const float*)part_o, (const float*)part_ml, positions, n_rows, n_heads, hd, window, chunk, max_splits, sinks,
-                    segment, out_f32);
+                    segment, out_f32, keep);
     else if (dtype == KLLM_BF16)
         kllm_launch((attn_simt_merge_kernel<bf16>), dim3((n_rows + 3) / 4), dim3(128), 0, s, (bf16*)out,
                     (const float*)part_o, (const float*)part_ml, positions, n_rows, n_heads, hd, window, chunk, max_splits, sinks,
-                    segment, out_f32);
+                    segment, out_f32, keep);
     else
         KLLM_FAIL("attention merge (simt): unknown element type %d", dtype);
     KLLM_LAUNCH_STATUS();

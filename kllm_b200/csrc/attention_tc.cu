@@ -35,7 +35,9 @@
 // Slots of a page beyond a request's length are never read: rows past the last
 // key are zero-filled instead of loaded.  The math is the reference's
 // (backend/model.cu:343-408): keys [max(0, p + 1 - window), p], scale after the
-// dot product, one division by the sum at the end.
+// dot product, one division by the sum at the end.  Beside a window the first `keep` keys of a
+// sequence may stay visible: the keys are then walked as the kept ones, in tiles of their own, and
+// the window (KeyLine).
 #include <mutex>
 #include "common.cuh"
 #include "attention_tc_static.h"
@@ -294,6 +296,8 @@ struct DecodeFusion {
     // n_kv * share as the kernel's n_kv: the cache is then addressed with kv head g / share of
     // n_kv / share, everything else goes by group.
     int share;
+    // beside a window: the first `keep` keys of the sequence stay visible (0: none)
+    int keep;
 };
 
 // Merge of the splits of one (token, kv head) by one CTA.  (m, l) of row r and split j
@@ -390,10 +394,12 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
     const int len = positions[t] + 1;
     if (whole_row) __syncthreads();
     const int start = (window > 0 && len > window) ? len - window : 0;
-    const int total = len - start;
+    // the token's keys as a line of numbers (the fused form has no kept keys: the line is the window)
+    const KeyLine line(start, len, FUSED ? 0 : fu.keep, TILE);
+    const int total = line.total();
     const int chunk = (((total + num_splits - 1) / num_splits) + TILE - 1) / TILE * TILE;
-    const int lo = start + split * chunk;
-    const int hi = min(len, lo + chunk);
+    const int lo = split * chunk;                          // this CTA's range of the line
+    const int hi = min(total, lo + chunk);
     const int ntiles = lo < hi ? (hi - lo + TILE - 1) / TILE : 0;
 
     // This range's slice of the block table, read once and together: otherwise every
@@ -405,7 +411,7 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
     if (whole_row) {
         pages = s_pages;
     } else if (ntiles > 0) {
-        const int first = lo / page_size, count = (hi - 1) / page_size - first + 1;
+        const int first = line.key(lo) / page_size, count = line.key(hi - 1) / page_size - first + 1;
         if (count <= DEC_PAGES) {
             for (int i = threadIdx.x; i < count; i += THREADS) s_pages[i] = table[first + i];
             __syncthreads();
@@ -416,7 +422,8 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
     // the tiles do not depend on the query: start them first
 #pragma unroll
     for (int s = 0; s < DEC_STAGES - 1; s++) {
-        if (s < ntiles) load_tile(smem + s * STAGE_ELEMS, kcache, vcache, pages, lo + s * TILE, hi, gk, nkc, page_size, page_base);
+        const int v = lo + s * TILE;
+        if (s < ntiles) load_tile(smem + s * STAGE_ELEMS, kcache, vcache, pages, line.key(v), line.limit(v), gk, nkc, page_size, page_base);
         cp_async_commit();
     }
     if (FUSED) l2_prefetch_slice(fu.prefetch, fu.prefetch_bytes, THREADS);   // after this kernel's own requests
@@ -455,7 +462,7 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
     // The CTA whose range holds the token's own position owns the new key and value:
     // it stores them into the page for later steps and, instead of reading them back,
     // writes them over their row of the shared-memory tile once that tile has landed.
-    const bool writer = FUSED && lo <= p_new && p_new < hi;
+    const bool writer = FUSED && ntiles > 0 && hi == total;
     if (FUSED) {
         // rotate_half on the query fragments: dims d and d + HD/2 sit in the same
         // register slot of k-steps ks and ks + KSTEPS/2 (rotation in float32, stored
@@ -505,21 +512,24 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
         cp_async_wait<DEC_STAGES - 2>();
         __syncthreads();
         const int nxt = i + DEC_STAGES - 1;
-        if (nxt < ntiles)
-            load_tile(smem + (nxt % DEC_STAGES) * STAGE_ELEMS, kcache, vcache, pages, lo + nxt * TILE, hi, gk, nkc, page_size, page_base);
+        if (nxt < ntiles) {
+            const int v = lo + nxt * TILE;
+            load_tile(smem + (nxt % DEC_STAGES) * STAGE_ELEMS, kcache, vcache, pages, line.key(v), line.limit(v), gk, nkc, page_size, page_base);
+        }
         cp_async_commit();
+        const int key0 = line.key(lo + i * TILE), lim = line.limit(lo + i * TILE);
         bf16* sk = smem + (i % DEC_STAGES) * STAGE_ELEMS;
         bf16* sv = sk + TILE * ROW;
         if (writer && i == ntiles - 1) {       // the token's own row: whatever the page held there is replaced
-            const int row = p_new - (lo + i * TILE);
+            const int row = p_new - key0;
             for (int j = threadIdx.x; j < HD; j += THREADS) {
                 sk[row * ROW + j] = s_newkv[j];
                 sv[row * ROW + j] = s_newkv[HD + j];
             }
             __syncthreads();
         }
-        const int key_base = lo + i * TILE + 16 * warp;
-        if (key_base < hi) {
+        const int key_base = key0 + 16 * warp;
+        if (key_base < lim) {
             float s[2][4];
             scores16(s, qa, sk, warp, lane);
             if (fu.slopes) {
@@ -533,7 +543,7 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
             for (int nt = 0; nt < 2; nt++)
 #pragma unroll
                 for (int j = 0; j < 4; j++)
-                    if (key_base + nt * 8 + 2 * tq + (j & 1) >= hi) s[nt][j] = -INFINITY;
+                    if (key_base + nt * 8 + 2 * tq + (j & 1) >= lim) s[nt][j] = -INFINITY;
             float mx0 = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1]));
             float mx1 = fmaxf(fmaxf(s[0][2], s[0][3]), fmaxf(s[1][2], s[1][3]));
             mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
@@ -664,7 +674,8 @@ constexpr int PRE_ROWS = 4 * 16 * MT;          // rows (token x head of the grou
 
 // `segment` C > 0: positions are cut into segments of C counted from 0 of the sequence and a row sees
 // only the keys of its own token's segment.  `v_heads`, `v_row`: shape of the value store (see
-// load_tile_wide).  `out_f32`: the output rows are float32 instead of bfloat16.
+// load_tile_wide).  `out_f32`: the output rows are float32 instead of bfloat16.  `keep` (beside a window): the first
+// `keep` keys of the sequence stay visible.
 __global__ void __launch_bounds__(THREADS)
 attn_prefill_kernel(void* __restrict__ out_, const bf16* __restrict__ q, int64_t q_stride,
                     const bf16* __restrict__ kcache, const bf16* __restrict__ vcache,
@@ -672,7 +683,7 @@ attn_prefill_kernel(void* __restrict__ out_, const bf16* __restrict__ q, int64_t
                     const int* __restrict__ block_table, int max_blocks, int n_requests, int n_heads,
                     int n_kv, int page_size, int window, float scale_log2e, int tokens_per_tile,
                     const float* __restrict__ slopes, float inv_scale, int split_p,
-                    const float* __restrict__ sinks, int segment, int v_heads, int v_row, int out_f32) {
+                    const float* __restrict__ sinks, int segment, int v_heads, int v_row, int out_f32, int keep) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* smem = reinterpret_cast<bf16*>(smem_raw);
     __shared__ int s_req, s_tok0;
@@ -707,7 +718,8 @@ attn_prefill_kernel(void* __restrict__ out_, const bf16* __restrict__ q, int64_t
     const bool plain_v = VD == HD && v_heads == n_kv && v_row == HD;
     const int gv = g / (n_kv / v_heads);
     const int* table = block_table + (int64_t)req * max_blocks;
-    const int ntiles = (hi - lo + TILE - 1) / TILE;
+    const KeyLine line(lo, hi, keep, TILE);
+    const int ntiles = (line.total() + TILE - 1) / TILE;
 
     // A tile whose rows all fit one warp (a decoding token's heads): every warp takes the same rows and every
     // fourth key tile, with a running (max, sum, output) of its own; the four are merged at the end in warp order.
@@ -780,8 +792,9 @@ attn_prefill_kernel(void* __restrict__ out_, const bf16* __restrict__ q, int64_t
 #pragma unroll
     for (int s = 0; s < PRE_STAGES - 1; s++) {
         if (s < ntiles) {
-            if (plain_v) load_tile(smem + s * STAGE_ELEMS, kcache, vcache, table, lo + s * TILE, hi, g, n_kv, page_size);
-            else load_tile_wide(smem + s * STAGE_ELEMS, kcache, vcache, table, lo + s * TILE, hi, g, n_kv, gv, v_heads, v_row, page_size);
+            const int k0 = line.key(s * TILE), lim = line.limit(s * TILE);
+            if (plain_v) load_tile(smem + s * STAGE_ELEMS, kcache, vcache, table, k0, lim, g, n_kv, page_size);
+            else load_tile_wide(smem + s * STAGE_ELEMS, kcache, vcache, table, k0, lim, g, n_kv, gv, v_heads, v_row, page_size);
         }
         cp_async_commit();
     }
@@ -792,16 +805,17 @@ attn_prefill_kernel(void* __restrict__ out_, const bf16* __restrict__ q, int64_t
         const int nxt = i + PRE_STAGES - 1;
         if (nxt < ntiles) {
             bf16* stage = smem + (nxt % PRE_STAGES) * STAGE_ELEMS;
-            if (plain_v) load_tile(stage, kcache, vcache, table, lo + nxt * TILE, hi, g, n_kv, page_size);
-            else load_tile_wide(stage, kcache, vcache, table, lo + nxt * TILE, hi, g, n_kv, gv, v_heads, v_row, page_size);
+            const int k0 = line.key(nxt * TILE), lim = line.limit(nxt * TILE);
+            if (plain_v) load_tile(stage, kcache, vcache, table, k0, lim, g, n_kv, page_size);
+            else load_tile_wide(stage, kcache, vcache, table, k0, lim, g, n_kv, gv, v_heads, v_row, page_size);
         }
         cp_async_commit();
         const bf16* sk = smem + (i % PRE_STAGES) * STAGE_ELEMS;
         const bf16* sv = sk + TILE * ROW;
-        const int key0 = lo + i * TILE;
-        if (!warp_active || key0 >= warp_hi || key0 + TILE <= warp_lo) continue;   // nothing of this tile is visible to the warp
+        const int key0 = line.key(i * TILE), lim = line.limit(i * TILE);
+        if (!warp_active || key0 >= warp_hi || (key0 + TILE <= warp_lo && key0 >= keep)) continue;   // nothing of this tile is visible to the warp
         if (spread && (i & 3) != warp) continue;                                   // another warp's tile
-        const bool need_mask = key0 < warp_lo_last || key0 + TILE - 1 > warp_full_below;
+        const bool need_mask = i * TILE < line.pad || key0 < warp_lo_last || key0 + TILE - 1 > warp_full_below;
         // scores of the warp's rows against the 64 keys: every key fragment serves all MT tiles
         float s[MT][8][4];
 #pragma unroll
@@ -843,8 +857,9 @@ attn_prefill_kernel(void* __restrict__ out_, const bf16* __restrict__ q, int64_t
 #pragma unroll
                     for (int j = 0; j < 2; j++) {
                         const int key = key0 + nt * 8 + 2 * tq + j;
-                        if (key > pr[m][0] || key < wr[m][0]) s[m][nt][j] = -INFINITY;
-                        if (key > pr[m][1] || key < wr[m][1]) s[m][nt][2 + j] = -INFINITY;
+                        const bool outside = key >= keep, none = key >= lim;     // outside the kept keys, past the tile's keys
+                        if (key > pr[m][0] || (key < wr[m][0] && outside) || none) s[m][nt][j] = -INFINITY;
+                        if (key > pr[m][1] || (key < wr[m][1] && outside) || none) s[m][nt][2 + j] = -INFINITY;
                     }
             }
             float t0 = -INFINITY, t1 = -INFINITY;
@@ -1046,8 +1061,9 @@ extern "C" int kllm_attention_decode(void* out, void* part_o, void* part_ml, con
                                      const int* token_req, const int* block_table, int max_blocks,
                                      int n_tokens, int n_heads, int n_kv, int hd, int page_size, int window,
                                      float scale, int num_splits, const float* slopes, int split_p,
-                                     const float* sinks, void* stream) {
+                                     const float* sinks, int keep, void* stream) {
     if (n_tokens <= 0) return 0;
+    if (keep < 0 || (keep > 0 && window <= 0)) KLLM_FAIL("attention decode: %d kept keys beside a window of %d", keep, window);
     int rc = check_common(n_heads, n_kv, hd, page_size, q, q_stride);
     if (rc) return rc;
     // more than 16 heads on a kv head: the fewest groups of equal size that fit a CTA's 16 rows
@@ -1062,6 +1078,7 @@ extern "C" int kllm_attention_decode(void* out, void* part_o, void* part_ml, con
     extra.sinks = sinks;
     extra.inv_scale = (slopes || sinks) ? 1.f / scale : 0.f;
     extra.split_p = split_p;
+    extra.keep = keep;
     if (n_tokens > 65535 || n_kv > 65535) KLLM_FAIL("attention decode: grid too large");
     if ((rc = set_attributes())) return rc;
     cudaStream_t s = (cudaStream_t)stream;
@@ -1183,20 +1200,20 @@ extern "C" int kllm_attention_decode_static(void* out, const void* q, int64_t q_
     }
     return kllm_attention_decode(out, part_o, part_ml, q, q_stride, kcache, vcache, positions, token_req,
                                  block_table, max_blocks, n_tokens, n_heads, n_kv, hd, page_size, window, scale,
-                                 num_splits, nullptr, 0, nullptr, stream);
+                                 num_splits, nullptr, 0, nullptr, 0, stream);
 }
 
 #endif  // KLLM_VD == KLLM_HD
 
 // Prefill form: requests' portions q_start[s]..q_start[s+1] (prefix sums, [n_requests+1])
 // starting at cache position start_pos[s].  `vd`: the value size this library was built for;
-// `segment`, `v_heads`, `v_row`, `out_f32` as the kernel describes them.
+// `segment`, `v_heads`, `v_row`, `out_f32`, `keep` as the kernel describes them.
 extern "C" int kllm_attention_prefill(void* out, const void* q, int64_t q_stride, const void* kcache,
                                       const void* vcache, const int* q_start, const int* start_pos,
                                       const int* block_table, int max_blocks, int n_tokens, int n_requests,
                                       int n_heads, int n_kv, int hd, int page_size, int window, float scale,
                                       const float* slopes, int split_p, const float* sinks, int vd, int segment,
-                                      int v_heads, int v_row, int out_f32, void* stream) {
+                                      int v_heads, int v_row, int out_f32, int keep, void* stream) {
     if (n_tokens <= 0) return 0;
     int rc = check_common(n_heads, n_kv, hd, page_size, q, q_stride);
     if (rc) return rc;
@@ -1204,6 +1221,8 @@ extern "C" int kllm_attention_prefill(void* out, const void* q, int64_t q_stride
     if (v_heads <= 0 || n_kv % v_heads || v_row < VD || v_row % 8 || ((uintptr_t)vcache & 15) || ((uintptr_t)kcache & 15))
         KLLM_FAIL("attention prefill: %d value heads under %d kv heads, value rows of %d elements", v_heads, n_kv, v_row);
     if (segment < 0) KLLM_FAIL("attention prefill: segment %d", segment);
+    if (keep < 0 || (keep > 0 && (window <= 0 || segment > 0)))
+        KLLM_FAIL("attention prefill: %d kept keys beside a window of %d, segments of %d", keep, window, segment);
     if (((uintptr_t)out & 7)) KLLM_FAIL("attention prefill: out must be 8-byte aligned");
     const int gs = n_heads / n_kv;
     if (gs > 64) KLLM_FAIL("attention prefill: %d heads per kv head, at most 64", gs);
@@ -1216,6 +1235,6 @@ extern "C" int kllm_attention_prefill(void* out, const void* q, int64_t q_stride
     kllm_launch((attn_prefill_kernel), dim3(grid), dim3(THREADS), PRE_SMEM_BYTES, (cudaStream_t)stream, 
         out, (const bf16*)q, q_stride, (const bf16*)kcache, (const bf16*)vcache, q_start, start_pos,
         block_table, max_blocks, n_requests, n_heads, n_kv, page_size, window, sl2e, tpt, slopes,
-        (slopes || sinks) ? 1.f / scale : 0.f, split_p, sinks, segment, v_heads, v_row, out_f32);
+        (slopes || sinks) ? 1.f / scale : 0.f, split_p, sinks, segment, v_heads, v_row, out_f32, keep);
     KLLM_LAUNCH_STATUS();
 }

@@ -160,6 +160,24 @@ template <typename T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
+// The keys that a tile of queries walks when it sees the window [lo, hi) and beside it the first `keep` keys of its
+// sequence: a line of numbers v in tiles of `tile`, first the kept keys [0, kept) padded to whole tiles, then the
+// window, so that no tile straddles the gap between them.  Where the window reaches down to the kept keys there is no
+// gap and the line is the keys [0, hi) themselves.  A tile at v holds the keys key(v), key(v) + 1, ... below limit(v).
+struct KeyLine {
+    int kept, pad, lo, hi;
+    __device__ __forceinline__ KeyLine(int lo_, int hi_, int keep, int tile) {
+        const bool gap = keep > 0 && lo_ > keep;
+        kept = gap ? keep : 0;
+        pad = gap ? (keep + tile - 1) / tile * tile : 0;
+        lo = keep > 0 && !gap ? 0 : lo_;
+        hi = hi_;
+    }
+    __device__ __forceinline__ int total() const { return pad + hi - lo; }
+    __device__ __forceinline__ int key(int v) const { return v < pad ? v : v - pad + lo; }
+    __device__ __forceinline__ int limit(int v) const { return v < pad ? kept : hi; }
+};
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -11,6 +11,8 @@
 //   1  y[M, N] float32  = acc
 //   2  y[M, N] float32 += acc                        (residual stream)
 //   3  y[M, N] bfloat16 = silu(acc_gate) * acc_up    (W = gate rows, W_up = up rows)
+//   4  the same with g = min(acc_gate, limit), u = clamp(acc_up, -limit, limit): g sigmoid(alpha g) (u + 1)
+//   5  y[M, N] bfloat16 = relu(acc)^2
 //
 // A persistent CTA per SM walks output tiles of 128 x BN.  BN, the accumulator's width,
 // is a multiple of 16 up to 256 (the gated epilogue spends half of the columns on
@@ -52,14 +54,16 @@ constexpr int TMEM_COLS = 2 * MAX_BN;
 constexpr int MAX_STAGES = 8;
 constexpr int SMEM_BYTES = 1024 + 4 * (A_BYTES + MAX_BN * 128);    // four stages of the widest tile
 
-enum Epilogue { EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU = 3 };
+enum Epilogue { EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU = 3, EPI_CLAMPED = 4, EPI_RELU2 = 5 };
+constexpr bool is_gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_CLAMPED; }
+constexpr bool is_bf16(int epi) { return epi != EPI_F32 && epi != EPI_ADD_F32; }
 
 // 32 consecutive results of one row, columns col..col+31 of the output, those below
 // `limit` (the end of the tile or of the matrix); res: what the float32 destination held
 template <int EPI>
 __device__ __forceinline__ void store_chunk(void* y, int64_t ldy, int row, int col, int limit, const float (&v)[32],
                                             const float4 (&res)[8]) {
-    if (EPI == EPI_BF16 || EPI == EPI_SWIGLU) {
+    if (is_bf16(EPI)) {
         bf16* p = (bf16*)y + (int64_t)row * ldy + col;
         if (col + 32 <= limit) {
 #pragma unroll
@@ -108,7 +112,7 @@ template <int EPI>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                 const __grid_constant__ CUtensorMap map_b2, void* __restrict__ y, int64_t ldy, int M, int N, int K,
-                int bn, int stages, int* status) {
+                int bn, int stages, float act_limit, float act_alpha, int* status) {
     extern __shared__ unsigned char smem_raw[];
     __shared__ __align__(8) uint64_t bar_full[MAX_STAGES], bar_empty[MAX_STAGES], bar_acc_full[2], bar_acc_empty[2];
     __shared__ unsigned s_tmem;
@@ -116,7 +120,7 @@ gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const unsigned base = (smem_u32(smem_raw) + 1023u) & ~1023u;
-    const int nout = (EPI == EPI_SWIGLU) ? bn / 2 : bn;            // output columns of a tile
+    const int nout = (is_gated(EPI)) ? bn / 2 : bn;            // output columns of a tile
     const int b_bytes = bn * 128, stage_bytes = A_BYTES + b_bytes;
     const int m_tiles = (M + BM - 1) / BM;
     const int n_tiles = (N + nout - 1) / nout;
@@ -145,7 +149,7 @@ gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
         if (lane == 0) {
             prefetch_map(&map_a);
             prefetch_map(&map_b);
-            if (EPI == EPI_SWIGLU) prefetch_map(&map_b2);
+            if (is_gated(EPI)) prefetch_map(&map_b2);
         }
         griddep_wait();
         int s = 0;
@@ -162,7 +166,7 @@ gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
                     mbar_expect_tx(&bar_full[s], (unsigned)stage_bytes);
                     tma_load_2d(a, &map_a, kb * BK, m0, &bar_full[s]);
                     tma_load_2d(b, &map_b, kb * BK, n0, &bar_full[s]);
-                    if (EPI == EPI_SWIGLU) tma_load_2d(b + (unsigned)(b_bytes / 2), &map_b2, kb * BK, n0, &bar_full[s]);
+                    if (is_gated(EPI)) tma_load_2d(b + (unsigned)(b_bytes / 2), &map_b2, kb * BK, n0, &bar_full[s]);
                 }
                 __syncwarp();
                 issued++;
@@ -238,15 +242,26 @@ gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
                 float v[32];
                 float4 res_next[8];
                 tmem_ld32(t + c * 32, v);
-                if (EPI == EPI_SWIGLU) {
+                if (is_gated(EPI)) {
                     float u[32];
                     tmem_ld32(t + bn / 2 + c * 32, u);
                     tmem_ld_wait();
 #pragma unroll
-                    for (int j = 0; j < 32; j++) v[j] = silu_mul(v[j], u[j]);
+                    for (int j = 0; j < 32; j++) {
+                        if (EPI == EPI_CLAMPED) {
+                            const float g = fminf(v[j], act_limit), w = fminf(fmaxf(u[j], -act_limit), act_limit);
+                            v[j] = g / (1.f + expf(-act_alpha * g)) * (w + 1.f);
+                        } else {
+                            v[j] = silu_mul(v[j], u[j]);
+                        }
+                    }
                 } else {
                     if (EPI == EPI_ADD_F32 && c + 1 < c_hi) load_residual(y, ldy, row, n0 + (c + 1) * 32, limit, row_ok, res_next);
                     tmem_ld_wait();
+                    if (EPI == EPI_RELU2) {
+#pragma unroll
+                        for (int j = 0; j < 32; j++) { v[j] = fmaxf(v[j], 0.f); v[j] *= v[j]; }
+                    }
                 }
                 const int col = n0 + c * 32;
                 if (row_ok && col < limit) store_chunk<EPI>(y, ldy, row, col, limit, v, res);
@@ -274,11 +289,11 @@ gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
 int pick_bn(int M, int N, int epilogue) {
     const int sms = sm_count();
     const int m_tiles = (M + BM - 1) / BM;
-    const int step = epilogue == EPI_SWIGLU ? 64 : 16;       // the up half starts on a 32-column chunk
+    const int step = is_gated(epilogue) ? 64 : 16;       // the up half starts on a 32-column chunk
     long long best = -1;
     int best_bn = MAX_BN;
     for (int bn = MAX_BN; bn >= 64; bn -= step) {
-        const int nout = epilogue == EPI_SWIGLU ? bn / 2 : bn;
+        const int nout = is_gated(epilogue) ? bn / 2 : bn;
         const long long tiles = (long long)m_tiles * ((N + nout - 1) / nout);
         const long long waves = (tiles + sms - 1) / sms;
         if (best < 0 || waves < best) { best = waves; best_bn = bn; }
@@ -288,7 +303,7 @@ int pick_bn(int M, int N, int epilogue) {
 
 template <int EPI>
 int launch(const CUtensorMap& ma, const CUtensorMap& mb, const CUtensorMap& mb2, void* y, int64_t ldy, int M, int N, int K,
-           int bn, int* status, cudaStream_t stream) {
+           int bn, float act_limit, float act_alpha, int* status, cudaStream_t stream) {
     static bool attr_set = false;
     if (!attr_set) {
         cudaError_t e = cudaFuncSetAttribute(gemm_tc5_kernel<EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
@@ -299,13 +314,13 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mb, const CUtensorMap& mb2,
         }
         attr_set = true;
     }
-    const int nout = (EPI == EPI_SWIGLU) ? bn / 2 : bn;
+    const int nout = (is_gated(EPI)) ? bn / 2 : bn;
     const long long tiles = (long long)((M + BM - 1) / BM) * ((N + nout - 1) / nout);
     const int grid = (int)(tiles < sm_count() ? tiles : sm_count());
     int stages = (SMEM_BYTES - 1024) / (A_BYTES + bn * 128);
     if (stages > MAX_STAGES) stages = MAX_STAGES;
     kllm_launch((gemm_tc5_kernel<EPI>), dim3(grid), dim3(THREADS), SMEM_BYTES, stream, ma, mb, mb2, y, ldy, M, N, K, bn, stages,
-                status);
+                act_limit, act_alpha, status);
     KLLM_LAUNCH_STATUS();
 }
 
@@ -316,7 +331,7 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mb, const CUtensorMap& mb2,
 // between this kernel and the library product.
 extern "C" int kllm_gemm_tcgen05_efficiency(int M, int N, int epilogue) {
     if (M <= 0 || N <= 0) return 0;
-    const int nout = epilogue == EPI_SWIGLU ? MAX_BN / 2 : MAX_BN;
+    const int nout = is_gated(epilogue) ? MAX_BN / 2 : MAX_BN;
     const double full = ((double)M / BM) * ((double)N / nout);
     const long long tiles = (long long)((M + BM - 1) / BM) * ((N + nout - 1) / nout);
     const long long waves = (tiles + sm_count() - 1) / sm_count();
@@ -328,34 +343,36 @@ extern "C" int kllm_gemm_tcgen05_efficiency(int M, int N, int epilogue) {
 extern "C" int kllm_gemm_tcgen05_fits(const void* x, int64_t ldx, const void* w, int64_t ldw, const void* w_up, int M,
                                       int N, int K, const void* y, int64_t ldy, int epilogue) {
     if (M <= 0 || N <= 0 || K <= 0) return 0;
-    if (epilogue < 0 || epilogue > 3) return 0;
+    if (epilogue < 0 || epilogue > 5) return 0;
     if ((K & 7) || (ldx & 7) || (ldw & 7)) return 0;                      // TMA: 16-byte rows
     if (((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ((uintptr_t)w_up & 15) || ((uintptr_t)y & 15)) return 0;
-    const bool bf16_out = epilogue == EPI_BF16 || epilogue == EPI_SWIGLU;
+    const bool bf16_out = is_bf16(epilogue);
     if (bf16_out ? (ldy & 7) : (ldy & 3)) return 0;                        // 16-byte vector stores
-    if (epilogue == EPI_SWIGLU && !w_up) return 0;
+    if (is_gated(epilogue) && !w_up) return 0;
     return 1;
 }
 
 // bn: accumulator width of a tile, 0 = chosen here, else a multiple of 16 (64 for the
-// gated epilogue) from 64 to 256.  status: device int that a wait which ran out sets
+// gated epilogues) from 64 to 256.  act_limit, act_alpha: of epilogue 4.  status: device int that a wait which ran out sets
 // (1: producer, 2: accumulator, 3: stage, 4: epilogue).
 extern "C" int kllm_gemm_tcgen05(const void* x, int64_t ldx, const void* w, int64_t ldw, const void* w_up, int M, int N,
-                                 int K, void* y, int64_t ldy, int epilogue, int bn, int* status, void* stream) {
+                                 int K, void* y, int64_t ldy, int epilogue, int bn, float act_limit, float act_alpha, int* status,
+                                 void* stream) {
     if (M <= 0 || N <= 0) return 0;
     if (!kllm_gemm_tcgen05_fits(x, ldx, w, ldw, w_up, M, N, K, y, ldy, epilogue))
         KLLM_FAIL("gemm (tcgen05): sizes %d x %d x %d, strides %lld/%lld/%lld or an address not taken (k and strides "
                   "multiples of 8, 16-byte aligned addresses)", M, N, K, (long long)ldx, (long long)ldw, (long long)ldy);
+    if (epilogue == EPI_CLAMPED && !(act_limit > 0.f)) KLLM_FAIL("gemm (tcgen05): the clamped epilogue needs a positive limit");
     if (bn == 0) bn = pick_bn(M, N, epilogue);
-    if (bn < 64 || bn > MAX_BN || bn % (epilogue == EPI_SWIGLU ? 64 : 16))
-        KLLM_FAIL("gemm (tcgen05): accumulator width %d, a multiple of %d from 64 to %d", bn, epilogue == EPI_SWIGLU ? 64 : 16, MAX_BN);
+    if (bn < 64 || bn > MAX_BN || bn % (is_gated(epilogue) ? 64 : 16))
+        KLLM_FAIL("gemm (tcgen05): accumulator width %d, a multiple of %d from 64 to %d", bn, is_gated(epilogue) ? 64 : 16, MAX_BN);
     CUtensorMap ma, mb, mb2;
-    const int b_rows = epilogue == EPI_SWIGLU ? bn / 2 : bn;
+    const int b_rows = is_gated(epilogue) ? bn / 2 : bn;
     int r = tensor_map(&ma, x, ldx, M, K, BM);
     if (r) return r;
     r = tensor_map(&mb, w, ldw, N, K, b_rows);
     if (r) return r;
-    if (epilogue == EPI_SWIGLU) {
+    if (is_gated(epilogue)) {
         r = tensor_map(&mb2, w_up, ldw, N, K, b_rows);
         if (r) return r;
     } else {
@@ -363,9 +380,11 @@ extern "C" int kllm_gemm_tcgen05(const void* x, int64_t ldx, const void* w, int6
     }
     cudaStream_t s = (cudaStream_t)stream;
     switch (epilogue) {
-        case EPI_BF16: return launch<EPI_BF16>(ma, mb, mb2, y, ldy, M, N, K, bn, status, s);
-        case EPI_F32: return launch<EPI_F32>(ma, mb, mb2, y, ldy, M, N, K, bn, status, s);
-        case EPI_ADD_F32: return launch<EPI_ADD_F32>(ma, mb, mb2, y, ldy, M, N, K, bn, status, s);
-        default: return launch<EPI_SWIGLU>(ma, mb, mb2, y, ldy, M, N, K, bn, status, s);
+        case EPI_BF16: return launch<EPI_BF16>(ma, mb, mb2, y, ldy, M, N, K, bn, 0.f, 0.f, status, s);
+        case EPI_F32: return launch<EPI_F32>(ma, mb, mb2, y, ldy, M, N, K, bn, 0.f, 0.f, status, s);
+        case EPI_ADD_F32: return launch<EPI_ADD_F32>(ma, mb, mb2, y, ldy, M, N, K, bn, 0.f, 0.f, status, s);
+        case EPI_CLAMPED: return launch<EPI_CLAMPED>(ma, mb, mb2, y, ldy, M, N, K, bn, act_limit, act_alpha, status, s);
+        case EPI_RELU2: return launch<EPI_RELU2>(ma, mb, mb2, y, ldy, M, N, K, bn, 0.f, 0.f, status, s);
+        default: return launch<EPI_SWIGLU>(ma, mb, mb2, y, ldy, M, N, K, bn, 0.f, 0.f, status, s);
     }
 }

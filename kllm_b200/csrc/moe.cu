@@ -3,6 +3,7 @@
 //   route     z = W_r h in float32 (h widened from the model's element type), score =
 //             sigmoid(z) or softmax(z); the `top` largest scores, the lower index first among
 //             equals; the weights are the chosen scores, as they are or divided by their sum.
+//             Optionally a correction per expert joins the scores for the choice alone.
 //             Optionally the experts form equal groups of neighbours, a group scores as its best
 //             expert, and only experts of the `keep` best groups can be chosen.
 //   sort      the (token, choice) pairs ordered by expert: offsets[E + 1] and perm[n * top]
@@ -16,9 +17,12 @@
 //             "gated" reads row `token` of the layer's input, times the row's weight if the
 //             weight acts on the expert's input, and stores act(gate) * up per sorted row;
 //             "down" reads the sorted rows and stores row token * top + choice of a float32
-//             matrix, times the weight if it acts on the output.
+//             matrix, times the weight if it acts on the output.  A third form, "plain", is the
+//             gated one for experts without a gate: the square of relu of the up product.
 //   combine   y[t] = sum over the choices of a token, in choice order; optionally plus the row of
 //             an expert that every token runs, times the sigmoid of a gate logit per token.
+//             Choices numbered from the number of experts on are identity experts: they have no
+//             matrices and no rows in the products, their output is the layer's input, times the weight.
 //   table     instead of a router: a table [vocab][top] that gives every token id its experts,
 //             each with the same weight.
 // The gated activation is silu(g) * u, or with a limit L and a slope a the clamped form
@@ -39,8 +43,9 @@ namespace {
 template <typename T>
 __global__ void __launch_bounds__(128)
 route_kernel(int* __restrict__ idx, float* __restrict__ wt, const T* __restrict__ h, const float* __restrict__ router,
-             int n, int d, int E, int top, int softmax, int renorm, int groups, int keep) {
-    extern __shared__ float zsh[];            // [E], then [2 * groups] when groups limit the choice
+             int n, int d, int E, int top, int softmax, int renorm, int groups, int keep, const float* __restrict__ corr,
+             float sum_eps) {
+    extern __shared__ float zsh[];            // [E], with a correction [E] scores, then [2 * groups] when groups limit the choice
     __shared__ float part[4][8];
     griddep_wait();
     griddep_launch();
@@ -86,11 +91,21 @@ route_kernel(int* __restrict__ idx, float* __restrict__ wt, const T* __restrict_
         for (int e = lane; e < E; e += 32) zsum += expf(z[e] - zmax);
         zsum = warp_sum(zsum);
     }
+    float* sc = zsh + E;
+    if (corr) {
+        // the choice is made among score + correction, the weights are the scores alone
+        for (int e = lane; e < E; e += 32) {
+            const float v = softmax ? expf(z[e] - zmax) / zsum : 1.f / (1.f + expf(-z[e]));
+            sc[e] = v;
+            z[e] = v + corr[e];
+        }
+        __syncwarp();
+    }
     if (groups > 1 && keep < groups) {
         // The experts form `groups` equal groups of neighbours; a group's score is its best expert's
         // (the logits order as the scores do).  Only experts of the `keep` best groups can be chosen,
         // the lower group first among equals; the scores themselves stay those over all experts.
-        float* gb = zsh + E;                              // a group's best logit, then whether it is kept
+        float* gb = zsh + (corr ? 2 * E : E);             // a group's best logit, then whether it is kept
         const int per = E / groups;
         for (int gi = lane; gi < groups; gi += 32) {
             float b = -INFINITY;
@@ -129,7 +144,7 @@ route_kernel(int* __restrict__ idx, float* __restrict__ wt, const T* __restrict_
             const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
         }
-        const float score = softmax ? expf(best - zmax) / zsum : 1.f / (1.f + expf(-best));
+        const float score = corr ? sc[bi] : softmax ? expf(best - zmax) / zsum : 1.f / (1.f + expf(-best));
         if (lane == 0) {
             idx[(int64_t)t * top + c] = bi;
             wt[(int64_t)t * top + c] = score;
@@ -139,7 +154,7 @@ route_kernel(int* __restrict__ idx, float* __restrict__ wt, const T* __restrict_
         __syncwarp();
     }
     if (renorm && lane == 0)
-        for (int c = 0; c < top; c++) wt[(int64_t)t * top + c] /= total;
+        for (int c = 0; c < top; c++) wt[(int64_t)t * top + c] /= total + sum_eps;
 }
 
 // ---- sort by expert ---------------------------------------------------------------
@@ -187,13 +202,21 @@ __device__ __forceinline__ float gated_act(float g, float u, const GatedAct& a) 
     return g / (1.f + expf(-a.alpha * g)) * (u + 1.f);
 }
 
-// GATED: W_e is [2 * N][K] (gate rows, then up rows), C [rows][N] in T, sorted order.
-// else : W_e is [N][K], C float32 [rows][N] at row perm[r].
-template <typename T, bool GATED>
+enum { DOWN = 0, GATE_UP = 1, PLAIN_UP = 2 };
+__device__ __forceinline__ float relu2(float v) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+}
+
+// GATE_UP : W_e is [2 * N][K] (gate rows, then up rows), C [rows][N] in T, sorted order.
+// PLAIN_UP: W_e is [N][K], C [rows][N] in T, sorted order.
+// DOWN    : W_e is [N][K], C float32 [rows][N] at row perm[r].
+template <typename T, int FORM>
 __global__ void __launch_bounds__(GT)
 expert_gemm_kernel(void* __restrict__ c_out, const T* __restrict__ a, int64_t a_stride, const T* __restrict__ w,
                    const int* __restrict__ offsets, const int* __restrict__ perm, const float* __restrict__ wt,
                    int E, int top, int N, int K, int scale_in, int scale_out, GatedAct act) {
+    constexpr bool GATED = FORM == GATE_UP, UP = FORM != DOWN;
     __shared__ float As[BK][BM + 1];
     __shared__ float Ws[GATED ? 2 : 1][BK][BN + 1];
     __shared__ int srow[BM];
@@ -218,8 +241,8 @@ expert_gemm_kernel(void* __restrict__ c_out, const T* __restrict__ a, int64_t a_
         float sc = 1.f;
         if (tid < nr) {
             const int flat = perm[r0 + tid];
-            src = GATED ? flat / top : r0 + tid;
-            if (GATED ? scale_in : scale_out) sc = wt[flat];
+            src = UP ? flat / top : r0 + tid;
+            if (UP ? scale_in : scale_out) sc = wt[flat];
         }
         srow[tid] = src;
         sscale[tid] = sc;
@@ -234,7 +257,7 @@ expert_gemm_kernel(void* __restrict__ c_out, const T* __restrict__ a, int64_t a_
             float v = 0.f;
             if (rr < nr && k0 + kk < K) {
                 v = to_f32(a[(int64_t)srow[rr] * a_stride + k0 + kk]);
-                if (GATED) v *= sscale[rr];
+                if (UP) v *= sscale[rr];
             }
             As[kk][rr] = v;
         }
@@ -272,6 +295,8 @@ expert_gemm_kernel(void* __restrict__ c_out, const T* __restrict__ a, int64_t a_
             if (cc >= N) continue;
             if (GATED) {
                 ((T*)c_out)[(int64_t)(r0 + rr) * N + cc] = from_f32<T>(gated_act(acc[0][i][j], acc[GATED ? 1 : 0][i][j], act));
+            } else if (UP) {
+                ((T*)c_out)[(int64_t)(r0 + rr) * N + cc] = from_f32<T>(relu2(acc[0][i][j]));
             } else {
                 ((float*)c_out)[(int64_t)perm[r0 + rr] * N + cc] = acc[0][i][j] * sscale[rr];
             }
@@ -302,18 +327,19 @@ __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], 
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-template <bool GATED, int MW>
+template <int FORM, int MW>
 constexpr size_t mma_smem_bytes() {
-    return (size_t)TSTAGES * (64 * MW + (GATED ? 2 : 1) * TN) * TLD * sizeof(bf16);
+    return (size_t)TSTAGES * (64 * MW + (FORM == GATE_UP ? 2 : 1) * TN) * TLD * sizeof(bf16);
 }
 
 // MW: 16-row tiles per warp; a CTA's tile has TM = 64 * MW rows (128 where an expert has many
 // rows, so that a weight fragment serves two row tiles; 64 otherwise).
-template <bool GATED, int MW>
+template <int FORM, int MW>
 __global__ void __launch_bounds__(TT)
 expert_gemm_mma_kernel(void* __restrict__ c_out, const bf16* __restrict__ a, int64_t a_stride, const bf16* __restrict__ w,
                        const int* __restrict__ offsets, const int* __restrict__ perm, const float* __restrict__ wt,
                        int E, int top, int N, int K, int scale_in, int scale_out, GatedAct act) {
+    constexpr bool GATED = FORM == GATE_UP, UP = FORM != DOWN;
     constexpr int NB = GATED ? 2 : 1, TM = 64 * MW;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16 (*As)[TM][TLD] = reinterpret_cast<bf16 (*)[TM][TLD]>(smem_raw);                           // [TSTAGES]
@@ -340,9 +366,9 @@ expert_gemm_mma_kernel(void* __restrict__ c_out, const bf16* __restrict__ a, int
         float sc = 1.f;
         if (i < nr) {
             const int flat = perm[r0 + i];
-            src = GATED ? flat / top : r0 + i;
+            src = UP ? flat / top : r0 + i;
             dst = flat;
-            if (GATED ? scale_in : scale_out) sc = wt[flat];
+            if (UP ? scale_in : scale_out) sc = wt[flat];
         }
         srow[i] = src;
         sdst[i] = dst;
@@ -417,6 +443,8 @@ expert_gemm_mma_kernel(void* __restrict__ c_out, const bf16* __restrict__ a, int
                     if (GATED) {
                         const float gv = acc[0][m][nt][2 * h + j] * sc, uv = acc[NB - 1][m][nt][2 * h + j] * sc;
                         ((bf16*)c_out)[(int64_t)(r0 + rr) * N + cc] = __float2bfloat16_rn(gated_act(gv, uv, act));
+                    } else if (UP) {
+                        ((bf16*)c_out)[(int64_t)(r0 + rr) * N + cc] = __float2bfloat16_rn(relu2(acc[0][m][nt][2 * h + j] * sc));
                     } else {
                         ((float*)c_out)[(int64_t)sdst[rr] * N + cc] = acc[0][m][nt][2 * h + j] * sc;
                     }
@@ -424,13 +452,13 @@ expert_gemm_mma_kernel(void* __restrict__ c_out, const bf16* __restrict__ a, int
         }
 }
 
-template <bool GATED, int MW>
+template <int FORM, int MW>
 int launch_mma(void* c, const void* a, int64_t a_stride, const void* w, const int* offsets, const int* perm,
                const float* wt, int rows, int E, int top, int N, int K, int scale_in, int scale_out, GatedAct act,
                cudaStream_t s) {
-    auto kern = expert_gemm_mma_kernel<GATED, MW>;
+    auto kern = expert_gemm_mma_kernel<FORM, MW>;
     static bool raised = false;
-    constexpr size_t smem = mma_smem_bytes<GATED, MW>();
+    constexpr size_t smem = mma_smem_bytes<FORM, MW>();
     if (!raised) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) {
@@ -446,19 +474,62 @@ int launch_mma(void* c, const void* a, int64_t a_stride, const void* w, const in
     KLLM_LAUNCH_STATUS();
 }
 
+// V consecutive columns per thread.  h, idx, wt: the layer's input and the routing, where choices from `experts` on are
+// identity experts (their rows of `parts` are never written); idx null: none are.
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
-combine_kernel(float* __restrict__ y, const float* __restrict__ parts, int64_t total, int d, int top,
-               const float* __restrict__ shared, const float* __restrict__ gate, int64_t gate_stride, float scale, int add) {
+combine_kernel(float* __restrict__ y, const float* __restrict__ parts, int64_t total, int dv, int top,
+               const float* __restrict__ shared, const float* __restrict__ gate, int64_t gate_stride, float scale, int add,
+               const T* __restrict__ h, const int* __restrict__ idx, const float* __restrict__ wt, int experts) {
     griddep_wait();
     griddep_launch();
     for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
-        const int64_t t = i / d;
-        const int c = (int)(i - t * d);
-        float s = 0.f;
-        for (int j = 0; j < top; j++) s += parts[(t * top + j) * d + c];
-        s *= scale;
-        if (shared) s += shared[i] * (gate ? 1.f / (1.f + expf(-gate[t * gate_stride])) : 1.f);
-        y[i] = add ? y[i] + s : s;
+        const int64_t t = total <= 0x7fffffff ? (int)i / dv : i / dv;
+        const int c = (int)(i - t * dv);
+        float s[V], v[V];
+        auto get = [&](const float* p) {
+            if constexpr (V == 4) {
+                const float4 q = *reinterpret_cast<const float4*>(p);
+                v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+            } else {
+                v[0] = *p;
+            }
+        };
+#pragma unroll
+        for (int u = 0; u < V; u++) s[u] = 0.f;
+        for (int j = 0; j < top; j++) {
+            const int64_t p = t * top + j;
+            if (idx && idx[p] >= experts) {
+                const T* hr = h + (t * dv + c) * V;
+                const float w = wt[p];
+                T hv[V];
+                if constexpr (V == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(hv) = *reinterpret_cast<const uint2*>(hr);
+                else
+#pragma unroll
+                    for (int u = 0; u < V; u++) hv[u] = hr[u];
+#pragma unroll
+                for (int u = 0; u < V; u++) s[u] += w * to_f32(hv[u]);
+            } else {
+                get(parts + (p * dv + c) * V);
+#pragma unroll
+                for (int u = 0; u < V; u++) s[u] += v[u];
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < V; u++) s[u] *= scale;
+        if (shared) {
+            const float g = gate ? 1.f / (1.f + expf(-gate[t * gate_stride])) : 1.f;
+            get(shared + i * V);
+#pragma unroll
+            for (int u = 0; u < V; u++) s[u] += v[u] * g;
+        }
+        if (add) {
+            get(y + i * V);
+#pragma unroll
+            for (int u = 0; u < V; u++) s[u] = v[u] + s[u];
+        }
+        if constexpr (V == 4) *reinterpret_cast<float4*>(y + i * 4) = make_float4(s[0], s[1], s[2], s[3]);
+        else y[i] = s[0];
     }
 }
 
@@ -483,22 +554,24 @@ table_route_kernel(int* __restrict__ idx, float* __restrict__ wt, const int* __r
 
 }  // namespace
 
-// idx int32 [n][top], wt float32 [n][top]; h [n][d] contiguous in `dtype`; router float32 [E][d].
+// idx int32 [n][top], wt float32 [n][top]; h [n][d] contiguous in `dtype`; router float32 [E][d]; corr float32 [E] or
+// NULL; sum_eps joins the sum that the weights are divided by.
 extern "C" int kllm_moe_route(int* idx, float* wt, const void* h, const float* router, int n, int d, int E, int top,
-                              int softmax, int renorm, int groups, int keep, int dtype, void* stream) {
+                              int softmax, int renorm, int groups, int keep, const float* corr, float sum_eps, int dtype,
+                              void* stream) {
     if (n <= 0) return 0;
     if (E <= 0 || E > 1024 || top <= 0 || top > E) KLLM_FAIL("moe route: %d of %d experts (at most 1024)", top, E);
     if (groups < 1) groups = keep = 1;
     if (E % groups || keep < 1 || keep > groups || top > keep * (E / groups))
         KLLM_FAIL("moe route: %d of %d experts in %d groups of which %d are kept", top, E, groups, keep);
     cudaStream_t s = (cudaStream_t)stream;
-    const size_t smem = (size_t)(E + 2 * groups) * sizeof(float);
+    const size_t smem = (size_t)((corr ? 2 : 1) * E + 2 * groups) * sizeof(float);
     if (dtype == KLLM_F32)
         kllm_launch((route_kernel<float>), dim3(n), dim3(128), smem, s, idx, wt, (const float*)h, router, n, d, E,
-                    top, softmax, renorm, groups, keep);
+                    top, softmax, renorm, groups, keep, corr, sum_eps);
     else if (dtype == KLLM_BF16)
         kllm_launch((route_kernel<bf16>), dim3(n), dim3(128), smem, s, idx, wt, (const bf16*)h, router, n, d, E,
-                    top, softmax, renorm, groups, keep);
+                    top, softmax, renorm, groups, keep, corr, sum_eps);
     else
         KLLM_FAIL("moe route: unknown element type %d", dtype);
     KLLM_LAUNCH_STATUS();
@@ -513,15 +586,17 @@ extern "C" int kllm_moe_sort(int* offsets, int* perm, int* rank, const int* idx,
     KLLM_LAUNCH_STATUS();
 }
 
-// gated != 0: a [tokens][K] (row stride a_stride), w [E][2N][K], c [rows][N] in `dtype`;
-// gated == 0: a [rows][K] sorted, w [E][N][K], c float32 [rows][N] indexed by perm.
+// form 1 (gated): a [tokens][K] (row stride a_stride), w [E][2N][K], c [rows][N] in `dtype`;
+// form 2 (plain): the same with w [E][N][K] and the square of relu;
+// form 0 (down): a [rows][K] sorted, w [E][N][K], c float32 [rows][N] indexed by perm.
+// offsets: [E + 1] at least; sorted rows from offsets[E] on belong to no expert here and are left alone.
 extern "C" int kllm_moe_gemm(void* c, const void* a, int64_t a_stride, const void* w, const int* offsets,
-                             const int* perm, const float* wt, int rows, int E, int top, int N, int K, int gated,
+                             const int* perm, const float* wt, int rows, int E, int top, int N, int K, int form,
                              int scale_in, int scale_out, int act_kind, float act_limit, float act_alpha, int dtype,
                              void* stream) {
     if (rows <= 0) return 0;
     if (N <= 0 || K <= 0 || E <= 0 || top <= 0) KLLM_FAIL("moe gemm: bad sizes");
-    if (act_kind < 0 || act_kind > 1) KLLM_FAIL("moe gemm: unknown activation %d", act_kind);
+    if (act_kind < 0 || act_kind > 1 || form < 0 || form > 2) KLLM_FAIL("moe gemm: unknown activation %d or form %d", act_kind, form);
     const GatedAct act = {act_kind, act_limit, act_alpha};
     const int row_tiles = (rows + BM - 1) / BM + E;
     if (row_tiles > 65535) KLLM_FAIL("moe gemm: %d rows in one launch", rows);
@@ -532,10 +607,12 @@ extern "C" int kllm_moe_gemm(void* c, const void* a, int64_t a_stride, const voi
         const bool tall = rows / E >= 128;
 #define KLLM_MOE_MMA(G, MW) \
     return launch_mma<G, MW>(c, a, a_stride, w, offsets, perm, wt, rows, E, top, N, K, scale_in, scale_out, act, s)
-        if (gated && tall) KLLM_MOE_MMA(true, 2);
-        if (gated) KLLM_MOE_MMA(true, 1);
-        if (tall) KLLM_MOE_MMA(false, 2);
-        KLLM_MOE_MMA(false, 1);
+        if (form == GATE_UP && tall) KLLM_MOE_MMA(GATE_UP, 2);
+        if (form == GATE_UP) KLLM_MOE_MMA(GATE_UP, 1);
+        if (form == PLAIN_UP && tall) KLLM_MOE_MMA(PLAIN_UP, 2);
+        if (form == PLAIN_UP) KLLM_MOE_MMA(PLAIN_UP, 1);
+        if (tall) KLLM_MOE_MMA(DOWN, 2);
+        KLLM_MOE_MMA(DOWN, 1);
 #undef KLLM_MOE_MMA
     }
     const dim3 grid((N + BN - 1) / BN, row_tiles);
@@ -543,9 +620,9 @@ extern "C" int kllm_moe_gemm(void* c, const void* a, int64_t a_stride, const voi
     kllm_launch((expert_gemm_kernel<T, G>), grid, dim3(GT), 0, s, c, (const T*)a, a_stride, (const T*)w, offsets, perm, \
                 wt, E, top, N, K, scale_in, scale_out, act)
     if (dtype == KLLM_F32) {
-        if (gated) KLLM_MOE(float, true); else KLLM_MOE(float, false);
+        if (form == GATE_UP) KLLM_MOE(float, GATE_UP); else if (form == PLAIN_UP) KLLM_MOE(float, PLAIN_UP); else KLLM_MOE(float, DOWN);
     } else if (dtype == KLLM_BF16) {
-        if (gated) KLLM_MOE(bf16, true); else KLLM_MOE(bf16, false);
+        if (form == GATE_UP) KLLM_MOE(bf16, GATE_UP); else if (form == PLAIN_UP) KLLM_MOE(bf16, PLAIN_UP); else KLLM_MOE(bf16, DOWN);
     } else {
         KLLM_FAIL("moe gemm: unknown element type %d", dtype);
     }
@@ -565,13 +642,25 @@ extern "C" int kllm_moe_table_route(int* idx, float* wt, const int* token_ids, c
 
 // y[t] = scale * (sum of parts[t * top + j] over j in order) (+ shared[t] * sigmoid(gate[t * gate_stride]) when
 // `shared` float32 [n][d] is given; gate NULL: the shared rows are added as they are).  add: the sum is added into y.
+// idx int32, wt float32 [n][top] and h [n][d] in `h_dtype` (all or none): choices from `experts` on add wt * h[t] in
+// place of a row of parts.
 extern "C" int kllm_moe_combine(float* y, const float* parts, int n, int d, int top, const float* shared,
-                                const float* gate, int64_t gate_stride, float scale, int add, void* stream) {
+                                const float* gate, int64_t gate_stride, float scale, int add, const void* h, const int* idx,
+                                const float* wt, int experts, int h_dtype, void* stream) {
     if (n <= 0) return 0;
-    const int64_t total = (int64_t)n * d;
+    if (idx && (!h || !wt || (h_dtype != KLLM_F32 && h_dtype != KLLM_BF16))) KLLM_FAIL("moe combine: identity experts need the input and the weights");
+    const bool vec = d % 4 == 0 && !(((uintptr_t)y | (uintptr_t)parts | (uintptr_t)shared | (uintptr_t)h) & 15);
+    const int64_t total = (int64_t)n * d / (vec ? 4 : 1);
     int64_t blocks = (total + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
-    kllm_launch((combine_kernel), dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, y, parts, total, d, top,
-                shared, gate, gate_stride, scale, add);
+#define KLLM_COMBINE(T, V)                                                                                               \
+    kllm_launch((combine_kernel<T, V>), dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, y, parts, total, d / V, top, \
+                shared, gate, gate_stride, scale, add, (const T*)h, idx, wt, experts)
+    if (idx && h_dtype == KLLM_BF16) {
+        if (vec) KLLM_COMBINE(bf16, 4); else KLLM_COMBINE(bf16, 1);
+    } else {
+        if (vec) KLLM_COMBINE(float, 4); else KLLM_COMBINE(float, 1);
+    }
+#undef KLLM_COMBINE
     KLLM_LAUNCH_STATUS();
 }

@@ -2,11 +2,12 @@
 //
 // The (token, choice) pairs of a step are sorted by expert (moe.cu: offsets[E + 1], perm[rows]);
 // expert e owns the sorted rows offsets[e] .. offsets[e + 1].  For those rows C = A W_e^T with
-// bfloat16 operands and float32 accumulation, in two forms:
+// bfloat16 operands and float32 accumulation, in three forms:
 //
 //   gated   A [rows, K] is the layer's input gathered into sorted order (gather kernel below),
 //           W [E, 2N, K] holds every expert's gate rows and then its up rows; the result
 //           act(gate) * up is stored as bfloat16 [rows, N] in sorted order;
+//   plain   the same for experts without a gate: W [E, N, K], the square of relu of the up product;
 //   down    A [rows, K] is that result, W [E, N, K]; the float32 result of sorted row r goes to
 //           row perm[r] = token * top + choice of C [rows, N], times the pair's weight if the
 //           weights act on the experts' outputs.
@@ -62,9 +63,10 @@ __device__ __forceinline__ int expert_of(const int* first, int E, int gm) {
 // rows of x [tokens, K] into sorted order: xs[r] = x[perm[r] / top], 16 bytes per thread and step
 __global__ void __launch_bounds__(256)
 gather_sorted_kernel(bf16* __restrict__ xs, const bf16* __restrict__ x, int64_t x_stride, const int* __restrict__ perm,
-                     int rows, int top, int K) {
+                     int rows, int top, int K, const int* __restrict__ count) {
     griddep_wait();
     griddep_launch();
+    rows = min(rows, *count);                            // rows behind the last expert's belong to nobody
     const int per_row = K / 8;
     for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < (int64_t)rows * per_row;
          i += (int64_t)gridDim.x * blockDim.x) {
@@ -74,12 +76,15 @@ gather_sorted_kernel(bf16* __restrict__ xs, const bf16* __restrict__ x, int64_t 
     }
 }
 
-template <bool GATED>
+enum { DOWN = 0, GATE_UP = 1, PLAIN_UP = 2 };
+
+template <int FORM>
 __global__ void __launch_bounds__(THREADS, 1)
 moe_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                void* __restrict__ y, const int* __restrict__ offsets, const int* __restrict__ perm,
                const float* __restrict__ wt, int E, int N, int K, int bn, int stages, int scale_out, GatedAct act,
                int* status) {
+    constexpr bool GATED = FORM == GATE_UP, UP = FORM != DOWN;
     extern __shared__ unsigned char smem_raw[];
     __shared__ __align__(8) uint64_t bar_full[MAX_STAGES], bar_empty[MAX_STAGES], bar_acc_full[2], bar_acc_empty[2];
     __shared__ unsigned s_tmem;
@@ -214,7 +219,7 @@ moe_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             const int limit = min(N, n0 + nout);
             int dst = row;
             float sc = 1.f;
-            if (!GATED && row_ok) {
+            if (!UP && row_ok) {
                 dst = perm[row];
                 if (scale_out) sc = wt[dst];
             }
@@ -233,10 +238,14 @@ moe_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     for (int j = 0; j < 32; j++) v[j] = gated_act(v[j], u[j], act);
                 } else {
                     tmem_ld_wait();
+                    if (FORM == PLAIN_UP) {
+#pragma unroll
+                        for (int j = 0; j < 32; j++) { v[j] = fmaxf(v[j], 0.f); v[j] *= v[j]; }
+                    }
                 }
                 const int col = n0 + c * 32;
                 if (!row_ok || col >= limit) continue;
-                if (GATED) {
+                if (UP) {
                     bf16* p = (bf16*)y + (int64_t)dst * N + col;
                     if (col + 32 <= limit) {
 #pragma unroll
@@ -295,12 +304,12 @@ int pick_bn(int row_tiles, int N, bool gated) {
     return best_bn;
 }
 
-template <bool GATED>
+template <int FORM>
 int launch(const CUtensorMap& ma, const CUtensorMap& mb, void* y, const int* offsets, const int* perm, const float* wt,
            int rows, int E, int N, int K, int bn, int scale_out, GatedAct act, int* status, cudaStream_t stream) {
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(moe_tc5_kernel<GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
+        cudaError_t e = cudaFuncSetAttribute(moe_tc5_kernel<FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
         if (e != cudaSuccess) {
             snprintf(g_kllm_err, sizeof(g_kllm_err), "moe gemm (tcgen05): %d bytes of shared memory refused: %s", SMEM_BYTES,
                      cudaGetErrorString(e));
@@ -309,12 +318,12 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mb, void* y, const int* off
         attr_set = true;
     }
     const int row_tiles = rows / BM + E;                   // >= the sum of the experts' tile counts
-    const int nout = GATED ? bn / 2 : bn;
+    const int nout = FORM == GATE_UP ? bn / 2 : bn;
     const long long tiles = (long long)row_tiles * ((N + nout - 1) / nout);
     const int grid = (int)(tiles < sm_count() ? tiles : sm_count());
     int stages = (SMEM_BYTES - 1024) / (A_BYTES + bn * 128);
     if (stages > MAX_STAGES) stages = MAX_STAGES;
-    kllm_launch((moe_tc5_kernel<GATED>), dim3(grid), dim3(THREADS), SMEM_BYTES, stream, ma, mb, y, offsets, perm, wt, E, N, K,
+    kllm_launch((moe_tc5_kernel<FORM>), dim3(grid), dim3(THREADS), SMEM_BYTES, stream, ma, mb, y, offsets, perm, wt, E, N, K,
                 bn, stages, scale_out, act, status);
     KLLM_LAUNCH_STATUS();
 }
@@ -324,47 +333,50 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mb, void* y, const int* off
 // 1 if the kernels take these sizes and addresses, else 0 (the caller then uses the grouped
 // mma.sync kernel).
 extern "C" int kllm_moe_gemm_tcgen05_fits(const void* a, const void* w, const void* c, int rows, int E, int N, int K,
-                                          int gated) {
+                                          int form) {
     if (rows <= 0 || E <= 0 || E > MAX_EXPERTS || N <= 0 || K <= 0) return 0;
     if ((K & 7) || (N & 7)) return 0;                                      // 16-byte rows for TMA and the vector stores
     if (((uintptr_t)a & 15) || ((uintptr_t)w & 15) || ((uintptr_t)c & 15)) return 0;
-    if ((long long)E * (gated ? 2 : 1) * N > 0x7fffffffLL) return 0;
+    if ((long long)E * (form == GATE_UP ? 2 : 1) * N > 0x7fffffffLL) return 0;
     return 1;
 }
 
-// xs [rows, K] = x[perm[r] / top], bfloat16.
+// xs [rows, K] = x[perm[r] / top], bfloat16, for the rows below *count.
 extern "C" int kllm_moe_gather_sorted(void* xs, const void* x, int64_t x_stride, const int* perm, int rows, int top, int K,
-                                      void* stream) {
+                                      const int* count, void* stream) {
     if (rows <= 0) return 0;
     if (K <= 0 || (K & 7) || (x_stride & 7) || top <= 0 || ((uintptr_t)xs & 15) || ((uintptr_t)x & 15))
         KLLM_FAIL("moe gather: rows of %d elements (stride %lld) are not whole 16-byte pieces", K, (long long)x_stride);
     const long long work = (long long)rows * (K / 8);
     const int grid = (int)((work + 255) / 256 < 148 * 8 ? (work + 255) / 256 : 148 * 8);
     kllm_launch((gather_sorted_kernel), dim3(grid), dim3(256), 0, (cudaStream_t)stream, (bf16*)xs, (const bf16*)x, x_stride, perm, rows,
-                top, K);
+                top, K, count);
     KLLM_LAUNCH_STATUS();
 }
 
-// a [rows, K] bfloat16 in sorted order (dense rows), w [E, (gated ? 2 : 1) * N, K] bfloat16 contiguous.
-// gated: c bfloat16 [rows, N] in sorted order; else c float32 [rows, N] at row perm[r], times wt[perm[r]]
+// a [rows, K] bfloat16 in sorted order (dense rows), w [E, (form 1 ? 2 : 1) * N, K] bfloat16 contiguous.
+// form 1 (gated), 2 (plain): c bfloat16 [rows, N] in sorted order; form 0 (down): c float32 [rows, N] at row perm[r], times wt[perm[r]]
 // when scale_out.  status: device int that a wait which ran out sets (1: producer, 2: accumulator,
 // 3: stage, 4: epilogue).
 extern "C" int kllm_moe_gemm_tcgen05(void* c, const void* a, const void* w, const int* offsets, const int* perm,
-                                     const float* wt, int rows, int E, int N, int K, int gated, int scale_out,
+                                     const float* wt, int rows, int E, int N, int K, int form, int scale_out,
                                      int act_kind, float act_limit, float act_alpha, int* status, void* stream) {
     if (rows <= 0) return 0;
-    if (!kllm_moe_gemm_tcgen05_fits(a, w, c, rows, E, N, K, gated))
+    if (!kllm_moe_gemm_tcgen05_fits(a, w, c, rows, E, N, K, form))
         KLLM_FAIL("moe gemm (tcgen05): sizes %d rows, %d experts, %d x %d or an address not taken", rows, E, N, K);
-    if (act_kind < 0 || act_kind > 1) KLLM_FAIL("moe gemm (tcgen05): unknown activation %d", act_kind);
+    if (act_kind < 0 || act_kind > 1 || form < 0 || form > 2)
+        KLLM_FAIL("moe gemm (tcgen05): unknown activation %d or form %d", act_kind, form);
+    const bool gated = form == GATE_UP;
     const GatedAct act = {act_kind, act_limit, act_alpha};
     const int row_tiles = rows / BM + E;
-    const int bn = pick_bn(row_tiles, N, gated != 0);
+    const int bn = pick_bn(row_tiles, N, gated);
     CUtensorMap ma, mb;
     int r = tensor_map(&ma, a, K, rows, K, BM);
     if (r) return r;
     r = tensor_map(&mb, w, K, E * (gated ? 2 : 1) * N, K, gated ? bn / 2 : bn);
     if (r) return r;
     cudaStream_t s = (cudaStream_t)stream;
-    if (gated) return launch<true>(ma, mb, c, offsets, perm, wt, rows, E, N, K, bn, scale_out, act, status, s);
-    return launch<false>(ma, mb, c, offsets, perm, wt, rows, E, N, K, bn, scale_out, act, status, s);
+    if (gated) return launch<GATE_UP>(ma, mb, c, offsets, perm, wt, rows, E, N, K, bn, scale_out, act, status, s);
+    if (form == PLAIN_UP) return launch<PLAIN_UP>(ma, mb, c, offsets, perm, wt, rows, E, N, K, bn, scale_out, act, status, s);
+    return launch<DOWN>(ma, mb, c, offsets, perm, wt, rows, E, N, K, bn, scale_out, act, status, s);
 }

@@ -199,7 +199,7 @@ rmsnorm_add_kernel(float* __restrict__ x, const float* __restrict__ y, const flo
     for (int i = threadIdx.x; i < d; i += blockDim.x) orow[i] = from_f32<T>(xr[i] * scale2 * gain2[i]);
 }
 
-// Layer norm with gain and bias, the residual sum folded in as in add_rmsnorm_kernel:
+// Layer norm with gain and an optional bias, the residual sum folded in as in add_rmsnorm_kernel:
 //
 //   x[r,:] (+)= res[r,:]
 //   out[r,:] = (x[r,:] - mean) * rsqrt(var + eps) * gain[:] + bias[:]
@@ -242,7 +242,7 @@ add_layernorm_kernel(float* __restrict__ x, const R* __restrict__ res, T* __rest
     for (int i = threadIdx.x; i < d; i += blockDim.x) {
         float v = xr[i];
         if (rr && !write_back) v += to_f32(rr[i]);
-        orow[i] = from_f32<T>((v - mean) * scale * gain[i] + bias[i]);
+        orow[i] = from_f32<T>((v - mean) * scale * gain[i] + (bias ? bias[i] : 0.f));
     }
 }
 
@@ -296,7 +296,7 @@ add_layernorm_vec4_kernel(float* __restrict__ x, const float* __restrict__ res, 
     for (int k = 0; k < kVec; k++) {
         const int i = threadIdx.x + k * kThreads;
         if (i < n4) {
-            const float4 g = g4[i], b = b4[i];
+            const float4 g = g4[i], b = bias ? b4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
             const float o0 = v[k].x * scale * g.x + b.x, o1 = v[k].y * scale * g.y + b.y;
             const float o2 = v[k].z * scale * g.z + b.z, o3 = v[k].w * scale * g.w + b.w;
             if (sizeof(T) == 4) {
@@ -313,7 +313,158 @@ add_layernorm_vec4_kernel(float* __restrict__ x, const float* __restrict__ res, 
     }
 }
 
+// four neighbouring elements of a row, stored at once
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(bf16* p, float4 v) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 pk;
+    pk.x = *reinterpret_cast<uint32_t*>(&lo);
+    pk.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = pk;
+}
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const bf16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+// Layer norm of a row y whose result joins or becomes the residual stream, one CTA per row:
+//
+//   v        = (y[r,:] - mean) * rsqrt(var + eps) * gain[:] (+ bias[:])
+//   ADD      x[r,:] += v, y float32 row r (a norm on a sublayer's OUTPUT)
+//   !ADD     x[r,:]  = v, y the table's row of token r times `mult` (the norm of an embedding; ids as in embedding.cu)
+//   rows[r,:] = x[r,:] in T, if `rows` is given: the next sublayer's input
+//
+// VEC: width a multiple of 4 up to kThreads * 4 * kVec, 16-byte rows; a thread keeps its elements in registers.  Which
+// form runs, and the block's size, follow from the width and the addresses alone.
+template <typename S, typename T, bool ADD, bool VEC>
+__global__ void __launch_bounds__(kThreads)
+layernorm_join_kernel(float* __restrict__ x, const S* __restrict__ src, const int* __restrict__ ids,
+                      const int* __restrict__ last_token, int vocab, float mult, const float* __restrict__ gain,
+                      const float* __restrict__ bias, float eps, T* __restrict__ rows, int d) {
+    __shared__ float red[32];
+    griddep_wait();
+    griddep_launch();
+    const int r = blockIdx.x;
+    int64_t at = r;
+    bool bad = false;
+    if (!ADD) {
+        int id = ids[r];
+        if (id < 0 && last_token != nullptr) id = last_token[-id - 1];
+        bad = id < 0 || id >= vocab;                         // such a row becomes NaN
+        at = bad ? 0 : id;
+    }
+    const S* yr = src + at * d;
+    float* xr = x + (int64_t)r * d;
+    T* orow = rows ? rows + (int64_t)r * d : nullptr;
+    const float nan = __int_as_float(0x7fc00000);
+    if constexpr (VEC) {
+        const int n4 = d >> 2;
+        float4 v[kVec];
+        float sum = 0.f;
+#pragma unroll
+        for (int k = 0; k < kVec; k++) {
+            const int i = threadIdx.x + k * blockDim.x;
+            if (i < n4) {
+                v[k] = load4(yr + 4 * i);
+                if (!ADD) { v[k].x *= mult; v[k].y *= mult; v[k].z *= mult; v[k].w *= mult; }
+                sum += (v[k].x + v[k].y) + (v[k].z + v[k].w);
+            }
+        }
+        const float mean = block_sum(sum, red) / (float)d;
+        float sq = 0.f;
+#pragma unroll
+        for (int k = 0; k < kVec; k++) {
+            if (threadIdx.x + k * blockDim.x < n4) {
+                v[k].x -= mean; v[k].y -= mean; v[k].z -= mean; v[k].w -= mean;
+                sq += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+            }
+        }
+        const float scale = bad ? nan : rsqrtf(block_sum(sq, red) / (float)d + eps);
+#pragma unroll
+        for (int k = 0; k < kVec; k++) {
+            const int i = threadIdx.x + k * blockDim.x;
+            if (i < n4) {
+                const float4 g = load4(gain + 4 * i);
+                float4 o = make_float4(v[k].x * scale * g.x, v[k].y * scale * g.y, v[k].z * scale * g.z, v[k].w * scale * g.w);
+                if (bias) {
+                    const float4 b = load4(bias + 4 * i);
+                    o.x += b.x; o.y += b.y; o.z += b.z; o.w += b.w;
+                }
+                if (ADD) {
+                    const float4 a = load4(xr + 4 * i);
+                    o.x += a.x; o.y += a.y; o.z += a.z; o.w += a.w;
+                }
+                store4(xr + 4 * i, o);
+                if (orow) store4(orow + 4 * i, o);
+            }
+        }
+    } else {
+        float sum = 0.f;
+        for (int i = threadIdx.x; i < d; i += blockDim.x) sum += to_f32(yr[i]) * (ADD ? 1.f : mult);
+        const float mean = block_sum(sum, red) / (float)d;
+        float sq = 0.f;
+        for (int i = threadIdx.x; i < d; i += blockDim.x) {
+            const float v = to_f32(yr[i]) * (ADD ? 1.f : mult) - mean;
+            sq += v * v;
+        }
+        const float scale = bad ? nan : rsqrtf(block_sum(sq, red) / (float)d + eps);
+        for (int i = threadIdx.x; i < d; i += blockDim.x) {
+            float o = (to_f32(yr[i]) * (ADD ? 1.f : mult) - mean) * scale * gain[i] + (bias ? bias[i] : 0.f);
+            if (ADD) o += xr[i];
+            xr[i] = o;
+            if (orow) orow[i] = from_f32<T>(o);
+        }
+    }
+}
+
+template <typename S, bool ADD>
+int launch_layernorm_join(float* x, const void* src, const int* ids, const int* last_token, int vocab, float mult,
+                          const float* gain, const float* bias, float eps, void* rows, int n_rows, int d, int rows_dtype,
+                          cudaStream_t s) {
+    const uintptr_t addr = (uintptr_t)x | (uintptr_t)src | (uintptr_t)gain | (uintptr_t)bias | (uintptr_t)rows;
+    const bool vec = (d & 3) == 0 && d <= kThreads * 4 * kVec && !(addr & 15);
+    const int threads = d <= 512 ? 64 : (d <= 2048 ? 128 : kThreads);
+#define KLLM_LNJ(T, VEC)                                                                                              \
+    kllm_launch((layernorm_join_kernel<S, T, ADD, VEC>), dim3(n_rows), dim3(threads), 0, s, x, (const S*)src, ids, last_token, \
+                vocab, mult, gain, bias, eps, (T*)rows, d)
+    if (rows && rows_dtype == KLLM_BF16) {
+        if (vec) KLLM_LNJ(bf16, true); else KLLM_LNJ(bf16, false);
+    } else {
+        if (vec) KLLM_LNJ(float, true); else KLLM_LNJ(float, false);
+    }
+#undef KLLM_LNJ
+    KLLM_LAUNCH_STATUS();
+}
+
 }  // namespace
+
+// x float32 [n][d] += layernorm(y) * gain (+ bias), y float32 [n][d]; rows (optional, element type `dtype`) [n][d]: the
+// updated rows.  gain, bias float32 [d], bias may be NULL.
+extern "C" int kllm_layernorm_add(float* x, const float* y, const float* gain, const float* bias, float eps, void* rows,
+                                  int n_rows, int d, int dtype, void* stream) {
+    if (n_rows <= 0) return 0;
+    if (d <= 0 || !gain || (dtype != KLLM_F32 && dtype != KLLM_BF16)) KLLM_FAIL("layernorm_add: width %d, element type %d, or no gain", d, dtype);
+    return launch_layernorm_join<float, true>(x, y, nullptr, nullptr, 0, 1.f, gain, bias, eps, rows, n_rows, d, dtype,
+                                              (cudaStream_t)stream);
+}
+
+// x float32 [n][d] = layernorm(table[ids[r]] * mult) * gain (+ bias); table [vocab][d] in `table_dtype`; rows (optional,
+// element type `dtype`) the same rows.  Ids as in kllm_embed.
+extern "C" int kllm_embed_layernorm(float* x, const void* table, const int* ids, const int* last_token, int vocab, float mult,
+                                    const float* gain, const float* bias, float eps, void* rows, int n_rows, int d,
+                                    int table_dtype, int dtype, void* stream) {
+    if (n_rows <= 0) return 0;
+    if (d <= 0 || !gain || (dtype != KLLM_F32 && dtype != KLLM_BF16)) KLLM_FAIL("embed_layernorm: width %d, element type %d, or no gain", d, dtype);
+    cudaStream_t s = (cudaStream_t)stream;
+    if (table_dtype == KLLM_F32)
+        return launch_layernorm_join<float, false>(x, table, ids, last_token, vocab, mult, gain, bias, eps, rows, n_rows, d, dtype, s);
+    if (table_dtype == KLLM_BF16)
+        return launch_layernorm_join<bf16, false>(x, table, ids, last_token, vocab, mult, gain, bias, eps, rows, n_rows, d, dtype, s);
+    KLLM_FAIL("embed_layernorm: unknown element type %d", table_dtype);
+}
 
 // x float32 [n][d] (updated), y float32 [n][d], gain float32 [d]; out (optional, element type
 // `dtype`) [n][d] with gain2 [d]; gain2 NULL: out gets the updated rows as they are, in its element type.
@@ -369,13 +520,13 @@ extern "C" int kllm_add_rmsnorm(void* x, const void* res, void* out, const void*
     KLLM_LAUNCH_STATUS();
 }
 
-// Layer norm with gain and bias (both float32 [d]); the other arguments as in kllm_add_rmsnorm.
+// Layer norm with gain and bias (both float32 [d]; bias may be NULL); the other arguments as in kllm_add_rmsnorm.
 extern "C" int kllm_add_layernorm(void* x, const void* res, void* out, const void* gain, const void* bias,
                                   const int* rows, int n_rows, int d, float eps, int dtype, int res_dtype,
                                   void* stream) {
     if (n_rows <= 0) return 0;
     if (d <= 0) KLLM_FAIL("layernorm: width %d must be positive", d);
-    if (!gain || !bias) KLLM_FAIL("layernorm: gain and bias are required");
+    if (!gain) KLLM_FAIL("layernorm: the gain is required");
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = d <= 512 ? 64 : (d <= 2048 ? 128 : kThreads);
     auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };

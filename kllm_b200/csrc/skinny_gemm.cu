@@ -19,8 +19,8 @@
 //                         silu(gate row) * (up row) as bfloat16 [n, F]
 //                         (backend/model.cu:477-483, :1112-1114)
 // Compiled with -DKLLM_BIAS=1 (a library of its own, so that the plain kernels keep their code) the
-// adding epilogue also adds a bias, and the gated one adds biases to both rows' sums and may take
-// the tanh gelu in place of silu.
+// adding epilogue also adds a bias, the gated one adds biases to both rows' sums and may take
+// the tanh gelu or the clamped form in place of silu, and the bfloat16 one may square the relu.
 //
 // Layout of the work: a tile is 16 weight rows (for SWIGLU 8 gate rows and the 8 up
 // rows that go with them).  A CTA of 16 warps, one per SM, walks tiles tile = blockIdx.x,
@@ -68,7 +68,8 @@ struct Args {
 #ifdef KLLM_BIAS
     const float* bias;      // ADD_F32: optional [N], joins the sum; SWIGLU: optional [N], to the gate rows' sums
     const float* bias_up;   // SWIGLU: optional [N], to the up rows' sums
-    int gelu;               // SWIGLU: the activation is the gelu with tanh instead of silu
+    int act;                // SWIGLU: 0 silu, 1 the gelu with tanh, 2 clamped (limit, alpha); STORE_BF16: 3 the square of relu
+    float limit, alpha;     // act 2: g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(alpha g') (u' + 1)
 #endif
 };
 
@@ -344,7 +345,13 @@ skinny_gemm_kernel(const Args a) {
 #ifdef KLLM_BIAS
                     if (a.bias) v += a.bias[col];
                     if (a.bias_up) u += a.bias_up[col];
-                    if (a.gelu) {
+                    if (a.act == 2) {
+                        v = fminf(v, a.limit);
+                        u = fminf(fmaxf(u, -a.limit), a.limit);
+                        a.y_bf16[(int64_t)c * a.y_stride + col] = __float2bfloat16_rn(v / (1.f + expf(-a.alpha * v)) * (u + 1.f));
+                        continue;
+                    }
+                    if (a.act == 1) {
                         const float act = 0.5f * v * (1.f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)));
                         a.y_bf16[(int64_t)c * a.y_stride + col] = __float2bfloat16_rn(act * u);
                         continue;
@@ -352,6 +359,12 @@ skinny_gemm_kernel(const Args a) {
 #endif
                     a.y_bf16[(int64_t)c * a.y_stride + col] = __float2bfloat16_rn((v / (1.f + expf(-v))) * u);
                 } else if (EPI == STORE_BF16) {
+#ifdef KLLM_BIAS
+                    if (a.act == 3) {
+                        v = fmaxf(v, 0.f);
+                        v *= v;
+                    }
+#endif
                     a.y_bf16[(int64_t)c * a.y_stride + col] = __float2bfloat16_rn(v);
                 } else if (EPI == STORE_F32) {
                     a.y_f32[(int64_t)c * a.y_stride + col] = v;
@@ -448,13 +461,13 @@ extern "C" int kllm_skinny_gemm_fits(int n, int K) {
 // w_stride: elements from one weight row to the next (>= K; more than K when the call
 // multiplies a slice of the columns of a wider matrix, which is how a K too long for
 // shared memory is taken: one call per slice, each adding into y_f32).
-// bias, bias_up, gelu: see Args; refused by a library compiled without KLLM_BIAS.
+// bias, bias_up, act, limit, alpha: see Args; refused by a library compiled without KLLM_BIAS.
 // prefetch: optional, `prefetch_bytes` bytes that a later kernel will stream; they are
 // requested into L2 before this kernel's own work.
 extern "C" int kllm_skinny_gemm(const void* w, const void* w_up, int64_t w_stride, int N, int K, int n, const void* x_bf16,
                                 int64_t x_stride, const float* x_f32, const float* gain, const int* rows,
                                 float eps, void* y_bf16, float* y_f32, int64_t y_stride, int prologue,
-                                int epilogue, const float* bias, const float* bias_up, int gelu,
+                                int epilogue, const float* bias, const float* bias_up, int act, float limit, float alpha,
                                 const void* prefetch, int64_t prefetch_bytes, void* stream) {
     if (n <= 0 || N <= 0) return 0;
     if (!kllm_skinny_gemm_fits(n, K))
@@ -475,9 +488,11 @@ extern "C" int kllm_skinny_gemm(const void* w, const void* w_up, int64_t w_strid
     if (prefetch && ((uintptr_t)prefetch & 15)) KLLM_FAIL("skinny_gemm: the matrix to prefetch must be 16-byte aligned");
     a.prefetch = prefetch; a.prefetch_bytes = prefetch ? prefetch_bytes : 0;
 #ifdef KLLM_BIAS
-    a.bias = bias; a.bias_up = bias_up; a.gelu = gelu;
+    if (act < 0 || act > 3 || (act && epilogue != (act == 3 ? STORE_BF16 : SWIGLU)) || (act == 2 && !(limit > 0.f)))
+        KLLM_FAIL("skinny_gemm: activation %d does not go with epilogue %d", act, epilogue);
+    a.bias = bias; a.bias_up = bias_up; a.act = act; a.limit = limit; a.alpha = alpha;
 #else
-    if (bias || bias_up || gelu) KLLM_FAIL("skinny_gemm: this library was built without biases");
+    if (bias || bias_up || act) KLLM_FAIL("skinny_gemm: this library was built without biases and activations");
 #endif
     a.tl_slot = TL_SLOT();
     cudaStream_t s = (cudaStream_t)stream;

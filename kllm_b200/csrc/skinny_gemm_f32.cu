@@ -52,7 +52,8 @@ struct Args {
 #ifdef KLLM_BIAS
     const float* bias;    // ADD: optional [N], joins the sum; SWIGLU: optional [N], to the gate rows' sums
     const float* bias_up; // SWIGLU: optional [N], to the up rows' sums
-    int gelu;             // SWIGLU: the activation is the gelu with tanh instead of silu
+    int act;              // SWIGLU: 0 silu, 1 the gelu with tanh, 2 clamped (limit, alpha); STORE: 3 the square of relu
+    float limit, alpha;   // act 2: g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(alpha g') (u' + 1)
 #endif
 };
 
@@ -204,7 +205,15 @@ skinny_f32_kernel(const Args a) {
 #ifdef KLLM_BIAS
                     if (EPI != STORE && a.bias) v += a.bias[col];
                     if (EPI == SWIGLU && a.bias_up) up += a.bias_up[col];
-                    if (EPI == SWIGLU && a.gelu)
+                    if (EPI == STORE && a.act == 3) {
+                        v = fmaxf(v, 0.f);
+                        v *= v;
+                    }
+                    if (EPI == SWIGLU && a.act == 2) {
+                        v = fminf(v, a.limit);
+                        up = fminf(fmaxf(up, -a.limit), a.limit);
+                        *dst = v / (1.f + expf(-a.alpha * v)) * (up + 1.f);
+                    } else if (EPI == SWIGLU && a.act == 1)
                         *dst = 0.5f * v * (1.f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v))) * up;
                     else
 #endif
@@ -260,11 +269,11 @@ extern "C" int kllm_skinny_gemm_f32_fits(int n, int K) {
 // given) normalised with gain [K] and eps.  epilogue 0: y written; 1: y += result; 2: w = gate
 // [N, K], w_up = up [N, K], y = silu(gate) * up.  w_stride: elements from one weight row to the
 // next (more than K when the call multiplies a slice of the columns of a wider matrix).
-// bias, bias_up, gelu: see Args; refused by a library compiled without KLLM_BIAS (as in skinny_gemm.cu).
+// bias, bias_up, act, limit, alpha: see Args; refused by a library compiled without KLLM_BIAS (as in skinny_gemm.cu).
 extern "C" int kllm_skinny_gemm_f32(const float* w, const float* w_up, int64_t w_stride, int N, int K, int n,
                                     const float* x, int64_t x_stride, const float* gain, const int* rows, float eps,
                                     float* y, int64_t y_stride, int prologue, int epilogue, const float* bias,
-                                    const float* bias_up, int gelu, void* stream) {
+                                    const float* bias_up, int act, float limit, float alpha, void* stream) {
     if (n <= 0 || N <= 0) return 0;
     if (!kllm_skinny_gemm_f32_fits(n, K))
         KLLM_FAIL("skinny_gemm_f32: %d rows of width %d not supported (1..8 rows, width a multiple of 128 that fits "
@@ -277,9 +286,11 @@ extern "C" int kllm_skinny_gemm_f32(const float* w, const float* w_up, int64_t w
     a.w = w; a.w_up = w_up; a.w_stride = w_stride; a.N = N; a.K = K; a.n = n; a.x = x; a.x_stride = x_stride;
     a.gain = gain; a.rows = rows; a.eps = eps; a.y = y; a.y_stride = y_stride;
 #ifdef KLLM_BIAS
-    a.bias = bias; a.bias_up = bias_up; a.gelu = gelu;
+    if (act < 0 || act > 3 || (act && epilogue != (act == 3 ? STORE : SWIGLU)) || (act == 2 && !(limit > 0.f)))
+        KLLM_FAIL("skinny_gemm_f32: activation %d does not go with epilogue %d", act, epilogue);
+    a.bias = bias; a.bias_up = bias_up; a.act = act; a.limit = limit; a.alpha = alpha;
 #else
-    if (bias || bias_up || gelu) KLLM_FAIL("skinny_gemm_f32: this library was built without biases");
+    if (bias || bias_up || act) KLLM_FAIL("skinny_gemm_f32: this library was built without biases and activations");
 #endif
     cudaStream_t s = (cudaStream_t)stream;
 #define KLLM_F32_CASE(P, E) if (prologue == P && epilogue == E) return launch<P, E>(a, s)

@@ -1,0 +1,810 @@
+// A state-space recurrence with one decay per head and token (Mamba-2), for mixed batches of prompt portions and
+// single tokens, with the state of every request in slots of two state tensors.
+//
+// A row of projections holds [z: H dv | x: H dv | B: G N | C: G N | dt: H].  x, B and C together pass a causal convolution
+// per channel and silu; then, per head h with its group g = h / (H / G) and a state S [N][dv] that starts at zero,
+//
+//     dt  = softplus(dt + dt_bias)            a_t = exp(-exp(A_log) dt_t)
+//     S_t = a_t S_(t-1) + dt_t B_t x_t^T      y_t = (S_t^T C_t + D x_t) * silu(z_t)
+//
+// and y is RMS-normed in equal parts of the row, times a gain.  Everything is float32; the normed row alone is stored in the
+// model's type.
+//
+// The convolution's inputs of the last `taps` positions live in a ring [taps][channels] per request, position p in entry
+// p mod taps: a step writes the entry of its own position and reads the others, so CTAs that share channels do not
+// depend on one another.
+//
+// Steps in which every request brings one row take one kernel (step_kernel) and the norm: a CTA per (slice of value
+// channels, head, request) forms its own channels of the convolution, updates its part of the state in registers
+// (requested before the projections are waited for) and gates its values.
+//
+// Steps with portions cut a request's rows into chunks of kC rows.  With c_i the sum of the chunk's decay logarithms
+// up to and including row i,
+//
+//     y_i   = exp(c_i) C_i^T S_in + sum over j <= i of (C_i . B_j) exp(c_i - c_j) dt_j x_j
+//     S_out = exp(c_last) S_in + sum over j of exp(c_last - c_j) dt_j B_j x_j^T
+//
+//   conv_kernel    convolution and silu of every channel; dt and the c_i of every head
+//   pairs_kernel   C_i . B_j per (chunk, group), which the group's heads share
+//   outer_kernel   every chunk's own addition to the state
+//   carry_kernel   the states at the chunks' starts, element by element over a request's chunks in order;
+//                  moves the slot on
+//   apply_kernel   y of every chunk, with D and the gate
+//   part_norm_kernel
+// The c_i may reach tens of thousands while their differences are small: they are summed in double precision and
+// kept as two floats, whose differences are formed pairwise.  Where a prompt is cut changes the order of float32 sums and
+// nothing else.
+#include "common.cuh"
+
+KLLM_EXPORT_LAST_ERROR(ssd)
+
+namespace {
+
+constexpr int kC = 64;          // rows of a chunk
+constexpr int kThreads = 256;
+
+struct SsdArgs {
+    const float* proj;                      // [n] rows at `stride`
+    int64_t stride;
+    const float *conv_w, *conv_b;           // [channels][taps], [channels]
+    const float *dt_bias, *a_log, *d;       // [H]
+    int taps, heads, groups, N, dv, inner, channels;
+    const int *q_start, *start_pos, *state_slots;
+    int n_requests;
+    float* state;                           // [slots][state_stride]: S as [H][N][dv]
+    int64_t state_stride;
+    float* ring;                            // [slots][ring_stride]: [taps][ch_pad]
+    int64_t ring_stride;
+    int ch_pad;                             // channels rounded up to a multiple of 4: row length of ring and xc
+    float* y;                               // [n][inner]: gated, before the norm
+    // work of the form for portions
+    float* xc;                              // [n][ch_pad]: x, B, C behind the convolution
+    float* dt;                              // [chunks][H][kC]
+    float2* cum;                            // [chunks][H][kC]
+    float* pairs;                           // [chunks][G][kC][kC]
+    float* s_in;                            // [chunks][H][N][dv]
+    bool vec;                               // sizes and addresses allow 16-byte accesses
+};
+
+__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// exp(a - b) of two sums kept as (high, low)
+__device__ __forceinline__ float exp_diff(float2 a, float2 b) { return expf((a.x - b.x) + (a.y - b.y)); }
+
+template <int V> struct Vec { float x[V]; };
+template <int V> __device__ __forceinline__ Vec<V> load_vec(const float* p) {
+    Vec<V> r;
+    if constexpr (V == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        r.x[0] = t.x; r.x[1] = t.y; r.x[2] = t.z; r.x[3] = t.w;
+    } else {
+#pragma unroll
+        for (int i = 0; i < V; i++) r.x[i] = p[i];
+    }
+    return r;
+}
+template <int V> __device__ __forceinline__ void store_vec(float* p, const Vec<V>& r) {
+    if constexpr (V == 4) {
+        *reinterpret_cast<float4*>(p) = make_float4(r.x[0], r.x[1], r.x[2], r.x[3]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < V; i++) p[i] = r.x[i];
+    }
+}
+
+// ---- one row per request -----------------------------------------------------------------------------------
+// grid (slices, heads, requests).  Thread (cg, nl): V value channels e0 + cg V ..., state channels nl, nl + lanes, ...
+// Shared memory: partial sums [kThreads * V], x [sl], B [N], C [N].  Started early, the kernel reads state and ring before
+// the kernel in front of it has ended: that kernel must write neither.
+template <int V>
+__global__ void __launch_bounds__(kThreads)
+step_kernel(const SsdArgs a, int sl) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int NB = V == 4 ? 8 : 16;                     // state channels in flight per thread
+    const int tid = threadIdx.x, slice = blockIdx.x, head = blockIdx.y, req = blockIdx.z;
+    const int N = a.N, dv = a.dv, per = a.heads / a.groups, group = head / per;
+    float* ps = sm;                                         // [kThreads * V], 16-byte aligned
+    float* xs = ps + kThreads * V;                          // [sl], a multiple of V
+    float* bs = xs + sl;                                    // B [N], then C [N]
+    const int t = a.q_start[req], p = a.start_pos[req], slot = a.state_slots[req];
+    const int nv = sl / V, lanes = kThreads / nv, cg = tid % nv, nl = tid / nv;
+    const bool on = nl < lanes;
+    const int e = slice * sl + cg * V;
+    float* Sg = a.state + (int64_t)slot * a.state_stride + (int64_t)head * N * dv + e;
+    Vec<V> s[NB];
+#pragma unroll
+    for (int i = 0; i < NB; i++) {
+        const int n = nl + i * lanes;
+        if (on && n < N) s[i] = load_vec<V>(Sg + (int64_t)n * dv);
+    }
+    float* ring = a.ring + (int64_t)slot * a.ring_stride;
+    const int mine = sl + 2 * N;                            // channels that this CTA convolves: x slice, B, C
+    auto channel = [&](int i) {
+        return i < sl ? head * dv + slice * sl + i : i < sl + N ? a.inner + group * N + (i - sl)
+                                                               : a.inner + a.groups * N + group * N + (i - sl - N);
+    };
+    // what earlier rows put into the first channel's sum, before the projections are waited for
+    auto before = [&](int c) {
+        float v = a.conv_b[c];
+        const float* w = a.conv_w + (int64_t)c * a.taps;
+        for (int i = 0; i < a.taps - 1; i++) {
+            const int q = p - (a.taps - 1) + i;
+            if (q >= 0) v = fmaf(w[i], ring[(int64_t)(q % a.taps) * a.ch_pad + c], v);
+        }
+        return v;
+    };
+    const float first = tid < mine ? before(channel(tid)) : 0.f;
+    const float rate = expf(a.a_log[head]), dbias = a.dt_bias[head], dskip = a.d[head];
+    griddep_wait();
+    griddep_launch();
+    const float* row = a.proj + (int64_t)t * a.stride;
+    const float* u = row + a.inner;
+    for (int i = tid; i < mine; i += kThreads) {
+        const int c = channel(i);
+        const float in = u[c];
+        const float v = silu_f(fmaf(a.conv_w[(int64_t)c * a.taps + a.taps - 1], in, i == tid ? first : before(c)));
+        xs[i] = v;                                          // x slice, B and C lie one behind the other
+        // one CTA moves each channel's ring on: x its own, B and C the group's first head
+        if (i < sl || (slice == 0 && head == group * per)) ring[(int64_t)(p % a.taps) * a.ch_pad + c] = in;
+    }
+    const float dt = softplus_f(row[a.inner + a.channels + head] + dbias);
+    const float al = expf(-rate * dt);
+    __syncthreads();
+    if (on) {
+        Vec<V> xv, acc;
+#pragma unroll
+        for (int j = 0; j < V; j++) {
+            xv.x[j] = xs[cg * V + j] * dt;
+            acc.x[j] = 0.f;
+        }
+        const float* cs = bs + N;
+        for (int n0 = nl; n0 < N; n0 += NB * lanes) {
+            if (n0 != nl) {
+#pragma unroll
+                for (int i = 0; i < NB; i++) {
+                    const int n = n0 + i * lanes;
+                    if (n < N) s[i] = load_vec<V>(Sg + (int64_t)n * dv);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < NB; i++) {
+                const int n = n0 + i * lanes;
+                if (n < N) {
+                    const float b = bs[n], c = cs[n];
+#pragma unroll
+                    for (int j = 0; j < V; j++) {
+                        s[i].x[j] = fmaf(al, s[i].x[j], b * xv.x[j]);
+                        acc.x[j] = fmaf(c, s[i].x[j], acc.x[j]);
+                    }
+                    store_vec<V>(Sg + (int64_t)n * dv, s[i]);
+                }
+            }
+        }
+        store_vec<V>(ps + nl * sl + cg * V, acc);
+    }
+    __syncthreads();
+    const float* z = row + head * dv + slice * sl;
+    float* yr = a.y + (int64_t)t * a.inner + head * dv + slice * sl;
+    for (int c = tid; c < sl; c += kThreads) {
+        float o = 0.f;
+        for (int l = 0; l < lanes; l++) o += ps[l * sl + c];
+        yr[c] = fmaf(dskip, xs[c], o) * silu_f(z[c]);
+    }
+}
+
+// ---- portions ------------------------------------------------------------------------------------------------
+
+// The request and first row of the step's chunk number `chunk`; false beyond the last chunk.
+__device__ __forceinline__ bool find_chunk(const SsdArgs& a, int chunk, int& req, int& row0, int& rows, int& index) {
+    for (req = 0; req < a.n_requests; req++) {
+        const int lo = a.q_start[req], len = a.q_start[req + 1] - lo, chunks = (len + kC - 1) / kC;
+        if (chunk < chunks) {
+            index = chunk;
+            row0 = lo + chunk * kC;
+            rows = min(kC, len - chunk * kC);
+            return true;
+        }
+        chunk -= chunks;
+    }
+    return false;
+}
+
+__device__ __forceinline__ void cp_async16(float* smem, const float* gmem, bool valid) {
+    const unsigned dst = (unsigned)__cvta_generic_to_shared(smem);
+    const int bytes = valid ? 16 : 0;                     // 0: the 16 bytes are filled with zeros, nothing is read
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst), "l"(gmem), "r"(bytes));
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
+
+// grid (chunk bound, blocks of kThreads channels, then blocks of kThreads heads).  A thread owns a channel of the
+// chunk's rows, or a head's decays.  TAPS > 0: that many taps, the inputs in registers; 0: any number.
+template <int TAPS>
+__global__ void __launch_bounds__(kThreads)
+conv_kernel(const SsdArgs a) {
+    griddep_wait();
+    griddep_launch();
+    int req, row0, rows, index;
+    if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
+    const int ch_blocks = (a.channels + kThreads - 1) / kThreads;
+    if ((int)blockIdx.y >= ch_blocks) {
+        const int h = (blockIdx.y - ch_blocks) * kThreads + threadIdx.x;
+        if (h >= a.heads) return;
+        const float rate = expf(a.a_log[h]), bias = a.dt_bias[h];
+        const float* src = a.proj + (int64_t)row0 * a.stride + a.inner + a.channels + h;
+        const int64_t at = ((int64_t)blockIdx.x * a.heads + h) * kC;
+        double sum = 0.0;
+#pragma unroll 8
+        for (int r = 0; r < rows; r++) {
+            const float dt = softplus_f(src[(int64_t)r * a.stride] + bias);
+            sum -= (double)(rate * dt);
+            const float hi = (float)sum;
+            a.dt[at + r] = dt;
+            a.cum[at + r] = make_float2(hi, (float)(sum - (double)hi));
+        }
+        return;
+    }
+    const int c = blockIdx.y * kThreads + threadIdx.x;
+    if (c >= a.channels) return;
+    const int taps = TAPS > 0 ? TAPS : a.taps;
+    const float* src = a.proj + (int64_t)row0 * a.stride + a.inner + c;
+    float* dst = a.xc + (int64_t)row0 * a.ch_pad + c;
+    float* ring = a.ring + (int64_t)a.state_slots[req] * a.ring_stride + c;
+    const int p0 = a.start_pos[req] + index * kC;           // position of the chunk's first row
+    const float* w = a.conv_w + (int64_t)c * taps;
+    const float bias = a.conv_b[c];
+    // input of row r, also in front of the chunk: an earlier row of the portion, or the ring
+    auto input = [&](int r) {
+        if (r >= 0 || index > 0) return src[(int64_t)r * a.stride];        // a chunk in front has kC >= taps - 1 rows
+        const int q = p0 + r;
+        return q >= 0 ? ring[(int64_t)(q % taps) * a.ch_pad] : 0.f;
+    };
+    if constexpr (TAPS > 0) {
+        float k[TAPS], u[TAPS];
+#pragma unroll
+        for (int i = 0; i < TAPS; i++) {
+            k[i] = w[i];
+            u[i] = i < TAPS - 1 ? input(i - (TAPS - 1)) : 0.f;
+        }
+        constexpr int AHEAD = 8;
+        for (int r0 = 0; r0 < rows; r0 += AHEAD) {
+            float in[AHEAD];
+#pragma unroll
+            for (int j = 0; j < AHEAD; j++) in[j] = r0 + j < rows ? src[(int64_t)(r0 + j) * a.stride] : 0.f;
+#pragma unroll
+            for (int j = 0; j < AHEAD; j++) {
+                if (r0 + j < rows) {
+                    u[TAPS - 1] = in[j];
+                    float v = bias;
+#pragma unroll
+                    for (int i = 0; i < TAPS; i++) v = fmaf(k[i], u[i], v);
+                    dst[(int64_t)(r0 + j) * a.ch_pad] = silu_f(v);
+#pragma unroll
+                    for (int i = 0; i < TAPS - 1; i++) u[i] = u[i + 1];
+                }
+            }
+        }
+    } else {
+        for (int r = 0; r < rows; r++) {
+            float v = bias;
+            for (int i = 0; i < taps; i++) v = fmaf(w[i], input(r - (taps - 1) + i), v);
+            dst[(int64_t)r * a.ch_pad] = silu_f(v);
+        }
+    }
+    if (index == 0) {
+        // the thread that has read the ring's old entries of this channel moves it on
+        const int len = a.q_start[req + 1] - a.q_start[req];
+        for (int r = max(0, len - taps); r < len; r++)
+            ring[(int64_t)((a.start_pos[req] + r) % taps) * a.ch_pad] = src[(int64_t)r * a.stride];
+    }
+}
+
+// grid (chunk bound, groups): pairs[i][j] = C_i . B_j.  Thread (ty, tx): rows 4 ty .., columns 4 tx .. .
+// Shared memory: C and B, kKP of their N values at a time, [kKP][kC + 4] each.
+constexpr int kKP = 32;
+
+__global__ void __launch_bounds__(kThreads)
+pairs_kernel(const SsdArgs a) {
+    __shared__ __align__(16) float Cs[kKP][kC + 4], Bs[kKP][kC + 4];
+    griddep_wait();
+    griddep_launch();
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4, group = blockIdx.y, N = a.N;
+    int req, row0, rows, index;
+    if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
+    const float* B = a.xc + (int64_t)row0 * a.ch_pad + a.inner + group * N;
+    const float* C = B + a.groups * N;
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+#pragma unroll
+        for (int j = 0; j < 4; j++) acc[i][j] = 0.f;
+    for (int k0 = 0; k0 < N; k0 += kKP) {
+        for (int i = tid; i < kC * kKP; i += kThreads) {
+            const int r = i / kKP, k = i - r * kKP;
+            const bool in = r < rows && k0 + k < N;
+            Cs[k][r] = in ? C[(int64_t)r * a.ch_pad + k0 + k] : 0.f;
+            Bs[k][r] = in ? B[(int64_t)r * a.ch_pad + k0 + k] : 0.f;
+        }
+        __syncthreads();
+        if (tx <= ty) {                                      // blocks of four that hold a pair j <= i
+#pragma unroll 8
+            for (int k = 0; k < kKP; k++) {
+                const float4 c4 = *reinterpret_cast<const float4*>(&Cs[k][4 * ty]);
+                const float4 b4 = *reinterpret_cast<const float4*>(&Bs[k][4 * tx]);
+                const float c[4] = {c4.x, c4.y, c4.z, c4.w}, b[4] = {b4.x, b4.y, b4.z, b4.w};
+#pragma unroll
+                for (int i = 0; i < 4; i++)
+#pragma unroll
+                    for (int j = 0; j < 4; j++) acc[i][j] = fmaf(c[i], b[j], acc[i][j]);
+            }
+        }
+        __syncthreads();
+    }
+    float* out = a.pairs + ((int64_t)blockIdx.x * a.groups + group) * kC * kC;
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+        *reinterpret_cast<float4*>(out + (4 * ty + i) * kC + 4 * tx) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+}
+
+// N consecutive values of shared memory as the register tile of thread `t` of 16: fours at 64 u + 4 t (N 4, 8), or two at 2 t
+template <int N> __device__ __forceinline__ int tile_at(int t, int i) { return N == 2 ? 2 * t + i : (i >> 2) * 64 + 4 * t + (i & 3); }
+
+// grid (chunk bound, heads, tiles of 16 RM state channels by 16 RN value channels): s_in = sum over the chunk's rows of
+// exp(c_last - c_j) dt_j B_j x_j^T.  Thread (ty, tx): an RM x RN tile.  Shared memory: B [kC][16 RM], x [kC][16 RN], weights [kC].
+template <int RM, int RN>
+__global__ void __launch_bounds__(kThreads)
+outer_kernel(const SsdArgs a, int e_tiles) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int TM = 16 * RM, TN = 16 * RN;
+    griddep_wait();
+    griddep_launch();
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    const int head = blockIdx.y, d0 = blockIdx.z / e_tiles * TM, e0 = blockIdx.z % e_tiles * TN, N = a.N, dv = a.dv;
+    int req, row0, rows, index;
+    if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
+    float* ks = sm;
+    float* vs = ks + kC * TM;
+    float* ws = vs + kC * TN;
+    const float* kg = a.xc + (int64_t)row0 * a.ch_pad + a.inner + (head / (a.heads / a.groups)) * N + d0;
+    const float* vg = a.xc + (int64_t)row0 * a.ch_pad + head * dv + e0;
+    if (a.vec) {
+        for (int i = tid; i < rows * (TM / 4); i += kThreads) {
+            const int r = i / (TM / 4), d = (i - r * (TM / 4)) * 4;
+            cp_async16(ks + r * TM + d, kg + (d0 + d < N ? (int64_t)r * a.ch_pad + d : 0), d0 + d < N);
+        }
+        for (int i = tid; i < rows * (TN / 4); i += kThreads) {
+            const int r = i / (TN / 4), c = (i - r * (TN / 4)) * 4;
+            cp_async16(vs + r * TN + c, vg + (e0 + c < dv ? (int64_t)r * a.ch_pad + c : 0), e0 + c < dv);
+        }
+        cp_async_commit();
+    } else {
+        for (int i = tid; i < rows * TM; i += kThreads) {
+            const int r = i / TM, d = i - r * TM;
+            ks[i] = d0 + d < N ? kg[(int64_t)r * a.ch_pad + d] : 0.f;
+        }
+        for (int i = tid; i < rows * TN; i += kThreads) {
+            const int r = i / TN, c = i - r * TN;
+            vs[i] = e0 + c < dv ? vg[(int64_t)r * a.ch_pad + c] : 0.f;
+        }
+    }
+    if (tid < rows) {
+        const int64_t at = ((int64_t)blockIdx.x * a.heads + head) * kC;
+        ws[tid] = exp_diff(a.cum[at + rows - 1], a.cum[at + tid]) * a.dt[at + tid];
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    float acc[RM][RN];
+#pragma unroll
+    for (int m = 0; m < RM; m++)
+#pragma unroll
+        for (int n = 0; n < RN; n++) acc[m][n] = 0.f;
+#pragma unroll 2
+    for (int r = 0; r < rows; r++) {
+        float k[RM], v[RN];
+        const float w = ws[r];
+        if constexpr (RM == 2) {
+            const float2 t = *reinterpret_cast<const float2*>(ks + r * TM + 2 * ty);
+            k[0] = t.x; k[1] = t.y;
+        } else {
+#pragma unroll
+            for (int u = 0; u < RM / 4; u++) {
+                const float4 t = *reinterpret_cast<const float4*>(ks + r * TM + u * 64 + 4 * ty);
+                k[4 * u] = t.x; k[4 * u + 1] = t.y; k[4 * u + 2] = t.z; k[4 * u + 3] = t.w;
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < RN / 4; u++) {
+            const float4 t = *reinterpret_cast<const float4*>(vs + r * TN + u * 64 + 4 * tx);
+            v[4 * u] = t.x * w; v[4 * u + 1] = t.y * w; v[4 * u + 2] = t.z * w; v[4 * u + 3] = t.w * w;
+        }
+#pragma unroll
+        for (int m = 0; m < RM; m++)
+#pragma unroll
+            for (int n = 0; n < RN; n++) acc[m][n] = fmaf(k[m], v[n], acc[m][n]);
+    }
+    float* S = a.s_in + ((int64_t)blockIdx.x * a.heads + head) * N * dv;
+#pragma unroll
+    for (int m = 0; m < RM; m++) {
+        const int d = d0 + tile_at<RM>(ty, m);
+        if (d >= N) continue;
+#pragma unroll
+        for (int u = 0; u < RN / 4; u++) {
+            const int e = e0 + u * 64 + 4 * tx;
+            if (a.vec) {
+                if (e < dv)
+                    *reinterpret_cast<float4*>(S + (int64_t)d * dv + e) =
+                        make_float4(acc[m][4 * u], acc[m][4 * u + 1], acc[m][4 * u + 2], acc[m][4 * u + 3]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < 4; i++)
+                    if (e + i < dv) S[(int64_t)d * dv + e + i] = acc[m][4 * u + i];
+            }
+        }
+    }
+}
+
+// grid (pieces of kThreads * V state elements, heads, requests): s_in turns from the chunks' own states into the
+// states at their starts.
+template <int V>
+__global__ void __launch_bounds__(kThreads)
+carry_kernel(const SsdArgs a) {
+    griddep_wait();
+    griddep_launch();
+    const int head = blockIdx.y, req = blockIdx.z;
+    const int64_t elems = (int64_t)a.N * a.dv, i = ((int64_t)blockIdx.x * kThreads + threadIdx.x) * V;
+    if (i >= elems) return;
+    int chunk = 0;
+    for (int r = 0; r < req; r++) chunk += (a.q_start[r + 1] - a.q_start[r] + kC - 1) / kC;
+    const int len = a.q_start[req + 1] - a.q_start[req], chunks = (len + kC - 1) / kC;
+    float* slot = a.state + (int64_t)a.state_slots[req] * a.state_stride + head * elems + i;
+    float* w = a.s_in + ((int64_t)chunk * a.heads + head) * elems + i;
+    const float2* cum = a.cum + ((int64_t)chunk * a.heads + head) * kC;
+    const int64_t step = a.heads * elems, cum_step = (int64_t)a.heads * kC;
+    Vec<V> s = load_vec<V>(slot);
+    constexpr int AHEAD = 8;
+    for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+        Vec<V> loc[AHEAD];
+        float d[AHEAD];
+#pragma unroll
+        for (int u = 0; u < AHEAD; u++)
+            if (c0 + u < chunks) {
+                loc[u] = load_vec<V>(w + (c0 + u) * step);
+                const float2 last = cum[(c0 + u) * cum_step + min(kC, len - (c0 + u) * kC) - 1];
+                d[u] = expf(last.x + last.y);
+            }
+#pragma unroll
+        for (int u = 0; u < AHEAD; u++)
+            if (c0 + u < chunks) {
+                store_vec<V>(w + (c0 + u) * step, s);
+#pragma unroll
+                for (int j = 0; j < V; j++) s.x[j] = fmaf(d[u], s.x[j], loc[u].x[j]);
+            }
+    }
+    store_vec<V>(slot, s);
+}
+
+// grid (chunk bound, heads, column blocks of 64 NJ): [exp(c) C | weights] [S_in ; x], in blocks of kKB inner elements, two of
+// them in shared memory.  Thread (rg, cg): rows 4 rg .. 4 rg + 3, value channels j * 64 + 4 cg .. + 3.
+// Shared memory, twice: left [kC][kKB + 4], right [kKB][64 NJ]; then the chunk's sums and steps [kC] each.
+constexpr int kKB = 32;
+
+template <int NJ>
+__global__ void __launch_bounds__(kThreads)
+apply_kernel(const SsdArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int QP = kKB + 4, CW = 64 * NJ, STAGE = kC * QP + kKB * CW;
+    griddep_wait();
+    griddep_launch();
+    const int tid = threadIdx.x, cg = tid & 15, rg = tid >> 4;
+    const int head = blockIdx.y, e0 = blockIdx.z * CW, N = a.N, dv = a.dv, group = head / (a.heads / a.groups);
+    const int ne = min(CW, dv - e0);
+    int req, row0, rows, index;
+    if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
+    float2* cum = reinterpret_cast<float2*>(sm + 2 * STAGE);
+    float* dts = reinterpret_cast<float*>(cum + kC);
+    if (tid < kC) {
+        const int64_t at = ((int64_t)blockIdx.x * a.heads + head) * kC + min(tid, rows - 1);
+        cum[tid] = a.cum[at];
+        dts[tid] = a.dt[at];
+    }
+    float acc[4][NJ * 4];
+#pragma unroll
+    for (int r = 0; r < 4; r++)
+#pragma unroll
+        for (int j = 0; j < NJ * 4; j++) acc[r][j] = 0.f;
+    const bool from_zero = index == 0 && a.start_pos[req] == 0;        // the state in front of a request's first chunk
+    const int nb_s = from_zero ? 0 : (N + kKB - 1) / kKB, nb = nb_s + (rows + kKB - 1) / kKB;
+    const float* S = a.s_in + ((int64_t)blockIdx.x * a.heads + head) * N * dv + e0;
+    const float* W = a.pairs + ((int64_t)blockIdx.x * a.groups + group) * kC * kC;
+    const float* xg = a.xc + (int64_t)row0 * a.ch_pad + head * dv + e0;
+    const float* Cg = a.xc + (int64_t)row0 * a.ch_pad + a.inner + (a.groups + group) * N;
+    auto load = [&](int b) {                // inner elements k0 .. k0 + kKB - 1 of the state's part, then of the chunk's own
+        float* left = sm + (b & 1) * STAGE;
+        float* right = left + kC * QP;
+        const bool state = b < nb_s;
+        const int k0 = (state ? b : b - nb_s) * kKB, nk = min(kKB, (state ? N : rows) - k0);
+        const float* lg = state ? Cg + k0 : W + k0;
+        const float* rg_ = state ? S + (int64_t)k0 * dv : xg + (int64_t)k0 * a.ch_pad;
+        const int64_t ls = state ? a.ch_pad : kC, rs = state ? dv : a.ch_pad;
+        if (a.vec) {
+            for (int i = tid; i < kC * (kKB / 4); i += kThreads) {
+                const int r = i / (kKB / 4), k = (i - r * (kKB / 4)) * 4;
+                const bool in = r < rows && (state ? k < nk : true);      // the pairs' rows are whole
+                cp_async16(left + r * QP + k, lg + (in ? r * ls + k : 0), in);
+            }
+            for (int i = tid; i < kKB * (CW / 4); i += kThreads) {
+                const int k = i / (CW / 4), c = (i - k * (CW / 4)) * 4;
+                const bool in = k < nk && c < ne;
+                cp_async16(right + k * CW + c, rg_ + (in ? k * rs + c : 0), in);
+            }
+        } else {
+            for (int i = tid; i < kC * kKB; i += kThreads) {
+                const int r = i / kKB, k = i - r * kKB;
+                left[r * QP + k] = (r < rows && k < nk) ? lg[r * ls + k] : 0.f;
+            }
+            for (int i = tid; i < kKB * CW; i += kThreads) {
+                const int k = i / CW, c = i - k * CW;
+                right[i] = (k < nk && c < ne) ? rg_[k * rs + c] : 0.f;
+            }
+        }
+        cp_async_commit();
+    };
+    load(0);
+    for (int b = 0; b < nb; b++) {
+        if (b + 1 < nb) {
+            load(b + 1);
+            cp_async_wait<1>();
+        } else {
+            cp_async_wait<0>();
+        }
+        __syncthreads();
+        float* qs = sm + (b & 1) * STAGE;
+        const float* ss = qs + kC * QP;
+        // the left block's decays, in place: a pair's, or the row's own towards the state
+        const bool state = b < nb_s;
+        const int k0 = state ? 0 : (b - nb_s) * kKB;
+        for (int i = tid; i < kC * kKB; i += kThreads) {
+            const int r = i / kKB, k = i - r * kKB, j = k0 + k;
+            float f;
+            if (state) f = expf(cum[r].x + cum[r].y);
+            else f = j <= r && r < rows ? exp_diff(cum[r], cum[j]) * dts[j] : 0.f;
+            qs[r * QP + k] = f == 0.f ? 0.f : qs[r * QP + k] * f;
+        }
+        __syncthreads();
+#pragma unroll 2
+        for (int d = 0; d < kKB; d += 4) {
+            float q[4][4];
+#pragma unroll
+            for (int r = 0; r < 4; r++) {
+                const float4 q4 = *reinterpret_cast<const float4*>(qs + (rg * 4 + r) * QP + d);
+                q[r][0] = q4.x; q[r][1] = q4.y; q[r][2] = q4.z; q[r][3] = q4.w;
+            }
+#pragma unroll
+            for (int j = 0; j < NJ; j++)
+#pragma unroll
+                for (int u = 0; u < 4; u++) {
+                    const float4 s4 = *reinterpret_cast<const float4*>(ss + (d + u) * CW + j * 64 + cg * 4);
+#pragma unroll
+                    for (int r = 0; r < 4; r++) {
+                        acc[r][j * 4 + 0] = fmaf(q[r][u], s4.x, acc[r][j * 4 + 0]);
+                        acc[r][j * 4 + 1] = fmaf(q[r][u], s4.y, acc[r][j * 4 + 1]);
+                        acc[r][j * 4 + 2] = fmaf(q[r][u], s4.z, acc[r][j * 4 + 2]);
+                        acc[r][j * 4 + 3] = fmaf(q[r][u], s4.w, acc[r][j * 4 + 3]);
+                    }
+                }
+        }
+        __syncthreads();                    // this stage may be loaded again
+    }
+    const float dskip = a.d[head];
+#pragma unroll
+    for (int r = 0; r < 4; r++) {
+        const int row = rg * 4 + r;
+        if (row >= rows) continue;
+        const float* xr = xg + (int64_t)row * a.ch_pad;
+        const float* zr = a.proj + (int64_t)(row0 + row) * a.stride + head * dv + e0;
+        float* yr = a.y + (int64_t)(row0 + row) * a.inner + head * dv + e0;
+#pragma unroll
+        for (int j = 0; j < NJ; j++) {
+            const int col = j * 64 + cg * 4;
+            if (a.vec) {
+                if (col >= ne) continue;
+                const float4 x4 = *reinterpret_cast<const float4*>(xr + col), z4 = *reinterpret_cast<const float4*>(zr + col);
+                *reinterpret_cast<float4*>(yr + col) =
+                    make_float4(fmaf(dskip, x4.x, acc[r][j * 4]) * silu_f(z4.x), fmaf(dskip, x4.y, acc[r][j * 4 + 1]) * silu_f(z4.y),
+                                fmaf(dskip, x4.z, acc[r][j * 4 + 2]) * silu_f(z4.z), fmaf(dskip, x4.w, acc[r][j * 4 + 3]) * silu_f(z4.w));
+            } else {
+#pragma unroll
+                for (int c = 0; c < 4; c++)
+                    if (col + c < ne) yr[col + c] = fmaf(dskip, xr[col + c], acc[r][j * 4 + c]) * silu_f(zr[col + c]);
+            }
+        }
+    }
+}
+
+// out[r][part] = y[r][part] / rms(y[r][part]) * gain: one CTA per (row, part) of w values; VEC: w a multiple of 4 up to
+// 4 * kVec * blockDim.x, 16-byte rows, the values in registers between the sum and the scaling.
+constexpr int kVec = 8;
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kThreads)
+part_norm_kernel(T* __restrict__ out, int64_t out_stride, const float* __restrict__ y, const float* __restrict__ gain, int parts,
+                 int w, float eps) {
+    __shared__ float red[32];
+    griddep_wait();
+    griddep_launch();
+    const int64_t r = blockIdx.x / parts;
+    const int part = blockIdx.x - (int)r * parts;
+    const float* src = y + (r * parts + part) * w;
+    const float* g = gain + (int64_t)part * w;
+    T* dst = out + r * out_stride + (int64_t)part * w;
+    float sq = 0.f;
+    if constexpr (VEC) {
+        const int w4 = w >> 2;
+        float4 v[kVec];
+#pragma unroll
+        for (int k = 0; k < kVec; k++) {
+            const int i = threadIdx.x + k * blockDim.x;
+            if (i < w4) {
+                v[k] = reinterpret_cast<const float4*>(src)[i];
+                sq += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+            }
+        }
+        const float scale = rsqrtf(block_sum(sq, red) / (float)w + eps);
+#pragma unroll
+        for (int k = 0; k < kVec; k++) {
+            const int i = threadIdx.x + k * blockDim.x;
+            if (i < w4) {
+                const float4 n4 = reinterpret_cast<const float4*>(g)[i];
+                const float o0 = v[k].x * scale * n4.x, o1 = v[k].y * scale * n4.y, o2 = v[k].z * scale * n4.z, o3 = v[k].w * scale * n4.w;
+                if constexpr (sizeof(T) == 4) {
+                    reinterpret_cast<float4*>(dst)[i] = make_float4(o0, o1, o2, o3);
+                } else {
+                    __nv_bfloat162 lo = __floats2bfloat162_rn(o0, o1), hi = __floats2bfloat162_rn(o2, o3);
+                    uint2 pk;
+                    pk.x = *reinterpret_cast<uint32_t*>(&lo);
+                    pk.y = *reinterpret_cast<uint32_t*>(&hi);
+                    reinterpret_cast<uint2*>(dst)[i] = pk;
+                }
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < w; i += blockDim.x) sq += src[i] * src[i];
+        const float scale = rsqrtf(block_sum(sq, red) / (float)w + eps);
+        for (int i = threadIdx.x; i < w; i += blockDim.x) dst[i] = from_f32<T>(src[i] * scale * g[i]);
+    }
+}
+
+template <int V>
+int launch_step(const SsdArgs& a, bool early, cudaStream_t s) {
+    // slices: a power of two, more of them while the launch would leave SMs idle
+    int slices = 1;
+    auto splits = [&](int n) { return a.dv % (n * V) == 0; };
+    while (a.dv / slices / V > kThreads && splits(slices * 2)) slices *= 2;
+    while (splits(slices * 2) && a.dv / (slices * 2) >= 16 && (int64_t)slices * a.heads * a.n_requests < 148) slices *= 2;
+    const int sl = a.dv / slices;
+    if (sl / V > kThreads) KLLM_FAIL("ssd step: a head of %d value channels does not fit", a.dv);
+    const size_t smem = sizeof(float) * ((size_t)kThreads * V + sl + 2 * (size_t)a.N);
+    if (smem > 200 * 1024) KLLM_FAIL("ssd step: a state of %d channels does not fit shared memory", a.N);
+    static bool raised = false;
+    if (!raised) {
+        cudaError_t e = cudaFuncSetAttribute(step_kernel<V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        if (e != cudaSuccess) KLLM_FAIL("ssd step: %s", cudaGetErrorString(e));
+        raised = true;
+    }
+    kllm_launch_dep(early, (step_kernel<V>), dim3(slices, a.heads, a.n_requests), dim3(kThreads), smem, s, a, sl);
+    KLLM_LAUNCH_STATUS();
+}
+
+template <typename K>
+int raise_smem(K kern, bool& raised) {
+    if (raised) return 0;
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+    if (e != cudaSuccess) KLLM_FAIL("ssd: %s", cudaGetErrorString(e));
+    raised = true;
+    return 0;
+}
+
+template <int RM, int RN>
+int launch_outer(const SsdArgs& a, int chunk_bound, cudaStream_t s) {
+    const int e_tiles = (a.dv + 16 * RN - 1) / (16 * RN), d_tiles = (a.N + 16 * RM - 1) / (16 * RM);
+    static bool raised = false;
+    int rc = raise_smem(outer_kernel<RM, RN>, raised);
+    if (rc) return rc;
+    kllm_launch((outer_kernel<RM, RN>), dim3(chunk_bound, a.heads, e_tiles * d_tiles), dim3(kThreads),
+                sizeof(float) * kC * (16 * (RM + RN) + 1), s, a, e_tiles);
+    KLLM_LAUNCH_STATUS();
+}
+
+template <int NJ>
+int launch_apply(const SsdArgs& a, int chunk_bound, cudaStream_t s) {
+    const size_t smem = sizeof(float) * (2 * (kC * (kKB + 4) + kKB * 64 * NJ) + 3 * kC);
+    static bool raised = false;
+    int rc = raise_smem(apply_kernel<NJ>, raised);
+    if (rc) return rc;
+    kllm_launch((apply_kernel<NJ>), dim3(chunk_bound, a.heads, (a.dv + 64 * NJ - 1) / (64 * NJ)), dim3(kThreads), smem, s, a);
+    KLLM_LAUNCH_STATUS();
+}
+
+int run_portions(const SsdArgs& a, int chunk_bound, cudaStream_t s) {
+    const dim3 grid(chunk_bound, (a.channels + kThreads - 1) / kThreads + (a.heads + kThreads - 1) / kThreads);
+    if (a.taps == 4) kllm_launch((conv_kernel<4>), grid, dim3(kThreads), 0, s, a);
+    else kllm_launch((conv_kernel<0>), grid, dim3(kThreads), 0, s, a);
+    kllm_launch((pairs_kernel), dim3(chunk_bound, a.groups), dim3(kThreads), 0, s, a);
+    int rc;
+    if (a.N <= 32) rc = a.dv <= 64 ? launch_outer<2, 4>(a, chunk_bound, s) : launch_outer<2, 8>(a, chunk_bound, s);
+    else if (a.N <= 64) rc = a.dv <= 64 ? launch_outer<4, 4>(a, chunk_bound, s) : launch_outer<4, 8>(a, chunk_bound, s);
+    else rc = a.dv <= 64 ? launch_outer<8, 4>(a, chunk_bound, s) : launch_outer<8, 8>(a, chunk_bound, s);
+    if (rc) return rc;
+    const int64_t elems = (int64_t)a.N * a.dv;
+    if (a.vec)
+        kllm_launch((carry_kernel<4>), dim3((unsigned)((elems / 4 + kThreads - 1) / kThreads), a.heads, a.n_requests), dim3(kThreads), 0, s, a);
+    else
+        kllm_launch((carry_kernel<1>), dim3((unsigned)((elems + kThreads - 1) / kThreads), a.heads, a.n_requests), dim3(kThreads), 0, s, a);
+    cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) KLLM_FAIL("ssd: %s", cudaGetErrorString(e));
+    return a.dv <= 64 ? launch_apply<1>(a, chunk_bound, s) : launch_apply<2>(a, chunk_bound, s);
+}
+
+}  // namespace
+
+extern "C" int kllm_ssd_chunk_rows() { return kC; }
+
+// proj float32 [n] rows at row stride `stride`: z, x (heads * dv each), B, C (groups * N each), dt (heads); conv_w float32
+// [channels][taps], conv_b [channels] over x, B and C; dt_bias, a_log, d float32 [heads]; state float32 [slots][state_stride] whose
+// first heads * N * dv values are S as [heads][N][dv]; ring float32 [slots][ring_stride] with taps rows of ch_pad (channels rounded
+// up to a multiple of 4); y float32 [n][heads * dv]: the gated values before the norm.  single: every request brings one
+// row; otherwise the work buffers xc [n][ch_pad], dt [chunk_bound][heads][C] (C: rows of a chunk), cum twice that, pairs
+// [chunk_bound][groups][C][C] and s_in [chunk_bound][heads][N][dv] are float32 and chunk_bound an upper bound of the chunks.
+// early (single): the kernel may start beside the end of the one before it in the stream, which must write neither
+// state nor ring.
+extern "C" int kllm_ssd(float* y, const float* proj, int64_t stride, const float* conv_w, const float* conv_b,
+                        const float* dt_bias, const float* a_log, const float* d, const int* q_start, const int* start_pos,
+                        const int* state_slots, float* state, int64_t state_stride, float* ring, int64_t ring_stride, int n,
+                        int n_requests, int heads, int groups, int N, int dv, int taps, int single, int early, int chunk_bound,
+                        float* xc, float* dt, float* cum, float* pairs, float* s_in, void* stream) {
+    if (n <= 0 || n_requests <= 0) return 0;
+    if (heads <= 0 || groups <= 0 || heads % groups || N <= 0 || dv <= 0) KLLM_FAIL("ssd: %d heads in %d groups of sizes %d, %d", heads, groups, N, dv);
+    if (taps < 1 || taps > kC) KLLM_FAIL("ssd: a convolution of %d taps (up to %d)", taps, kC);
+    if (heads > 65535 || groups > 65535 || n_requests > 65535) KLLM_FAIL("ssd: %d heads, %d requests in one launch", heads, n_requests);
+    SsdArgs a;
+    a.proj = proj; a.stride = stride; a.conv_w = conv_w; a.conv_b = conv_b; a.dt_bias = dt_bias; a.a_log = a_log; a.d = d;
+    a.taps = taps; a.heads = heads; a.groups = groups; a.N = N; a.dv = dv; a.inner = heads * dv;
+    a.channels = a.inner + 2 * groups * N; a.ch_pad = (a.channels + 3) / 4 * 4;
+    a.q_start = q_start; a.start_pos = start_pos; a.state_slots = state_slots; a.n_requests = n_requests;
+    a.state = state; a.state_stride = state_stride; a.ring = ring; a.ring_stride = ring_stride; a.y = y;
+    a.xc = xc; a.dt = dt; a.cum = (float2*)cum; a.pairs = pairs; a.s_in = s_in;
+    if (state_stride < (int64_t)heads * N * dv || ring_stride < (int64_t)taps * a.ch_pad)
+        KLLM_FAIL("ssd: slots of %lld and %lld values are too small", (long long)state_stride, (long long)ring_stride);
+    if (single && n != n_requests) KLLM_FAIL("ssd: %d rows of %d requests that bring one row each", n, n_requests);
+    if (!single && (!xc || !dt || !cum || !pairs || !s_in || chunk_bound <= 0)) KLLM_FAIL("ssd: portions need work buffers");
+    cudaStream_t s = (cudaStream_t)stream;
+    const bool rows_vec = dv % 4 == 0 && state_stride % 4 == 0 && !((uintptr_t)state & 15);
+    if (single) return rows_vec ? launch_step<4>(a, early != 0, s) : launch_step<1>(a, early != 0, s);
+    a.vec = rows_vec && N % 4 == 0 && stride % 4 == 0 &&
+            !(((uintptr_t)proj | (uintptr_t)xc | (uintptr_t)s_in | (uintptr_t)pairs | (uintptr_t)y) & 15);
+    return run_portions(a, chunk_bound, s);
+}
+
+// out [n] rows of parts * w values in `dtype` at out_stride = y / rms(y) * gain, each of the `parts` pieces of a row by its own
+// root mean square; y float32 [n][parts * w], gain float32 [parts * w].
+extern "C" int kllm_part_norm(void* out, int64_t out_stride, const float* y, const float* gain, int n, int parts, int w, float eps,
+                              int dtype, void* stream) {
+    if (n <= 0) return 0;
+    if (parts <= 0 || w <= 0) KLLM_FAIL("part norm: %d parts of %d values", parts, w);
+    if ((int64_t)n * parts > 0x7fffffffLL) KLLM_FAIL("part norm: %d rows of %d parts in one launch", n, parts);
+    const int threads = w <= 256 ? 64 : (w <= 1024 ? 128 : kThreads);
+    const int esize = dtype == KLLM_F32 ? 4 : 2;
+    const bool vec = w % 4 == 0 && w <= threads * 4 * kVec && out_stride % 4 == 0 && !(((uintptr_t)y | (uintptr_t)gain) & 15) &&
+                     !((uintptr_t)out & (4 * esize - 1));
+    cudaStream_t s = (cudaStream_t)stream;
+#define KLLM_PN(T, VEC) kllm_launch((part_norm_kernel<T, VEC>), dim3(n * parts), dim3(threads), 0, s, (T*)out, out_stride, y, gain, parts, w, eps)
+    if (dtype == KLLM_F32) {
+        if (vec) KLLM_PN(float, true); else KLLM_PN(float, false);
+    } else if (dtype == KLLM_BF16) {
+        if (vec) KLLM_PN(bf16, true); else KLLM_PN(bf16, false);
+    } else {
+        KLLM_FAIL("part norm: unknown element type %d", dtype);
+    }
+#undef KLLM_PN
+    KLLM_LAUNCH_STATUS();
+}

@@ -144,8 +144,8 @@ def add_rmsnorm(x: torch.Tensor, res: Optional[torch.Tensor], out: torch.Tensor,
 
 
 def add_layernorm(x: torch.Tensor, res: Optional[torch.Tensor], out: torch.Tensor, gain: torch.Tensor,
-                  bias: torch.Tensor, eps: float, rows: Optional[torch.Tensor] = None) -> None:
-    """x (+)= res in float32, out = (x - mean) / sqrt(var + eps) * gain + bias; ``rows`` as in
+                  bias: Optional[torch.Tensor], eps: float, rows: Optional[torch.Tensor] = None) -> None:
+    """x (+)= res in float32, out = (x - mean) / sqrt(var + eps) * gain (+ bias); ``rows`` as in
     ``add_rmsnorm`` (csrc/norm.cu)."""
     _cuda(x, res, out, gain, bias, rows)
     _i32(rows, "rows")
@@ -153,7 +153,7 @@ def add_layernorm(x: torch.Tensor, res: Optional[torch.Tensor], out: torch.Tenso
     if x.dtype != torch.float32 or not x.is_contiguous() or not out.is_contiguous() or out.shape[1] != d:
         raise KernelError("add_layernorm: x must be contiguous float32, out contiguous of the same width")
     for t in (gain, bias):
-        if t.dtype != torch.float32 or t.numel() != d or not t.is_contiguous():
+        if t is not None and (t.dtype != torch.float32 or t.numel() != d or not t.is_contiguous()):
             raise KernelError("add_layernorm: gain and bias must be contiguous float32 [d]")
     if res is not None and (res.dtype not in (out.dtype, torch.float32) or not res.is_contiguous() or res.shape != x.shape):
         raise KernelError("add_layernorm: res must match x in shape and be float32 or of out's dtype")
@@ -163,6 +163,42 @@ def add_layernorm(x: torch.Tensor, res: Optional[torch.Tensor], out: torch.Tenso
     lib = load_library("norm")
     rc = lib.kllm_add_layernorm(_p(x), _p(res), _p(out), _p(gain), _p(bias), _p(rows), n_rows, d, ctypes.c_float(eps),
                                 dtype_code(out.dtype), dtype_code(res.dtype if res is not None else out.dtype), _stream())
+    _check(lib, "norm", rc)
+
+
+def layernorm_add(x: torch.Tensor, y: torch.Tensor, gain: torch.Tensor, bias: Optional[torch.Tensor], eps: float,
+                  out: Optional[torch.Tensor] = None) -> None:
+    """x += (y - mean) / sqrt(var + eps) * gain (+ bias), all float32 [n, d]: a layer norm on a sublayer's output as it
+    joins the residual stream.  With ``out`` [n, d] also the updated rows in out's dtype."""
+    _cuda(x, y, gain, bias, out)
+    d = x.shape[1]
+    for t in (x, y):
+        if t.dtype != torch.float32 or not t.is_contiguous() or t.shape != x.shape:
+            raise KernelError("layernorm_add: x and y must be contiguous float32 of one shape")
+    _bias(gain, d, "layernorm_add"); _bias(bias, d, "layernorm_add")
+    if out is not None and (not out.is_contiguous() or out.shape != x.shape):
+        raise KernelError("layernorm_add: out contiguous like x")
+    lib = load_library("norm")
+    rc = lib.kllm_layernorm_add(_p(x), _p(y), _p(gain), _p(bias), ctypes.c_float(eps), _p(out), x.shape[0], d,
+                                dtype_code(out.dtype if out is not None else torch.float32), _stream())
+    _check(lib, "norm", rc)
+
+
+def embed_layernorm(out_x: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, gain: torch.Tensor,
+                    bias: Optional[torch.Tensor], eps: float, last_token: Optional[torch.Tensor] = None, scale: float = 1.0,
+                    rows: Optional[torch.Tensor] = None) -> None:
+    """``embed`` with a layer norm of every row in the same kernel; with ``rows`` [n, d] also the normed rows in its dtype."""
+    _cuda(out_x, table, ids, last_token, gain, bias, rows)
+    _i32(ids, "ids"); _i32(last_token, "last_token")
+    n, d = out_x.shape
+    if out_x.dtype != torch.float32 or not out_x.is_contiguous() or not table.is_contiguous() or table.shape[1] != d \
+            or ids.numel() != n or (rows is not None and (not rows.is_contiguous() or rows.shape != out_x.shape)):
+        raise KernelError("embed_layernorm: contiguous operands, x float32 [n, d], table [vocab, d], one id per row")
+    _bias(gain, d, "embed_layernorm"); _bias(bias, d, "embed_layernorm")
+    lib = load_library("norm")
+    rc = lib.kllm_embed_layernorm(_p(out_x), _p(table), _p(ids), _p(last_token), table.shape[0], ctypes.c_float(scale), _p(gain),
+                                  _p(bias), ctypes.c_float(eps), _p(rows), n, d, dtype_code(table.dtype),
+                                  dtype_code(rows.dtype if rows is not None else torch.float32), _stream())
     _check(lib, "norm", rc)
 
 
@@ -441,12 +477,12 @@ def attention_generic(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, 
                       positions: torch.Tensor, token_req: torch.Tensor, block_table: torch.Tensor,
                       n_heads: int, n_kv: int, head_dim: int, window: int, scale: float,
                       score_slopes: Optional[torch.Tensor] = None, v_head_dim: Optional[int] = None,
-                      sinks: Optional[torch.Tensor] = None, segment: int = 0) -> None:
+                      sinks: Optional[torch.Tensor] = None, segment: int = 0, keep: int = 0) -> None:
     """Causal GQA attention of every new token over its request's cached keys: one warp per
     (token, head), any head size up to 512, values of their own size, optional score slopes and
     sinks (float32 [n_heads]: exp(sinks[h]) joins the denominator of head h's softmax).
-    ``segment``, fewer value heads than key heads, value rows that head longer rows and a float32
-    ``out`` as in ``attention_simt``."""
+    ``segment``, fewer value heads than key heads, value rows that head longer rows, a float32
+    ``out`` and ``keep`` as in ``attention_simt``."""
     _cuda(out, q, kcache, vcache, positions, token_req, block_table, score_slopes, sinks)
     vd = int(v_head_dim or head_dim)
     v_heads, v_row = _value_layout(kcache, vcache, n_kv, vd)
@@ -464,8 +500,8 @@ def attention_generic(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, 
                                     n, n_heads, n_kv, head_dim, vd, kcache.shape[2], int(window or 0),
                                     ctypes.c_float(scale), _slopes_arg(score_slopes, n_heads),
                                     _slopes_arg(sinks, n_heads, "sinks"), int(segment or 0), v_heads, v_row,
-                                    int(out.dtype == torch.float32 and q.dtype != torch.float32), dtype_code(q.dtype),
-                                    _stream())
+                                    int(out.dtype == torch.float32 and q.dtype != torch.float32), int(keep or 0),
+                                    dtype_code(q.dtype), _stream())
     _check(lib, "attention_generic", rc)
 
 
@@ -481,13 +517,18 @@ def _value_layout(kcache, vcache, n_kv, vd):
     return int(vcache.shape[1]), int(vcache.shape[3])
 
 
+def _kept_room(keep) -> int:
+    """Places that the kept first keys of a window take in the kernels' walk: whole tiles of 64."""
+    return -(-int(keep or 0) // 64) * 64
+
+
 SIMT_CHUNK = 256      # keys per CTA when a decoding token's context is cut (attention_simt)
 
 
 def attention_simt(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, ctx,
                    block_table: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, window: int,
                    scale: float, score_slopes: Optional[torch.Tensor] = None, v_head_dim: Optional[int] = None,
-                   sinks: Optional[torch.Tensor] = None, segment: int = 0, upto: Optional[int] = None) -> None:
+                   sinks: Optional[torch.Tensor] = None, segment: int = 0, upto: Optional[int] = None, keep: int = 0) -> None:
     """Causal GQA attention of the step's tokens on the CUDA cores, float32 arithmetic
     (csrc/attention_simt.cu): the attention of the float32 path.  The requests that bring
     one token each at the head of the batch (decoding requests, which the scheduler puts
@@ -504,7 +545,8 @@ def attention_simt(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vca
     ``v_head_dim`` (the values are then the head of each row: a store whose rows are keys and, in
     their first part, values).  ``out`` may be float32 beside bfloat16 operands.  ``upto``: only the
     first ``upto`` requests are served, which bring one token each (the caller gives the portions
-    after them to another kernel)."""
+    after them to another kernel).  ``keep`` (beside a window): the first ``keep`` keys of a request stay
+    visible when the window has passed them."""
     _cuda(out, q, kcache, vcache, block_table, score_slopes, sinks)
     _slopes_arg(sinks, n_heads, "sinks")
     vd = int(v_head_dim or head_dim)
@@ -531,7 +573,7 @@ def attention_simt(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vca
             singles += 1
     bound = ctx.split_bound or ctx.max_ctx
     if window:
-        bound = min(bound, int(window))
+        bound = min(bound, int(window) + _kept_room(keep))
     if segment:
         bound = min(bound, segment)
     splits = max(1, -(-bound // SIMT_CHUNK))
@@ -544,12 +586,12 @@ def attention_simt(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vca
         rc = lib.kllm_attention_simt(_p(out), _p(part_o), _p(part_ml), _p(q), ctypes.c_int64(q.stride(0)), _p(kcache),
                                      _p(vcache), _p(ctx.q_start), _p(ctx.start_pos), _p(block_table),
                                      block_table.shape[1], singles, singles, *common, 1, SIMT_CHUNK, splits,
-                                     _p(score_slopes), _p(sinks), segment, v_heads, v_row, out_f32, dtype_code(q.dtype),
-                                     _stream())
+                                     _p(score_slopes), _p(sinks), segment, v_heads, v_row, out_f32, int(keep or 0),
+                                     dtype_code(q.dtype), _stream())
         _check(lib, "attention_simt", rc)
         rc = lib.kllm_attention_simt_merge(_p(out), _p(part_o), _p(part_ml), _p(ctx.positions), singles, n_heads,
                                            vd, int(window or 0), SIMT_CHUNK, splits, _p(sinks), segment, out_f32,
-                                           dtype_code(q.dtype), _stream())
+                                           int(keep or 0), dtype_code(q.dtype), _stream())
         _check(lib, "attention_simt", rc)
         first = singles
     if first < n_req:
@@ -558,8 +600,8 @@ def attention_simt(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vca
         rc = lib.kllm_attention_simt(_p(out), None, None, _p(q), ctypes.c_int64(q.stride(0)), _p(kcache), _p(vcache),
                                      _p(ctx.q_start[first:]), _p(ctx.start_pos[first:]), _p(block_table[first:]),
                                      block_table.shape[1], n_req - first, rest // qt + (n_req - first), *common, qt, 0, 1,
-                                     _p(score_slopes), _p(sinks), segment, v_heads, v_row, out_f32, dtype_code(q.dtype),
-                                     _stream())
+                                     _p(score_slopes), _p(sinks), segment, v_heads, v_row, out_f32, int(keep or 0),
+                                     dtype_code(q.dtype), _stream())
         _check(lib, "attention_simt", rc)
 
 
@@ -619,7 +661,7 @@ def decode_splits(n_tokens: int, n_kv: int, ctx_bound: int) -> int:
 def attention(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, ctx,
               block_table: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, window: int,
               scale: float, score_slopes: Optional[torch.Tensor] = None, v_head_dim: Optional[int] = None,
-              exact_weights: bool = False, sinks: Optional[torch.Tensor] = None, segment: int = 0) -> None:
+              exact_weights: bool = False, sinks: Optional[torch.Tensor] = None, segment: int = 0, keep: int = 0) -> None:
     """Causal GQA attention of the step's tokens over the paged cache, by the
     kernel that fits: bfloat16 with a head size in TC_HEAD_DIMS runs on tensor cores
     (the decode form when every request brings one token, else the prefill form: on
@@ -640,11 +682,17 @@ def attention(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: 
     ``segment`` (a query sees only the keys of its own segment of that many positions), values of
     another size than the keys, a value store with fewer heads than the key store or with rows that
     the values only head, and a float32 ``out`` beside bfloat16 operands are taken by the CUDA-core
-    kernels and, for portions in bfloat16 with sizes in steps of 16, by the ``mma.sync`` prefill kernel."""
+    kernels and, for portions in bfloat16 with sizes in steps of 16, by the ``mma.sync`` prefill kernel.
+    ``keep`` (beside a window): the first ``keep`` keys of a request stay visible when the window has
+    passed them; taken by the CUDA-core kernels and the ``mma.sync`` kernels."""
+    keep = int(keep or 0) if window else 0
+    if keep and segment:
+        raise KernelError("attention: kept first keys go with a window, not with segments")
     group = n_heads // max(1, n_kv)
     vd = int(v_head_dim or head_dim)
     special = score_slopes is not None or exact_weights
-    special = special or sinks is not None
+    special = special or sinks is not None or keep > 0
+    seen = (int(window) + _kept_room(keep)) if window else 1 << 30      # most places of a token's walk
     plain_values = vcache.shape[1] == n_kv and vcache.shape[3] == vd and out.dtype == q.dtype
     tc = (q.dtype == torch.bfloat16 and (head_dim in TC_HEAD_DIMS or head_dim in TC_WIDE_HEAD_DIMS) and vd == head_dim
           and not (special and scale <= 0) and not segment and plain_values)
@@ -655,7 +703,7 @@ def attention(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: 
     wide = (not tc and q.dtype == torch.bfloat16 and (head_dim in TC_HEAD_DIMS or head_dim in TC_WIDE_HEAD_DIMS)
             and vd % 16 == 0 and 16 <= vd <= 256 and group <= 64 and not (special and scale <= 0)
             and vcache.dim() == 4 and vcache.shape[3] % 8 == 0)
-    short = min(int(segment or (1 << 30)), int(window or (1 << 30))) <= WIDE_SINGLE_KEYS
+    short = min(int(segment or (1 << 30)), seen) <= WIDE_SINGLE_KEYS
     # the decode kernel takes 16 heads per CTA: more heads on a kv head are cut into groups of equal size
     groups = n_kv * next((s for s in range(1, group + 1) if group % s == 0 and group // s <= 16), 1)
     # single tokens of the wide form: the decode kernel where the values have a plain store of their own size
@@ -665,8 +713,8 @@ def attention(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: 
         # token t of the first `singles` is request t: no token-to-request table needed
         attention_decode(out[:singles], q[:singles], kcache, vcache, ctx.positions[:singles], None, block_table[:singles],
                          n_heads, n_kv, head_dim, window, scale,
-                         decode_splits(singles, groups, min(bound, window or (1 << 30))), slopes=score_slopes,
-                         split_weights=exact_weights, sinks=sinks, v_head_dim=vd)
+                         decode_splits(singles, groups, min(bound, seen)), slopes=score_slopes,
+                         split_weights=exact_weights, sinks=sinks, v_head_dim=vd, keep=keep)
     if wide and not short and (ctx.all_single or not ctx.host_n_new):
         if wide_decode and ctx.all_single:
             return decode(ctx.n_tokens, ctx.split_bound or ctx.max_ctx)
@@ -682,26 +730,26 @@ def attention(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: 
                 wide = False
             else:
                 attention_simt(out, q, kcache, vcache, ctx, block_table, n_heads, n_kv, head_dim, window, scale,
-                               score_slopes, vd, sinks, segment, upto=singles)
+                               score_slopes, vd, sinks, segment, upto=singles, keep=keep)
     if wide:
         if singles < ctx.n_requests:
             attention_prefill(out, q, kcache, vcache, ctx.q_start[singles:], ctx.start_pos[singles:],
                               block_table[singles:], ctx.n_requests - singles, n_heads, n_kv, head_dim, window, scale,
                               slopes=score_slopes, split_weights=exact_weights, sinks=sinks, v_head_dim=vd,
-                              segment=segment)
+                              segment=segment, keep=keep)
         return
     if (special or vd != head_dim or segment or not plain_values) and not (tc and group <= 64):
         if not simt_fits(q, n_heads, n_kv, head_dim, vd) or vcache.shape[3] % 4:
             # head sizes that are no multiples of 4, very wide groups: one warp per (token, head)
             return attention_generic(out, q, kcache, vcache, ctx.positions, ctx.token_req, block_table, n_heads, n_kv,
-                                     head_dim, window, scale, score_slopes, vd, sinks, segment)
+                                     head_dim, window, scale, score_slopes, vd, sinks, segment, keep)
         return attention_simt(out, q, kcache, vcache, ctx, block_table, n_heads, n_kv, head_dim, window, scale,
-                              score_slopes, vd, sinks, segment)
+                              score_slopes, vd, sinks, segment, keep=keep)
     if tc and ctx.all_single and group <= 64:
         return attention_decode(out, q, kcache, vcache, ctx.positions, ctx.token_req, block_table, n_heads,
                                 n_kv, head_dim, window, scale,
-                                decode_splits(ctx.n_tokens, groups, min(ctx.split_bound or ctx.max_ctx, window or (1 << 30))),
-                                slopes=score_slopes, split_weights=exact_weights, sinks=sinks)
+                                decode_splits(ctx.n_tokens, groups, min(ctx.split_bound or ctx.max_ctx, seen)),
+                                slopes=score_slopes, split_weights=exact_weights, sinks=sinks, keep=keep)
     singles = 0
     if tc and group <= 64 and ctx.host_n_new:
         while singles < ctx.n_requests and ctx.host_n_new[singles] == 1:
@@ -719,7 +767,7 @@ def attention(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vcache: 
     if tc and group <= 64:
         return attention_prefill(out, q, kcache, vcache, q_start, start_pos, table,
                                  n_req, n_heads, n_kv, head_dim, window, scale, slopes=score_slopes,
-                                 split_weights=exact_weights, sinks=sinks)
+                                 split_weights=exact_weights, sinks=sinks, keep=keep)
     if simt_fits(q, n_heads, n_kv, head_dim):
         return attention_simt(out, q, kcache, vcache, ctx, block_table, n_heads, n_kv, head_dim, window, scale)
     return attention_generic(out, q, kcache, vcache, ctx.positions, ctx.token_req, block_table, n_heads, n_kv,
@@ -746,13 +794,13 @@ def _slopes_arg(slopes, n_heads, what="score slopes"):
 def attention_decode(out, q, kcache, vcache, positions, token_req, block_table, n_heads, n_kv, head_dim,
                      window, scale, num_splits: int, slopes: Optional[torch.Tensor] = None,
                      split_weights: bool = False, sinks: Optional[torch.Tensor] = None,
-                     v_head_dim: Optional[int] = None) -> None:
+                     v_head_dim: Optional[int] = None, keep: int = 0) -> None:
     """Tensor-core decode attention: every token attends on its own, its keys cut
     into ``num_splits`` ranges that are merged in a fixed order.  ``slopes`` (float32 [heads]):
     slope[h] * (key position - query position) is added to the scaled scores; ``split_weights``:
     the probabilities enter the second product as two bfloat16 terms instead of one; ``sinks``
     (float32 [heads]): exp(sinks[h]) joins the denominator of head h's softmax; ``v_head_dim``: values of another
-    size than the keys (a library of its own per pair of sizes)."""
+    size than the keys (a library of its own per pair of sizes); ``keep``: first keys that stay visible beside a window."""
     _cuda(out, q, kcache, vcache, positions, token_req, block_table, slopes, sinks)
     vd = int(v_head_dim or head_dim)
     _check_attention(out, q, kcache, vcache, block_table, n_kv, head_dim, vd)
@@ -769,7 +817,7 @@ def attention_decode(out, q, kcache, vcache, positions, token_req, block_table, 
                                    _p(kcache), _p(vcache), _p(positions), _p(token_req), _p(block_table),
                                    block_table.shape[1], n, n_heads, n_kv, head_dim, kcache.shape[2],
                                    int(window or 0), ctypes.c_float(scale), int(num_splits), _slopes_arg(slopes, n_heads),
-                                   int(bool(split_weights)), _slopes_arg(sinks, n_heads, "sinks"), _stream())
+                                   int(bool(split_weights)), _slopes_arg(sinks, n_heads, "sinks"), int(keep or 0), _stream())
     _check(lib, "attention_tc", rc)
     global launches
     if num_splits > 1:
@@ -813,12 +861,12 @@ def attention_decode_fused(out, q, k_new, v_new, cos_sin, kcache, vcache, positi
 def attention_prefill(out, q, kcache, vcache, q_start, start_pos, block_table, n_requests, n_heads, n_kv,
                       head_dim, window, scale, slopes: Optional[torch.Tensor] = None,
                       split_weights: bool = False, sinks: Optional[torch.Tensor] = None,
-                      v_head_dim: Optional[int] = None, segment: int = 0) -> None:
+                      v_head_dim: Optional[int] = None, segment: int = 0, keep: int = 0) -> None:
     """Tensor-core attention of portions: request s brings rows q_start[s]..q_start[s+1]
     that start at cache position start_pos[s].  ``slopes``, ``split_weights`` and ``sinks`` as in
     ``attention_decode``.  ``v_head_dim`` (values of another size than the keys: a library of its
-    own per pair of sizes), ``segment``, a value store of another shape than the key store and a
-    float32 ``out`` as in ``attention_simt``."""
+    own per pair of sizes), ``segment``, a value store of another shape than the key store, a
+    float32 ``out`` and ``keep`` as in ``attention_simt``."""
     _cuda(out, q, kcache, vcache, q_start, start_pos, block_table, slopes, sinks)
     vd = int(v_head_dim or head_dim)
     if q.dtype != torch.bfloat16 or out.dtype not in (torch.bfloat16, torch.float32) or kcache.dtype != torch.bfloat16:
@@ -836,7 +884,7 @@ def attention_prefill(out, q, kcache, vcache, q_start, start_pos, block_table, n
                                     q.shape[0], int(n_requests), n_heads, n_kv, head_dim, kcache.shape[2],
                                     int(window or 0), ctypes.c_float(scale), _slopes_arg(slopes, n_heads),
                                     int(bool(split_weights)), _slopes_arg(sinks, n_heads, "sinks"), vd,
-                                    int(segment or 0), v_heads, v_row, int(out.dtype == torch.float32), _stream())
+                                    int(segment or 0), v_heads, v_row, int(out.dtype == torch.float32), int(keep or 0), _stream())
     _check(lib, "attention_tc", rc)
 
 
@@ -989,9 +1037,12 @@ def biased_glu(out: torch.Tensor, gate: torch.Tensor, up: torch.Tensor, bias_gat
     _check(lib, "activation", rc)
 
 
+_SKINNY_ACT = {"silu": 0, "gelu_tanh": 1, "clamped": 2, "relu2": 3}
+
+
 def _bias_form(bias, bias_up, activation):
     """Compile-time definitions of the weight-streaming library that a call takes: the plain kernels are a library
-    without biases and the gelu."""
+    without biases and other activations than silu."""
     return {"KLLM_BIAS": 1} if bias is not None or bias_up is not None or activation != "silu" else None
 
 
@@ -1027,6 +1078,8 @@ def sample(out: torch.Tensor, logits: torch.Tensor, temperature: Optional[torch.
 SKINNY_MAX_ROWS = 16
 _PRO = {"bf16": 0, "norm": 1}
 _EPI = {"bf16": 0, "f32": 1, "add": 2, "swiglu": 3}
+_GEMM_EPI = dict(_EPI, clamped=4, relu2=5)
+_GATED_EPI = ("swiglu", "clamped")
 
 
 SKINNY_F32_MAX_ROWS = 8
@@ -1070,7 +1123,7 @@ def skinny_gemm(weight: torch.Tensor, *, x: Optional[torch.Tensor] = None, x_f32
                 n_rows: Optional[int] = None, weight_up: Optional[torch.Tensor] = None, epilogue: str = "bf16",
                 out: Optional[torch.Tensor] = None, prefetch: Optional[torch.Tensor] = None,
                 bias: Optional[torch.Tensor] = None, bias_up: Optional[torch.Tensor] = None,
-                activation: str = "silu") -> torch.Tensor:
+                activation: str = "silu", limit: float = 0.0, alpha: float = 1.0) -> torch.Tensor:
     """y = X @ weight^T for at most 16 rows, the weights streamed once (csrc/skinny_gemm.cu
     for bfloat16 weights, csrc/skinny_gemm_f32.cu for float32 weights: true float32 FMAs,
     at most 8 rows).
@@ -1080,8 +1133,8 @@ def skinny_gemm(weight: torch.Tensor, *, x: Optional[torch.Tensor] = None, x_f32
     [n, N] in the weights' dtype ("bf16" / "f32" name the dtype); "add" adds y into the
     float32 ``out``; "swiglu" takes ``weight`` as gate and ``weight_up`` as up matrix and
     stores silu(gate) * up [n, N] in the weights' dtype.  ``bias`` (float32 [N]) joins the sum of
-    "add", or the gate's sums of "swiglu" (``bias_up``: the up sums'); ``activation`` "gelu_tanh" takes
-    silu's place there.
+    "add", or the gate's sums of "swiglu" (``bias_up``: the up sums'); ``activation`` "gelu_tanh" or "clamped" (with
+    ``limit`` and ``alpha``, as in ``clamped_glu``) takes silu's place there, "relu2" squares the relu of what "store" stores.
     ``prefetch``: a contiguous tensor that a later kernel will stream (the next weight
     matrix); the kernel asks for it to be brought into L2 before its own work.
     A width K too long for shared memory is taken in column slices, one launch each, when
@@ -1092,13 +1145,14 @@ def skinny_gemm(weight: torch.Tensor, *, x: Optional[torch.Tensor] = None, x_f32
     N, K = weight.shape
     _bias(bias, N, "skinny_gemm"); _bias(bias_up, N, "skinny_gemm")
     if (bias is not None and epilogue not in ("add", "swiglu")) or (bias_up is not None and epilogue != "swiglu") \
-            or activation not in ("silu", "gelu_tanh"):
-        raise KernelError("skinny_gemm: biases go with 'add' and 'swiglu', the activation is silu or gelu_tanh")
+            or activation not in _SKINNY_ACT or (activation == "relu2" and epilogue != "store"):
+        raise KernelError("skinny_gemm: biases go with 'add' and 'swiglu', the activation is silu, gelu_tanh or clamped there, "
+                          "relu2 with 'store'")
     if epilogue == "store":
         epilogue = "f32" if weight.dtype == torch.float32 else "bf16"
     if weight.dtype == torch.float32:
         return _skinny_gemm_f32(weight, x, x_f32, gain, eps, rows, n_rows, weight_up, epilogue, out, bias, bias_up,
-                                activation)
+                                activation, limit, alpha)
     if weight.dtype != torch.bfloat16 or weight.stride(1) != 1 or weight.stride(0) % 8:
         raise KernelError("skinny_gemm: the weight must be bfloat16 with dense rows at a stride that is a multiple of 8")
     if weight_up is not None and weight_up.stride() != weight.stride():
@@ -1145,13 +1199,14 @@ def skinny_gemm(weight: torch.Tensor, *, x: Optional[torch.Tensor] = None, x_f32
     rc = lib.kllm_skinny_gemm(_p(weight), _p(weight_up), ctypes.c_int64(weight.stride(0)), N, K, n, _p(x),
                               ctypes.c_int64(x.stride(0) if x is not None else 0), _p(x_f32), _p(gain), _p(rows),
                               ctypes.c_float(eps), _p(y16), _p(y32), ctypes.c_int64(out.stride(0)), pro, epi,
-                              _p(bias), _p(bias_up), int(activation == "gelu_tanh"), *_prefetch_args(prefetch), _stream())
+                              _p(bias), _p(bias_up), _SKINNY_ACT[activation], ctypes.c_float(limit), ctypes.c_float(alpha),
+                              *_prefetch_args(prefetch), _stream())
     _check(lib, "skinny_gemm", rc)
     return out
 
 
 def _skinny_gemm_f32(weight, x, x_f32, gain, eps, rows, n_rows, weight_up, epilogue, out, bias=None, bias_up=None,
-                     activation="silu"):
+                     activation="silu", limit=0.0, alpha=1.0):
     """The float32 form of ``skinny_gemm`` (same arguments; no prefetch hint)."""
     N, K = weight.shape
     if weight.stride(1) != 1 or weight.stride(0) % 4:
@@ -1193,7 +1248,8 @@ def _skinny_gemm_f32(weight, x, x_f32, gain, eps, rows, n_rows, weight_up, epilo
     rc = lib.kllm_skinny_gemm_f32(_p(weight), _p(weight_up), ctypes.c_int64(weight.stride(0)), N, K, n, _p(src),
                                   ctypes.c_int64(stride), _p(gain), _p(rows), ctypes.c_float(eps), _p(out),
                                   ctypes.c_int64(out.stride(0)), pro, {"f32": 0, "add": 1, "swiglu": 2}[epilogue],
-                                  _p(bias), _p(bias_up), int(activation == "gelu_tanh"), _stream())
+                                  _p(bias), _p(bias_up), _SKINNY_ACT[activation], ctypes.c_float(limit), ctypes.c_float(alpha),
+                                  _stream())
     _check(lib, "skinny_gemm_f32", rc)
     return out
 
@@ -1231,7 +1287,7 @@ def linear_into(acc: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, bias: 
 
 def _gemm_args(x, weight, weight_up, out, epilogue):
     return (_p(x), ctypes.c_int64(x.stride(0)), _p(weight), ctypes.c_int64(weight.stride(0)), _p(weight_up),
-            x.shape[0], weight.shape[0], x.shape[1], _p(out), ctypes.c_int64(out.stride(0)), _EPI[epilogue])
+            x.shape[0], weight.shape[0], x.shape[1], _p(out), ctypes.c_int64(out.stride(0)), _GEMM_EPI[epilogue])
 
 
 def gemm_fits(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epilogue: str = "bf16",
@@ -1257,20 +1313,21 @@ def gemm_pays(n: int, N: int, epilogue: str = "bf16", least: int = 75) -> bool:
     if not USE_TCGEN05 or n <= 0 or N <= 0:
         return False
     sms = sm_count()
-    nout = 128 if epilogue == "swiglu" else 256
+    nout = 128 if epilogue in _GATED_EPI else 256
     tiles = -(-n // 128) * -(-N // nout)
     waves = -(-tiles // sms)
     return 100.0 * (n / 128.0) * (N / float(nout)) / (waves * sms) >= least
 
 
 def gemm(x: torch.Tensor, weight: torch.Tensor, *, epilogue: str = "bf16", out: Optional[torch.Tensor] = None,
-         weight_up: Optional[torch.Tensor] = None, bn: int = 0) -> torch.Tensor:
+         weight_up: Optional[torch.Tensor] = None, bn: int = 0, limit: float = 0.0, alpha: float = 1.0) -> torch.Tensor:
     """y = x @ weight^T on the tcgen05 tensor cores (csrc/gemm_tcgen05.cu), x bfloat16
     [n, K], weight bfloat16 [N, K].
 
     ``epilogue``: "bf16" / "f32" store y [n, N]; "add" adds y into the float32 ``out``;
     "swiglu" takes ``weight`` as gate and ``weight_up`` as up matrix and stores
-    silu(gate) * up as bfloat16 [n, N].  ``bn``: accumulator width of a tile (0 = chosen
+    silu(gate) * up as bfloat16 [n, N]; "clamped" likewise with the activation of ``clamped_glu`` (``limit``, ``alpha``);
+    "relu2" stores the square of relu(y) as bfloat16.  ``bn``: accumulator width of a tile (0 = chosen
     by the tile count).
     """
     _cuda(x, weight, weight_up, out)
@@ -1282,14 +1339,14 @@ def gemm(x: torch.Tensor, weight: torch.Tensor, *, epilogue: str = "bf16", out: 
         out = torch.empty((n, N), dtype=want, device=x.device)
     if out.dtype != want or out.shape[0] != n or out.shape[1] != N:
         raise KernelError("gemm: out has the wrong dtype or shape")
-    if epilogue == "swiglu" and weight_up is None:
-        raise KernelError("gemm: swiglu needs an up matrix like the gate matrix")
+    if epilogue in _GATED_EPI and weight_up is None:
+        raise KernelError(f"gemm: {epilogue} needs an up matrix like the gate matrix")
     if not gemm_fits(x, weight, out, epilogue, weight_up):
         raise KernelError(f"gemm: operands {tuple(x.shape)} x {tuple(weight.shape)} (strides {x.stride()}, "
                           f"{weight.stride()}, out {out.stride()}) are not supported")
     lib = load_library("gemm_tcgen05")
-    rc = lib.kllm_gemm_tcgen05(*_gemm_args(x, weight, weight_up, out, epilogue), int(bn), _p(status_word(x.device)),
-                               _stream())
+    rc = lib.kllm_gemm_tcgen05(*_gemm_args(x, weight, weight_up, out, epilogue), int(bn), ctypes.c_float(limit),
+                               ctypes.c_float(alpha), _p(status_word(x.device)), _stream())
     _check(lib, "gemm_tcgen05", rc)
     return out
 
@@ -1354,6 +1411,22 @@ def linear_per_head(x: torch.Tensor, weight: torch.Tensor, transposed: bool = Fa
     torch.bmm(x.transpose(0, 1), weight if transposed else weight.transpose(1, 2),
               out=y.view(n, H, b).transpose(0, 1))
     return y
+
+
+def linear_relu2(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """The square of relu(x @ weight^T) in x's dtype, the activation applied to the float32 sums: in the epilogue of the
+    weight-streaming product (a few rows) or of the tcgen05 product (steps that fill its tiles), else by a kernel
+    behind the library's product."""
+    _cuda(x, weight)
+    n = x.shape[0]
+    if (x.dtype == weight.dtype and x.stride(1) == 1 and weight.stride(1) == 1 and skinny_fits(n, x.shape[1], x.dtype)
+            and weight.stride(0) % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0):
+        return skinny_gemm(weight, x=x, epilogue="store", activation="relu2")
+    if x.dtype == torch.bfloat16 and gemm_pays(n, weight.shape[0], "relu2"):
+        out = torch.empty((n, weight.shape[0]), dtype=x.dtype, device=x.device)
+        if gemm_fits(x, weight, out, "relu2"):
+            return gemm(x, weight, epilogue="relu2", out=out)
+    return unary(linear(x, weight, out_dtype=torch.float32), "relu2", x.dtype)
 
 
 def linear(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor] = None,
@@ -1605,6 +1678,69 @@ def gla(y: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: t
         launches += 3 if dv <= 256 else 4
 
 
+# ---- a state-space recurrence (csrc/ssd.cu) --------------------------------------------------
+
+def ssd(proj: torch.Tensor, conv: torch.Tensor, conv_bias: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+        d: torch.Tensor, state: torch.Tensor, ring: torch.Tensor, ctx, heads: int, groups: int, N: int, dv: int,
+        early: bool = False) -> torch.Tensor:
+    """float32 [n, heads * dv]: (S_t^T C_t + D x_t) * silu(z_t) of the recurrence S_t = exp(-exp(a_log) dt_t) S_(t-1) +
+    dt_t B_t x_t^T per head.  ``proj`` float32 [n, >= 2 heads dv + 2 groups N + heads] with dense rows holds z, x, B, C and dt; x, B and
+    C pass a causal convolution (``conv`` float32 [channels, taps], last column the current row's, ``conv_bias``) and silu, dt
+    a softplus behind ``dt_bias``.  ``state`` float32 [slots, >= heads * N * dv] holds S as [heads, N, dv] per request slot,
+    ``ring`` float32 [slots, >= taps * row] (row: the channels rounded up to a multiple of 4) the convolution's inputs of
+    the last taps positions, position p in row p mod taps; both are carried on.  ``early``: a step of one row per request
+    may read them beside the end of the kernel before it, which then must not write them."""
+    _cuda(proj, conv, conv_bias, dt_bias, a_log, d, state, ring)
+    n, inner, taps = proj.shape[0], heads * dv, conv.shape[1]
+    channels = inner + 2 * groups * N
+    row = -(-channels // 4) * 4
+    if proj.dtype != torch.float32 or proj.stride(1) != 1 or proj.shape[1] < inner + channels + heads:
+        raise KernelError("ssd: the projections must be float32 rows of z, x, B, C and dt")
+    if conv.dtype != torch.float32 or not conv.is_contiguous() or conv.shape[0] != channels:
+        raise KernelError("ssd: the convolution must be contiguous float32 [channels, taps]")
+    _bias(conv_bias, channels, "ssd")
+    for t in (dt_bias, a_log, d):
+        _bias(t, heads, "ssd")
+    for t, size in ((state, heads * N * dv), (ring, taps * row)):
+        if t.dtype != torch.float32 or t.dim() != 2 or t.stride(1) != 1 or t.shape[1] < size:
+            raise KernelError(f"ssd: a state must be float32 [slots, >= {size}]")
+    for t in (ctx.q_start, ctx.start_pos, ctx.state_slots):
+        _i32(t, "ssd: request table")
+    f32 = dict(dtype=torch.float32, device=proj.device)
+    y = torch.empty((n, inner), **f32)
+    lib = load_library("ssd")
+    xc = dt = cum = pairs = s_in = None
+    bound = 0
+    if not ctx.all_single:
+        C = lib.kllm_ssd_chunk_rows()
+        bound = n // C + ctx.n_requests
+        xc, dt, cum = torch.empty((n, row), **f32), torch.empty((bound, heads, C), **f32), torch.empty((bound, heads, C, 2), **f32)
+        pairs, s_in = torch.empty((bound, groups, C, C), **f32), torch.empty((bound, heads, N, dv), **f32)
+    rc = lib.kllm_ssd(_p(y), _p(proj), ctypes.c_int64(proj.stride(0)), _p(conv), _p(conv_bias), _p(dt_bias), _p(a_log), _p(d),
+                      _p(ctx.q_start), _p(ctx.start_pos), _p(ctx.state_slots), _p(state), ctypes.c_int64(state.stride(0)),
+                      _p(ring), ctypes.c_int64(ring.stride(0)), n, ctx.n_requests, heads, groups, N, dv, taps,
+                      int(ctx.all_single), int(early), bound, _p(xc), _p(dt), _p(cum), _p(pairs), _p(s_in), _stream())
+    _check(lib, "ssd", rc)
+    if not ctx.all_single:
+        global launches
+        launches += 4
+    return y
+
+
+def part_norm(out: torch.Tensor, y: torch.Tensor, gain: torch.Tensor, parts: int, eps: float) -> None:
+    """out = y / rms(y) * gain, every one of ``parts`` equal pieces of a row by its own root mean square; y contiguous
+    float32 [n, width], out [n, width] (model dtype, dense rows), gain float32 [width] (csrc/ssd.cu)."""
+    _cuda(out, y, gain)
+    n, width = y.shape
+    if y.dtype != torch.float32 or not y.is_contiguous() or out.shape != y.shape or out.stride(1) != 1 or width % parts:
+        raise KernelError("part_norm: y contiguous float32 [n, width], out alike with dense rows, the parts dividing the width")
+    _bias(gain, width, "part_norm")
+    lib = load_library("ssd")
+    rc = lib.kllm_part_norm(_p(out), ctypes.c_int64(out.stride(0)), _p(y), _p(gain), n, int(parts), width // parts,
+                            ctypes.c_float(eps), dtype_code(out.dtype), _stream())
+    _check(lib, "ssd", rc)
+
+
 # ---- what stands in front of a layer (csrc/shift_norm.cu) --------------------------------------
 
 def norm_shift(x: torch.Tensor, gain: torch.Tensor, eps: float, mu: torch.Tensor, state: torch.Tensor, ctx,
@@ -1725,13 +1861,22 @@ def attention_mixed(out: torch.Tensor, q: torch.Tensor, kcache: torch.Tensor, vc
 
 _GATED_ACT = {"silu": 0, "clamped": 1}
 
+
+def _expert_form(gated: bool, activation: str) -> int:
+    """Which of the experts' products a call is: 0 the down product, 1 gate and up with a gated activation, 2 the up
+    product of experts without a gate (the square of relu)."""
+    return (2 if activation == "relu2" else 1) if gated else 0
+
+
 def moe_route(h: torch.Tensor, router: torch.Tensor, top: int, score: str = "sigmoid", renormalize: bool = False,
-              groups: int = 1, keep: int = 1):
+              groups: int = 1, keep: int = 1, correction: Optional[torch.Tensor] = None, sum_eps: float = 0.0):
     """(idx int32 [n, top], weights float32 [n, top]): logits router @ h in float32, scores by
     ``score`` ("sigmoid" or "softmax"), the ``top`` largest, the lower index among equals.  With
     ``groups`` > 1 the experts form that many equal groups of neighbours, a group scores as its best
-    expert, and only experts of the ``keep`` best groups can be chosen."""
-    _cuda(h, router)
+    expert, and only experts of the ``keep`` best groups can be chosen.  ``correction`` (float32 [experts]) joins the
+    scores for the choice, not for the weights; ``sum_eps`` joins the sum that ``renormalize`` divides by."""
+    _cuda(h, router, correction)
+    _bias(correction, router.shape[0], "moe_route")
     n, d = h.shape
     if not h.is_contiguous() or router.dtype != torch.float32 or not router.is_contiguous() or router.shape[1] != d:
         raise KernelError("moe_route: h contiguous [n, d], router float32 [experts, d]")
@@ -1742,7 +1887,7 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, top: int, score: str = "sig
     lib = load_library("moe")
     rc = lib.kllm_moe_route(_p(idx), _p(wt), _p(h), _p(router), n, d, router.shape[0], int(top),
                             int(score == "softmax"), int(bool(renormalize)), int(groups or 1), int(keep or 1),
-                            dtype_code(h.dtype), _stream())
+                            _p(correction), ctypes.c_float(sum_eps), dtype_code(h.dtype), _stream())
     _check(lib, "moe", rc)
     return idx, wt
 
@@ -1772,14 +1917,16 @@ def moe_gemm(a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, perm: torc
     Otherwise a is [rows, K] in sorted order, w [E, N, K]; returns float32 [rows, N] with row
     token * top + choice, times its weight when ``scale_out``.  ``activation`` of the gated
     form: "silu" (silu(g) * u) or "clamped" (with g' = min(g, limit) and u' = clamp(u, -limit,
-    limit): g' * sigmoid(alpha g') * (u' + 1))."""
+    limit): g' * sigmoid(alpha g') * (u' + 1)); "relu2": the experts have no gate, w [E, N, K] holds their up
+    rows and the result is the square of relu.  Sorted rows behind the last of w's experts are left alone."""
     _cuda(a, w, offsets, perm, wt)
-    if activation not in _GATED_ACT or (activation == "clamped" and not limit > 0):
-        raise KernelError(f"moe_gemm: activation {activation!r} (silu, or clamped with a positive limit)")
+    form = _expert_form(gated, activation)
+    if activation not in (*_GATED_ACT, "relu2") or (activation == "clamped" and not limit > 0):
+        raise KernelError(f"moe_gemm: activation {activation!r} (silu, relu2, or clamped with a positive limit)")
     _i32(offsets, "offsets"); _i32(perm, "perm")
     rows = perm.numel()
     E, N, K = w.shape
-    if gated:
+    if form == 1:
         N //= 2
     if a.dtype != w.dtype or a.stride(1) != 1 or a.shape[1] != K or not w.is_contiguous():
         raise KernelError("moe_gemm: a [., K] with dense rows and w [E, ., K] contiguous, of one dtype")
@@ -1788,7 +1935,7 @@ def moe_gemm(a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, perm: torc
     c = torch.empty((rows, N), dtype=a.dtype if gated else torch.float32, device=a.device)
     lib = load_library("moe")
     rc = lib.kllm_moe_gemm(_p(c), _p(a), ctypes.c_int64(a.stride(0)), _p(w), _p(offsets), _p(perm), _p(wt), rows, E,
-                           int(top), N, K, int(gated), int(scale_in), int(scale_out), _GATED_ACT[activation],
+                           int(top), N, K, form, int(scale_in), int(scale_out), _GATED_ACT.get(activation, 0),
                            ctypes.c_float(limit), ctypes.c_float(alpha), dtype_code(a.dtype), _stream())
     _check(lib, "moe", rc)
     return c
@@ -1797,13 +1944,14 @@ def moe_gemm(a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, perm: torc
 MOE_TCGEN05_ROWS = 64      # rows per expert on average from which a step's experts run on the tcgen05 kernel
 
 
-def moe_gemm_tcgen05_pays(a: torch.Tensor, w: torch.Tensor, rows: int, gated: bool, scale_in: bool) -> bool:
+def moe_gemm_tcgen05_pays(a: torch.Tensor, w: torch.Tensor, rows: int, gated: bool, scale_in: bool,
+                          activation: str = "silu") -> bool:
     """Whether ``moe_gemm_tcgen05`` takes these operands and the step is large enough for tiles of 128
     rows per expert: bfloat16, no weight on the experts' inputs (TMA brings the rows to the tensor
     cores as they are), rows and matrices in whole 16-byte pieces and at least as wide as one 64-column k
     block (a layer's two products have the same two widths, so one answer holds for both)."""
     E, N, K = w.shape
-    if gated:
+    if _expert_form(gated, activation) == 1:
         N //= 2
     return (USE_TCGEN05 and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and not scale_in and E <= 512
             and rows >= 512 and rows >= MOE_TCGEN05_ROWS * E and K % 8 == 0 and N % 8 == 0 and min(K, N) >= 64
@@ -1818,43 +1966,48 @@ def moe_gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, pe
     operands and results; the weights may act on the experts' outputs only.  The gated form first gathers
     the layer's input into sorted order, one row per (token, choice)."""
     _cuda(a, w, offsets, perm, wt)
-    if activation not in _GATED_ACT or (activation == "clamped" and not limit > 0):
-        raise KernelError(f"moe_gemm: activation {activation!r} (silu, or clamped with a positive limit)")
+    form = _expert_form(gated, activation)
+    if activation not in (*_GATED_ACT, "relu2") or (activation == "clamped" and not limit > 0):
+        raise KernelError(f"moe_gemm: activation {activation!r} (silu, relu2, or clamped with a positive limit)")
     _i32(offsets, "offsets"); _i32(perm, "perm")
     rows = perm.numel()
     E, N, K = w.shape
-    if gated:
+    if form == 1:
         N //= 2
-    if not moe_gemm_tcgen05_pays(a, w, rows, gated, False) or a.shape[1] != K:
+    if not moe_gemm_tcgen05_pays(a, w, rows, gated, False, activation) or a.shape[1] != K:
         raise KernelError("moe_gemm_tcgen05: operands not taken (bfloat16, rows of whole 16-byte pieces, a large step)")
     if wt.dtype != torch.float32 or not wt.is_contiguous() or wt.numel() != rows:
         raise KernelError("moe_gemm: one float32 weight per (token, choice)")
     lib = load_library("moe_gemm_tcgen05")
     if gated:
         xs = torch.empty((rows, K), dtype=a.dtype, device=a.device)
-        rc = lib.kllm_moe_gather_sorted(_p(xs), _p(a), ctypes.c_int64(a.stride(0)), _p(perm), rows, int(top), K, _stream())
+        rc = lib.kllm_moe_gather_sorted(_p(xs), _p(a), ctypes.c_int64(a.stride(0)), _p(perm), rows, int(top), K,
+                                        _p(offsets[E:]), _stream())
         _check(lib, "moe_gemm_tcgen05", rc)
         a = xs
     elif not a.is_contiguous() or a.shape[0] != rows:
         raise KernelError("moe_gemm_tcgen05: the sorted rows must be contiguous")
     c = torch.empty((rows, N), dtype=a.dtype if gated else torch.float32, device=a.device)
-    rc = lib.kllm_moe_gemm_tcgen05(_p(c), _p(a), _p(w), _p(offsets), _p(perm), _p(wt), rows, E, N, K, int(gated),
-                                   int(scale_out), _GATED_ACT[activation], ctypes.c_float(limit), ctypes.c_float(alpha),
+    rc = lib.kllm_moe_gemm_tcgen05(_p(c), _p(a), _p(w), _p(offsets), _p(perm), _p(wt), rows, E, N, K, form,
+                                   int(scale_out), _GATED_ACT.get(activation, 0), ctypes.c_float(limit), ctypes.c_float(alpha),
                                    _p(status_word(a.device)), _stream())
     _check(lib, "moe_gemm_tcgen05", rc)
     return c
 
 
 def moe_combine(parts: torch.Tensor, top: int, shared: Optional[torch.Tensor] = None,
-                gate: Optional[torch.Tensor] = None, scale: float = 1.0,
-                into: Optional[torch.Tensor] = None) -> torch.Tensor:
+                gate: Optional[torch.Tensor] = None, scale: float = 1.0, into: Optional[torch.Tensor] = None,
+                identity: Optional[tuple] = None) -> torch.Tensor:
     """y[t] = sum of parts[t * top + j] over j in order; float32.  With ``shared`` (float32
     [n, d], the output of an expert that every token runs) also + shared[t] * sigmoid(gate[t]),
     ``gate`` being a float32 column of one logit per token (None: the rows are added as they are).
     ``scale`` multiplies the sum over j (one weight that all of a token's choices share).  ``into``: a float32
-    [n, d] matrix (the residual stream) to which the sum is added; it is what is returned."""
-    _cuda(parts, shared, gate, into)
-    if top == 1 and shared is None and scale == 1.0 and into is None:
+    [n, d] matrix (the residual stream) to which the sum is added; it is what is returned.  ``identity`` (idx, wt,
+    h, experts): a choice idx[t, j] from ``experts`` on is an identity expert, which adds wt[t, j] * h[t] (h [n, d] the
+    layer's input); its row of ``parts`` is never read."""
+    idx, wt, h, experts = identity or (None, None, None, 0)
+    _cuda(parts, shared, gate, into, idx, wt, h)
+    if top == 1 and shared is None and scale == 1.0 and into is None and identity is None:
         return parts            # nothing to add up: the rows themselves
     n, d = parts.shape[0] // top, parts.shape[1]
     if not parts.is_contiguous() or parts.dtype != torch.float32:
@@ -1865,11 +2018,17 @@ def moe_combine(parts: torch.Tensor, top: int, shared: Optional[torch.Tensor] = 
         raise KernelError("moe_combine: the gate is a float32 column [n, 1] beside a shared expert")
     if into is not None and (into.dtype != torch.float32 or not into.is_contiguous() or into.shape != (n, d)):
         raise KernelError("moe_combine: the matrix added into must be contiguous float32 [n, d]")
+    if identity is not None:
+        _i32(idx, "idx")
+        if idx.numel() != n * top or wt.dtype != torch.float32 or not wt.is_contiguous() or wt.numel() != n * top \
+                or not h.is_contiguous() or h.shape != (n, d):
+            raise KernelError("moe_combine: identity experts take idx int32, wt float32 [n, top] and h contiguous [n, d]")
     y = into if into is not None else torch.empty((n, d), dtype=torch.float32, device=parts.device)
     lib = load_library("moe")
     rc = lib.kllm_moe_combine(_p(y), _p(parts), n, d, int(top), _p(shared), _p(gate),
                               ctypes.c_int64(gate.stride(0) if gate is not None else 0), ctypes.c_float(scale),
-                              int(into is not None), _stream())
+                              int(into is not None), _p(h), _p(idx), _p(wt), int(experts),
+                              dtype_code(h.dtype if h is not None else torch.float32), _stream())
     _check(lib, "moe", rc)
     return y
 

@@ -2,6 +2,7 @@
 
 params: ``hidden``, ``n_heads``, ``n_kv_heads``, ``head_dim``; optional ``window``
 (None: every earlier key is visible; W: the last W keys, the query's own included),
+``keep_first`` (beside a window, K: the first K keys of the sequence stay visible when the window has passed them),
 ``scale`` (default 1/sqrt(head_dim)), ``position`` (a PartSpec of the position
 family, e.g. rotary; None for no position encoding), ``qk_transform`` (a PartSpec of
 the qk_transform family, None for Llama: something applied to the projected queries
@@ -82,6 +83,7 @@ class PagedAttention:
         if self.n_heads % self.n_kv:
             raise ValueError(f"{self.n_heads} heads are not a multiple of {self.n_kv} kv heads")
         self.window = p.get("window")
+        self.keep_first = int(p.get("keep_first") or 0) if self.window else 0
         self.scale = float(p.get("scale") or 1.0 / math.sqrt(self.head_dim))
         self.v_head_dim = int(p.get("v_head_dim") or self.head_dim)
         self.exact_weights = bool(p.get("exact_weights", False))
@@ -117,6 +119,8 @@ class PagedAttention:
         if self.mix_name and (not self._prepares or self.differential or self.segment or p.get("score_slopes")):
             raise ValueError("attention: mixed scores need a qk_transform that stores keys and values (prepare) and go "
                              "without differential maps, segments and score slopes")
+        if self.keep_first and (self.mix_name or self.segment):
+            raise ValueError("attention: kept first keys go without mixed scores and segments")
         if self.sink_name and not self._prepares:
             raise ValueError("attention: a sink needs a qk_transform that stores keys and values (prepare)")
         self.gate_name = p.get("out_gate")
@@ -207,7 +211,7 @@ class PagedAttention:
     def cache_need(self):
         return PagedKVNeed(self.n_kv * self.maps, self.head_dim, self.window,
                            None if self.v_head_dim == self.head_dim else self.v_head_dim,
-                           n_v_heads=self.n_kv if self.maps > 1 else None)
+                           n_v_heads=self.n_kv if self.maps > 1 else None, keep_first=self.keep_first)
 
     def _split(self, qkv, writes):
         q = qkv[:, :self.q_dim]
@@ -245,14 +249,14 @@ class PagedAttention:
             kernels.attention(attn, q, cache.k, cache.v, ctx, cache.block_table, self.n_heads, self.n_kv,
                               self.head_dim, self.window or 0, self.scale, score_slopes=self.score_slopes,
                               v_head_dim=self.v_head_dim, exact_weights=self.exact_weights, segment=self.segment,
-                              sinks=self.sinks)
+                              sinks=self.sinks, keep=self.keep_first)
             return attn
         # two maps per head: 2H query heads over 2G key heads and G value heads, combined afterwards
         both = torch.empty((n, self.maps * self.o_dim), dtype=torch.float32, device=q.device)
         kernels.attention(both, q, cache.k, cache.v, ctx, cache.block_table, self.n_heads * self.maps,
                           self.n_kv * self.maps, self.head_dim, self.window or 0, self.scale,
                           score_slopes=self.score_slopes, v_head_dim=self.v_head_dim, exact_weights=True,
-                          segment=self.segment)
+                          segment=self.segment, keep=self.keep_first)
         kernels.maps_combine(attn, both, self.n_kv, self.n_heads // self.n_kv, self.v_head_dim, self.lam,
                              float(self.differential["eps"]), 1.0 - float(self.differential["diff"]))
         return attn
@@ -264,8 +268,9 @@ class PagedAttention:
         if self.qk_transform is not None:
             self.qk_transform.apply(q, k if cache.writes else None, ctx, self.n_heads, self.n_kv, self.head_dim)
             table = None          # the fused decode kernel takes the raw projections
-        if self.score_slopes is not None or self.v_head_dim != self.head_dim or self.exact_weights or self.segment:
-            table = None          # ... and has no bias on its scores, one head size, bfloat16 weights, no segments
+        if (self.score_slopes is not None or self.v_head_dim != self.head_dim or self.exact_weights or self.segment
+                or self.keep_first):
+            table = None          # ... and has no bias on its scores, one head size, bfloat16 weights, a plain window
         if (table is not None and cache.writes and ctx.all_single and self.dtype == torch.bfloat16 and group <= 16
                 and self.head_dim in kernels.TC_HEAD_DIMS and self.head_dim % 32 == 0):
             # decode: rotary encoding, cache write and attention in one kernel
@@ -287,7 +292,8 @@ class PagedAttention:
         attn = torch.empty((n, self.o_dim), dtype=self.dtype, device=q.device)
         kernels.attention(attn, q, cache.k, cache.v, ctx, cache.block_table, self.n_heads, self.n_kv,
                           self.head_dim, self.window or 0, self.scale, score_slopes=self.score_slopes,
-                          v_head_dim=self.v_head_dim, exact_weights=self.exact_weights, segment=self.segment)
+                          v_head_dim=self.v_head_dim, exact_weights=self.exact_weights, segment=self.segment,
+                          keep=self.keep_first)
         return attn
 
     @property

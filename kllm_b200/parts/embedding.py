@@ -1,7 +1,8 @@
 """Token embedding and output head.
 
 Embedding: params ``vocab``, ``width``, optional ``scale`` (every row is multiplied by it,
-default 1) and ``tensor`` (the table's full name where it is not ``<prefix>.weight``); tensor
+default 1), ``tensor`` (the table's full name where it is not ``<prefix>.weight``) and ``norm`` (a PartSpec of a norm
+that offers ``embed``: the rows are normed, and ``forward_rows(ids) -> (x, rows)`` also gives them in the model dtype); tensor
 ``<prefix>.weight`` [vocab, width]; ``forward(ids) -> x`` float32 [n, width], the residual
 stream (reference backend/model.cu:89-95, no scaling for Llama).
 
@@ -16,7 +17,7 @@ from __future__ import annotations
 import torch
 
 from .. import kernels
-from .spec import BuildEnv, PartSpec, TensorSpec, register_part
+from .spec import BuildEnv, PartSpec, TensorSpec, part_factory, register_part
 
 
 class TokenEmbedding:
@@ -25,15 +26,24 @@ class TokenEmbedding:
         self.width = int(spec.params["width"])
         self.scale = float(spec.params.get("scale", 1.0))
         self.name = spec.params.get("tensor") or spec.prefix + ".weight"
+        ns = spec.params.get("norm")
+        self.norm = part_factory("norm", ns.kind)(ns, env) if ns is not None else None
         self.table = None
 
     def tensor_specs(self):
-        return [TensorSpec(self.name, (self.vocab, self.width))]
+        return [TensorSpec(self.name, (self.vocab, self.width))] + (self.norm.tensor_specs() if self.norm else [])
 
     def bind(self, tensors):
         self.table = tensors[self.name]
+        if self.norm:
+            self.norm.bind(tensors)
+
+    def forward_rows(self, ids, last_token=None):
+        return self.norm.embed(self.table, ids, last_token, self.scale)
 
     def forward(self, ids, last_token=None):
+        if self.norm:
+            return self.forward_rows(ids, last_token)[0]
         x = torch.empty((ids.numel(), self.width), dtype=torch.float32, device=ids.device)
         kernels.embed(x, self.table, ids, last_token, self.scale)
         return x

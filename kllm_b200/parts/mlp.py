@@ -1,6 +1,7 @@
 """Gated feed-forward (SwiGLU): down( act(x Wg^T) * (x Wu^T) ).
 
-params: ``hidden``, ``intermediate``, ``activation`` ("silu"; "gelu_tanh": the tanh form of the gelu), optional
+params: ``hidden``, ``intermediate``, ``activation`` ("silu"; "gelu_tanh": the tanh form of the gelu; "clamped" with
+``limit`` L and ``alpha`` a: g sigmoid(a g) (u + 1) with g = min(x Wg^T, L) and u = clamp(x Wu^T, -L, L), no biases), optional
 ``tensors`` (gate, up, down -> full names), ``bias`` (True: all three projections have float32 biases,
 ``<weight name>.b``).  Tensors:
 ``<prefix>.{gate,up}_proj.weight`` [f, d] and ``<prefix>.down_proj.weight`` [d, f],
@@ -34,9 +35,12 @@ class GatedMLP:
         self.hidden = int(p["hidden"])
         self.inter = int(p["intermediate"])
         self.activation = p.get("activation", "silu")
-        if self.activation not in ("silu", "gelu_tanh"):
-            raise ValueError(f"gated feed-forward: activation {self.activation!r} has no kernel (silu, gelu_tanh)")
+        if self.activation not in ("silu", "gelu_tanh", "clamped"):
+            raise ValueError(f"gated feed-forward: activation {self.activation!r} has no kernel (silu, gelu_tanh, clamped)")
         self.has_bias = bool(p.get("bias", False))
+        self.limit, self.alpha = float(p.get("limit") or 0.0), float(p.get("alpha", 1.0))
+        if self.activation == "clamped" and (self.has_bias or not self.limit > 0):
+            raise ValueError("gated feed-forward: the clamped activation needs a positive limit and goes without biases")
         self.plain = self.activation == "silu" and not self.has_bias
         self.b_gate = self.b_up = self.b_down = None
         self.prefix = spec.prefix
@@ -84,14 +88,18 @@ class GatedMLP:
                 and w_gate.data_ptr() % 16 == 0 and w_up.data_ptr() % 16 == 0):
             # a step of a few rows: the weights streamed once, biases and activation in the product's epilogue
             return kernels.skinny_gemm(w_gate, weight_up=w_up, x=xn, epilogue="swiglu", prefetch=self._target(0),
-                                       bias=self.b_gate, bias_up=self.b_up, activation=self.activation)
-        if (self.plain and self.dtype == torch.bfloat16 and kernels.gemm_pays(n, self.inter, "swiglu")
-                and kernels.gemm_fits(xn, w_gate, act, "swiglu", w_up)):
+                                       bias=self.b_gate, bias_up=self.b_up, activation=self.activation, limit=self.limit,
+                                       alpha=self.alpha)
+        epilogue = "clamped" if self.activation == "clamped" else "swiglu" if self.plain else None
+        if (epilogue and self.dtype == torch.bfloat16 and kernels.gemm_pays(n, self.inter, epilogue)
+                and kernels.gemm_fits(xn, w_gate, act, epilogue, w_up)):
             # large portions: both products and the activation in one tcgen05 kernel
-            kernels.gemm(xn, w_gate, weight_up=w_up, epilogue="swiglu", out=act)
+            kernels.gemm(xn, w_gate, weight_up=w_up, epilogue=epilogue, out=act, limit=self.limit, alpha=self.alpha)
         else:
             gu = kernels.linear(xn, self.w_gate_up, out_dtype=torch.float32)
-            if self.plain:
+            if self.activation == "clamped":
+                kernels.clamped_glu(act, gu[:, :self.inter], gu[:, self.inter:], self.limit, self.alpha)
+            elif self.plain:
                 kernels.silu_mul(act, gu[:, :self.inter], gu[:, self.inter:])
             else:
                 kernels.biased_glu(act, gu[:, :self.inter], gu[:, self.inter:], self.b_gate, self.b_up, self.activation)
@@ -104,6 +112,8 @@ class GatedMLP:
         # gate and up stay float32 until the activation has been applied; the down
         # projection's float32 result goes into the residual stream unrounded
         n = xn.shape[0]
+        if self.activation == "clamped":
+            return kernels.linear(self._activation(xn), self.w_down, out_dtype=torch.float32, small_ok=True)
         if not self.plain:
             y = torch.zeros((n, self.hidden), dtype=torch.float32, device=xn.device)
             self.forward_add(y, xn, ctx)

@@ -15,7 +15,7 @@ import torch
 
 # registering the built-in part kinds
 from . import (attention, block, embedding, gla, latent_attention, lightning, mlp, moe, norm, qk_norm, rotary,  # noqa: F401
-               side_by_side, side_input, stream_entry, streams, wkv)
+               side_by_side, side_input, ssd, stream_entry, streams, wkv)
 from .context import LayerCache, StepContext
 from .spec import BuildEnv, ModelSpec, PagedKVNeed, StateNeed, TensorSpec, part_factory
 
@@ -104,8 +104,14 @@ class DecoderModel:
     def forward(self, ctx: StepContext, caches: List[LayerCache]) -> Optional[torch.Tensor]:
         """Logits float32 [ctx.n_want, vocab] at ``ctx.want_rows`` (None when no row
         is wanted; the cache is still filled)."""
-        x = self.embedding.forward(ctx.token_ids, ctx.last_token)
         pending = None
+        first = self.blocks[self.schedule[0].block] if self.schedule and not self.entries else None
+        if getattr(self.embedding, "norm", None) is not None and getattr(first, "accepts_ready_rows", False):
+            # the kernel that norms the embedding's rows also leaves them in the first layer's dtype
+            x, rows = self.embedding.forward_rows(ctx.token_ids, ctx.last_token)
+            pending = block.ReadyRows(rows)
+        else:
+            x = self.embedding.forward(ctx.token_ids, ctx.last_token)
         held = [e.begin(x, bool(self.schedule) and self.schedule[0].entry is not None
                         and self.schedule[0].entry[0] == j) for j, e in enumerate(self.entries)]
         for i, call in enumerate(self.schedule):
@@ -113,7 +119,7 @@ class DecoderModel:
             if cache.writes != call.writes_cache:
                 cache = LayerCache(cache.k, cache.v, cache.block_table, cache.state,
                                    writes=call.writes_cache, page_size=cache.page_size, states=cache.states)
-            block = self.blocks[call.block]
+            layer = self.blocks[call.block]
             if call.entry is not None:
                 if hasattr(pending, "settle"):
                     pending = pending.settle(x)
@@ -121,10 +127,10 @@ class DecoderModel:
                     x.add_(pending)
                     pending = None
                 self.entries[call.entry[0]].apply(x, held[call.entry[0]], call.entry[1])
-            if hasattr(pending, "settle") and not getattr(block, getattr(pending, "accepted_by", "accepts_deferred_norm"),
+            if hasattr(pending, "settle") and not getattr(layer, getattr(pending, "accepted_by", "accepts_deferred_norm"),
                                                            False):
                 pending = pending.settle(x)
-            pending = block.forward(x, pending, ctx, cache)
+            pending = layer.forward(x, pending, ctx, cache)
             if self.tap is not None:
                 if hasattr(pending, "peek"):
                     self.tap(i, pending.peek(x))       # what settle() would leave in x, without settling

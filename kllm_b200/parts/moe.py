@@ -7,7 +7,7 @@ gated feed-forwards, chosen by a router.
      or sum over the chosen e of  s_e expert_e(h)        (``weight_on`` "output")
 
 params: ``hidden``, ``experts``, ``top``, ``expert_ff``, ``score`` ("sigmoid" | "softmax"),
-``renormalize`` (divide the chosen scores by their sum), ``weight_on`` ("input" | "output"),
+``renormalize`` (divide the chosen scores by their sum, plus ``sum_eps`` if given), ``weight_on`` ("input" | "output"),
 optional ``router_tensor`` and ``expert_tensors`` (a format string with ``{e}`` and ``{m}``
 for the expert's number and matrix gate/up/down; default ``<prefix>.e{e}.{m}``).
 The router table stays float32 in both dtypes.  At bind time the experts' matrices are
@@ -34,6 +34,13 @@ optionally gate_logit -> full names)}: one more expert that every token runs, ad
 routed ones, multiplied by sigmoid(w . x) when ``gate_logit`` names a [1, d] tensor.  Its gate,
 up and logit rows are one product; the sigmoid and the sum are part of the combine kernel.
 
+``activation`` "relu2": the experts have no gate, W_down relu(W_up x)^2, and no gate tensors; a ``shared`` expert with
+this activation likewise.
+``correction`` (the full name of a float32 vector, one value per expert, identity experts included): joins the scores
+when the experts are chosen, not in their weights.
+``identity`` (I): the choice is among ``experts`` + I, of which the last I have no tensors: their output is the layer's
+input (with ``weight_on`` "output", times the weight).  The router has a row for each of them.
+
 A step sorts its (token, choice) pairs by expert on the device and runs two grouped
 products over the sorted rows (csrc/moe.cu); shapes and launch sizes depend on the number
 of tokens alone, never on the routing, so decode steps can be replayed as CUDA graphs.
@@ -54,8 +61,12 @@ class RoutedExperts:
         self.experts = int(p["experts"])
         self.top = int(p["top"])
         self.ff = int(p["expert_ff"])
-        if not (1 <= self.top <= self.experts <= 1024):
-            raise ValueError(f"routed experts: {self.top} of {self.experts} (at most 1024 experts)")
+        self.identity = int(p.get("identity") or 0)
+        self.choices = self.experts + self.identity
+        if not (1 <= self.top <= self.choices <= 1024):
+            raise ValueError(f"routed experts: {self.top} of {self.choices} (at most 1024 experts)")
+        self.correction_name, self.correction = p.get("correction"), None
+        self.sum_eps = float(p.get("sum_eps") or 0.0)
         self.score = p.get("score", "sigmoid")
         self.renormalize = bool(p.get("renormalize", False))
         self.weight_on = p.get("weight_on", "input")
@@ -78,7 +89,11 @@ class RoutedExperts:
                                 or self.top > self.groups_keep * (self.experts // self.groups)):
             raise ValueError(f"routed experts: {self.top} of {self.experts} experts in {self.groups} groups of which "
                              f"{self.groups_keep} are kept")
+        if (self.identity or self.correction_name) and (self.routing == "table" or self.weight_on == "input"):
+            raise ValueError("routed experts: identity experts and corrections go with scores that weigh the outputs")
         self.act = self._activation(p)
+        self.plain = self.act["activation"] == "relu2"              # experts without a gate
+        self.matrices = ("up", "down") if self.plain else ("gate", "up", "down")
         # a step with at least this many rows per expert on average, a table and ids that the host knows runs
         # the library's products expert by expert (``_forward_planned``); below it the grouped kernels
         self.planned_rows = int(p.get("planned_rows") or 128)
@@ -90,8 +105,8 @@ class RoutedExperts:
     @staticmethod
     def _activation(p):
         kind = p.get("activation", "silu")
-        if kind not in ("silu", "clamped"):
-            raise ValueError(f"routed experts: activation {kind!r} (silu, clamped)")
+        if kind not in ("silu", "clamped", "relu2"):
+            raise ValueError(f"routed experts: activation {kind!r} (silu, clamped, relu2)")
         limit, alpha = float(p.get("limit") or 0.0), float(p.get("alpha") or 1.0)
         if kind == "clamped" and not limit > 0:
             raise ValueError("routed experts: the clamped activation needs a positive limit")
@@ -105,17 +120,18 @@ class RoutedExperts:
             out = [TensorSpec(self.table_name, (self.table_vocab, self.top), store="int32",
                               init=f"distinct:{self.experts}")]
         else:
-            out = [TensorSpec(self.router_name, (self.experts, self.hidden), store="float32")]
+            out = [TensorSpec(self.router_name, (self.choices, self.hidden), store="float32")]
+        if self.correction_name:
+            out.append(TensorSpec(self.correction_name, (self.choices,), store="float32", init="zeros"))
         if self.shared:
             f, n = self.shared["ff"], self.shared["names"]
-            out += [TensorSpec(n["gate"], (f, self.hidden)), TensorSpec(n["up"], (f, self.hidden)),
-                    TensorSpec(n["down"], (self.hidden, f))]
+            out += [TensorSpec(n["gate"], (f, self.hidden))] if n.get("gate") else []
+            out += [TensorSpec(n["up"], (f, self.hidden)), TensorSpec(n["down"], (self.hidden, f))]
             if n.get("gate_logit"):
                 out.append(TensorSpec(n["gate_logit"], (1, self.hidden)))
         for e in range(self.experts):
-            out += [TensorSpec(self._name(e, "gate"), (self.ff, self.hidden)),
-                    TensorSpec(self._name(e, "up"), (self.ff, self.hidden)),
-                    TensorSpec(self._name(e, "down"), (self.hidden, self.ff))]
+            out += [TensorSpec(self._name(e, m), (self.hidden, self.ff) if m == "down" else (self.ff, self.hidden))
+                    for m in self.matrices]
         return out
 
     def bind(self, tensors):
@@ -125,10 +141,12 @@ class RoutedExperts:
         self.table_host = self.table.cpu().numpy().astype("int16") if self.routing == "table" else None
         if self.shared:
             n = self.shared["names"]
-            rows = [tensors[n["gate"]], tensors[n["up"]]] + ([tensors[n["gate_logit"]]] if n.get("gate_logit") else [])
+            rows = [tensors[n[m]] for m in ("gate", "up") if n.get(m)] + ([tensors[n["gate_logit"]]] if n.get("gate_logit") else [])
             self.shared["w_in"] = torch.cat(rows, dim=0).contiguous()       # gate rows, up rows, the logit's row
             self.shared["w_down"] = tensors[n["down"]]
-        self.w_gate_up = torch.stack([torch.cat([tensors[self._name(e, "gate")], tensors[self._name(e, "up")]], dim=0)
+        self.correction = tensors[self.correction_name].contiguous() if self.correction_name else None
+        # the experts' up rows, behind their gate rows where they have a gate
+        self.w_gate_up = torch.stack([torch.cat([tensors[self._name(e, m)] for m in self.matrices[:-1]], dim=0)
                                       for e in range(self.experts)]).contiguous()
         self.w_down = torch.stack([tensors[self._name(e, "down")] for e in range(self.experts)]).contiguous()
 
@@ -136,6 +154,8 @@ class RoutedExperts:
         """(activation rows [n, f], gate logits float32 [n, 1] or None) of the expert that every token runs."""
         sh, f = self.shared, self.shared["ff"]
         w = sh["w_in"]
+        if sh["act"]["activation"] == "relu2":
+            return kernels.linear_relu2(xn, w), None
         if sh["act"]["activation"] == "silu" and w.shape[0] == 2 * f and xn.is_contiguous():
             # no gate logit among the rows: the activation in the product's epilogue
             w_gate, w_up = w[:f], w[f:]
@@ -210,7 +230,8 @@ class RoutedExperts:
         if self.routing == "table" or (self.shared and self.shared["names"].get("gate_logit")):
             x.add_(self.forward(h, ctx))
             return
-        kernels.moe_combine(self._routed(h, ctx), self.top, into=x)
+        parts, identity = self._routed(h, ctx)
+        kernels.moe_combine(parts, self.top, into=x, identity=identity)
         if self.shared is not None:
             act, _ = self._shared_act(h)
             kernels.linear_into(x, act, self.shared["w_down"])
@@ -221,27 +242,30 @@ class RoutedExperts:
             plan = self._plan(ctx, xn.shape[0])
             if plan is not None:
                 return self._forward_planned(xn, plan)
-        parts = self._routed(xn, ctx)
+        parts, identity = self._routed(xn, ctx)
         if self.shared is None:
-            return kernels.moe_combine(parts, self.top)
+            return kernels.moe_combine(parts, self.top, identity=identity)
         rows, logit = self._shared(xn)
-        return kernels.moe_combine(parts, self.top, shared=rows, gate=logit)
+        return kernels.moe_combine(parts, self.top, shared=rows, gate=logit, identity=identity)
 
     def _routed(self, xn, ctx):
-        """Float32 rows token * top + choice of the chosen experts' weighted outputs."""
+        """(float32 rows token * top + choice of the chosen experts' weighted outputs, what ``moe_combine`` needs for
+        identity experts or None)."""
         if self.routing == "table":
             idx, wt = kernels.moe_table_route(ctx.token_ids, self.table, self.experts, self.table_weight, ctx.last_token)
         else:
             idx, wt = kernels.moe_route(xn, self.router, self.top, self.score, self.renormalize, self.groups,
-                                        self.groups_keep)
-        offsets, perm = kernels.moe_sort(idx, self.experts)
+                                        self.groups_keep, correction=self.correction, sum_eps=self.sum_eps)
+        # pairs of identity experts sort behind those of the experts, beyond the rows that the products walk
+        offsets, perm = kernels.moe_sort(idx, self.choices)
+        identity = (idx, wt, xn, self.experts) if self.identity else None
         on_input = self.weight_on == "input"
-        if kernels.moe_gemm_tcgen05_pays(xn, self.w_gate_up, perm.numel(), True, on_input):
+        if kernels.moe_gemm_tcgen05_pays(xn, self.w_gate_up, perm.numel(), True, on_input, self.act["activation"]):
             # a large step in bfloat16: tiles of 128 rows per expert on the tcgen05 tensor cores
             act = kernels.moe_gemm_tcgen05(xn, self.w_gate_up, offsets, perm, wt, self.top, gated=True, **self.act)
-            return kernels.moe_gemm_tcgen05(act, self.w_down, offsets, perm, wt, self.top, gated=False, scale_out=True)
+            return kernels.moe_gemm_tcgen05(act, self.w_down, offsets, perm, wt, self.top, gated=False, scale_out=True), identity
         act = kernels.moe_gemm(xn, self.w_gate_up, offsets, perm, wt, self.top, gated=True, scale_in=on_input, **self.act)
-        return kernels.moe_gemm(act, self.w_down, offsets, perm, wt, self.top, gated=False, scale_out=not on_input)
+        return kernels.moe_gemm(act, self.w_down, offsets, perm, wt, self.top, gated=False, scale_out=not on_input), identity
 
 
 register_part("feed_forward", "routed_experts", RoutedExperts)

@@ -1,4 +1,4 @@
-"""RMSNorm with the residual sum folded in, and layer norm with gain and bias (``LayerNorm``, at the end).
+"""RMSNorm with the residual sum folded in, and layer norm with gain and optional bias (``LayerNorm``, at the end).
 
 params: ``width``, ``eps``, optional ``tensor`` (the gain's full name where it is not
 ``<prefix>.weight``), optional ``offset`` (the files hold the gain minus this number, e.g. a weight
@@ -68,30 +68,60 @@ class RMSNorm:
 class LayerNorm:
     """Layer norm with gain and bias: (x - mean) / sqrt(var + eps) * w + b, the variance being the
     mean of the squared deviations.  params: ``width``, ``eps``, optional ``tensor`` (the gain's
-    full name where it is not ``<prefix>.weight``) and ``bias_tensor`` (default: the gain's name
-    + ``.b``).  Both tensors stay float32; mean, variance and scale are float32 in both dtypes.
-    Same interface as ``RMSNorm.forward``; no part folds this norm into its own kernels."""
+    full name where it is not ``<prefix>.weight``), ``bias_tensor`` (default: the gain's name
+    + ``.b``), ``bias`` (False: there is none), ``layer_scale`` (full name of a vector [width] that multiplies the
+    result element by element, the scale of a sublayer whose output this norms) and ``factor`` (a number that
+    multiplies it, default 1): both act on gain and bias once, in float32, when the weights are bound.
+    All tensors stay float32; mean, variance and scale are float32 in both dtypes.
+    Same interface as ``RMSNorm``; no part folds this norm into its own kernels.  ``embed(table, ids, last_token, scale)
+    -> (x, rows)``: the norm of an embedding's rows, with the look-up in the same kernel; x float32, rows the same in
+    the model dtype (x itself when that is float32)."""
 
     def __init__(self, spec: PartSpec, env: BuildEnv):
         self.width = int(spec.params["width"])
         self.eps = float(spec.params["eps"])
         self.name = spec.params.get("tensor") or spec.prefix + ".weight"
-        self.bias_name = spec.params.get("bias_tensor") or self.name + ".b"
+        self.bias_name = (spec.params.get("bias_tensor") or self.name + ".b") if spec.params.get("bias", True) else None
+        self.scale_name = spec.params.get("layer_scale")
+        self.factor = float(spec.params.get("factor", 1.0))
         self.dtype = env.dtype
         self.gain = self.bias = None
 
     def tensor_specs(self):
-        return [TensorSpec(self.name, (self.width,), store="float32", init="gain"),
-                TensorSpec(self.bias_name, (self.width,), store="float32", init="zeros")]
+        out = [TensorSpec(self.name, (self.width,), store="float32", init="gain")]
+        if self.bias_name:
+            out.append(TensorSpec(self.bias_name, (self.width,), store="float32", init="zeros"))
+        if self.scale_name:
+            out.append(TensorSpec(self.scale_name, (self.width,), store="float32", init="gain"))
+        return out
 
     def bind(self, tensors):
-        self.gain, self.bias = tensors[self.name], tensors[self.bias_name]
+        def scaled(t):
+            t = t * tensors[self.scale_name] if self.scale_name else t
+            return (t * self.factor if self.factor != 1.0 else t).contiguous()
+        self.gain = scaled(tensors[self.name])
+        self.bias = scaled(tensors[self.bias_name]) if self.bias_name else None
 
     def forward(self, x, res=None, rows=None):
         n = x.shape[0] if rows is None else rows.numel()
         out = torch.empty((n, self.width), dtype=self.dtype, device=x.device)
         kernels.add_layernorm(x, res, out, self.gain, self.bias, self.eps, rows=rows)
         return out
+
+    def add_normed(self, x, y, then=None):
+        out = None
+        if isinstance(then, str):
+            if then != "rows":
+                raise ValueError(f"add_normed: then={then!r} (a norm, or 'rows')")
+            out = torch.empty(x.shape, dtype=self.dtype, device=x.device)
+        kernels.layernorm_add(x, y, self.gain, self.bias, self.eps, out=out)
+        return out if then is None or isinstance(then, str) else then.forward(x, None)
+
+    def embed(self, table, ids, last_token, scale):
+        x = torch.empty((ids.numel(), self.width), dtype=torch.float32, device=ids.device)
+        rows = None if self.dtype == torch.float32 else torch.empty(x.shape, dtype=self.dtype, device=ids.device)
+        kernels.embed_layernorm(x, table, ids, self.gain, self.bias, self.eps, last_token, scale, rows=rows)
+        return x, (x if rows is None else rows)
 
 
 register_part("norm", "rmsnorm", RMSNorm)

@@ -28,6 +28,8 @@ def rotary_frequencies(dims: int, base: float, scaling=None):
     f stays where l < original / high, becomes f / factor where l > original / low, and in between,
     with s = (original / l - low) / (high - low), (1 - s) f / factor + s f.
 
+    ``kind`` "linear" (``factor``): every f is divided by the factor.
+
     ``kind`` "ramp" (``factor``, ``original``, ``fast``, ``slow``): with where(t) = dims ln(original /
     (2 pi t)) / (2 ln base), lo = max(floor(where(fast)), 0), hi = min(ceil(where(slow)), dims - 1) and
     ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1): f_i / factor * ramp_i + f_i (1 - ramp_i); the
@@ -38,7 +40,12 @@ def rotary_frequencies(dims: int, base: float, scaling=None):
     freq = [float(base) ** (-2.0 * i / dims) for i in range(half)]
     if not scaling:
         return torch.tensor(freq, dtype=torch.float64), 1.0
-    kind, factor, orig = scaling["kind"], float(scaling["factor"]), float(scaling["original"])
+    kind, factor = scaling["kind"], float(scaling["factor"])
+    if kind == "linear":
+        return torch.tensor([f / factor for f in freq], dtype=torch.float64), 1.0
+    if kind not in ("wavelength", "ramp"):
+        raise ValueError(f"rotary scaling of kind {kind!r} (linear, wavelength, ramp)")
+    orig = float(scaling["original"])
     if kind == "wavelength":
         low, high = float(scaling["low"]), float(scaling["high"])
         out = []
@@ -52,7 +59,7 @@ def rotary_frequencies(dims: int, base: float, scaling=None):
                 s = (orig / wave - low) / (high - low)
                 out.append((1.0 - s) * f / factor + s * f)
         return torch.tensor(out, dtype=torch.float64), 1.0
-    if kind == "ramp":
+    else:
         def where(turns):
             return dims * math.log(orig / (2.0 * math.pi * turns)) / (2.0 * math.log(float(base)))
         lo = max(math.floor(where(float(scaling["fast"]))), 0)
@@ -62,7 +69,6 @@ def rotary_frequencies(dims: int, base: float, scaling=None):
             ramp = min(1.0, max(0.0, (i - lo) / max(hi - lo, 0.001)))
             out.append(f / factor * ramp + f * (1.0 - ramp))
         return torch.tensor(out, dtype=torch.float64), 0.1 * math.log(factor) + 1.0
-    raise ValueError(f"rotary scaling of kind {kind!r} (wavelength, ramp)")
 
 
 class RotaryEmbedding:

@@ -94,6 +94,7 @@ class ModelSpec:
 class PagedKVNeed:
     """Keys and values in pages.  window None: every key is kept; window W: only
     the last W keys of a request are ever read, older pages may be given back.
+    keep_first: beside a window, the first so many keys of a request are read as well and their pages stay.
     v_head_dim: the size of a head's values where it differs from the keys' (None: the same).
     values_are_keys: one row per token serves as key and as value (a layer that attends
     through a cached low-rank latent): no value store is kept, the views of the values are the
@@ -107,6 +108,7 @@ class PagedKVNeed:
     v_head_dim: Optional[int] = None
     values_are_keys: bool = False
     n_v_heads: Optional[int] = None
+    keep_first: int = 0
 
     @property
     def value_dim(self) -> int:
