@@ -52,6 +52,8 @@ output norms, a token side input) beside a dense Sozarax model of equal size, th
 (a recurrent mixer, attention with norms over the whole projections, a plain feed-forward), and beside a Llama.
 ``--design dirarax`` measures the Dirarax design (gated linear attention, attention and retention side by side, one norm
 for both sublayers with a token shift, biased and routed feed-forwards) beside a Sozarax and a Llama.
+``--design rupenex`` measures the Rupenex design (Mamba-2 layers, window attention with kept first keys and sinks, layer norms
+with layer scales on the sublayers' output, clamped and routed feed-forwards with identity experts) beside a Dirarax and a Llama.
 """
 from __future__ import annotations
 
@@ -258,8 +260,8 @@ def main():
     ap.add_argument("--workload", default="", choices=["", "llama2-7b-mixed"],
                     help="llama2-7b-mixed: 32 requests, prompts uniform in [128, 3072], 128 new tokens each, through "
                          "the scheduler (a record of its own, not the bench line)")
-    ap.add_argument("--design", default="", choices=["", "sozarax", "nutizen", "ronurax", "senulix", "dirarax"],
-                    help="sozarax, nutizen, ronurax, senulix, dirarax: prefill and decode of that design at two layer sizes beside a Llama of equal size, and "
+    ap.add_argument("--design", default="", choices=["", "sozarax", "nutizen", "ronurax", "senulix", "dirarax", "rupenex"],
+                    help="sozarax, nutizen, ronurax, senulix, dirarax, rupenex: prefill and decode of that design at two layer sizes beside a Llama of equal size, and "
                          "its kernels against their rooflines (a record of its own, not the bench line)")
     args = ap.parse_args()
     if args.timeline:
@@ -720,6 +722,29 @@ def dirarax_config(width, layers, heads, kv_heads, head_dim, ff, experts, top, e
             "layers": [{"type": "parallel" if i % 4 == 3 else "gla", "mixer": dict(par if i % 4 == 3 else gla),
                         "mlp": dict(dense if i % 2 == 0 else moe)} for i in range(layers)],
             "loop": {"start": 0, "stop": layers, "times": 1}}
+
+
+def rupenex_config(width, layers, heads, kv_heads, head_dim, ff, experts, top, expert_ff, vocab, window, keep):
+    """A Rupenex model of ``layers`` layers in the pattern of three Mamba-2 layers (twice the width, heads of 64 values,
+    128 state channels, a group for every 8 heads) and one of window attention; dense and routed feed-forwards in turn, half
+    as many identity experts as experts."""
+    mh = 2 * width // 64
+    mamba = {"heads": mh, "vdim": 64, "state": 128, "groups": mh // 8, "conv": 4, "norm_groups": mh // 8}
+    attn = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+            "mask": {"size": window, "keep_first": keep}, "rot": {"base": 500000.0, "dims": head_dim, "scaling": {"factor": 8.0}}}
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top, "identity": experts // 2},
+           "shared": {"ff": expert_ff}}
+    return {"architecture": "Rupenex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "layers": [{"type": "attention" if i % 4 == 3 else "mamba2", "mixer": dict(attn if i % 4 == 3 else mamba),
+                        "mlp": dict(dense if i % 2 == 0 else moe)} for i in range(layers)]}
+
+
+RUPENEX_EXTRA = {
+    # name: window, kept first keys
+    "2048-wide": (1024, 64),
+    "4096-wide": (1024, 64),
+}
 
 
 SENULIX_EXTRA = {
@@ -1529,8 +1554,230 @@ def design_comparison(args):
             del wgu
         return rows
 
+    def rupenex_rows(width, heads, kv, hd, ff, E, top, eff, window, keep):
+        """The Rupenex design's own kernels, each beside the kernels of the closest design that do the like work."""
+        import itertools
+        import types
+        rows = []
+        dev, f32 = "cuda", torch.float32
+        A = heads * hd
+        esz = 2 if dtype == "bfloat16" else 4
+        hbm, tens = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+        cores = 2 * 128 * kernels.sm_count() * 1.9e9        # float32 operations a second of the CUDA cores
+
+        def ctx_of(n_new, start):
+            S = len(n_new)
+            qs = torch.tensor([0] + list(itertools.accumulate(n_new)), dtype=torch.int32, device=dev)
+            return types.SimpleNamespace(
+                n_tokens=sum(n_new), n_requests=S, q_start=qs,
+                token_req=torch.repeat_interleave(torch.arange(S, dtype=torch.int32), torch.tensor(n_new)).to(dev),
+                start_pos=torch.tensor(start, dtype=torch.int32, device=dev),
+                positions=torch.cat([torch.arange(s, s + c, dtype=torch.int32) for s, c in zip(start, n_new)]).to(dev),
+                state_slots=torch.arange(S, dtype=torch.int32, device=dev), host_n_new=list(n_new),
+                host_start_pos=list(start), all_single=all(c == 1 for c in n_new),
+                max_ctx=max(s + c for s, c in zip(start, n_new)), split_bound=0, max_new=max(n_new))
+
+        def row(name, us, by, like=None, tensor=0.0, core=0.0):
+            floor, bound = max((by / hbm * 1e6, "memory"), (tensor / tens * 1e6 if dtype == "bfloat16" else 0.0, "tensor"),
+                               (core / cores * 1e6, "float32 cores"))
+            rows.append({"kernel": name, "us": round(us, 1), "floor_us": round(floor, 2), "bound": bound,
+                         "times_floor": round(us / floor, 1), "like": like})
+
+        def each(call, inner=16):
+            # recorded once and replayed: the host's launches do not stand between the kernels
+            for k in range(3):
+                call(k)
+            torch.cuda.synchronize()
+            graph = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(graph):
+                for k in range(inner):
+                    call(k)
+            return timed(graph.replay) * 1e3 / inner
+        mh, mv, N = 2 * width // 64, 64, 128
+        G = mh // 8
+        gh, gk, gv, R = width // 256, 128, 256, 16
+        for name, n_new, start in (("prefill", [T], [0]), ("decode", [1] * B, [ctx - 1] * B)):
+            c, S, n = ctx_of(n_new, start), len(n_new), sum(n_new)
+            # ---- recurrences up to the normed and gated row: the state read and written once, the rows read and
+            # written once, and four float32 operations per state element and row on the CUDA cores ----
+            inner, chn = mh * mv, mh * mv + 2 * G * N
+            P = inner + chn + mh
+            projs = rotate(lambda: torch.randn(n, P, device=dev) * 0.3, 4 * n * P)
+            states = rotate(lambda: (torch.zeros(S, mh * N * mv, device=dev), torch.zeros(S, 4 * chn, device=dev)), 4 * S * mh * N * mv)
+            conv, cb = torch.randn(chn, 4, device=dev) * 0.4, torch.zeros(chn, device=dev)
+            dtb, alog, dsk, gain = (torch.full((mh,), v, device=dev) for v in (-4.0, 1.0, 1.0, 1.0))
+            gain = torch.ones(inner, device=dev)
+            y = torch.empty((n, inner), dtype=tdt, device=dev)
+
+            def ssd(i):
+                st, ring = states[i % len(states)]
+                o = kernels.ssd(projs[i % len(projs)], conv, cb, dtb, alog, dsk, st, ring, c, mh, G, N, mv)
+                kernels.part_norm(y, o, gain, G, 1e-6)
+            row(f"mamba2 {name} (convolution, scan, gate and norm)", each(ssd), 8.0 * S * mh * N * mv + 4.0 * n * P + esz * n * inner,
+                like=f"gated linear attention {name}", core=4.0 * n * mh * N * mv)
+            del projs, states
+            KA, VB = gh * gk, gh * gv
+            P2 = 2 * KA + 2 * VB + R
+            projs = rotate(lambda: torch.randn(n, P2, device=dev) * 0.3, 4 * n * P2)
+            states = rotate(lambda: torch.zeros(S, KA * gv, device=dev), 4 * S * KA * gv)
+            w2, b2, g2 = (torch.randn(KA, R, device=dev) * 0.1).to(tdt), torch.full((KA,), 4.0, device=dev), torch.ones(VB, device=dev)
+            y2 = torch.empty((n, VB), dtype=tdt, device=dev)
+
+            def gla(i):
+                p = projs[i % len(projs)]
+                kernels.gla(y2, p[:, :KA], p[:, KA:2 * KA], p[:, 2 * KA:2 * KA + VB], p[:, 2 * KA + VB:2 * (KA + VB)],
+                            states[i % len(states)], c, gh, gk, gv, g2, 1e-6, low=p[:, P2 - R:], w2=w2, w2_bias=b2, tau=16.0,
+                            q_scale=gk ** -0.5)
+            row(f"gated linear attention {name}", each(gla), 8.0 * S * KA * gv + 4.0 * n * P2 + esz * n * VB,
+                core=4.0 * n * KA * gv)
+            del projs, states
+            # ---- norms on a sublayer's output, with the next sublayer's rows ----
+            xs = rotate(lambda: (torch.randn(n, width, device=dev), torch.randn(n, width, device=dev)), 8 * n * width)
+            gw = torch.ones(width, device=dev)
+            orow = torch.empty((n, width), dtype=tdt, device=dev)
+            row(f"layer norm into the stream {name}", each(lambda i: kernels.layernorm_add(*xs[i % len(xs)], gw, None, 1e-6, out=orow)),
+                n * width * (12.0 + esz), like=f"senulix norm into the stream {name}")
+            row(f"senulix norm into the stream {name}", each(lambda i: kernels.rmsnorm_add(*xs[i % len(xs)], gw, 1e-6, out=orow)),
+                n * width * (12.0 + esz))
+            del xs
+            # ---- window attention with kept keys and sinks ----
+            per = -(-max(s + m for s, m in zip(start, n_new)) // page)
+            table = torch.arange(S * per, dtype=torch.int32, device=dev).view(S, per).contiguous()
+            caches = rotate(lambda: tuple(torch.randn(S * per, kv, page, hd, device=dev).to(tdt) for _ in range(2)),
+                            S * per * kv * page * 2 * hd * esz)
+            q = (torch.randn(n, A, device=dev) * 0.2).to(tdt)
+            out = torch.empty(n, A, device=dev, dtype=tdt)
+            sinks = torch.zeros(heads, device=dev)
+
+            def seen(p, kept):
+                return min(p + 1, window) + min(kept, max(0, p + 1 - window))
+            for what, kept, kw in (("kept-keys attention", keep, dict(sinks=sinks, exact_weights=True, keep=keep)),
+                                   ("nutizen-form attention", 0, dict(sinks=sinks, exact_weights=True)), ("llama attention", 0, {})):
+                pairs = sum(seen(p, kept) for s, m in zip(start, n_new) for p in range(s, s + m))
+                keys = sum(min(s + m, window + m - 1 + kept) for s, m in zip(start, n_new))
+                row(f"{what} {name} (window {window})",
+                    each(lambda i: kernels.attention(out, q, *caches[i % len(caches)], c, table, heads, kv, hd, window, hd ** -0.5, **kw)),
+                    keys * kv * 2 * hd * esz + 2 * n * A * esz, tensor=4.0 * pairs * heads * hd,
+                    like=f"nutizen-form attention {name} (window {window})" if kept else None)
+            # ---- norm, rotation and cache write ----
+            W = A + 2 * kv * hd
+            projs = rotate(lambda: torch.randn(n, W, device=dev), 4 * n * W)
+            freq = (5e5 ** (-2.0 * torch.arange(hd // 2, dtype=torch.float64) / hd) / 8).to(dev)
+            qo, hg = torch.empty((n, A), dtype=tdt, device=dev), torch.ones(hd, device=dev)
+            for what, gains, inter, like in (("head norms, rotation and cache write", (hg, hg), False, f"dirarax rotation and cache write {name}"),
+                                             ("dirarax rotation and cache write", (None, None), True, None)):
+                row(f"{what} {name}",
+                    each(lambda i: kernels.headnorm_rope_append(qo, projs[i % len(projs)], None, *gains, 1e-6, freq, 1.0, hd,
+                                                                c.positions, c.token_req, table, *caches[0], heads, kv, kv, hd, hd,
+                                                                interleaved=inter)), n * W * (4 + esz), like=like)
+            del caches, projs
+            # ---- the dense feed-forward's gate and up half, clamped, beside Llama's silu ----
+            wgu = rotate(lambda: (torch.randn(2 * ff, width, device=dev) * 0.02).to(tdt), 2 * ff * width * esz)
+            h = (torch.randn(n, width, device=dev)).to(tdt)
+
+            def glu(clamped):
+                def call(i):
+                    w = wgu[i % len(wgu)]
+                    kw = dict(limit=7.0, alpha=1.702) if clamped else {}
+                    if kernels.skinny_fits(n, width, tdt):
+                        kernels.skinny_gemm(w[:ff], weight_up=w[ff:], x=h, epilogue="swiglu", activation="clamped" if clamped else "silu", **kw)
+                        return
+                    o = torch.empty((n, ff), dtype=tdt, device=dev)
+                    epi = "clamped" if clamped else "swiglu"
+                    if tdt == torch.bfloat16 and kernels.gemm_pays(n, ff, epi):
+                        kernels.gemm(h, w[:ff], weight_up=w[ff:], epilogue=epi, out=o, **kw)
+                        return
+                    gu = kernels.linear(h, w, out_dtype=f32)
+                    if clamped:
+                        kernels.clamped_glu(o, gu[:, :ff], gu[:, ff:], 7.0, 1.702)
+                    else:
+                        kernels.silu_mul(o, gu[:, :ff], gu[:, ff:])
+                return call
+            by, fl = 2.0 * ff * width * esz + n * (width + ff) * esz, 4.0 * n * ff * width
+            row(f"clamped gate and up {name}", each(glu(True)), by, like=f"llama gate and up {name}", tensor=fl)
+            row(f"llama gate and up {name}", each(glu(False)), by, tensor=fl)
+            del wgu
+            # ---- routed experts: routing, sort, products and sum ----
+            I = E // 2
+            router, corr = torch.randn(E + I, width, device=dev) * 0.05, torch.zeros(E + I, device=dev)
+            idx, wt = kernels.moe_route(h, router, top, "softmax", True, correction=corr, sum_eps=1e-20)
+            real = int((idx < E).sum())
+            used = int(torch.unique(idx[idx < E]).numel())
+            wu = rotate(lambda: ((torch.randn(E, eff, width, device=dev) * 0.02).to(tdt), (torch.randn(E, width, eff, device=dev) * 0.02).to(tdt)),
+                        2 * E * eff * width * esz)
+
+            def experts(plain, wts, rt, cr):
+                act = "relu2" if plain else "silu"
+
+                def call(i):
+                    w_in, w_dn = wts[i % len(wts)]
+                    ix, ww = kernels.moe_route(h, rt, top, "softmax", True, correction=cr, sum_eps=1e-20 if plain else 0.0)
+                    off, perm = kernels.moe_sort(ix, rt.shape[0])
+                    if kernels.moe_gemm_tcgen05_pays(h, w_in, perm.numel(), True, False, act):
+                        a = kernels.moe_gemm_tcgen05(h, w_in, off, perm, ww, top, gated=True, activation=act)
+                        p = kernels.moe_gemm_tcgen05(a, w_dn, off, perm, ww, top, gated=False, scale_out=True)
+                    else:
+                        a = kernels.moe_gemm(h, w_in, off, perm, ww, top, gated=True, activation=act)
+                        p = kernels.moe_gemm(a, w_dn, off, perm, ww, top, gated=False, scale_out=True)
+                    kernels.moe_combine(p, top, identity=(ix, ww, h, E) if plain else None)
+                return call
+            row(f"experts without gates {name}", each(experts(True, wu, router, corr), inner=8), 2.0 * used * eff * width * esz + n * width * (esz + 4)
+                + (E + I) * width * 4.0, like=f"dirarax experts {name}", tensor=4.0 * real * eff * width)
+            del wu
+            router2 = torch.randn(E, width, device=dev) * 0.05
+            idx2, _ = kernels.moe_route(h, router2, top, "softmax", True)
+            used2 = int(torch.unique(idx2).numel())
+            wg = rotate(lambda: ((torch.randn(E, 2 * eff, width, device=dev) * 0.02).to(tdt), (torch.randn(E, width, eff, device=dev) * 0.02).to(tdt)),
+                        3 * E * eff * width * esz)
+            row(f"dirarax experts {name}", each(experts(False, wg, router2, None), inner=8), 3.0 * used2 * eff * width * esz + n * width * (esz + 4)
+                + E * width * 4.0, tensor=6.0 * n * top * eff * width)
+            del wg
+            # ---- the expert that every token runs: its up half ----
+            ws = rotate(lambda: (torch.randn(2 * eff, width, device=dev) * 0.02).to(tdt), 2 * eff * width * esz)
+
+            def shared(plain):
+                def call(i):
+                    w = ws[i % len(ws)]
+                    if plain:
+                        kernels.linear_relu2(h, w[:eff])
+                    elif kernels.skinny_fits(n, width, tdt):
+                        kernels.skinny_gemm(w[:eff], weight_up=w[eff:], x=h, epilogue="swiglu")
+                    else:
+                        o = torch.empty((n, eff), dtype=tdt, device=dev)
+                        if tdt == torch.bfloat16 and kernels.gemm_pays(n, eff, "swiglu"):
+                            kernels.gemm(h, w[:eff], weight_up=w[eff:], epilogue="swiglu", out=o)
+                        else:
+                            gu = kernels.linear(h, w, out_dtype=f32)
+                            kernels.silu_mul(o, gu[:, :eff], gu[:, eff:])
+                return call
+            row(f"common expert's up half {name}", each(shared(True)), eff * width * esz + n * (width + eff) * esz,
+                like=f"dirarax common expert's gate and up {name}", tensor=2.0 * n * eff * width)
+            row(f"dirarax common expert's gate and up {name}", each(shared(False)), 2.0 * eff * width * esz + n * (width + eff) * esz,
+                tensor=4.0 * n * eff * width)
+            del ws
+        return rows
+
     sizes = {}
     for name, (width, layers, heads, kv, hd, ff, E, top, eff, vocab) in DESIGN_SIZES.items():
+        if args.design == "rupenex":
+            window, keep = RUPENEX_EXTRA[name]
+            rup = rupenex_config(width, layers, heads, kv, hd, ff, E, top, eff, vocab, window, keep)
+            dira = dirarax_config(width, layers, heads, kv, hd, ff, E, top, eff, vocab)
+            llama = dict(TINYLLAMA, num_hidden_layers=layers, hidden_size=width, num_attention_heads=heads,
+                         num_key_value_heads=kv, head_dim=hd, intermediate_size=ff, vocab_size=vocab,
+                         max_position_embeddings=max(ctx, T))
+            m = rup["layers"][0]["mixer"]
+            rec = {"layers": layers, "recurrent_heads": f"{m['heads']} of 64 values x {m['state']}, {m['groups']} groups",
+                   "attention": f"{heads} heads of {hd} over {kv} kv heads, window {window} + {keep} first keys", "ff": ff,
+                   "experts": f"{top} of {E} x {eff} + {E // 2} identity, common {eff}"}
+            for key, cfg in (("rupenex", rup), ("dirarax", dira), ("llama", llama)):
+                print(f"[bench] {name}: {key}", file=sys.stderr, flush=True)
+                rec[key] = model_run(cfg, vocab)
+            print(f"[bench] {name}: kernels", file=sys.stderr, flush=True)
+            rec["kernels"] = rupenex_rows(width, heads, kv, hd, ff, E, top, eff, window, keep)
+            sizes[name] = rec
+            torch.cuda.empty_cache()
+            continue
         if args.design == "dirarax":
             dira = dirarax_config(width, layers, heads, kv, hd, ff, E, top, eff, vocab)
             soz = sozarax_config(width, layers, heads, kv, hd, ff, E, top, eff, vocab)
@@ -1618,7 +1865,7 @@ def design_comparison(args):
         sizes[name] = rec
         torch.cuda.empty_cache()
     sampler.stop()
-    beside = {"senulix": "a dense Sozarax and a Llama", "dirarax": "a Sozarax and a Llama"}.get(args.design, "a Llama")
+    beside = {"senulix": "a dense Sozarax and a Llama", "dirarax": "a Sozarax and a Llama", "rupenex": "a Dirarax and a Llama"}.get(args.design, "a Llama")
     print(json.dumps({"partial": f"{args.design.capitalize()} beside {beside} of equal size", "dtype": dtype, "prefill_tokens": T,
                       "decode_batch": B, "decode_context": ctx, "data": "synthetic, random weights",
                       "peaks": pk, "clocks": sampler.summary(t_begin, time.time()), "sizes": sizes}))

@@ -269,7 +269,7 @@ def random_weights(cfg, seed, std=0.12, qk_gain=2.0):
         elif name.endswith(".dt_bias"):
             t = rng.uniform(-4.0, 0.5, shape)
         elif name.endswith(".D"):
-            t = 0.5 + 0.5 * rng.standard_normal(shape)
+            t = rng.uniform(1.5, 3.0, shape)       # a head's value D x + S^T C does not cross zero as a whole
         elif name.endswith(".correction"):
             t = rng.uniform(-0.1, 0.1, shape)
         elif name.endswith(".conv"):
