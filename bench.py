@@ -1611,7 +1611,7 @@ def design_comparison(args):
 
             def ssd(i):
                 st, ring = states[i % len(states)]
-                o = kernels.ssd(projs[i % len(projs)], conv, cb, dtb, alog, dsk, st, ring, c, mh, G, N, mv)
+                o = kernels.ssd(projs[i % len(projs)], conv, cb, dtb, alog, dsk, st, ring, c, mh, G, N, mv, dtype=tdt)
                 kernels.part_norm(y, o, gain, G, 1e-6)
             row(f"mamba2 {name} (convolution, scan, gate and norm)", each(ssd), 8.0 * S * mh * N * mv + 4.0 * n * P + esz * n * inner,
                 like=f"gated linear attention {name}", core=4.0 * n * mh * N * mv)

@@ -36,50 +36,88 @@ KLLM_EXPORT_LAST_ERROR(moe)
 namespace {
 
 // ---- router ----------------------------------------------------------------------
-// one CTA of four warps per token: the warps share the columns of the router's rows, so that a step of
+// One CTA of eight warps per TOK tokens (four in a large step, whose CTAs then read the router's rows once for
+// all four): the warps share the columns of the router's rows, V neighbours per thread and load, so that a step of
 // few tokens still has many loads in flight (the router's rows come from HBM in every decode step: the
-// weights streamed between two steps push them out of L2); warp 0 then makes the choice.  E logits in
+// weights streamed between two steps push them out of L2); one warp per token then makes the choice.  E logits per token in
 // shared memory (E <= 1024).  A logit's sum has one order, fixed by the width.
-template <typename T>
-__global__ void __launch_bounds__(128)
+constexpr int kRouteThreads = 256;
+
+template <typename T, int TOK, int V>
+__global__ void __launch_bounds__(kRouteThreads)
 route_kernel(int* __restrict__ idx, float* __restrict__ wt, const T* __restrict__ h, const float* __restrict__ router,
              int n, int d, int E, int top, int softmax, int renorm, int groups, int keep, const float* __restrict__ corr,
-             float sum_eps) {
-    extern __shared__ float zsh[];            // [E], with a correction [E] scores, then [2 * groups] when groups limit the choice
-    __shared__ float part[4][8];
+             float sum_eps, int per_token) {
+    extern __shared__ float zall[];           // per token: [E], with a correction [E] scores, then [2 * groups] when groups limit the choice
+    constexpr int EB = TOK == 1 ? 8 : 4, WARPS = kRouteThreads / 32;
+    __shared__ float part[WARPS][TOK * EB];
     griddep_wait();
     griddep_launch();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int t = blockIdx.x;
-    float* z = zsh;
-    const T* hr = h + (int64_t)t * d;
-    // eight experts at a time: their loads are independent of one another, and the token's row is read
-    // once for all eight; every expert's sum still runs over its columns in the one order
-    for (int e0 = 0; e0 < E; e0 += 8) {
-        const float* wr[8];
-        float acc[8];
+    const int t0 = blockIdx.x * TOK;
+    const T* hr[TOK];
 #pragma unroll
-        for (int j = 0; j < 8; j++) {
+    for (int i = 0; i < TOK; i++) hr[i] = h + (int64_t)min(t0 + i, n - 1) * d;
+    // EB experts at a time: their loads are independent of one another; every expert's sum still runs over its
+    // columns in the one order
+    for (int e0 = 0; e0 < E; e0 += EB) {
+        const float* wr[EB];
+        float acc[TOK][EB];
+#pragma unroll
+        for (int j = 0; j < EB; j++) {
             wr[j] = router + (int64_t)min(e0 + j, E - 1) * d;
-            acc[j] = 0.f;
-        }
-#pragma unroll 4
-        for (int c = threadIdx.x; c < d; c += 128) {
-            const float hv = to_f32(hr[c]);
 #pragma unroll
-            for (int j = 0; j < 8; j++) acc[j] += hv * wr[j][c];
+            for (int i = 0; i < TOK; i++) acc[i][j] = 0.f;
+        }
+#pragma unroll 2
+        for (int c = threadIdx.x * V; c < d; c += kRouteThreads * V) {
+            float w[EB][V], hv[TOK][V];
+#pragma unroll
+            for (int j = 0; j < EB; j++) {
+                if constexpr (V == 4) {
+                    const float4 q = *reinterpret_cast<const float4*>(wr[j] + c);
+                    w[j][0] = q.x; w[j][1] = q.y; w[j][2] = q.z; w[j][3] = q.w;
+                } else {
+                    w[j][0] = wr[j][c];
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < TOK; i++) {
+                T raw[V];
+                if constexpr (V == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(raw) = *reinterpret_cast<const uint2*>(hr[i] + c);
+                else if constexpr (V == 4) *reinterpret_cast<float4*>(raw) = *reinterpret_cast<const float4*>(hr[i] + c);
+                else raw[0] = hr[i][c];
+#pragma unroll
+                for (int u = 0; u < V; u++) hv[i][u] = to_f32(raw[u]);
+            }
+#pragma unroll
+            for (int i = 0; i < TOK; i++)
+#pragma unroll
+                for (int j = 0; j < EB; j++)
+#pragma unroll
+                    for (int u = 0; u < V; u++) acc[i][j] += hv[i][u] * w[j][u];
         }
 #pragma unroll
-        for (int j = 0; j < 8; j++) {
-            const float a = warp_sum(acc[j]);
-            if (lane == 0) part[warp][j] = a;
-        }
+        for (int i = 0; i < TOK; i++)
+#pragma unroll
+            for (int j = 0; j < EB; j++) {
+                const float v = warp_sum(acc[i][j]);
+                if (lane == 0) part[warp][i * EB + j] = v;
+            }
         __syncthreads();
-        if (threadIdx.x < 8 && e0 + threadIdx.x < E)
-            z[e0 + threadIdx.x] = (part[0][threadIdx.x] + part[1][threadIdx.x]) + (part[2][threadIdx.x] + part[3][threadIdx.x]);
+        if (threadIdx.x < TOK * EB) {
+            const int i = threadIdx.x / EB, e = e0 + threadIdx.x % EB;
+            float v = 0.f;
+#pragma unroll
+            for (int q = 0; q < WARPS; q++) v += part[q][threadIdx.x];
+            if (e < E) zall[i * per_token + e] = v;
+        }
         __syncthreads();
     }
-    if (warp != 0) return;
+    const int t = t0 + warp;
+    if (warp >= TOK || t >= n) return;
+    float* zsh = zall + warp * per_token;
+    float* z = zsh;
     // the choice is made among the logits: both scores grow with them, and a sigmoid that has
     // reached 1.0f no longer tells two experts apart
     float zmax = 0.f, zsum = 1.f;
@@ -565,15 +603,26 @@ extern "C" int kllm_moe_route(int* idx, float* wt, const void* h, const float* r
     if (E % groups || keep < 1 || keep > groups || top > keep * (E / groups))
         KLLM_FAIL("moe route: %d of %d experts in %d groups of which %d are kept", top, E, groups, keep);
     cudaStream_t s = (cudaStream_t)stream;
-    const size_t smem = (size_t)((corr ? 2 : 1) * E + 2 * groups) * sizeof(float);
-    if (dtype == KLLM_F32)
-        kllm_launch((route_kernel<float>), dim3(n), dim3(128), smem, s, idx, wt, (const float*)h, router, n, d, E,
-                    top, softmax, renorm, groups, keep, corr, sum_eps);
-    else if (dtype == KLLM_BF16)
-        kllm_launch((route_kernel<bf16>), dim3(n), dim3(128), smem, s, idx, wt, (const bf16*)h, router, n, d, E,
-                    top, softmax, renorm, groups, keep, corr, sum_eps);
-    else
+    const int per_token = (corr ? 2 : 1) * E + 2 * groups;
+    const bool vec = d % 4 == 0 && !(((uintptr_t)h | (uintptr_t)router) & 15);
+    const bool many = n >= 4 * 148 && per_token * 4 * sizeof(float) <= 40 * 1024;
+#define KLLM_ROUTE(T, TOK, V)                                                                                                  \
+    kllm_launch((route_kernel<T, TOK, V>), dim3((n + TOK - 1) / TOK), dim3(kRouteThreads), (size_t)TOK * per_token * sizeof(float), s, \
+                idx, wt, (const T*)h, router, n, d, E, top, softmax, renorm, groups, keep, corr, sum_eps, per_token)
+#define KLLM_ROUTE_T(T)                        \
+    if (many && vec) KLLM_ROUTE(T, 4, 4);      \
+    else if (many) KLLM_ROUTE(T, 4, 1);        \
+    else if (vec) KLLM_ROUTE(T, 1, 4);         \
+    else KLLM_ROUTE(T, 1, 1)
+    if (dtype == KLLM_F32) {
+        KLLM_ROUTE_T(float);
+    } else if (dtype == KLLM_BF16) {
+        KLLM_ROUTE_T(bf16);
+    } else {
         KLLM_FAIL("moe route: unknown element type %d", dtype);
+    }
+#undef KLLM_ROUTE_T
+#undef KLLM_ROUTE
     KLLM_LAUNCH_STATUS();
 }
 

@@ -12,8 +12,8 @@
 //   caches [pages][k heads][page_size][dk] and [pages][v heads][page_size][dv] at position p.
 //
 // The number of value heads is independent of the number of key heads (several key heads may
-// attend over one value head).  The angle is formed in double precision from a double frequency,
-// once per token and pair, so that it is as exact as a table computed on the host would be; sums
+// attend over one value head).  The angle is formed in double precision from a double frequency and
+// reduced to a turn there, once per token and pair, so that it is as exact at any position as at the first; sums
 // of squares, scales and the rotation are float32.  One CTA per token, one warp per head; a
 // head's sums depend on its size alone.
 //
@@ -44,10 +44,12 @@ headnorm_rope_append_kernel(T* __restrict__ q_out, const float* __restrict__ qkv
     const int t = blockIdx.x, p = positions[t], half = rot >> 1;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
-        double s, c;
-        sincos((double)p * freq[i], &s, &c);
-        cs[i] = (float)c * amplitude;
-        cs[half + i] = (float)s * amplitude;
+        // the angle and its rest from whole turns in double precision, cos and sin of the rest in float32
+        const double angle = (double)p * freq[i];
+        float s, c;
+        sincosf((float)(angle - rint(angle * 0.15915494309189533577) * 6.28318530717958647693), &s, &c);
+        cs[i] = c * amplitude;
+        cs[half + i] = s * amplitude;
     }
     __syncthreads();
     int64_t page = -1;

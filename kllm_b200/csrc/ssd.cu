@@ -8,7 +8,7 @@
 //     S_t = a_t S_(t-1) + dt_t B_t x_t^T      y_t = (S_t^T C_t + D x_t) * silu(z_t)
 //
 // and y is RMS-normed in equal parts of the row, times a gain.  Everything is float32; the normed row alone is stored in the
-// model's type.
+// model's type.  (In bfloat16 models portions round x, B and C to it behind silu, where their sizes suit the tensor cores.)
 //
 // The convolution's inputs of the last `taps` positions live in a ring [taps][channels] per request, position p in entry
 // p mod taps: a step writes the entry of its own position and reads the others, so CTAs that share channels do not
@@ -25,12 +25,20 @@
 //     S_out = exp(c_last) S_in + sum over j of exp(c_last - c_j) dt_j B_j x_j^T
 //
 //   conv_kernel    convolution and silu of every channel; dt and the c_i of every head
+//   ring_kernel    the ring takes the portions' last inputs
 //   pairs_kernel   C_i . B_j per (chunk, group), which the group's heads share
 //   outer_kernel   every chunk's own addition to the state
 //   carry_kernel   the states at the chunks' starts, element by element over a request's chunks in order;
 //                  moves the slot on
 //   apply_kernel   y of every chunk, with D and the gate
 //   part_norm_kernel
+// In bfloat16 models with N and dv in steps of 16 the products run on the tensor cores (mma.sync m16n8k16, chunks of kT
+// rows): x, B and C are bfloat16, and what is float32 enters as two bfloat16 terms, high and low (16 bits of mantissa):
+//
+//   outer_tc_kernel   B^T (exp(c_last - c_j) dt_j x_j), the weighted rows split
+//   carry_kernel      leaves the states at the chunks' starts split, float32 in the slot and in every sum
+//   apply_tc_kernel   C S_in with the state split, rows times exp(c_i); then, key tile by key tile, C B^T in registers, times the
+//                     float32 decays and steps, split, times x
 // The c_i may reach tens of thousands while their differences are small: they are summed in double precision and
 // kept as two floats, whose differences are formed pairwise.  Where a prompt is cut changes the order of float32 sums and
 // nothing else.
@@ -41,6 +49,7 @@ KLLM_EXPORT_LAST_ERROR(ssd)
 namespace {
 
 constexpr int kC = 64;          // rows of a chunk
+constexpr int kT = 128;         // ... of the tensor-core form
 constexpr int kThreads = 256;
 
 struct SsdArgs {
@@ -58,11 +67,14 @@ struct SsdArgs {
     int ch_pad;                             // channels rounded up to a multiple of 4: row length of ring and xc
     float* y;                               // [n][inner]: gated, before the norm
     // work of the form for portions
-    float* xc;                              // [n][ch_pad]: x, B, C behind the convolution
-    float* dt;                              // [chunks][H][kC]
-    float2* cum;                            // [chunks][H][kC]
+    void* xc;                               // [n][xc_pad] float32, or bfloat16 in the tensor-core form: x, B, C behind the convolution
+    int xc_pad;
+    float* dt;                              // [chunks][H][rows of a chunk]
+    float2* cum;                            // [chunks][H][rows of a chunk]
     float* pairs;                           // [chunks][G][kC][kC]
     float* s_in;                            // [chunks][H][N][dv]
+    bf16* s_split;                          // tensor-core form: [2][chunks][H][N][dv], high and low terms
+    int64_t split_plane;                    // elements of one of the two
     bool vec;                               // sizes and addresses allow 16-byte accesses
 };
 
@@ -97,7 +109,7 @@ template <int V> __device__ __forceinline__ void store_vec(float* p, const Vec<V
 // Shared memory: partial sums [kThreads * V], x [sl], B [N], C [N].  Started early, the kernel reads state and ring before
 // the kernel in front of it has ended: that kernel must write neither.
 template <int V>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, 4)
 step_kernel(const SsdArgs a, int sl) {
     extern __shared__ __align__(16) float sm[];
     constexpr int NB = V == 4 ? 8 : 16;                     // state channels in flight per thread
@@ -123,31 +135,60 @@ step_kernel(const SsdArgs a, int sl) {
         return i < sl ? head * dv + slice * sl + i : i < sl + N ? a.inner + group * N + (i - sl)
                                                                : a.inner + a.groups * N + group * N + (i - sl - N);
     };
-    // what earlier rows put into the first channel's sum, before the projections are waited for
+    // what earlier rows put into a channel's sum: of the first kEarly channels of a thread before the projections are waited
+    // for, all loads of four taps at once
     auto before = [&](int c) {
         float v = a.conv_b[c];
         const float* w = a.conv_w + (int64_t)c * a.taps;
-        for (int i = 0; i < a.taps - 1; i++) {
-            const int q = p - (a.taps - 1) + i;
-            if (q >= 0) v = fmaf(w[i], ring[(int64_t)(q % a.taps) * a.ch_pad + c], v);
+        for (int i0 = 0; i0 < a.taps - 1; i0 += 4) {
+            float wv[4], rv[4];
+#pragma unroll
+            for (int u = 0; u < 4; u++) {
+                const int i = i0 + u, q = p - (a.taps - 1) + i;
+                const bool in = i < a.taps - 1 && q >= 0;
+                wv[u] = in ? w[i] : 0.f;
+                rv[u] = in ? ring[(int64_t)(q % a.taps) * a.ch_pad + c] : 0.f;
+            }
+#pragma unroll
+            for (int u = 0; u < 4; u++) v = fmaf(wv[u], rv[u], v);
         }
         return v;
     };
-    const float first = tid < mine ? before(channel(tid)) : 0.f;
+    constexpr int kEarly = 2;
+    float sum[kEarly], wlast[kEarly];
+    int ch[kEarly];
+#pragma unroll
+    for (int u = 0; u < kEarly; u++) {
+        const int i = tid + u * kThreads;
+        ch[u] = i < mine ? channel(i) : -1;
+        sum[u] = ch[u] >= 0 ? before(ch[u]) : 0.f;
+        wlast[u] = ch[u] >= 0 ? a.conv_w[(int64_t)ch[u] * a.taps + a.taps - 1] : 0.f;
+    }
     const float rate = expf(a.a_log[head]), dbias = a.dt_bias[head], dskip = a.d[head];
     griddep_wait();
     griddep_launch();
     const float* row = a.proj + (int64_t)t * a.stride;
-    const float* u = row + a.inner;
-    for (int i = tid; i < mine; i += kThreads) {
-        const int c = channel(i);
-        const float in = u[c];
-        const float v = silu_f(fmaf(a.conv_w[(int64_t)c * a.taps + a.taps - 1], in, i == tid ? first : before(c)));
-        xs[i] = v;                                          // x slice, B and C lie one behind the other
+    const float* u_row = row + a.inner;
+    float in[kEarly];
+#pragma unroll
+    for (int u = 0; u < kEarly; u++) in[u] = ch[u] >= 0 ? u_row[ch[u]] : 0.f;
+    const float dt_in = row[a.inner + a.channels + head];
+    const float* z = row + head * dv + slice * sl;
+    const float z_first = tid < sl ? z[tid] : 0.f;
+    auto keep = [&](int i, int c, float x, float v) {
+        xs[i] = silu_f(v);                                  // x slice, B and C lie one behind the other
         // one CTA moves each channel's ring on: x its own, B and C the group's first head
-        if (i < sl || (slice == 0 && head == group * per)) ring[(int64_t)(p % a.taps) * a.ch_pad + c] = in;
+        if (i < sl || (slice == 0 && head == group * per)) ring[(int64_t)(p % a.taps) * a.ch_pad + c] = x;
+    };
+#pragma unroll
+    for (int u = 0; u < kEarly; u++)
+        if (ch[u] >= 0) keep(tid + u * kThreads, ch[u], in[u], fmaf(wlast[u], in[u], sum[u]));
+    for (int i = tid + kEarly * kThreads; i < mine; i += kThreads) {
+        const int c = channel(i);
+        const float x = u_row[c];
+        keep(i, c, x, fmaf(a.conv_w[(int64_t)c * a.taps + a.taps - 1], x, before(c)));
     }
-    const float dt = softplus_f(row[a.inner + a.channels + head] + dbias);
+    const float dt = softplus_f(dt_in + dbias);
     const float al = expf(-rate * dt);
     __syncthreads();
     if (on) {
@@ -183,25 +224,25 @@ step_kernel(const SsdArgs a, int sl) {
         store_vec<V>(ps + nl * sl + cg * V, acc);
     }
     __syncthreads();
-    const float* z = row + head * dv + slice * sl;
     float* yr = a.y + (int64_t)t * a.inner + head * dv + slice * sl;
     for (int c = tid; c < sl; c += kThreads) {
         float o = 0.f;
         for (int l = 0; l < lanes; l++) o += ps[l * sl + c];
-        yr[c] = fmaf(dskip, xs[c], o) * silu_f(z[c]);
+        yr[c] = fmaf(dskip, xs[c], o) * silu_f(c == tid ? z_first : z[c]);
     }
 }
 
 // ---- portions ------------------------------------------------------------------------------------------------
 
-// The request and first row of the step's chunk number `chunk`; false beyond the last chunk.
+// The request and first row of the step's chunk number `chunk` of KC rows; false beyond the last chunk.
+template <int KC>
 __device__ __forceinline__ bool find_chunk(const SsdArgs& a, int chunk, int& req, int& row0, int& rows, int& index) {
     for (req = 0; req < a.n_requests; req++) {
-        const int lo = a.q_start[req], len = a.q_start[req + 1] - lo, chunks = (len + kC - 1) / kC;
+        const int lo = a.q_start[req], len = a.q_start[req + 1] - lo, chunks = (len + KC - 1) / KC;
         if (chunk < chunks) {
             index = chunk;
-            row0 = lo + chunk * kC;
-            rows = min(kC, len - chunk * kC);
+            row0 = lo + chunk * KC;
+            rows = min(KC, len - chunk * KC);
             return true;
         }
         chunk -= chunks;
@@ -217,45 +258,71 @@ __device__ __forceinline__ void cp_async16(float* smem, const float* gmem, bool 
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
 
-// grid (chunk bound, blocks of kThreads channels, then blocks of kThreads heads).  A thread owns a channel of the
-// chunk's rows, or a head's decays.  TAPS > 0: that many taps, the inputs in registers; 0: any number.
-template <int TAPS>
+// grid (chunk bound * KC / kRun, blocks of kThreads channels, then blocks of 8 heads).  A thread owns a channel of kRun of the
+// chunk's rows; of the further blocks those of a chunk's first run form its decays, one warp per head.  TAPS > 0: that many
+// taps, the inputs in registers; 0: any number.
+constexpr int kRun = 32;
+
+template <int TAPS, typename T, int KC>
 __global__ void __launch_bounds__(kThreads)
 conv_kernel(const SsdArgs a) {
     griddep_wait();
     griddep_launch();
     int req, row0, rows, index;
-    if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
+    const int chunk = blockIdx.x / (KC / kRun), run0 = (blockIdx.x % (KC / kRun)) * kRun;
+    if (!find_chunk<KC>(a, chunk, req, row0, rows, index)) return;
     const int ch_blocks = (a.channels + kThreads - 1) / kThreads;
     if ((int)blockIdx.y >= ch_blocks) {
-        const int h = (blockIdx.y - ch_blocks) * kThreads + threadIdx.x;
-        if (h >= a.heads) return;
+        constexpr int R = KC / 32;                          // rows of a lane, one behind the other
+        const int h = (blockIdx.y - ch_blocks) * (kThreads / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+        if (run0 > 0 || h >= a.heads) return;
         const float rate = expf(a.a_log[h]), bias = a.dt_bias[h];
         const float* src = a.proj + (int64_t)row0 * a.stride + a.inner + a.channels + h;
-        const int64_t at = ((int64_t)blockIdx.x * a.heads + h) * kC;
-        double sum = 0.0;
-#pragma unroll 8
-        for (int r = 0; r < rows; r++) {
-            const float dt = softplus_f(src[(int64_t)r * a.stride] + bias);
-            sum -= (double)(rate * dt);
-            const float hi = (float)sum;
-            a.dt[at + r] = dt;
-            a.cum[at + r] = make_float2(hi, (float)(sum - (double)hi));
+        float dt[R];
+#pragma unroll
+        for (int i = 0; i < R; i++) {
+            const int r = lane * R + i;
+            dt[i] = r < rows ? src[(int64_t)r * a.stride] : 0.f;
+        }
+        double part[R], mine = 0.0;
+#pragma unroll
+        for (int i = 0; i < R; i++) {
+            dt[i] = softplus_f(dt[i] + bias);
+            mine -= (double)(rate * dt[i]);
+            part[i] = mine;
+        }
+        double sum = mine;                                  // over the lanes up to and including this one
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const double other = __shfl_up_sync(0xffffffffu, sum, o);
+            if (lane >= o) sum += other;
+        }
+        const double base = sum - mine;
+        const int64_t at = ((int64_t)chunk * a.heads + h) * KC + lane * R;
+#pragma unroll
+        for (int i = 0; i < R; i++) {
+            if (lane * R + i < rows) {
+                const double v = base + part[i];
+                const float hi = (float)v;
+                a.dt[at + i] = dt[i];
+                a.cum[at + i] = make_float2(hi, (float)(v - (double)hi));
+            }
         }
         return;
     }
-    const int c = blockIdx.y * kThreads + threadIdx.x;
-    if (c >= a.channels) return;
+    const int c = blockIdx.y * kThreads + threadIdx.x, n = min(kRun, rows - run0);
+    if (c >= a.channels || n <= 0) return;
     const int taps = TAPS > 0 ? TAPS : a.taps;
-    const float* src = a.proj + (int64_t)row0 * a.stride + a.inner + c;
-    float* dst = a.xc + (int64_t)row0 * a.ch_pad + c;
+    const int first = index * KC + run0;                    // the run's first row, counted from the portion's start
+    const float* src = a.proj + (int64_t)(row0 + run0) * a.stride + a.inner + c;
+    T* dst = reinterpret_cast<T*>(a.xc) + (int64_t)(row0 + run0) * a.xc_pad + c;
     float* ring = a.ring + (int64_t)a.state_slots[req] * a.ring_stride + c;
-    const int p0 = a.start_pos[req] + index * kC;           // position of the chunk's first row
+    const int p0 = a.start_pos[req] + first;                // position of the run's first row
     const float* w = a.conv_w + (int64_t)c * taps;
     const float bias = a.conv_b[c];
-    // input of row r, also in front of the chunk: an earlier row of the portion, or the ring
+    // input of row r, also in front of the run: an earlier row of the portion, or the ring
     auto input = [&](int r) {
-        if (r >= 0 || index > 0) return src[(int64_t)r * a.stride];        // a chunk in front has kC >= taps - 1 rows
+        if (first + r >= 0) return src[(int64_t)r * a.stride];
         const int q = p0 + r;
         return q >= 0 ? ring[(int64_t)(q % taps) * a.ch_pad] : 0.f;
     };
@@ -266,37 +333,44 @@ conv_kernel(const SsdArgs a) {
             k[i] = w[i];
             u[i] = i < TAPS - 1 ? input(i - (TAPS - 1)) : 0.f;
         }
-        constexpr int AHEAD = 8;
-        for (int r0 = 0; r0 < rows; r0 += AHEAD) {
+        constexpr int AHEAD = 16;
+        for (int r0 = 0; r0 < n; r0 += AHEAD) {
             float in[AHEAD];
 #pragma unroll
-            for (int j = 0; j < AHEAD; j++) in[j] = r0 + j < rows ? src[(int64_t)(r0 + j) * a.stride] : 0.f;
+            for (int j = 0; j < AHEAD; j++) in[j] = r0 + j < n ? src[(int64_t)(r0 + j) * a.stride] : 0.f;
 #pragma unroll
             for (int j = 0; j < AHEAD; j++) {
-                if (r0 + j < rows) {
+                if (r0 + j < n) {
                     u[TAPS - 1] = in[j];
                     float v = bias;
 #pragma unroll
                     for (int i = 0; i < TAPS; i++) v = fmaf(k[i], u[i], v);
-                    dst[(int64_t)(r0 + j) * a.ch_pad] = silu_f(v);
+                    dst[(int64_t)(r0 + j) * a.xc_pad] = from_f32<T>(silu_f(v));
 #pragma unroll
                     for (int i = 0; i < TAPS - 1; i++) u[i] = u[i + 1];
                 }
             }
         }
     } else {
-        for (int r = 0; r < rows; r++) {
+        for (int r = 0; r < n; r++) {
             float v = bias;
             for (int i = 0; i < taps; i++) v = fmaf(w[i], input(r - (taps - 1) + i), v);
-            dst[(int64_t)r * a.ch_pad] = silu_f(v);
+            dst[(int64_t)r * a.xc_pad] = from_f32<T>(silu_f(v));
         }
     }
-    if (index == 0) {
-        // the thread that has read the ring's old entries of this channel moves it on
-        const int len = a.q_start[req + 1] - a.q_start[req];
-        for (int r = max(0, len - taps); r < len; r++)
-            ring[(int64_t)((a.start_pos[req] + r) % taps) * a.ch_pad] = src[(int64_t)r * a.stride];
-    }
+}
+
+// grid (blocks of kThreads channels, requests), behind conv_kernel: the ring takes the portion's last inputs.
+__global__ void __launch_bounds__(kThreads)
+ring_kernel(const SsdArgs a) {
+    griddep_wait();
+    griddep_launch();
+    const int c = blockIdx.x * kThreads + threadIdx.x, req = blockIdx.y;
+    if (c >= a.channels) return;
+    const int lo = a.q_start[req], len = a.q_start[req + 1] - lo;
+    float* ring = a.ring + (int64_t)a.state_slots[req] * a.ring_stride + c;
+    for (int r = max(0, len - a.taps); r < len; r++)
+        ring[(int64_t)((a.start_pos[req] + r) % a.taps) * a.ch_pad] = a.proj[(int64_t)(lo + r) * a.stride + a.inner + c];
 }
 
 // grid (chunk bound, groups): pairs[i][j] = C_i . B_j.  Thread (ty, tx): rows 4 ty .., columns 4 tx .. .
@@ -310,8 +384,8 @@ pairs_kernel(const SsdArgs a) {
     griddep_launch();
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4, group = blockIdx.y, N = a.N;
     int req, row0, rows, index;
-    if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
-    const float* B = a.xc + (int64_t)row0 * a.ch_pad + a.inner + group * N;
+    if (!find_chunk<kC>(a, blockIdx.x, req, row0, rows, index)) return;
+    const float* B = reinterpret_cast<const float*>(a.xc) + (int64_t)row0 * a.xc_pad + a.inner + group * N;
     const float* C = B + a.groups * N;
     float acc[4][4];
 #pragma unroll
@@ -322,8 +396,8 @@ pairs_kernel(const SsdArgs a) {
         for (int i = tid; i < kC * kKP; i += kThreads) {
             const int r = i / kKP, k = i - r * kKP;
             const bool in = r < rows && k0 + k < N;
-            Cs[k][r] = in ? C[(int64_t)r * a.ch_pad + k0 + k] : 0.f;
-            Bs[k][r] = in ? B[(int64_t)r * a.ch_pad + k0 + k] : 0.f;
+            Cs[k][r] = in ? C[(int64_t)r * a.xc_pad + k0 + k] : 0.f;
+            Bs[k][r] = in ? B[(int64_t)r * a.xc_pad + k0 + k] : 0.f;
         }
         __syncthreads();
         if (tx <= ty) {                                      // blocks of four that hold a pair j <= i
@@ -361,30 +435,30 @@ outer_kernel(const SsdArgs a, int e_tiles) {
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
     const int head = blockIdx.y, d0 = blockIdx.z / e_tiles * TM, e0 = blockIdx.z % e_tiles * TN, N = a.N, dv = a.dv;
     int req, row0, rows, index;
-    if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
+    if (!find_chunk<kC>(a, blockIdx.x, req, row0, rows, index)) return;
     float* ks = sm;
     float* vs = ks + kC * TM;
     float* ws = vs + kC * TN;
-    const float* kg = a.xc + (int64_t)row0 * a.ch_pad + a.inner + (head / (a.heads / a.groups)) * N + d0;
-    const float* vg = a.xc + (int64_t)row0 * a.ch_pad + head * dv + e0;
+    const float* kg = reinterpret_cast<const float*>(a.xc) + (int64_t)row0 * a.xc_pad + a.inner + (head / (a.heads / a.groups)) * N + d0;
+    const float* vg = reinterpret_cast<const float*>(a.xc) + (int64_t)row0 * a.xc_pad + head * dv + e0;
     if (a.vec) {
         for (int i = tid; i < rows * (TM / 4); i += kThreads) {
             const int r = i / (TM / 4), d = (i - r * (TM / 4)) * 4;
-            cp_async16(ks + r * TM + d, kg + (d0 + d < N ? (int64_t)r * a.ch_pad + d : 0), d0 + d < N);
+            cp_async16(ks + r * TM + d, kg + (d0 + d < N ? (int64_t)r * a.xc_pad + d : 0), d0 + d < N);
         }
         for (int i = tid; i < rows * (TN / 4); i += kThreads) {
             const int r = i / (TN / 4), c = (i - r * (TN / 4)) * 4;
-            cp_async16(vs + r * TN + c, vg + (e0 + c < dv ? (int64_t)r * a.ch_pad + c : 0), e0 + c < dv);
+            cp_async16(vs + r * TN + c, vg + (e0 + c < dv ? (int64_t)r * a.xc_pad + c : 0), e0 + c < dv);
         }
         cp_async_commit();
     } else {
         for (int i = tid; i < rows * TM; i += kThreads) {
             const int r = i / TM, d = i - r * TM;
-            ks[i] = d0 + d < N ? kg[(int64_t)r * a.ch_pad + d] : 0.f;
+            ks[i] = d0 + d < N ? kg[(int64_t)r * a.xc_pad + d] : 0.f;
         }
         for (int i = tid; i < rows * TN; i += kThreads) {
             const int r = i / TN, c = i - r * TN;
-            vs[i] = e0 + c < dv ? vg[(int64_t)r * a.ch_pad + c] : 0.f;
+            vs[i] = e0 + c < dv ? vg[(int64_t)r * a.xc_pad + c] : 0.f;
         }
     }
     if (tid < rows) {
@@ -444,8 +518,8 @@ outer_kernel(const SsdArgs a, int e_tiles) {
 }
 
 // grid (pieces of kThreads * V state elements, heads, requests): s_in turns from the chunks' own states into the
-// states at their starts.
-template <int V>
+// states at their starts; SPLIT: those go to s_split.
+template <int V, int KC, bool SPLIT>
 __global__ void __launch_bounds__(kThreads)
 carry_kernel(const SsdArgs a) {
     griddep_wait();
@@ -454,12 +528,12 @@ carry_kernel(const SsdArgs a) {
     const int64_t elems = (int64_t)a.N * a.dv, i = ((int64_t)blockIdx.x * kThreads + threadIdx.x) * V;
     if (i >= elems) return;
     int chunk = 0;
-    for (int r = 0; r < req; r++) chunk += (a.q_start[r + 1] - a.q_start[r] + kC - 1) / kC;
-    const int len = a.q_start[req + 1] - a.q_start[req], chunks = (len + kC - 1) / kC;
+    for (int r = 0; r < req; r++) chunk += (a.q_start[r + 1] - a.q_start[r] + KC - 1) / KC;
+    const int len = a.q_start[req + 1] - a.q_start[req], chunks = (len + KC - 1) / KC;
     float* slot = a.state + (int64_t)a.state_slots[req] * a.state_stride + head * elems + i;
     float* w = a.s_in + ((int64_t)chunk * a.heads + head) * elems + i;
-    const float2* cum = a.cum + ((int64_t)chunk * a.heads + head) * kC;
-    const int64_t step = a.heads * elems, cum_step = (int64_t)a.heads * kC;
+    const float2* cum = a.cum + ((int64_t)chunk * a.heads + head) * KC;
+    const int64_t step = a.heads * elems, cum_step = (int64_t)a.heads * KC;
     Vec<V> s = load_vec<V>(slot);
     constexpr int AHEAD = 8;
     for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
@@ -469,13 +543,26 @@ carry_kernel(const SsdArgs a) {
         for (int u = 0; u < AHEAD; u++)
             if (c0 + u < chunks) {
                 loc[u] = load_vec<V>(w + (c0 + u) * step);
-                const float2 last = cum[(c0 + u) * cum_step + min(kC, len - (c0 + u) * kC) - 1];
+                const float2 last = cum[(c0 + u) * cum_step + min(KC, len - (c0 + u) * KC) - 1];
                 d[u] = expf(last.x + last.y);
             }
 #pragma unroll
         for (int u = 0; u < AHEAD; u++)
             if (c0 + u < chunks) {
-                store_vec<V>(w + (c0 + u) * step, s);
+                if constexpr (SPLIT) {
+                    bf16 hi[V], lo[V];
+#pragma unroll
+                    for (int j = 0; j < V; j++) {
+                        hi[j] = __float2bfloat16_rn(s.x[j]);
+                        lo[j] = __float2bfloat16_rn(s.x[j] - __bfloat162float(hi[j]));
+                    }
+                    bf16* dst = a.s_split + (w - a.s_in) + (c0 + u) * step;
+                    static_assert(V == 4, "eight bytes at a time");
+                    *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(hi);
+                    *reinterpret_cast<uint2*>(dst + a.split_plane) = *reinterpret_cast<const uint2*>(lo);
+                } else {
+                    store_vec<V>(w + (c0 + u) * step, s);
+                }
 #pragma unroll
                 for (int j = 0; j < V; j++) s.x[j] = fmaf(d[u], s.x[j], loc[u].x[j]);
             }
@@ -499,7 +586,7 @@ apply_kernel(const SsdArgs a) {
     const int head = blockIdx.y, e0 = blockIdx.z * CW, N = a.N, dv = a.dv, group = head / (a.heads / a.groups);
     const int ne = min(CW, dv - e0);
     int req, row0, rows, index;
-    if (!find_chunk(a, blockIdx.x, req, row0, rows, index)) return;
+    if (!find_chunk<kC>(a, blockIdx.x, req, row0, rows, index)) return;
     float2* cum = reinterpret_cast<float2*>(sm + 2 * STAGE);
     float* dts = reinterpret_cast<float*>(cum + kC);
     if (tid < kC) {
@@ -516,16 +603,16 @@ apply_kernel(const SsdArgs a) {
     const int nb_s = from_zero ? 0 : (N + kKB - 1) / kKB, nb = nb_s + (rows + kKB - 1) / kKB;
     const float* S = a.s_in + ((int64_t)blockIdx.x * a.heads + head) * N * dv + e0;
     const float* W = a.pairs + ((int64_t)blockIdx.x * a.groups + group) * kC * kC;
-    const float* xg = a.xc + (int64_t)row0 * a.ch_pad + head * dv + e0;
-    const float* Cg = a.xc + (int64_t)row0 * a.ch_pad + a.inner + (a.groups + group) * N;
+    const float* xg = reinterpret_cast<const float*>(a.xc) + (int64_t)row0 * a.xc_pad + head * dv + e0;
+    const float* Cg = reinterpret_cast<const float*>(a.xc) + (int64_t)row0 * a.xc_pad + a.inner + (a.groups + group) * N;
     auto load = [&](int b) {                // inner elements k0 .. k0 + kKB - 1 of the state's part, then of the chunk's own
         float* left = sm + (b & 1) * STAGE;
         float* right = left + kC * QP;
         const bool state = b < nb_s;
         const int k0 = (state ? b : b - nb_s) * kKB, nk = min(kKB, (state ? N : rows) - k0);
         const float* lg = state ? Cg + k0 : W + k0;
-        const float* rg_ = state ? S + (int64_t)k0 * dv : xg + (int64_t)k0 * a.ch_pad;
-        const int64_t ls = state ? a.ch_pad : kC, rs = state ? dv : a.ch_pad;
+        const float* rg_ = state ? S + (int64_t)k0 * dv : xg + (int64_t)k0 * a.xc_pad;
+        const int64_t ls = state ? a.xc_pad : kC, rs = state ? dv : a.xc_pad;
         if (a.vec) {
             for (int i = tid; i < kC * (kKB / 4); i += kThreads) {
                 const int r = i / (kKB / 4), k = (i - r * (kKB / 4)) * 4;
@@ -600,7 +687,7 @@ apply_kernel(const SsdArgs a) {
     for (int r = 0; r < 4; r++) {
         const int row = rg * 4 + r;
         if (row >= rows) continue;
-        const float* xr = xg + (int64_t)row * a.ch_pad;
+        const float* xr = xg + (int64_t)row * a.xc_pad;
         const float* zr = a.proj + (int64_t)(row0 + row) * a.stride + head * dv + e0;
         float* yr = a.y + (int64_t)(row0 + row) * a.inner + head * dv + e0;
 #pragma unroll
@@ -621,38 +708,304 @@ apply_kernel(const SsdArgs a) {
     }
 }
 
-// out[r][part] = y[r][part] / rms(y[r][part]) * gain: one CTA per (row, part) of w values; VEC: w a multiple of 4 up to
-// 4 * kVec * blockDim.x, 16-byte rows, the values in registers between the sum and the scaling.
+// ---- portions in bfloat16 on the tensor cores -------------------------------------------------------------------
+
+__device__ __forceinline__ void cp16(bf16* smem, const bf16* gmem, bool valid) {
+    cp_async16(reinterpret_cast<float*>(smem), reinterpret_cast<const float*>(gmem), valid);
+}
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const bf16* p) {
+    const unsigned a = (unsigned)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void ldsm4_trans(uint32_t (&r)[4], const bf16* p) {
+    const unsigned a = (unsigned)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// two values as a pair of bfloat16, and what that rounding left as another
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    const __nv_bfloat162 l = __floats2bfloat162_rn(a - __low2float(h), b - __high2float(h));
+    hi = *reinterpret_cast<const uint32_t*>(&h);
+    lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+
+constexpr int kDB = 64;                     // value channels of a CTA
+constexpr int kXP = kDB + 8;                // padded row of such a block, in elements
+
+// acc[2 p], acc[2 p + 1] += A (16 rows, 16 inner) times columns 16 p .. of rows k0 .. k0 + 15 of a block at row length kXP
+__device__ __forceinline__ void rows_times_block(float (&acc)[8][4], const uint32_t (&a)[4], const bf16* block, int k0, int lane) {
+    const int mi = lane >> 3;
+    const bf16* base = block + (k0 + (mi & 1) * 8 + (lane & 7)) * kXP + (mi >> 1) * 8;
+#pragma unroll
+    for (int p = 0; p < kDB / 16; p++) {
+        uint32_t b[4];
+        ldsm4_trans(b, base + p * 16);
+        mma16816(acc[2 * p], a, b[0], b[1]);
+        mma16816(acc[2 * p + 1], a, b[2], b[3]);
+    }
+}
+
+// grid (chunk bound, heads, blocks of kDB value channels): s_in = sum over the chunk's rows of exp(c_last - c_j) dt_j B_j x_j^T.
+// Warp w: state channels 16 w .., 16 (w + 8) .., ...  Shared memory: B [kT][N + 8], the weighted rows [kT][kXP] high and low, weights [kT].
+__global__ void __launch_bounds__(kThreads)
+outer_tc_kernel(const SsdArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    griddep_wait();
+    griddep_launch();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tq = lane & 3, mi = lane >> 3;
+    const int head = blockIdx.y, e0 = blockIdx.z * kDB, N = a.N, dv = a.dv, NP = N + 8, ne = min(kDB, dv - e0);
+    int req, row0, rows, index;
+    if (!find_chunk<kT>(a, blockIdx.x, req, row0, rows, index)) return;
+    bf16* Bs = reinterpret_cast<bf16*>(sm);
+    bf16* xh = Bs + kT * NP;
+    bf16* xl = xh + kT * kXP;
+    float* ws = reinterpret_cast<float*>(xl + kT * kXP);
+    const bf16* xg = reinterpret_cast<const bf16*>(a.xc) + (int64_t)row0 * a.xc_pad;
+    const bf16* bg = xg + a.inner + (head / (a.heads / a.groups)) * N;
+    const int steps = (rows + 15) / 16, per = N / 8;
+    for (int i = tid; i < steps * 16 * per; i += kThreads) {
+        const int r = i / per, c = (i - r * per) * 8;
+        cp16(Bs + r * NP + c, bg + (r < rows ? (int64_t)r * a.xc_pad + c : 0), r < rows);
+    }
+    cp_async_commit();
+    if (tid < kT) {
+        const int64_t at = ((int64_t)blockIdx.x * a.heads + head) * kT;
+        ws[tid] = tid < rows ? exp_diff(a.cum[at + rows - 1], a.cum[at + tid]) * a.dt[at + tid] : 0.f;
+    }
+    __syncthreads();
+    for (int i = tid; i < steps * 16 * (kDB / 8); i += kThreads) {
+        const int r = i / (kDB / 8), c = (i - r * (kDB / 8)) * 8;
+        uint4 h = make_uint4(0, 0, 0, 0), l = h;
+        if (r < rows && c < ne) {
+            const uint4 v = *reinterpret_cast<const uint4*>(xg + (int64_t)r * a.xc_pad + head * dv + e0 + c);
+            const float w = ws[r];
+            auto part = [&](uint32_t in, uint32_t& hi, uint32_t& lo) {
+                const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&in));
+                split2(f.x * w, f.y * w, hi, lo);
+            };
+            part(v.x, h.x, l.x); part(v.y, h.y, l.y); part(v.z, h.z, l.z); part(v.w, h.w, l.w);
+        }
+        *reinterpret_cast<uint4*>(xh + r * kXP + c) = h;
+        *reinterpret_cast<uint4*>(xl + r * kXP + c) = l;
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    float* S = a.s_in + ((int64_t)blockIdx.x * a.heads + head) * N * dv + e0;
+    for (int m0 = warp * 16; m0 < N; m0 += 16 * (kThreads / 32)) {
+        float acc[8][4];
+#pragma unroll
+        for (int i = 0; i < 8; i++)
+#pragma unroll
+            for (int j = 0; j < 4; j++) acc[i][j] = 0.f;
+        for (int k = 0; k < steps; k++) {
+            uint32_t af[4];
+            ldsm4_trans(af, Bs + (k * 16 + (mi >> 1) * 8 + (lane & 7)) * NP + m0 + (mi & 1) * 8);
+            rows_times_block(acc, af, xh, k * 16, lane);
+            rows_times_block(acc, af, xl, k * 16, lane);
+        }
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            const int c = i * 8 + 2 * tq;
+            if (c >= ne) continue;
+            *reinterpret_cast<float2*>(S + (int64_t)(m0 + gid) * dv + c) = make_float2(acc[i][0], acc[i][1]);
+            *reinterpret_cast<float2*>(S + (int64_t)(m0 + gid + 8) * dv + c) = make_float2(acc[i][2], acc[i][3]);
+        }
+    }
+}
+
+// grid (chunk bound, heads, blocks of kDB value channels).  Warp w: rows 16 w .. 16 w + 15 of the chunk.
+// Shared memory: C [kT][N + 8]; the state's two terms [N][kXP] each, then B [kT][N + 8] in their place; x [kT][kXP]; sums and steps [kT].
+__global__ void __launch_bounds__(kThreads, 2)
+apply_tc_kernel(const SsdArgs a, int shared_place) {
+    extern __shared__ __align__(16) float sm[];
+    griddep_wait();
+    griddep_launch();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tq = lane & 3, mi = lane >> 3;
+    const int head = blockIdx.y, e0 = blockIdx.z * kDB, N = a.N, dv = a.dv, NP = N + 8, ne = min(kDB, dv - e0);
+    const int group = head / (a.heads / a.groups), per = N / 8;
+    int req, row0, rows, index;
+    if (!find_chunk<kT>(a, blockIdx.x, req, row0, rows, index)) return;
+    bf16* Cs = reinterpret_cast<bf16*>(sm);
+    bf16* Us = Cs + kT * NP;
+    bf16* xs = Us + shared_place;
+    float2* cum = reinterpret_cast<float2*>(xs + kT * kXP);
+    float* dts = reinterpret_cast<float*>(cum + kT);
+    const bf16* xg = reinterpret_cast<const bf16*>(a.xc) + (int64_t)row0 * a.xc_pad;
+    const bf16* bg = xg + a.inner + group * N;
+    const bf16* cg = bg + a.groups * N;
+    const int rows16 = (rows + 15) / 16 * 16;
+    const bool from_zero = index == 0 && a.start_pos[req] == 0;        // the state in front of a request's first chunk
+    for (int i = tid; i < rows16 * per; i += kThreads) {
+        const int r = i / per, c = (i - r * per) * 8;
+        cp16(Cs + r * NP + c, cg + (r < rows ? (int64_t)r * a.xc_pad + c : 0), r < rows);
+    }
+    auto load_b = [&]() {
+        for (int i = tid; i < rows16 * per; i += kThreads) {
+            const int r = i / per, c = (i - r * per) * 8;
+            cp16(Us + r * NP + c, bg + (r < rows ? (int64_t)r * a.xc_pad + c : 0), r < rows);
+        }
+    };
+    if (from_zero) {
+        load_b();
+    } else {
+        const bf16* S = a.s_split + ((int64_t)blockIdx.x * a.heads + head) * N * dv + e0;
+        for (int i = tid; i < 2 * N * (kDB / 8); i += kThreads) {
+            const int r = i / (kDB / 8), c = (i - r * (kDB / 8)) * 8, n = r < N ? r : r - N;
+            const bool in = c < ne;
+            cp16(Us + r * kXP + c, S + (in ? (r < N ? 0 : a.split_plane) + (int64_t)n * dv + c : 0), in);
+        }
+    }
+    for (int i = tid; i < rows16 * (kDB / 8); i += kThreads) {
+        const int r = i / (kDB / 8), c = (i - r * (kDB / 8)) * 8;
+        const bool in = r < rows && c < ne;
+        cp16(xs + r * kXP + c, xg + (in ? (int64_t)r * a.xc_pad + head * dv + e0 + c : 0), in);
+    }
+    cp_async_commit();
+    if (tid < kT) {
+        const int64_t at = ((int64_t)blockIdx.x * a.heads + head) * kT + min(tid, rows - 1);
+        cum[tid] = a.cum[at];
+        dts[tid] = a.dt[at];
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    const bool active = 16 * warp < rows;
+    const bf16* ca = Cs + (16 * warp + (lane & 15)) * NP + (lane >> 4) * 8;
+    float acc[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; i++)
+#pragma unroll
+        for (int j = 0; j < 4; j++) acc[i][j] = 0.f;
+    const int i0 = 16 * warp + gid, i1 = i0 + 8;
+    const float2 ci0 = cum[min(i0, kT - 1)], ci1 = cum[min(i1, kT - 1)];
+    if (!from_zero) {
+        if (active) {
+            for (int k = 0; k < N; k += 16) {
+                uint32_t af[4];
+                ldsm4(af, ca + k);
+                rows_times_block(acc, af, Us, k, lane);
+                rows_times_block(acc, af, Us + N * kXP, k, lane);
+            }
+            const float f0 = expf(ci0.x + ci0.y), f1 = expf(ci1.x + ci1.y);
+#pragma unroll
+            for (int i = 0; i < 8; i++) { acc[i][0] *= f0; acc[i][1] *= f0; acc[i][2] *= f1; acc[i][3] *= f1; }
+        }
+        __syncthreads();                    // the state's place takes B
+        load_b();
+        cp_async_commit();
+        cp_async_wait<0>();
+        __syncthreads();
+    }
+    if (!active) return;
+    for (int key0 = 0; key0 <= 16 * warp; key0 += 64) {
+        const int slices = min(4, (16 * warp - key0) / 16 + 1);          // slices of 16 keys that hold a pair j <= i
+        float s[8][4];
+#pragma unroll
+        for (int i = 0; i < 8; i++)
+#pragma unroll
+            for (int j = 0; j < 4; j++) s[i][j] = 0.f;
+        const bf16* kb = Us + (key0 + (mi >> 1) * 8 + (lane & 7)) * NP + (mi & 1) * 8;
+        for (int k = 0; k < N; k += 16) {
+            uint32_t af[4];
+            ldsm4(af, ca + k);
+#pragma unroll
+            for (int sl = 0; sl < 4; sl++) {
+                if (sl < slices) {
+                    uint32_t b[4];
+                    ldsm4(b, kb + 16 * sl * NP + k);
+                    mma16816(s[2 * sl], af, b[0], b[1]);
+                    mma16816(s[2 * sl + 1], af, b[2], b[3]);
+                }
+            }
+        }
+#pragma unroll
+        for (int sl = 0; sl < 4; sl++) {
+            if (sl < slices) {
+                uint32_t ph[4], pl[4];
+#pragma unroll
+                for (int h = 0; h < 2; h++) {
+                    float p[4];
+#pragma unroll
+                    for (int u = 0; u < 2; u++) {
+                        const int j = key0 + 16 * sl + 8 * h + 2 * tq + u;
+                        const float2 cj = cum[j];
+                        const float d = dts[j];
+                        p[u] = j <= i0 ? s[2 * sl + h][u] * (exp_diff(ci0, cj) * d) : 0.f;
+                        p[2 + u] = j <= i1 ? s[2 * sl + h][2 + u] * (exp_diff(ci1, cj) * d) : 0.f;
+                    }
+                    split2(p[0], p[1], ph[2 * h], pl[2 * h]);
+                    split2(p[2], p[3], ph[2 * h + 1], pl[2 * h + 1]);
+                }
+                rows_times_block(acc, ph, xs, key0 + 16 * sl, lane);
+                rows_times_block(acc, pl, xs, key0 + 16 * sl, lane);
+            }
+        }
+    }
+    const float dskip = a.d[head];
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+        const int r = h ? i1 : i0;
+        if (r >= rows) continue;
+        const float* zr = a.proj + (int64_t)(row0 + r) * a.stride + head * dv + e0;
+        float* yr = a.y + (int64_t)(row0 + r) * a.inner + head * dv + e0;
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            const int c = i * 8 + 2 * tq;
+            if (c >= ne) continue;
+            const float2 z = *reinterpret_cast<const float2*>(zr + c);
+            const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(xs + r * kXP + c));
+            *reinterpret_cast<float2*>(yr + c) =
+                make_float2(fmaf(dskip, x.x, acc[i][2 * h]) * silu_f(z.x), fmaf(dskip, x.y, acc[i][2 * h + 1]) * silu_f(z.y));
+        }
+    }
+}
+
+// out[r][part] = y[r][part] / rms(y[r][part]) * gain of w values.  WARP: one warp per (row, part), eight to a CTA; else one
+// CTA.  VEC: w a multiple of 4 up to 4 * kVec * (threads of a part), 16-byte rows, the values in registers between the
+// sum and the scaling.
 constexpr int kVec = 8;
 
-template <typename T, bool VEC>
+template <typename T, bool VEC, bool WARP>
 __global__ void __launch_bounds__(kThreads)
 part_norm_kernel(T* __restrict__ out, int64_t out_stride, const float* __restrict__ y, const float* __restrict__ gain, int parts,
-                 int w, float eps) {
+                 int w, float eps, int64_t items) {
     __shared__ float red[32];
     griddep_wait();
     griddep_launch();
-    const int64_t r = blockIdx.x / parts;
-    const int part = blockIdx.x - (int)r * parts;
-    const float* src = y + (r * parts + part) * w;
+    const int64_t item = WARP ? (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5) : blockIdx.x;
+    if (item >= items) return;
+    const int me = WARP ? threadIdx.x & 31 : threadIdx.x, all = WARP ? 32 : blockDim.x;
+    const int64_t r = item / parts;
+    const int part = (int)(item - r * parts);
+    const float* src = y + item * w;
     const float* g = gain + (int64_t)part * w;
     T* dst = out + r * out_stride + (int64_t)part * w;
     float sq = 0.f;
+    auto total = [&](float v) {
+        if constexpr (WARP) return warp_sum(v);
+        else return block_sum(v, red);
+    };
     if constexpr (VEC) {
         const int w4 = w >> 2;
         float4 v[kVec];
 #pragma unroll
         for (int k = 0; k < kVec; k++) {
-            const int i = threadIdx.x + k * blockDim.x;
+            const int i = me + k * all;
             if (i < w4) {
                 v[k] = reinterpret_cast<const float4*>(src)[i];
                 sq += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
             }
         }
-        const float scale = rsqrtf(block_sum(sq, red) / (float)w + eps);
+        const float scale = rsqrtf(total(sq) / (float)w + eps);
 #pragma unroll
         for (int k = 0; k < kVec; k++) {
-            const int i = threadIdx.x + k * blockDim.x;
+            const int i = me + k * all;
             if (i < w4) {
                 const float4 n4 = reinterpret_cast<const float4*>(g)[i];
                 const float o0 = v[k].x * scale * n4.x, o1 = v[k].y * scale * n4.y, o2 = v[k].z * scale * n4.z, o3 = v[k].w * scale * n4.w;
@@ -668,9 +1021,9 @@ part_norm_kernel(T* __restrict__ out, int64_t out_stride, const float* __restric
             }
         }
     } else {
-        for (int i = threadIdx.x; i < w; i += blockDim.x) sq += src[i] * src[i];
-        const float scale = rsqrtf(block_sum(sq, red) / (float)w + eps);
-        for (int i = threadIdx.x; i < w; i += blockDim.x) dst[i] = from_f32<T>(src[i] * scale * g[i]);
+        for (int i = me; i < w; i += all) sq += src[i] * src[i];
+        const float scale = rsqrtf(total(sq) / (float)w + eps);
+        for (int i = me; i < w; i += all) dst[i] = from_f32<T>(src[i] * scale * g[i]);
     }
 }
 
@@ -725,64 +1078,100 @@ int launch_apply(const SsdArgs& a, int chunk_bound, cudaStream_t s) {
     KLLM_LAUNCH_STATUS();
 }
 
+template <typename T, int KC>
+void launch_conv(const SsdArgs& a, int chunk_bound, cudaStream_t s) {
+    const int blocks = (a.channels + kThreads - 1) / kThreads;
+    const dim3 grid(chunk_bound * (KC / kRun), blocks + (a.heads * 32 + kThreads - 1) / kThreads);
+    if (a.taps == 4) kllm_launch((conv_kernel<4, T, KC>), grid, dim3(kThreads), 0, s, a);
+    else kllm_launch((conv_kernel<0, T, KC>), grid, dim3(kThreads), 0, s, a);
+    kllm_launch((ring_kernel), dim3(blocks, a.n_requests), dim3(kThreads), 0, s, a);
+}
+
+template <int V, int KC, bool SPLIT>
+void launch_carry(const SsdArgs& a, cudaStream_t s) {
+    const int64_t elems = (int64_t)a.N * a.dv;
+    kllm_launch((carry_kernel<V, KC, SPLIT>), dim3((unsigned)((elems / V + kThreads - 1) / kThreads), a.heads, a.n_requests), dim3(kThreads), 0,
+                s, a);
+}
+
 int run_portions(const SsdArgs& a, int chunk_bound, cudaStream_t s) {
-    const dim3 grid(chunk_bound, (a.channels + kThreads - 1) / kThreads + (a.heads + kThreads - 1) / kThreads);
-    if (a.taps == 4) kllm_launch((conv_kernel<4>), grid, dim3(kThreads), 0, s, a);
-    else kllm_launch((conv_kernel<0>), grid, dim3(kThreads), 0, s, a);
+    launch_conv<float, kC>(a, chunk_bound, s);
     kllm_launch((pairs_kernel), dim3(chunk_bound, a.groups), dim3(kThreads), 0, s, a);
     int rc;
     if (a.N <= 32) rc = a.dv <= 64 ? launch_outer<2, 4>(a, chunk_bound, s) : launch_outer<2, 8>(a, chunk_bound, s);
     else if (a.N <= 64) rc = a.dv <= 64 ? launch_outer<4, 4>(a, chunk_bound, s) : launch_outer<4, 8>(a, chunk_bound, s);
     else rc = a.dv <= 64 ? launch_outer<8, 4>(a, chunk_bound, s) : launch_outer<8, 8>(a, chunk_bound, s);
     if (rc) return rc;
-    const int64_t elems = (int64_t)a.N * a.dv;
-    if (a.vec)
-        kllm_launch((carry_kernel<4>), dim3((unsigned)((elems / 4 + kThreads - 1) / kThreads), a.heads, a.n_requests), dim3(kThreads), 0, s, a);
-    else
-        kllm_launch((carry_kernel<1>), dim3((unsigned)((elems + kThreads - 1) / kThreads), a.heads, a.n_requests), dim3(kThreads), 0, s, a);
+    if (a.vec) launch_carry<4, kC, false>(a, s);
+    else launch_carry<1, kC, false>(a, s);
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) KLLM_FAIL("ssd: %s", cudaGetErrorString(e));
     return a.dv <= 64 ? launch_apply<1>(a, chunk_bound, s) : launch_apply<2>(a, chunk_bound, s);
 }
 
+int run_portions_tc(const SsdArgs& a, int chunk_bound, cudaStream_t s) {
+    const int place = max(2 * a.N * kXP, kT * (a.N + 8));              // elements that the state's terms and B share
+    const size_t outer_bytes = sizeof(bf16) * (size_t)kT * (a.N + 8 + 2 * kXP) + sizeof(float) * kT;
+    const size_t apply_bytes = sizeof(bf16) * ((size_t)kT * (a.N + 8 + kXP) + place) + 3 * sizeof(float) * kT;
+    static bool raised_outer = false, raised_apply = false;
+    int rc = raise_smem(outer_tc_kernel, raised_outer);
+    if (!rc) rc = raise_smem(apply_tc_kernel, raised_apply);
+    if (rc) return rc;
+    const dim3 grid(chunk_bound, a.heads, (a.dv + kDB - 1) / kDB);
+    launch_conv<bf16, kT>(a, chunk_bound, s);
+    kllm_launch((outer_tc_kernel), grid, dim3(kThreads), outer_bytes, s, a);
+    launch_carry<4, kT, true>(a, s);
+    kllm_launch((apply_tc_kernel), grid, dim3(kThreads), apply_bytes, s, a, place);
+    KLLM_LAUNCH_STATUS();
+}
+
+// bfloat16 models whose sizes the tensor-core form takes (its shared memory bounds N)
+bool tensor_cores(int dtype, int N, int dv) { return dtype == KLLM_BF16 && N % 16 == 0 && dv % 16 == 0 && N <= 256; }
+
 }  // namespace
 
-extern "C" int kllm_ssd_chunk_rows() { return kC; }
+// Rows of a chunk of the form for portions that these sizes take; kT of the tensor-core form.
+extern "C" int kllm_ssd_chunk_rows(int N, int dv, int dtype) { return tensor_cores(dtype, N, dv) ? kT : kC; }
 
 // proj float32 [n] rows at row stride `stride`: z, x (heads * dv each), B, C (groups * N each), dt (heads); conv_w float32
 // [channels][taps], conv_b [channels] over x, B and C; dt_bias, a_log, d float32 [heads]; state float32 [slots][state_stride] whose
-// first heads * N * dv values are S as [heads][N][dv]; ring float32 [slots][ring_stride] with taps rows of ch_pad (channels rounded
-// up to a multiple of 4); y float32 [n][heads * dv]: the gated values before the norm.  single: every request brings one
-// row; otherwise the work buffers xc [n][ch_pad], dt [chunk_bound][heads][C] (C: rows of a chunk), cum twice that, pairs
-// [chunk_bound][groups][C][C] and s_in [chunk_bound][heads][N][dv] are float32 and chunk_bound an upper bound of the chunks.
+// first heads * N * dv values are S as [heads][N][dv]; ring float32 [slots][ring_stride] with taps rows of the channels rounded
+// up to a multiple of 4; y float32 [n][heads * dv]: the gated values before the norm; dtype: the model's.  single: every request
+// brings one row; otherwise work buffers, C the rows of a chunk (kllm_ssd_chunk_rows) and chunk_bound an upper bound of the
+// chunks: xc [n][channels rounded up to a multiple of 4] float32, or bfloat16 rounded up to a multiple of 8 with the
+// tensor-core form; dt [chunk_bound][heads][C] float32, cum twice that; s_in [chunk_bound][heads][N][dv] float32; pairs
+// [chunk_bound][groups][C][C] float32, or with the tensor-core form s_split [2][chunk_bound][heads][N][dv] bfloat16.
 // early (single): the kernel may start beside the end of the one before it in the stream, which must write neither
 // state nor ring.
 extern "C" int kllm_ssd(float* y, const float* proj, int64_t stride, const float* conv_w, const float* conv_b,
                         const float* dt_bias, const float* a_log, const float* d, const int* q_start, const int* start_pos,
                         const int* state_slots, float* state, int64_t state_stride, float* ring, int64_t ring_stride, int n,
                         int n_requests, int heads, int groups, int N, int dv, int taps, int single, int early, int chunk_bound,
-                        float* xc, float* dt, float* cum, float* pairs, float* s_in, void* stream) {
+                        void* xc, float* dt, float* cum, float* pairs, float* s_in, void* s_split, int dtype, void* stream) {
     if (n <= 0 || n_requests <= 0) return 0;
     if (heads <= 0 || groups <= 0 || heads % groups || N <= 0 || dv <= 0) KLLM_FAIL("ssd: %d heads in %d groups of sizes %d, %d", heads, groups, N, dv);
     if (taps < 1 || taps > kC) KLLM_FAIL("ssd: a convolution of %d taps (up to %d)", taps, kC);
     if (heads > 65535 || groups > 65535 || n_requests > 65535) KLLM_FAIL("ssd: %d heads, %d requests in one launch", heads, n_requests);
+    const bool tc = tensor_cores(dtype, N, dv);
     SsdArgs a;
     a.proj = proj; a.stride = stride; a.conv_w = conv_w; a.conv_b = conv_b; a.dt_bias = dt_bias; a.a_log = a_log; a.d = d;
     a.taps = taps; a.heads = heads; a.groups = groups; a.N = N; a.dv = dv; a.inner = heads * dv;
     a.channels = a.inner + 2 * groups * N; a.ch_pad = (a.channels + 3) / 4 * 4;
     a.q_start = q_start; a.start_pos = start_pos; a.state_slots = state_slots; a.n_requests = n_requests;
     a.state = state; a.state_stride = state_stride; a.ring = ring; a.ring_stride = ring_stride; a.y = y;
-    a.xc = xc; a.dt = dt; a.cum = (float2*)cum; a.pairs = pairs; a.s_in = s_in;
+    a.xc = xc; a.xc_pad = tc ? (a.channels + 7) / 8 * 8 : a.ch_pad; a.dt = dt; a.cum = (float2*)cum; a.pairs = pairs; a.s_in = s_in;
+    a.s_split = (bf16*)s_split; a.split_plane = (int64_t)chunk_bound * heads * N * dv;
     if (state_stride < (int64_t)heads * N * dv || ring_stride < (int64_t)taps * a.ch_pad)
         KLLM_FAIL("ssd: slots of %lld and %lld values are too small", (long long)state_stride, (long long)ring_stride);
     if (single && n != n_requests) KLLM_FAIL("ssd: %d rows of %d requests that bring one row each", n, n_requests);
-    if (!single && (!xc || !dt || !cum || !pairs || !s_in || chunk_bound <= 0)) KLLM_FAIL("ssd: portions need work buffers");
+    if (!single && (!xc || !dt || !cum || !s_in || chunk_bound <= 0 || !(tc ? s_split : (void*)pairs))) KLLM_FAIL("ssd: portions need work buffers");
     cudaStream_t s = (cudaStream_t)stream;
     const bool rows_vec = dv % 4 == 0 && state_stride % 4 == 0 && !((uintptr_t)state & 15);
     if (single) return rows_vec ? launch_step<4>(a, early != 0, s) : launch_step<1>(a, early != 0, s);
     a.vec = rows_vec && N % 4 == 0 && stride % 4 == 0 &&
-            !(((uintptr_t)proj | (uintptr_t)xc | (uintptr_t)s_in | (uintptr_t)pairs | (uintptr_t)y) & 15);
-    return run_portions(a, chunk_bound, s);
+            !(((uintptr_t)proj | (uintptr_t)xc | (uintptr_t)s_in | (uintptr_t)pairs | (uintptr_t)s_split | (uintptr_t)y) & 15);
+    if (tc && !a.vec) KLLM_FAIL("ssd: the tensor-core form needs 16-byte aligned operands with row strides in multiples of 4");
+    return tc ? run_portions_tc(a, chunk_bound, s) : run_portions(a, chunk_bound, s);
 }
 
 // out [n] rows of parts * w values in `dtype` at out_stride = y / rms(y) * gain, each of the `parts` pieces of a row by its own
@@ -792,19 +1181,30 @@ extern "C" int kllm_part_norm(void* out, int64_t out_stride, const float* y, con
     if (n <= 0) return 0;
     if (parts <= 0 || w <= 0) KLLM_FAIL("part norm: %d parts of %d values", parts, w);
     if ((int64_t)n * parts > 0x7fffffffLL) KLLM_FAIL("part norm: %d rows of %d parts in one launch", n, parts);
-    const int threads = w <= 256 ? 64 : (w <= 1024 ? 128 : kThreads);
+    // the form follows from the part's width and the addresses alone
+    const bool warp = w <= 32 * 4 * kVec;
+    const int threads = warp ? kThreads : (w <= 4096 ? 128 : kThreads), per_part = warp ? 32 : threads;
     const int esize = dtype == KLLM_F32 ? 4 : 2;
-    const bool vec = w % 4 == 0 && w <= threads * 4 * kVec && out_stride % 4 == 0 && !(((uintptr_t)y | (uintptr_t)gain) & 15) &&
+    const bool vec = w % 4 == 0 && w <= per_part * 4 * kVec && out_stride % 4 == 0 && !(((uintptr_t)y | (uintptr_t)gain) & 15) &&
                      !((uintptr_t)out & (4 * esize - 1));
+    const int64_t items = (int64_t)n * parts;
+    const int grid = (int)(warp ? (items + kThreads / 32 - 1) / (kThreads / 32) : items);
     cudaStream_t s = (cudaStream_t)stream;
-#define KLLM_PN(T, VEC) kllm_launch((part_norm_kernel<T, VEC>), dim3(n * parts), dim3(threads), 0, s, (T*)out, out_stride, y, gain, parts, w, eps)
+#define KLLM_PN(T, VEC, WARP) \
+    kllm_launch((part_norm_kernel<T, VEC, WARP>), dim3(grid), dim3(threads), 0, s, (T*)out, out_stride, y, gain, parts, w, eps, items)
+#define KLLM_PN_T(T)                                       \
+    if (warp && vec) KLLM_PN(T, true, true);               \
+    else if (warp) KLLM_PN(T, false, true);                \
+    else if (vec) KLLM_PN(T, true, false);                 \
+    else KLLM_PN(T, false, false)
     if (dtype == KLLM_F32) {
-        if (vec) KLLM_PN(float, true); else KLLM_PN(float, false);
+        KLLM_PN_T(float);
     } else if (dtype == KLLM_BF16) {
-        if (vec) KLLM_PN(bf16, true); else KLLM_PN(bf16, false);
+        KLLM_PN_T(bf16);
     } else {
         KLLM_FAIL("part norm: unknown element type %d", dtype);
     }
+#undef KLLM_PN_T
 #undef KLLM_PN
     KLLM_LAUNCH_STATUS();
 }

@@ -1682,14 +1682,16 @@ def gla(y: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: t
 
 def ssd(proj: torch.Tensor, conv: torch.Tensor, conv_bias: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
         d: torch.Tensor, state: torch.Tensor, ring: torch.Tensor, ctx, heads: int, groups: int, N: int, dv: int,
-        early: bool = False) -> torch.Tensor:
+        early: bool = False, dtype: torch.dtype = torch.float32) -> torch.Tensor:
     """float32 [n, heads * dv]: (S_t^T C_t + D x_t) * silu(z_t) of the recurrence S_t = exp(-exp(a_log) dt_t) S_(t-1) +
     dt_t B_t x_t^T per head.  ``proj`` float32 [n, >= 2 heads dv + 2 groups N + heads] with dense rows holds z, x, B, C and dt; x, B and
     C pass a causal convolution (``conv`` float32 [channels, taps], last column the current row's, ``conv_bias``) and silu, dt
     a softplus behind ``dt_bias``.  ``state`` float32 [slots, >= heads * N * dv] holds S as [heads, N, dv] per request slot,
     ``ring`` float32 [slots, >= taps * row] (row: the channels rounded up to a multiple of 4) the convolution's inputs of
     the last taps positions, position p in row p mod taps; both are carried on.  ``early``: a step of one row per request
-    may read them beside the end of the kernel before it, which then must not write them."""
+    may read them beside the end of the kernel before it, which then must not write them.  ``dtype`` is the model's: with
+    bfloat16 the products of portions run on the tensor cores where the sizes allow it (N and dv in steps of 16), x, B and
+    C rounded to bfloat16 behind silu, everything else float32 (as two bfloat16 terms where it enters a product)."""
     _cuda(proj, conv, conv_bias, dt_bias, a_log, d, state, ring)
     n, inner, taps = proj.shape[0], heads * dv, conv.shape[1]
     channels = inner + 2 * groups * N
@@ -1709,21 +1711,27 @@ def ssd(proj: torch.Tensor, conv: torch.Tensor, conv_bias: torch.Tensor, dt_bias
     f32 = dict(dtype=torch.float32, device=proj.device)
     y = torch.empty((n, inner), **f32)
     lib = load_library("ssd")
-    xc = dt = cum = pairs = s_in = None
-    bound = 0
+    xc = dt = cum = pairs = s_in = s_split = None
+    bound, tc = 0, False
     if not ctx.all_single:
-        C = lib.kllm_ssd_chunk_rows()
+        C = lib.kllm_ssd_chunk_rows(N, dv, dtype_code(dtype))
+        tc = C == lib.kllm_ssd_chunk_rows(16, 16, dtype_code(torch.bfloat16))
         bound = n // C + ctx.n_requests
-        xc, dt, cum = torch.empty((n, row), **f32), torch.empty((bound, heads, C), **f32), torch.empty((bound, heads, C, 2), **f32)
-        pairs, s_in = torch.empty((bound, groups, C, C), **f32), torch.empty((bound, heads, N, dv), **f32)
+        dt, cum, s_in = (torch.empty((bound, heads) + t, **f32) for t in ((C,), (C, 2), (N, dv)))
+        if tc:
+            xc = torch.empty((n, -(-channels // 8) * 8), dtype=torch.bfloat16, device=proj.device)
+            s_split = torch.empty((2, bound, heads, N, dv), dtype=torch.bfloat16, device=proj.device)
+        else:
+            xc, pairs = torch.empty((n, row), **f32), torch.empty((bound, groups, C, C), **f32)
     rc = lib.kllm_ssd(_p(y), _p(proj), ctypes.c_int64(proj.stride(0)), _p(conv), _p(conv_bias), _p(dt_bias), _p(a_log), _p(d),
                       _p(ctx.q_start), _p(ctx.start_pos), _p(ctx.state_slots), _p(state), ctypes.c_int64(state.stride(0)),
                       _p(ring), ctypes.c_int64(ring.stride(0)), n, ctx.n_requests, heads, groups, N, dv, taps,
-                      int(ctx.all_single), int(early), bound, _p(xc), _p(dt), _p(cum), _p(pairs), _p(s_in), _stream())
+                      int(ctx.all_single), int(early), bound, _p(xc), _p(dt), _p(cum), _p(pairs), _p(s_in), _p(s_split),
+                      dtype_code(dtype), _stream())
     _check(lib, "ssd", rc)
     if not ctx.all_single:
         global launches
-        launches += 4
+        launches += 4 if tc else 5
     return y
 
 

@@ -16,8 +16,8 @@ params: ``hidden``, ``heads``, ``head_dim`` (dv), ``state`` (N), ``groups``, ``t
 
 State (``StateNeed``), float32, zero when a request opens: S as [heads][N][dv], and under the name "conv" the convolution's
 inputs of the last ``taps`` positions, position p in row p mod taps.  The projections are one product whose float32
-result feeds the kernels; convolution, decays, state, sums, gate and norm are float32 in both dtypes.  The mixer
-has the split form (``gla.SplitMixer``).
+result feeds the kernels; convolution, decays, state, sums, gate and norm are float32 in both dtypes; in bfloat16 portions round
+x, B and C behind silu where their products run on the tensor cores.  The mixer has the split form (``gla.SplitMixer``).
 """
 from __future__ import annotations
 
@@ -71,7 +71,7 @@ class StateSpaceMixer(SplitMixer):
 
     def core(self, proj, ctx, cache, y):
         g = kernels.ssd(proj, self.conv, self.conv_bias, self.dt_bias, self.a_log, self.d, cache.state, cache.states["conv"], ctx,
-                        self.heads, self.groups, self.N, self.dv, early=True)
+                        self.heads, self.groups, self.N, self.dv, early=True, dtype=self.dtype)
         kernels.part_norm(y, g, self.gain, self.parts, self.eps)
 
 
