@@ -11,7 +11,8 @@
 //             shapes do not depend on the routing.
 //   gemm      for the sorted rows of every expert e, C = A W_e^T with float32 accumulation:
 //             bfloat16 operands as tiles of 64 rows x 64 columns on the tensor cores
-//             (mma.sync m16n8k16, operands through a three-stage cp.async ring), float32
+//             (mma.sync m16n8k16, operands through a three-stage cp.async ring; a step of few rows
+//             streams the experts' weights through registers instead), float32
 //             operands (and bfloat16 ones whose rows are not 16-byte aligned) as tiles of 32 x
 //             64 on the CUDA cores.  Two forms:
 //             "gated" reads row `token` of the layer's input, times the row's weight if the
@@ -490,6 +491,126 @@ expert_gemm_mma_kernel(void* __restrict__ c_out, const bf16* __restrict__ a, int
         }
 }
 
+// ---- a step of few rows, bfloat16: the experts' weights streamed ---------------------------------------------
+// A CTA takes 16 weight rows of one expert (GATE_UP: 8 gate rows and the 8 up rows that go with them) as the 16 rows of an MMA
+// tile and that expert's rows of A, eight at a time, as its columns.  The eight warps share k in steps of 32: a lane loads 16
+// bytes of weight rows g and g + 8 straight into registers, kSteps steps of them on their way at once, and takes the same 16
+// bytes' worth of k of row g of A from shared memory (a permutation of k that both operands share).  The warps' partial
+// tiles are added in warp order: a row's sums have one order, fixed by K.
+constexpr int STREAM_ROWS = 64;                             // most (token, choice) pairs of a step that takes this form
+constexpr int SW = 8, kSteps = 8;                           // warps, steps in flight
+// elements between rows of A in shared memory: an odd number of 64-byte pieces
+__host__ __device__ constexpr int stream_row(int K) { return K % 64 ? K : K + 32; }
+
+__device__ __forceinline__ uint4 ldg_stream(const bf16* p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];\n" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+
+template <int FORM>
+__global__ void __launch_bounds__(SW * 32)
+expert_stream_kernel(void* __restrict__ c_out, const bf16* __restrict__ a, int64_t a_stride, const bf16* __restrict__ w,
+                     const int* __restrict__ offsets, const int* __restrict__ perm, const float* __restrict__ wt, int top, int N,
+                     int K, int scale_in, int scale_out, GatedAct act) {
+    constexpr bool GATED = FORM == GATE_UP, UP = FORM != DOWN;
+    constexpr int OUT = GATED ? 8 : 16;                     // output columns of a CTA
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    bf16* xs = reinterpret_cast<bf16*>(smem_raw);           // [8][stream_row(K)]
+    __shared__ float red[SW][16][8];
+    griddep_wait();
+    griddep_launch();
+    const int e = blockIdx.y, n0 = blockIdx.x * OUT, lo = offsets[e], hi = offsets[e + 1];
+    if (lo >= hi) return;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int XP = stream_row(K);
+    const bf16* we = w + (int64_t)e * (GATED ? 2 : 1) * N * K;
+    const int ra = min(n0 + g, N - 1), rb = GATED ? N + ra : min(n0 + g + 8, N - 1);     // rows past the end: not stored
+    const bf16 *wa = we + (int64_t)ra * K + t * 8, *wb = we + (int64_t)rb * K + t * 8;
+    for (int r0 = lo; r0 < hi; r0 += 8) {
+        const int nr = min(8, hi - r0);
+        for (int i = tid; i < nr * (K / 8); i += SW * 32) {
+            const int r = i / (K / 8), c = (i - r * (K / 8)) * 8;
+            const int64_t src = UP ? perm[r0 + r] / top : r0 + r;
+            cp16(xs + r * XP + c, a + src * a_stride + c, true);
+        }
+        asm volatile("cp.async.commit_group;\n" ::: "memory");
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        bool staged = false;
+        for (int k0 = warp * 32; k0 < K; k0 += SW * 32 * kSteps) {
+            uint4 va[kSteps], vb[kSteps];
+#pragma unroll
+            for (int u = 0; u < kSteps; u++) {
+                const int k = k0 + u * SW * 32;
+                if (k < K) {
+                    va[u] = ldg_stream(wa + k);
+                    vb[u] = ldg_stream(wb + k);
+                }
+            }
+            if (!staged) {                                  // the first weights are on their way before A is waited for
+                asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+                __syncthreads();
+                staged = true;
+            }
+#pragma unroll
+            for (int u = 0; u < kSteps; u++) {
+                const int k = k0 + u * SW * 32;
+                if (k < K) {
+                    const uint4 x = *reinterpret_cast<const uint4*>(xs + g * XP + k + t * 8);
+                    const uint32_t lo4[4] = {va[u].x, vb[u].x, va[u].y, vb[u].y}, hi4[4] = {va[u].z, vb[u].z, va[u].w, vb[u].w};
+                    mma16816(acc, lo4, x.x, x.y);
+                    mma16816(acc, hi4, x.z, x.w);
+                }
+            }
+        }
+        if (!staged) {
+            asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+            __syncthreads();
+        }
+        red[warp][g][2 * t] = acc[0];
+        red[warp][g][2 * t + 1] = acc[1];
+        red[warp][g + 8][2 * t] = acc[2];
+        red[warp][g + 8][2 * t + 1] = acc[3];
+        __syncthreads();
+        for (int i = tid; i < OUT * 8; i += SW * 32) {
+            const int c = i / OUT, r = i - c * OUT, col = n0 + r;         // row of A, weight row
+            if (c < nr && col < N) {
+                float v = 0.f, u = 0.f;
+#pragma unroll
+                for (int q = 0; q < SW; q++) {
+                    v += red[q][r][c];
+                    if (GATED) u += red[q][r + 8][c];
+                }
+                const int row = r0 + c, flat = perm[row];
+                const float sc = (UP ? scale_in : scale_out) ? wt[flat] : 1.f;
+                if (GATED) ((bf16*)c_out)[(int64_t)row * N + col] = __float2bfloat16_rn(gated_act(v * sc, u * sc, act));
+                else if (UP) ((bf16*)c_out)[(int64_t)row * N + col] = __float2bfloat16_rn(relu2(v * sc));
+                else ((float*)c_out)[(int64_t)flat * N + col] = v * sc;
+            }
+        }
+        __syncthreads();                                    // A's rows and the partial tiles are no longer read
+    }
+}
+
+template <int FORM>
+int launch_stream(void* c, const void* a, int64_t a_stride, const void* w, const int* offsets, const int* perm,
+                  const float* wt, int E, int top, int N, int K, int scale_in, int scale_out, GatedAct act, cudaStream_t s) {
+    auto kern = expert_stream_kernel<FORM>;
+    static bool raised = false;
+    if (!raised) {
+        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        if (e != cudaSuccess) {
+            snprintf(g_kllm_err, sizeof(g_kllm_err), "moe gemm: shared memory limit: %s", cudaGetErrorString(e));
+            return (int)e;
+        }
+        raised = true;
+    }
+    constexpr int OUT = FORM == GATE_UP ? 8 : 16;
+    kllm_launch(kern, dim3((N + OUT - 1) / OUT, E), dim3(SW * 32), (size_t)8 * stream_row(K) * sizeof(bf16), s, c, (const bf16*)a, a_stride,
+                (const bf16*)w, offsets, perm, wt, top, N, K, scale_in, scale_out, act);
+    KLLM_LAUNCH_STATUS();
+}
+
 template <int FORM, int MW>
 int launch_mma(void* c, const void* a, int64_t a_stride, const void* w, const int* offsets, const int* perm,
                const float* wt, int rows, int E, int top, int N, int K, int scale_in, int scale_out, GatedAct act,
@@ -651,6 +772,14 @@ extern "C" int kllm_moe_gemm(void* c, const void* a, int64_t a_stride, const voi
     if (row_tiles > 65535) KLLM_FAIL("moe gemm: %d rows in one launch", rows);
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == KLLM_BF16 && K % 8 == 0 && a_stride % 8 == 0 && (((uintptr_t)a | (uintptr_t)w) & 15) == 0) {
+        // few rows: the weights streamed (which form runs depends on the sizes and the number of rows alone)
+        if (rows <= STREAM_ROWS && K % 32 == 0 && (size_t)8 * stream_row(K) * sizeof(bf16) <= 200 * 1024 && E <= 65535) {
+#define KLLM_MOE_STREAM(G) return launch_stream<G>(c, a, a_stride, w, offsets, perm, wt, E, top, N, K, scale_in, scale_out, act, s)
+            if (form == GATE_UP) KLLM_MOE_STREAM(GATE_UP);
+            if (form == PLAIN_UP) KLLM_MOE_STREAM(PLAIN_UP);
+            KLLM_MOE_STREAM(DOWN);
+#undef KLLM_MOE_STREAM
+        }
         // tiles of 128 rows where the experts have that many rows on average (which tile a row
         // falls into changes no sum of that row)
         const bool tall = rows / E >= 128;
