@@ -739,16 +739,19 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
 constexpr int kDB = 64;                     // value channels of a CTA
 constexpr int kXP = kDB + 8;                // padded row of such a block, in elements
 
-// acc[2 p], acc[2 p + 1] += A (16 rows, 16 inner) times columns 16 p .. of rows k0 .. k0 + 15 of a block at row length kXP
-__device__ __forceinline__ void rows_times_block(float (&acc)[8][4], const uint32_t (&a)[4], const bf16* block, int k0, int lane) {
+// Fragments of rows k0 .. k0 + 15 of a block at row length kXP, as the second operand: b[p] for columns 16 p .. 16 p + 15.  All
+// loads go out before the first product that needs one.
+__device__ __forceinline__ void load_block(uint32_t (&b)[4][4], const bf16* block, int k0, int lane) {
     const int mi = lane >> 3;
     const bf16* base = block + (k0 + (mi & 1) * 8 + (lane & 7)) * kXP + (mi >> 1) * 8;
 #pragma unroll
+    for (int p = 0; p < kDB / 16; p++) ldsm4_trans(b[p], base + p * 16);
+}
+__device__ __forceinline__ void times_block(float (&acc)[8][4], const uint32_t (&a)[4], const uint32_t (&b)[4][4]) {
+#pragma unroll
     for (int p = 0; p < kDB / 16; p++) {
-        uint32_t b[4];
-        ldsm4_trans(b, base + p * 16);
-        mma16816(acc[2 * p], a, b[0], b[1]);
-        mma16816(acc[2 * p + 1], a, b[2], b[3]);
+        mma16816(acc[2 * p], a, b[p][0], b[p][1]);
+        mma16816(acc[2 * p + 1], a, b[p][2], b[p][3]);
     }
 }
 
@@ -807,8 +810,11 @@ outer_tc_kernel(const SsdArgs a) {
         for (int k = 0; k < steps; k++) {
             uint32_t af[4];
             ldsm4_trans(af, Bs + (k * 16 + (mi >> 1) * 8 + (lane & 7)) * NP + m0 + (mi & 1) * 8);
-            rows_times_block(acc, af, xh, k * 16, lane);
-            rows_times_block(acc, af, xl, k * 16, lane);
+            uint32_t bh[4][4], bl[4][4];
+            load_block(bh, xh, k * 16, lane);
+            load_block(bl, xl, k * 16, lane);
+            times_block(acc, af, bh);
+            times_block(acc, af, bl);
         }
 #pragma unroll
         for (int i = 0; i < 8; i++) {
@@ -889,8 +895,11 @@ apply_tc_kernel(const SsdArgs a, int shared_place) {
             for (int k = 0; k < N; k += 16) {
                 uint32_t af[4];
                 ldsm4(af, ca + k);
-                rows_times_block(acc, af, Us, k, lane);
-                rows_times_block(acc, af, Us + N * kXP, k, lane);
+                uint32_t bh[4][4], bl[4][4];
+                load_block(bh, Us, k, lane);
+                load_block(bl, Us + N * kXP, k, lane);
+                times_block(acc, af, bh);
+                times_block(acc, af, bl);
             }
             const float f0 = expf(ci0.x + ci0.y), f1 = expf(ci1.x + ci1.y);
 #pragma unroll
@@ -912,22 +921,24 @@ apply_tc_kernel(const SsdArgs a, int shared_place) {
             for (int j = 0; j < 4; j++) s[i][j] = 0.f;
         const bf16* kb = Us + (key0 + (mi >> 1) * 8 + (lane & 7)) * NP + (mi & 1) * 8;
         for (int k = 0; k < N; k += 16) {
-            uint32_t af[4];
+            uint32_t af[4], b[4][4];
             ldsm4(af, ca + k);
+#pragma unroll
+            for (int sl = 0; sl < 4; sl++)
+                if (sl < slices) ldsm4(b[sl], kb + 16 * sl * NP + k);
 #pragma unroll
             for (int sl = 0; sl < 4; sl++) {
                 if (sl < slices) {
-                    uint32_t b[4];
-                    ldsm4(b, kb + 16 * sl * NP + k);
-                    mma16816(s[2 * sl], af, b[0], b[1]);
-                    mma16816(s[2 * sl + 1], af, b[2], b[3]);
+                    mma16816(s[2 * sl], af, b[sl][0], b[sl][1]);
+                    mma16816(s[2 * sl + 1], af, b[sl][2], b[sl][3]);
                 }
             }
         }
 #pragma unroll
         for (int sl = 0; sl < 4; sl++) {
             if (sl < slices) {
-                uint32_t ph[4], pl[4];
+                uint32_t ph[4], pl[4], xb[4][4];
+                load_block(xb, xs, key0 + 16 * sl, lane);
 #pragma unroll
                 for (int h = 0; h < 2; h++) {
                     float p[4];
@@ -942,23 +953,29 @@ apply_tc_kernel(const SsdArgs a, int shared_place) {
                     split2(p[0], p[1], ph[2 * h], pl[2 * h]);
                     split2(p[2], p[3], ph[2 * h + 1], pl[2 * h + 1]);
                 }
-                rows_times_block(acc, ph, xs, key0 + 16 * sl, lane);
-                rows_times_block(acc, pl, xs, key0 + 16 * sl, lane);
+                times_block(acc, ph, xb);
+                times_block(acc, pl, xb);
             }
         }
     }
     const float dskip = a.d[head];
+    float2 zv[2][8];                        // all of the gate's loads before the first store
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+        const float* zr = a.proj + (int64_t)(row0 + min(h ? i1 : i0, rows - 1)) * a.stride + head * dv + e0;
+#pragma unroll
+        for (int i = 0; i < 8; i++) zv[h][i] = *reinterpret_cast<const float2*>(zr + min(i * 8 + 2 * tq, ne - 2));
+    }
 #pragma unroll
     for (int h = 0; h < 2; h++) {
         const int r = h ? i1 : i0;
         if (r >= rows) continue;
-        const float* zr = a.proj + (int64_t)(row0 + r) * a.stride + head * dv + e0;
         float* yr = a.y + (int64_t)(row0 + r) * a.inner + head * dv + e0;
 #pragma unroll
         for (int i = 0; i < 8; i++) {
             const int c = i * 8 + 2 * tq;
             if (c >= ne) continue;
-            const float2 z = *reinterpret_cast<const float2*>(zr + c);
+            const float2 z = zv[h][i];
             const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(xs + r * kXP + c));
             *reinterpret_cast<float2*>(yr + c) =
                 make_float2(fmaf(dskip, x.x, acc[i][2 * h]) * silu_f(z.x), fmaf(dskip, x.y, acc[i][2 * h + 1]) * silu_f(z.y));
