@@ -323,7 +323,7 @@ attn_simt_decode_kernel(float* __restrict__ part_o, float* __restrict__ part_ml,
                         const int* __restrict__ q_start, const int* __restrict__ start_pos,
                         const int* __restrict__ block_table, int max_blocks, int n_requests, int n_heads, int n_kv,
                         int page_size, int window, float scale, int chunk, int max_splits,
-                        const float* __restrict__ slopes) {
+                        const float* __restrict__ slopes, int keep) {
     constexpr int KT = dec_keys(HD), LD = HD + 4, D4 = HD / 4;
     constexpr int HGRP = DEC_THREADS / KT;                  // head groups of the first product
     constexpr int HPG = (GS + HGRP - 1) / HGRP;             // heads of a group
@@ -344,16 +344,18 @@ attn_simt_decode_kernel(float* __restrict__ part_o, float* __restrict__ part_ml,
     if (s >= n_requests) return;
     const int tok = q_start[s], pos = start_pos[s];
     const int lo_all = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
-    const int lo = lo_all + split * chunk, hi = min(pos + 1, lo + chunk);
+    const KeyLine line(lo_all, pos + 1, keep, KEYS);        // kept keys, then the window; a sub-tile may hold the border
+    const int lo = split * chunk, hi = min(line.total(), lo + chunk);
     if (lo >= hi) return;
+    auto there = [&](int v) { return v < hi && (v >= line.pad || v < line.kept); };
     const int* table = block_table + (int64_t)s * max_blocks;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
-    auto load_tile = [&](int key0) {
+    auto load_tile = [&](int v0) {
 #pragma unroll
         for (int u = 0; u < KT * D4 / DEC_THREADS; u++) {
-            const int e = tid + u * DEC_THREADS, k = e / D4, c = e - k * D4, kp = key0 + k;
-            const bool ok = kp < hi;
+            const int e = tid + u * DEC_THREADS, k = e / D4, c = e - k * D4, kp = line.key(v0 + k);
+            const bool ok = there(v0 + k);
             int64_t off = 0;
             if (ok) {
                 const int lp = kp / page_size;
@@ -378,7 +380,7 @@ attn_simt_decode_kernel(float* __restrict__ part_o, float* __restrict__ part_ml,
 #pragma unroll
     for (int i = 0; i < HPT; i++) acc[i] = make_float4(0.f, 0.f, 0.f, 0.f);
 
-    for (int key0 = lo; key0 < hi; key0 += KT) {
+    for (int v0 = lo; v0 < hi; v0 += KT) {
         asm volatile("cp.async.wait_group 0;\n" ::: "memory");
         __syncthreads();
         // ---- scores of key k1 with the heads of group hg1 ----
@@ -399,14 +401,15 @@ attn_simt_decode_kernel(float* __restrict__ part_o, float* __restrict__ part_ml,
                         }
                     }
                 }
-                const int kp = key0 + k1;
+                const int kp = line.key(v0 + k1);
+                const bool ok = there(v0 + k1);
 #pragma unroll
                 for (int i = 0; i < HPG; i++) {
                     const int h = hg1 * HPG + i;
                     if (h < GS) {
                         float v = ((sc[i].x + sc[i].y) + (sc[i].z + sc[i].w)) * scale;
                         if (slopes) v += slopes[g * GS + h] * (float)(kp - pos);
-                        Ps[k1 * GS + h] = kp < hi ? v : -INFINITY;
+                        Ps[k1 * GS + h] = ok ? v : -INFINITY;
                     }
                 }
             }
@@ -422,7 +425,7 @@ attn_simt_decode_kernel(float* __restrict__ part_o, float* __restrict__ part_ml,
             }
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-            const float m_old = m_s[h], m_new = fmaxf(m_old, mx);        // finite: key0 itself is below hi
+            const float m_old = m_s[h], m_new = fmaxf(m_old, mx);        // finite: the key at v0 itself is there
             float sum = 0.f;
 #pragma unroll
             for (int j = 0; j < KT / 32; j++) {
@@ -466,7 +469,7 @@ attn_simt_decode_kernel(float* __restrict__ part_o, float* __restrict__ part_ml,
             }
         }
         __syncthreads();                                    // K, V and P of this sub-tile are no longer read
-        if (key0 + KT < hi) load_tile(key0 + KT);
+        if (v0 + KT < hi) load_tile(v0 + KT);
     }
     // ---- the key groups' sums, added in group order ----
     float* red = Ks;                                        // [KG][GS][HD]
@@ -492,7 +495,7 @@ template <int HD, int GS>
 int launch_decode(float* part_o, float* part_ml, const void* q, int64_t q_stride, const void* kcache, const void* vcache,
                   const int* q_start, const int* start_pos, const int* block_table, int max_blocks, int n_requests,
                   int n_heads, int n_kv, int page_size, int window, float scale, int chunk, int max_splits,
-                  const float* slopes, cudaStream_t s) {
+                  const float* slopes, int keep, cudaStream_t s) {
     auto kern = attn_simt_decode_kernel<HD, GS>;
     static bool raised = false;
     constexpr size_t smem = dec_smem_floats(HD, GS) * sizeof(float);
@@ -506,7 +509,7 @@ int launch_decode(float* part_o, float* part_ml, const void* q, int64_t q_stride
     }
     kllm_launch(kern, dim3(n_requests * n_kv, 1, max_splits), dim3(DEC_THREADS), smem, s, part_o, part_ml, (const float*)q,
                 q_stride, (const float*)kcache, (const float*)vcache, q_start, start_pos, block_table, max_blocks,
-                n_requests, n_heads, n_kv, page_size, window, scale, chunk, max_splits, slopes);
+                n_requests, n_heads, n_kv, page_size, window, scale, chunk, max_splits, slopes, keep);
     KLLM_LAUNCH_STATUS();
 }
 
@@ -644,12 +647,12 @@ extern "C" int kllm_attention_simt(void* out, void* part_o, void* part_ml, const
     cudaStream_t s = (cudaStream_t)stream;
     // decoding tokens in float32 at the common head sizes and group widths: the kernel in which every thread works
     if (chunk > 0 && dtype == KLLM_F32 && (hd == 64 || hd == 128) && vd == hd && n_requests == max_tiles && segment == 0 &&
-        v_heads == n_kv && v_row == vd && keep == 0) {
+        v_heads == n_kv && v_row == vd) {
 #define KLLM_SIMT_DEC(HD_, GS_)                                                                                        \
     if (hd == HD_ && gs == GS_)                                                                                       \
         return launch_decode<HD_, GS_>((float*)part_o, (float*)part_ml, q, q_stride, kcache, vcache, q_start, start_pos, \
                                        block_table, max_blocks, n_requests, n_heads, n_kv, page_size, window, scale,  \
-                                       chunk, max_splits, slopes, s)
+                                       chunk, max_splits, slopes, keep, s)
         KLLM_SIMT_DEC(64, 1); KLLM_SIMT_DEC(64, 2); KLLM_SIMT_DEC(64, 4); KLLM_SIMT_DEC(64, 8); KLLM_SIMT_DEC(64, 16);
         KLLM_SIMT_DEC(128, 1); KLLM_SIMT_DEC(128, 2); KLLM_SIMT_DEC(128, 4); KLLM_SIMT_DEC(128, 8); KLLM_SIMT_DEC(128, 16);
 #undef KLLM_SIMT_DEC

@@ -449,7 +449,7 @@ ATTN_SIZES = [(4, 2, 128, 128), (4, 2, 16, 24), (3, 1, 10, 6), (8, 2, 64, 64), (
 # every pair of window and kept keys at four sizes, two of them at the others, the one beyond every tile's reach at two
 ATTN_MASKS = [(40, 20), (130, 7), (1, 3), (64, 64), (100, 65), (299, 1), (17, 0), (40, 400)]
 ATTN_CASES = [(m, z) for z in ATTN_SIZES[:4] for m in ATTN_MASKS] + [(m, z) for z in ATTN_SIZES[4:] for m in ATTN_MASKS[:2]] + \
-    [((2100, 16), z) for z in (ATTN_SIZES[3], ATTN_SIZES[1])]
+    [((2100, 16), z) for z in (ATTN_SIZES[3], ATTN_SIZES[1])] + [((260, 100), ATTN_SIZES[3]), ((270, 10), ATTN_SIZES[0]), ((262, 30), ATTN_SIZES[1])]
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -463,7 +463,7 @@ def test_window_edges_kept_keys_and_sinks(dtype, mask, sizes):
     (window, keep), (H, G, dk, dv) = mask, sizes
     long = window > 300
     rng = np.random.default_rng(H * 100 + dk + window)
-    T, page, scale = (2400 if long else 300), 16, 0.5
+    T, page, scale = (2400 if long else 380 if 256 < window < 290 else 300), 16, 0.5
     q, k = rng.standard_normal((T, H, dk)) * 0.2, rng.standard_normal((T, G, dk)) * 0.2
     v = rng.standard_normal((T, G, dv))
     probes = [T - 1, T - 2, T - 3, T - 4, T - 5, T - 6, T - 7, T - 60, T - 61, T - 62]
