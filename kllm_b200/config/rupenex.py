@@ -3,7 +3,7 @@
     architecture   "Rupenex"
     vocab, width   sizes of the embedding
     norm           {eps}: of every norm of the model
-    logit_scale    the logits are multiplied by it
+    logit_scale    the logits are multiplied by it (absent: 1)
     layers         a list; each entry {type, mixer, mlp}:
                    type "attention": mixer {heads, kv_heads, dim, vdim, scale, mask {size, keep_first},
                        rot {base, dims, scaling {factor}}}
@@ -182,7 +182,7 @@ class RupenexConfig(ModelConfig):
         eps = take_float(_obj(d, "norm"), "eps")
         if eps <= 0:
             raise ConfigError(f"config.json: norm.eps must be positive, got {eps}")
-        scale = take_float(d, "logit_scale")
+        scale = take_float(d, "logit_scale", 1.0)
         raw = d.get("layers")
         if not isinstance(raw, list) or not raw:
             raise ConfigError("config.json: 'layers' must be a non-empty list")

@@ -29,7 +29,7 @@ def test_config_round_trip_and_refusals():
             at[path[-1]] = value
         return c
     attn, mamba, moe = ("layers", 0, "mixer"), ("layers", 1, "mixer"), ("layers", 0, "mlp")
-    for path, value in ((("vocab",), KeyError), (("norm", "eps"), 0.0), (("layers",), []), (("logit_scale",), KeyError),
+    for path, value in ((("vocab",), KeyError), (("norm", "eps"), 0.0), (("layers",), []), (("logit_scale",), "2"),
                         (attn + ("heads",), 3), (attn + ("kv_heads",), 0), (attn + ("rot", "dims"), 3), (attn + ("rot", "dims"), 18),
                         (attn + ("rot", "scaling", "factor"), 0), (attn + ("rot", "scaling"), {}), (attn + ("scale",), KeyError),
                         (attn + ("mask", "size"), 0), (attn + ("mask", "keep_first"), -1), (attn + ("mask",), 5),
@@ -39,6 +39,7 @@ def test_config_round_trip_and_refusals():
                         (moe + ("router", "identity"), -1), (moe + ("shared",), {"ff": 0}), (moe + ("expert",), KeyError)):
         with pytest.raises(ConfigError):
             parse_config(broken(path, value))
+    assert parse_config(broken(("logit_scale",), KeyError)).logit_scale == 1.0
     # all of what a router chooses among may be chosen, identity experts included
     assert parse_config(broken(moe + ("router", "top"), 8)).layers[0].mlp.top == 8
 
